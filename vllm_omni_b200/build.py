@@ -43,16 +43,19 @@ def _compile(src: Path, force: bool, checked: bool = False) -> str:
     dep_m = max(src.stat().st_mtime, _newest_header_mtime())
     if not force and out.exists() and out.stat().st_mtime >= dep_m:
         return f"up-to-date {out.name}"
+    tmp = out.with_name(f".{out.name}.{os.getpid()}")
     if src.suffix == ".cu":
         nvcc = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
-        cmd = [nvcc, *NVCC_FLAGS, *(["-DOMNI_BOUNDS_CHECK"] if checked else []), "-I", str(CSRC), "-o", str(out), str(src)]
+        cmd = [nvcc, *NVCC_FLAGS, *(["-DOMNI_BOUNDS_CHECK"] if checked else []), "-I", str(CSRC), "-o", str(tmp), str(src)]
     else:
         cuda_inc = os.path.join(os.environ.get("CUDA_HOME", "/usr/local/cuda"), "include")     # NVTX v3 headers
         inc = ["-I", cuda_inc] if os.path.isdir(cuda_inc) else []
-        cmd = [os.environ.get("CXX", "g++"), *CXX_FLAGS, "-I", str(CSRC), *inc, "-o", str(out), str(src), "-lrt", "-ldl"]
+        cmd = [os.environ.get("CXX", "g++"), *CXX_FLAGS, "-I", str(CSRC), *inc, "-o", str(tmp), str(src), "-lrt", "-ldl"]
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
+        tmp.unlink(missing_ok=True)
         raise RuntimeError(f"build failed: {' '.join(cmd)}\n{r.stdout}\n{r.stderr}")
+    os.replace(tmp, out)                     # a process that starts meanwhile never loads half a library
     return f"built {out.name}"
 
 
@@ -77,6 +80,16 @@ def build_one(name: str, force: bool = False) -> str:
         if src.exists():
             return _compile(src, force)
     raise FileNotFoundError(f"no source for library {name!r} under {CSRC}")
+
+
+def build_set(names) -> list[str]:
+    """Build the named libraries that are missing or older than their sources, one process at a time."""
+    import fcntl
+    LIB.mkdir(exist_ok=True)
+    with open(LIB / ".lock", "w") as lk:
+        fcntl.flock(lk, fcntl.LOCK_EX)
+        with ThreadPoolExecutor(max_workers=min(8, len(names) or 1)) as ex:
+            return list(ex.map(build_one, names))
 
 
 if __name__ == "__main__":

@@ -1,0 +1,32 @@
+// Operands of the windowed paged attention family (attn_window.cu, attn_window_sm100.cu).
+//
+// Position i of a sequence attends to j <= i with i - j < window or j < keep_first.  The score is
+// (q . k) * scale, optionally bounded to cap * tanh(score / cap), minus r1[h] * ln(1 + r2[h] * (i - j)).
+// `sink[h]` joins the softmax denominator as exp(sink[h]).  `gate` multiplies head h's result by
+// sigmoid(gate[row, h]).  Heads are padded to dp (query / key) and vp (value) channels, multiples of 16
+// with zero padding.
+#pragma once
+#include <cuda_runtime.h>
+
+namespace omni {
+
+struct WinAttn {
+  const void* q; long q_rs;            // [T, H, dp], row pitch in elements
+  const void* k_cache; const void* v_cache;     // [num_blocks, block_size, G, dp | vp]
+  const int* block_tables; int bt_stride;       // [S, bt_stride]
+  const int* q_start; const int* context;       // [S + 1], [S]
+  const int* row_seq;                  // [T] (row-per-block kernel)
+  const int* seq_list; int n_list;     // decode kernel: sequences with exactly one row
+  const int* items; int n_items;       // prefill kernel: (sequence, first token of the block) pairs
+  void* out; long o_rs;                // [T, H, vp]
+  const void* gate; long g_rs;         // [T, H] logits or nullptr
+  const float* r1; const float* r2;    // [H] or nullptr
+  const float* sink;                   // [H] or nullptr
+  float scale, cap;                    // cap <= 0: no bound
+  int window, keep_first;              // window <= 0: unbounded
+  int T, H, G, dp, vp, num_seqs, num_blocks, block_size;
+  int splits; float* part_o; float* part_ml;    // decode: shares of the visible keys, merged by a second kernel
+  int* status;
+};
+
+}  // namespace omni

@@ -1,0 +1,467 @@
+// Row-wise steps of decoder-only language models whose residual stream is kept in fp32, for bf16
+// activations (serving) and fp32 activations (exact mode):
+//
+//   omni_embed_norm     x = embed[id] (+ position table), xn = rms(x) * g            (one launch)
+//   omni_add_norm       x += rms(y) * g_y, xn = rms(x) * g_n                          (one launch)
+//   omni_poly_norm      a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's rms
+//   omni_conv_heads     short causal convolution over time of the packed q/k/v projection, per-head
+//                       RMS norm of q and k, mixing of v with an earlier layer's values, K/V rows
+//                       written to their pages, convolution history written to the state pool
+//   omni_logit_softcap  cap * tanh(logit / cap) -> fp32
+//
+// Norm gains are fp32, either one number for the whole row (stride 0) or one per channel (stride 1).
+// Rows are padded to a multiple of 8 channels; padding channels hold zeros and do not count in means.
+#include "host_util.h"
+#include "ptx_sm100.cuh"
+
+namespace omni {
+
+// eight consecutive elements as fp32
+template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]);
+template <> __device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 f = unpack_bf16(w[j]);
+    v[2 * j] = f.x;
+    v[2 * j + 1] = f.y;
+  }
+}
+template <typename T> __device__ __forceinline__ void store8(T* p, const float (&v)[8]);
+template <> __device__ __forceinline__ void store8<float>(float* p, const float (&v)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <> __device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]),
+                                            pack_bf16(v[6], v[7]));
+}
+
+// Sum of NV values over the block; every thread gets the totals.  `sh` holds 32 * NV floats.
+template <int NV>
+__device__ __forceinline__ void block_sum(float (&s)[NV], float* sh) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) s[i] += __shfl_xor_sync(0xffffffffu, s[i], o);
+  __syncthreads();          // the previous use of `sh` is over
+  if (lane == 0)
+#pragma unroll
+    for (int i = 0; i < NV; ++i) sh[warp * NV + i] = s[i];
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    float t = 0.f;
+    for (int w = 0; w < nw; ++w) t += sh[w * NV + i];
+    s[i] = t;
+  }
+}
+
+__device__ __forceinline__ float rms_scale(float sumsq, int n, float eps) {
+  return 1.0f / sqrtf(sumsq / (float)n + eps);
+}
+
+// multiply eight values by `s` and the gains of their channels
+__device__ __forceinline__ void scale_gain8(float (&v)[8], float s, const float* g, int gs, int c) {
+  if (gs == 0) {
+    const float k = s * g[0];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= k;
+  } else {
+    float w[8];
+    load8<float>(g + c, w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= s * w[e];
+  }
+}
+
+// ------------------------------------------------------------------ embedding + first norm
+template <typename T, int NV>
+__global__ void __launch_bounds__(1024)
+embed_norm_kernel(const long* __restrict__ ids, const long* __restrict__ pos, const T* __restrict__ embed, int vocab,
+                  const T* __restrict__ pos_table, int max_pos, const T* __restrict__ overlay,
+                  const unsigned char* __restrict__ overlay_mask, float* __restrict__ x, T* __restrict__ xn,
+                  const float* __restrict__ g, int gs, int D, int Dp, int ld_embed, float eps) {
+  __shared__ float sh[32];
+  const long r = blockIdx.x;
+  long id = ids[r];
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  long p = pos_table ? pos[r] : 0;
+  p = p < 0 ? 0 : (p >= max_pos ? max_pos - 1 : p);
+  const bool over = overlay != nullptr && (overlay_mask == nullptr || overlay_mask[r]);
+  const T* src = over ? overlay + r * ld_embed : embed + id * ld_embed;
+  float v[NV][8];
+  float ss[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Dp) {
+      load8<T>(src + c, v[i]);
+      if (pos_table) {
+        float pe[8];
+        load8<T>(pos_table + p * ld_embed + c, pe);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] += pe[e];
+      }
+      store8<float>(x + r * Dp + c, v[i]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss[0] = fmaf(v[i][e], v[i][e], ss[0]);
+    }
+  }
+  block_sum<1>(ss, sh);
+  const float s = rms_scale(ss[0], D, eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Dp) {
+      scale_gain8(v[i], s, g, gs, c);
+      store8<T>(xn + r * Dp + c, v[i]);
+    }
+  }
+}
+
+// ------------------------------------------------- residual add of a normed branch + next norm
+// x += rms(y) * g_y; xn = rms(x) * g_n.  xn == nullptr: no second norm.
+template <typename T, int NV>
+__global__ void __launch_bounds__(1024)
+add_norm_kernel(float* __restrict__ x, const T* __restrict__ y, int ldy, const float* __restrict__ gy, int gys,
+                T* __restrict__ xn, const float* __restrict__ gn, int gns, int D, int Dp, float eps) {
+  __shared__ float sh[32];
+  const long r = blockIdx.x;
+  float yv[NV][8], xv[NV][8];
+  float ss[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Dp) {
+      load8<T>(y + r * ldy + c, yv[i]);
+      load8<float>(x + r * Dp + c, xv[i]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss[0] = fmaf(yv[i][e], yv[i][e], ss[0]);
+    }
+  }
+  block_sum<1>(ss, sh);
+  const float sy = rms_scale(ss[0], D, eps);
+  ss[0] = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Dp) {
+      scale_gain8(yv[i], sy, gy, gys, c);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        xv[i][e] += yv[i][e];
+        ss[0] = fmaf(xv[i][e], xv[i][e], ss[0]);
+      }
+      store8<float>(x + r * Dp + c, xv[i]);
+    }
+  }
+  if (xn == nullptr) return;
+  block_sum<1>(ss, sh);
+  const float sn = rms_scale(ss[0], D, eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Dp) {
+      scale_gain8(xv[i], sn, gn, gns, c);
+      store8<T>(xn + r * Dp + c, xv[i]);
+    }
+  }
+}
+
+// --------------------------------------------------------------------------------- PolyNorm
+template <typename T, int NV>
+__global__ void __launch_bounds__(1024)
+poly_norm_kernel(const T* __restrict__ z, int ldz, T* __restrict__ out, int ldo, const float* __restrict__ coef, int F,
+                 int Fp, float eps) {
+  __shared__ float sh[96];
+  const long r = blockIdx.x;
+  float v[NV][8];
+  float ss[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Fp) {
+      load8<T>(z + r * ldz + c, v[i]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float q = v[i][e] * v[i][e];
+        ss[0] += q;
+        ss[1] = fmaf(q, q, ss[1]);
+        ss[2] = fmaf(q * q, q, ss[2]);
+      }
+    }
+  }
+  block_sum<3>(ss, sh);
+  const float k1 = coef[0] * rms_scale(ss[0], F, eps), k2 = coef[1] * rms_scale(ss[1], F, eps);
+  const float k3 = coef[2] * rms_scale(ss[2], F, eps), k0 = coef[3];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Fp) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] = fmaf(v[i][e], fmaf(v[i][e], fmaf(v[i][e], k3, k2), k1), k0);
+      store8<T>(out + r * ldo + c, v[i]);
+    }
+  }
+}
+
+// ------------------------------------------ short convolution, head norms, value mixing, pages
+// The packed projection has columns [q: H * dp | k: G * dp | v: G * vp | ...], heads padded to dp / vp
+// channels (multiples of 8).  A group of `lph` lanes owns one (row, head); a lane holds 8 channels.
+// The history of a sequence (its last K-1 projected rows) comes from the state pool when it lies before
+// the rows of this launch; pool rows are double-buffered (read index != write index), so the groups that
+// read a sequence's old history never race with the one that writes its new one.
+struct ConvHeads {
+  const void* proj; long ldp;
+  int T, H, G, dp, vp, d, taps;
+  const float* conv;        // [taps, H * dp + G * dp + G * vp] or nullptr
+  const float* q_norm;      // [dp] or nullptr (no norm)
+  const float* k_norm;
+  float eps;
+  const int* row_seq;       // [T] sequence of each row
+  const int* q_start;       // [S + 1] first row of each sequence
+  const int* context;       // [S] tokens of the sequence before its first row
+  const int* slots;         // [T] page slot of each row, < 0: not written
+  void* state;              // [pool rows, taps - 1, channels]
+  const int* state_in;      // [S]
+  const int* state_out;     // [S], < 0: not written
+  void* q_out;              // [T, H * dp]
+  void* k_cache; void* v_cache;     // [slots, G, dp], [slots, G, vp]
+  void* v_first;            // [T, G * vp]
+  int v_mode;               // 0: as they are, 1: also saved to v_first, 2: mixed with v_first
+  const float* lambda;
+  long num_slots;           // page slots of the caches / rows of the pool (bounds of the index operands)
+  int num_state, num_seqs;
+  int* status;
+  int lph;                  // lanes per head: a power of two, 32 at most
+};
+
+template <typename T, int IT>
+__global__ void __launch_bounds__(256)
+conv_heads_kernel(ConvHeads p) {
+  const int lane = threadIdx.x & (p.lph - 1);
+  const int t = blockIdx.x * (blockDim.x / p.lph) + threadIdx.x / p.lph;
+  const int head = blockIdx.y;
+  const bool live = t < p.T;
+  const int row = live ? t : p.T - 1;                     // idle groups keep the shuffles company
+  const int kind = head < p.H ? 0 : (head < p.H + p.G ? 1 : 2);
+  const int width = kind == 2 ? p.vp : p.dp;
+  const int hk = kind == 0 ? head : (kind == 1 ? head - p.H : head - p.H - p.G);
+  const int C = (p.H + p.G) * p.dp + p.G * p.vp;
+  const int col0 = kind == 0 ? hk * p.dp : (kind == 1 ? (p.H + hk) * p.dp : (p.H + p.G) * p.dp + hk * p.vp);
+  const T* proj = static_cast<const T*>(p.proj);
+  T* state = static_cast<T*>(p.state);
+  int seq = p.row_seq[row];
+  seq = min(max(seq, 0), p.num_seqs - 1);
+  const int q0 = p.q_start[seq], ctx = p.context[seq];
+  const int off = row - q0;                               // row within the sequence's portion
+  const int hist = p.taps - 1;
+  int sin = 0, sout = -1;
+  if (hist > 0) {
+    sin = p.state_in[seq];
+    sout = p.state_out[seq];
+    if (sin < 0 || sin >= p.num_state || sout >= p.num_state) {
+      if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+      sin = 0;
+      sout = -1;
+    }
+  }
+  float v[IT][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < IT; ++i) {
+    const int c = (i * p.lph + lane) * 8;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[i][e] = 0.f;
+    if (c < width) {
+      const int col = col0 + c;
+      if (p.conv == nullptr) {
+        load8<T>(proj + (long)row * p.ldp + col, v[i]);
+      } else {
+        for (int j = 0; j < p.taps; ++j) {
+          const int b = off - hist + j;                   // row of the portion; negative: history
+          float u[8], w[8];
+          if (b >= 0) load8<T>(proj + (long)(q0 + b) * p.ldp + col, u);
+          else if (ctx + b >= 0) load8<T>(state + ((long)sin * hist + hist + b) * C + col, u);
+          else continue;
+          load8<float>(p.conv + (long)j * C + col, w);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[i][e] = fmaf(w[e], u[e], v[i][e]);
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[i][e], v[i][e], ss);
+    }
+  }
+  // new history: the group of the portion's last row writes all of it
+  if (live && hist > 0 && sout >= 0 && row == p.q_start[seq + 1] - 1) {
+    const int n = off + 1;
+    for (int m = 0; m < hist; ++m) {
+      const int b = n - hist + m;
+#pragma unroll
+      for (int i = 0; i < IT; ++i) {
+        const int c = (i * p.lph + lane) * 8;
+        if (c < width) {
+          float u[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+          if (b >= 0) load8<T>(proj + (long)(q0 + b) * p.ldp + col0 + c, u);
+          else if (ctx + b >= 0) load8<T>(state + ((long)sin * hist + hist + b) * C + col0 + c, u);
+          store8<T>(state + ((long)sout * hist + m) * C + col0 + c, u);
+        }
+      }
+    }
+  }
+  const float* nw = kind == 0 ? p.q_norm : (kind == 1 ? p.k_norm : nullptr);
+  if (nw != nullptr) {                                    // uniform over the block (one head per block row)
+    for (int o = p.lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float s = rms_scale(ss, p.d, p.eps);
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+      const int c = (i * p.lph + lane) * 8;
+      if (c < width) scale_gain8(v[i], s, nw, 1, c);
+    }
+  }
+  if (!live) return;
+  int slot = kind == 0 ? 0 : p.slots[row];
+  if (slot >= p.num_slots && kind != 0) {
+    if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+    slot = -1;
+  }
+  const float lam = p.v_mode == 2 ? p.lambda[0] : 0.f;
+#pragma unroll
+  for (int i = 0; i < IT; ++i) {
+    const int c = (i * p.lph + lane) * 8;
+    if (c >= width) continue;
+    if (kind == 0) {
+      store8<T>(static_cast<T*>(p.q_out) + (long)row * p.H * p.dp + col0 + c, v[i]);
+    } else if (kind == 1) {
+      if (slot >= 0) store8<T>(static_cast<T*>(p.k_cache) + ((long)slot * p.G + hk) * p.dp + c, v[i]);
+    } else {
+      T* vf = static_cast<T*>(p.v_first) + (long)row * p.G * p.vp + hk * p.vp + c;
+      if (p.v_mode == 1) store8<T>(vf, v[i]);
+      if (p.v_mode == 2) {
+        float f[8];
+        load8<T>(vf, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = (1.f - lam) * v[i][e] + lam * f[e];
+      }
+      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + ((long)slot * p.G + hk) * p.vp + c, v[i]);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------ logit cap
+template <typename T>
+__global__ void __launch_bounds__(256)
+logit_softcap_kernel(const T* __restrict__ in, long ldi, float* __restrict__ out, long ldo, long rows, int V, float cap) {
+  const long total = rows * V;
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
+    const long r = i / V;
+    const int c = (int)(i - r * V);
+    const float z = (float)in[r * ldi + c];
+    out[r * ldo + c] = cap > 0.f ? cap * tanhf(z / cap) : z;
+  }
+}
+
+// threads and vectors per thread for a row of n channels (n <= 32768)
+static bool row_shape(int n, int& threads, int& nv) {
+  const int vec = n / 8;
+  for (threads = 64; threads < 1024 && threads < vec; threads *= 2) {
+    if (threads >= 256 && vec <= threads * 2) break;
+  }
+  nv = (vec + threads - 1) / threads;
+  nv = nv <= 1 ? 1 : (nv <= 2 ? 2 : 4);
+  return vec <= threads * nv;
+}
+
+}  // namespace omni
+
+using namespace omni;
+typedef __nv_bfloat16 bf16;
+
+#define OMNI_ROW_DISPATCH(KERNEL, ROWS, ...)                                                            \
+  do {                                                                                                  \
+    cudaStream_t st_ = (cudaStream_t)stream;                                                            \
+    if (is_bf16) {                                                                                      \
+      typedef bf16 T;                                                                                   \
+      if (nv == 1) KERNEL<T, 1><<<(unsigned)(ROWS), threads, 0, st_>>>(__VA_ARGS__);                    \
+      else if (nv == 2) KERNEL<T, 2><<<(unsigned)(ROWS), threads, 0, st_>>>(__VA_ARGS__);               \
+      else KERNEL<T, 4><<<(unsigned)(ROWS), threads, 0, st_>>>(__VA_ARGS__);                            \
+    } else {                                                                                            \
+      typedef float T;                                                                                  \
+      if (nv == 1) KERNEL<T, 1><<<(unsigned)(ROWS), threads, 0, st_>>>(__VA_ARGS__);                    \
+      else if (nv == 2) KERNEL<T, 2><<<(unsigned)(ROWS), threads, 0, st_>>>(__VA_ARGS__);               \
+      else KERNEL<T, 4><<<(unsigned)(ROWS), threads, 0, st_>>>(__VA_ARGS__);                            \
+    }                                                                                                   \
+  } while (0)
+
+extern "C" int omni_embed_norm(const long* ids, const long* pos, const void* embed, int vocab, const void* pos_table,
+                               int max_pos, const void* overlay, const void* overlay_mask, float* x, void* xn,
+                               const float* g, int gs, int rows, int D, int Dp, int ld_embed, float eps, int is_bf16,
+                               void* stream) {
+  if (rows <= 0) return RC_OK;
+  int threads, nv;
+  if ((Dp & 7) || (ld_embed & 7) || D > Dp || vocab < 1 || !row_shape(Dp, threads, nv)) return RC_BAD_ARG;
+  OMNI_ROW_DISPATCH(embed_norm_kernel, rows, ids, pos, (const T*)embed, vocab, (const T*)pos_table, max_pos,
+                    (const T*)overlay, (const unsigned char*)overlay_mask, x, (T*)xn, g, gs, D, Dp, ld_embed, eps);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_add_norm(float* x, const void* y, int ldy, const float* gy, int gys, void* xn, const float* gn,
+                             int gns, int rows, int D, int Dp, float eps, int is_bf16, void* stream) {
+  if (rows <= 0) return RC_OK;
+  int threads, nv;
+  if ((Dp & 7) || (ldy & 7) || D > Dp || !row_shape(Dp, threads, nv)) return RC_BAD_ARG;
+  OMNI_ROW_DISPATCH(add_norm_kernel, rows, x, (const T*)y, ldy, gy, gys, (T*)xn, gn, gns, D, Dp, eps);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_poly_norm(const void* z, int ldz, void* out, int ldo, const float* coef, int rows, int F, int Fp,
+                              float eps, int is_bf16, void* stream) {
+  if (rows <= 0) return RC_OK;
+  int threads, nv;
+  if ((Fp & 7) || (ldz & 7) || (ldo & 7) || F > Fp || !row_shape(Fp, threads, nv)) return RC_BAD_ARG;
+  OMNI_ROW_DISPATCH(poly_norm_kernel, rows, (const T*)z, ldz, (T*)out, ldo, coef, F, Fp, eps);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_conv_heads(const ConvHeads* args, int is_bf16, void* stream) {
+  ConvHeads p = *args;
+  if (p.T <= 0) return RC_OK;
+  if (p.num_seqs <= 0 || p.H <= 0 || p.G <= 0 || (p.dp & 7) || (p.vp & 7) || (p.ldp & 7) || p.d > p.dp || p.taps < 1)
+    return RC_BAD_ARG;
+  if ((p.conv == nullptr && p.taps != 1) || (p.taps > 1 && (p.state == nullptr || p.num_state <= 0))) return RC_BAD_ARG;
+  if (p.v_mode != 0 && p.v_first == nullptr) return RC_BAD_ARG;
+  const int lanes = (p.dp > p.vp ? p.dp : p.vp) / 8;
+  if (lanes > 128) return RC_BAD_ARG;
+  p.lph = 1;
+  while (p.lph < lanes && p.lph < 32) p.lph *= 2;
+  const int rows_per_cta = 256 / p.lph;
+  dim3 grid((p.T + rows_per_cta - 1) / rows_per_cta, p.H + 2 * p.G);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (is_bf16) {
+    if (lanes <= 32) conv_heads_kernel<bf16, 1><<<grid, 256, 0, st>>>(p);
+    else conv_heads_kernel<bf16, 4><<<grid, 256, 0, st>>>(p);
+  } else {
+    if (lanes <= 32) conv_heads_kernel<float, 1><<<grid, 256, 0, st>>>(p);
+    else conv_heads_kernel<float, 4><<<grid, 256, 0, st>>>(p);
+  }
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_logit_softcap(const void* in, long ldi, float* out, long ldo, long rows, int V, float cap, int is_bf16,
+                                  void* stream) {
+  if (rows <= 0) return RC_OK;
+  long blocks = (rows * V + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (is_bf16) logit_softcap_kernel<bf16><<<(unsigned)blocks, 256, 0, st>>>((const bf16*)in, ldi, out, ldo, rows, V, cap);
+  else logit_softcap_kernel<float><<<(unsigned)blocks, 256, 0, st>>>((const float*)in, ldi, out, ldo, rows, V, cap);
+  return (int)cudaGetLastError();
+}

@@ -19,6 +19,7 @@ from __future__ import annotations
 import torch
 
 from ..models.qwen_decoder import ModelBatch
+from ..models.seq_table import SeqTable
 
 DEFAULT_BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 256)
 
@@ -39,10 +40,21 @@ class _Bucket:
         self.hidden = None
         self.captured: dict = {}
         self.warm = False
+        self.seqs = None
+
+    def add_seq_table(self, max_context: int, stateful: bool):
+        """Static SeqTable of n one-token sequences over this bucket's tables."""
+        dev = self.ids.device
+        i32 = lambda *s, v=0: torch.full(s, v, dtype=torch.int32, device=dev)
+        self.starts = torch.arange(self.n + 1, dtype=torch.int32, device=dev)
+        self.ctx = i32(self.n)
+        state = (i32(self.n), i32(self.n, v=-1)) if stateful else (None, None)
+        self.seqs = SeqTable(self.starts, self.ctx, self.tables, self.starts[:self.n], self.starts[:self.n], self.n, self.n,
+                             max_context, *state)
 
     def batch(self) -> ModelBatch:
         return ModelBatch(self.ids, self.pos, self.slots, [], decode_rows=self.rows, decode_block_tables=self.tables,
-                          decode_seq_lens=self.lens, input_embeds=self.embeds, embeds_mask=self.emask)
+                          decode_seq_lens=self.lens, input_embeds=self.embeds, embeds_mask=self.emask, seqs=self.seqs)
 
 
 class DecodeGraphRunner:
@@ -71,6 +83,8 @@ class DecodeGraphRunner:
         if st is None:
             cfg = self.decoder.cfg
             st = _Bucket(size, cfg.hidden_size, self.max_blocks, cfg.mrope_section is not None, self.dtype, self.device)
+            if getattr(self.decoder, "uses_seq_table", False):
+                st.add_seq_table(self.max_blocks * self.kv_caches[0][0].shape[1], any(len(c) > 2 for c in self.kv_caches))
             self._state[size] = st
         return st
 
@@ -104,6 +118,13 @@ class DecodeGraphRunner:
         if pad:
             st.tables[n:].copy_(st.tables[:1].expand(pad, -1))
             st.lens[n:].copy_(st.lens[:1].expand(pad))
+        if st.seqs is not None:
+            put(st.ctx, b.seqs.context)
+            if st.seqs.state_in is not None:
+                put(st.seqs.state_in, b.seqs.state_in)
+                st.seqs.state_out[:n].copy_(b.seqs.state_out)
+                if pad:
+                    st.seqs.state_out[n:].fill_(-1)    # padding rows never write a sequence's state
         if b.input_embeds is not None:
             put(st.embeds, b.input_embeds.to(st.embeds.dtype))
             put(st.emask, b.embeds_mask if b.embeds_mask is not None else torch.ones_like(order, dtype=torch.bool))

@@ -1,5 +1,5 @@
-"""Paged KV cache bookkeeping: block pool (C++ allocator in csrc/rt_host.cpp, Python fallback)
-and the per-request block tables.  The device tensors themselves belong to the model runner;
+"""Paged KV cache bookkeeping: block pool (C++ allocator in csrc/rt_host.cpp, Python fallback),
+the per-request block tables and the slots of per-sequence state.  The device tensors themselves belong to the model runner;
 this class only decides which pages a request owns."""
 from __future__ import annotations
 
@@ -83,10 +83,51 @@ class BlockPool:
                 pass
 
 
+class StateSlots:
+    """Fixed-size per-sequence state (convolution histories, recurrent states) beside the pages.  A slot is
+    two rows of the runner's state tensors: a step reads one and writes the other, so that within one launch
+    the readers of a sequence's old state never race with the writer of its new one."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self._free = list(range(num_slots - 1, -1, -1))
+
+    @property
+    def num_rows(self) -> int:
+        return 2 * self.num_slots
+
+    @property
+    def num_free(self) -> int:
+        return len(self._free)
+
+    def acquire(self, request) -> bool:
+        if request.state_slot is not None:
+            return True
+        if not self._free:
+            return False
+        request.state_slot, request.state_phase = self._free.pop(), 0
+        return True
+
+    def rows(self, request) -> tuple[int, int]:
+        """(row the next step reads, row it writes).  A sequence's first step reads a stale row: kernels take
+        history only where the position says there is one."""
+        base = 2 * request.state_slot
+        return base + request.state_phase, base + 1 - request.state_phase
+
+    def advance(self, request) -> None:
+        request.state_phase ^= 1
+
+    def release(self, request) -> None:
+        if request.state_slot is not None:
+            self._free.append(request.state_slot)
+            request.state_slot = None
+
+
 class KVCacheManager:
-    def __init__(self, num_blocks: int, block_size: int):
+    def __init__(self, num_blocks: int, block_size: int, num_state_slots: int = 0):
         self.block_size = block_size
         self.pool = BlockPool(num_blocks)
+        self.state = StateSlots(num_state_slots) if num_state_slots else None
 
     def blocks_needed(self, request, num_new_tokens: int) -> int:
         total = request.num_computed_tokens + num_new_tokens
@@ -96,10 +137,15 @@ class KVCacheManager:
     def allocate_slots(self, request, num_new_tokens: int) -> bool:
         """Make sure ``request`` owns pages for its next ``num_new_tokens`` tokens."""
         n = self.blocks_needed(request, num_new_tokens)
+        fresh = self.state is not None and request.state_slot is None
+        if fresh and not self.state.acquire(request):
+            return False
         if n == 0:
             return True
         got = self.pool.alloc(n)
         if got is None:
+            if fresh:
+                self.state.release(request)
             return False
         request.block_ids.extend(got)
         return True
@@ -111,6 +157,8 @@ class KVCacheManager:
     def free(self, request) -> None:
         self.pool.free(request.block_ids)
         request.block_ids = []
+        if self.state is not None:
+            self.state.release(request)
 
     @property
     def usage(self) -> float:

@@ -30,7 +30,8 @@ class LLMEngine:
     def __init__(self, model, tokenizer=None, device=None, dtype=torch.bfloat16, block_size: int = 16,
                  num_gpu_blocks: int | None = None, gpu_memory_utilization: float = 0.9, max_num_seqs: int = 64,
                  max_num_batched_tokens: int = 8192, max_model_len: int = 32768, kv_transfer_criteria=None,
-                 chunk_adapter=None, kv_transfer_manager=None, stage_id: int = 0, engine_output_type: str | None = None):
+                 chunk_adapter=None, kv_transfer_manager=None, stage_id: int = 0, engine_output_type: str | None = None,
+                 scheduler_cls=None):
         self.model = model
         self.device = torch.device(device) if device is not None else torch.device(
             "cuda" if torch.cuda.is_available() else "cpu")
@@ -52,10 +53,17 @@ class LLMEngine:
             if num_gpu_blocks is None:
                 num_gpu_blocks = self._profile_num_blocks(dec, block_size, gpu_memory_utilization, max_model_len,
                                                           max_num_seqs)
-            self.kv = KVCacheManager(num_gpu_blocks, block_size)
-            self.runner = ARModelRunner(model, self.device, dtype, num_gpu_blocks, block_size)
-            self.scheduler = OmniARScheduler(self.kv, max_num_seqs, max_num_batched_tokens, kv_transfer_criteria,
-                                             chunk_adapter)
+            # models that carry per-sequence state beside the pages have a slot for every running sequence
+            stateful = any(s is not None for s in dec.state_shapes()) if hasattr(dec, "state_shapes") else False
+            self.kv = KVCacheManager(num_gpu_blocks, block_size, max_num_seqs if stateful else 0)
+            self.runner = ARModelRunner(model, self.device, dtype, num_gpu_blocks, block_size,
+                                        self.kv.state.num_rows if stateful else 0)
+            self.scheduler = (scheduler_cls or OmniARScheduler)(self.kv, max_num_seqs, max_num_batched_tokens,
+                                                                kv_transfer_criteria, chunk_adapter)
+            hard = getattr(dec, "max_positions", None)
+            if hard is not None:
+                max_model_len = min(max_model_len, hard)
+                self.scheduler.max_model_len = hard
         self.kv_transfer_manager = kv_transfer_manager
         self.max_model_len = max_model_len
         self._detok: dict[str, IncrementalDetokenizer] = {}
@@ -79,7 +87,7 @@ class LLMEngine:
         return int(rows * per_row * es) + (2 << 30)
 
     def _profile_num_blocks(self, dec, block_size, util, max_model_len, max_num_seqs) -> int:
-        per_block = 2 * dec.num_hidden_layers * block_size * dec.num_key_value_heads * dec.head_dim * \
+        per_block = block_size * sum(h * (dk + dv) for h, dk, dv in dec.kv_layer_shapes()) * \
             torch.empty(0, dtype=self.dtype).element_size()
         if self.device.type == "cuda":
             from ..utils.gpu_memory import kv_cache_budget

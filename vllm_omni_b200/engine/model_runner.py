@@ -19,21 +19,29 @@ import zlib
 import torch
 
 from ..models.qwen_decoder import ModelBatch, PrefillSeg
+from ..models.seq_table import SeqTable
 from ..ops import kv_cache as KC
 from ..ops.sampler import RowParams, sample
 from .scheduler import SchedulerOutput
 
 
 class ARModelRunner:
-    def __init__(self, model, device, dtype, num_blocks: int, block_size: int):
+    def __init__(self, model, device, dtype, num_blocks: int, block_size: int, num_state_rows: int = 0):
+        """``num_state_rows``: rows of the per-sequence state pool, for models that carry state beside the pages."""
         self.model, self.device, self.dtype = model, device, dtype
         self.block_size = block_size
         dec = model.decoder_config
         # under tensor parallelism a rank keeps the pages of its own KV heads only
-        kvh = getattr(getattr(model, "decoder", None), "kv_heads_local", dec.num_key_value_heads)
-        self.kv_caches = [(torch.zeros(num_blocks, block_size, kvh, dec.head_dim, dtype=dtype, device=device),
-                           torch.zeros(num_blocks, block_size, kvh, dec.head_dim, dtype=dtype, device=device))
-                          for _ in range(dec.num_hidden_layers)]
+        decoder = getattr(model, "decoder", None)
+        local = getattr(decoder, "kv_heads_local", None)
+        self.seq_table = bool(getattr(decoder, "uses_seq_table", False))
+        z = lambda *s: torch.zeros(*s, dtype=dtype, device=device)
+        self.kv_caches = [(z(num_blocks, block_size, local or h, dk), z(num_blocks, block_size, local or h, dv))
+                          for h, dk, dv in dec.kv_layer_shapes()]
+        if num_state_rows:
+            # a layer's cache entry is (k pages, v pages, state rows) where the layer carries state
+            self.kv_caches = [kv if s is None else kv + (z(num_state_rows, *s),)
+                              for kv, s in zip(self.kv_caches, dec.state_shapes())]
         self.tp_group = None        # set by OmniLLM: sampled ids of every step come from rank 0
         # decode-only steps replay a captured graph per batch-size bucket (on by default on a GPU,
         # ``OMNI_AR_CUDA_GRAPH=0`` switches it off); contexts longer than ``OMNI_AR_GRAPH_MAX_TOKENS``
@@ -53,7 +61,7 @@ class ARModelRunner:
         embeds, emask = [], []
         any_embeds = False
         row = 0
-        sample_rows, sample_reqs = [], []
+        sample_rows, sample_reqs, want_rows = [], [], []
         max_blocks = 1
         for s in sched.scheduled:
             r = s.request
@@ -64,8 +72,8 @@ class ARModelRunner:
             p = self.model.positions_for(r, s.start, s.num_new_tokens)
             pos.append(p)
             slots.extend(kv_mgr.slot_mapping(r, s.start, s.num_new_tokens))
-            bt = torch.tensor(r.block_ids, dtype=torch.int32)
             if s.is_prefill:
+                bt = None if self.seq_table else torch.tensor(r.block_ids, dtype=torch.int32)
                 prefills.append(PrefillSeg(row, s.num_new_tokens, s.start, bt))
             else:
                 dec_rows.append(row)
@@ -76,6 +84,7 @@ class ARModelRunner:
             if e is not None:
                 any_embeds = True
                 embeds.append((row, e))
+            want_rows.extend(row + w for w in s.want)
             if s.samples:
                 sample_rows.append(row + s.num_new_tokens - 1)
                 sample_reqs.append(r)
@@ -87,8 +96,14 @@ class ARModelRunner:
         batch = ModelBatch(torch.tensor(ids, dtype=torch.long, device=dev), positions.to(dev),
                            torch.tensor(slots, dtype=torch.int32, device=dev))
         for seg in prefills:
-            seg.block_table = seg.block_table.to(dev)
+            if seg.block_table is not None:
+                seg.block_table = seg.block_table.to(dev)
         batch.prefills = prefills
+        if self.seq_table:
+            live = [s.request for s in sched.scheduled]
+            states = [kv_mgr.state.rows(r) for r in live] if kv_mgr.state is not None else None
+            batch.seqs = SeqTable.build([s.num_new_tokens for s in sched.scheduled], [s.start for s in sched.scheduled],
+                                        [r.block_ids for r in live], states, dev)
         if dec_rows:
             batch.decode_rows = torch.tensor(dec_rows, dtype=torch.long, device=dev)
             batch.decode_block_tables = torch.tensor([t + [0] * (max_blocks - len(t)) for t in dec_tables],
@@ -102,7 +117,7 @@ class ARModelRunner:
                 buf[r0:r0 + e.shape[0]] = e.to(dev, self.dtype)
                 mask[r0:r0 + e.shape[0]] = True
             batch.input_embeds, batch.embeds_mask = buf, mask
-        return batch, sample_rows, sample_reqs
+        return batch, sample_rows, sample_reqs, want_rows
 
     # ------------------------------------------------------------------ step
     @torch.no_grad()
@@ -110,11 +125,16 @@ class ARModelRunner:
         """Runs one engine step; returns ({request_id: sampled token}, kv_extracted_request_ids)."""
         if sched.empty:
             return {}, []
-        batch, sample_rows, sample_reqs = self._build_batch(sched, kv_mgr)
+        batch, sample_rows, sample_reqs, want_rows = self._build_batch(sched, kv_mgr)
         if self.graph_runner is not None and self.graph_runner.supports(batch):
             hidden, captured = self.graph_runner.run(batch)
         else:
             hidden, captured = self.model.forward_batch(batch, self.kv_caches, sched)
+        if getattr(kv_mgr, "state", None) is not None:
+            for s in sched.scheduled:
+                kv_mgr.state.advance(s.request)
+        if want_rows:
+            sched.logits = self.model.compute_logits(hidden[torch.tensor(want_rows, dtype=torch.long, device=self.device)])
         sampled: dict[str, int] = {}
         if sample_rows:
             rows_t = torch.tensor(sample_rows, dtype=torch.long, device=self.device)
@@ -150,10 +170,14 @@ class ARModelRunner:
         T = request.num_computed_tokens
         bt = torch.tensor(request.block_ids, dtype=torch.int32, device=self.device)
         layers = []
-        for li, (kc, vc) in enumerate(self.kv_caches):
+        for li, (kc, vc, *_) in enumerate(self.kv_caches):
             ok, ov = (out_buffers[li] if out_buffers is not None else (None, None))
             layers.append(KC.kv_gather(kc, vc, bt, T, ok, ov))
-        return {"num_tokens": T, "layers": layers}
+        out = {"num_tokens": T, "layers": layers}
+        if request.state_slot is not None:
+            row = 2 * request.state_slot + request.state_phase
+            out["state"] = [c[2][row].clone() if len(c) > 2 else None for c in self.kv_caches]
+        return out
 
 
 class GenerationModelRunner:

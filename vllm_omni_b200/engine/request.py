@@ -49,6 +49,8 @@ class Request:
     output_token_ids: list[int] = field(default_factory=list)
     num_computed_tokens: int = 0                           # tokens whose KV is in the cache
     block_ids: list[int] = field(default_factory=list)
+    state_slot: int | None = None                          # slot of the per-sequence state (models that carry one)
+    state_phase: int = 0                                   # which of the slot's two rows holds the current state
     num_emitted_tokens: int = 0                            # output tokens already reported (streaming)
     multimodal_outputs: dict[str, list] = field(default_factory=dict)
     first_token_time: float | None = None

@@ -29,6 +29,7 @@ class ScheduledRequest:
     start: int                   # == request.num_computed_tokens
     is_prefill: bool
     samples: bool                # whether this step produces a token for the request
+    want: list[int] = field(default_factory=list)    # rows of this portion whose logits the caller asks for
 
 
 @dataclass
@@ -37,6 +38,7 @@ class SchedulerOutput:
     finished_ids: list[str] = field(default_factory=list)
     kv_transfer_ids: list[str] = field(default_factory=list)     # extract KV for these after the step
     total_tokens: int = 0
+    logits: object | None = None          # [wanted rows, vocab] in batch order, set by the runner
 
     @property
     def empty(self) -> bool:
@@ -56,6 +58,7 @@ class OmniARScheduler:
         self.chunk_adapter = chunk_adapter
         self.waiting_for_kv_extract: dict[str, Request] = {}
         self.finished_since_last: list[str] = []
+        self.max_model_len: int | None = None      # hard limit of a sequence's length (learned position tables)
 
     # ------------------------------------------------------------------ admission
     def add_request(self, req: Request) -> None:
@@ -216,7 +219,7 @@ class OmniARScheduler:
             if sp.stop_token_ids and tok in sp.stop_token_ids:
                 req.status, req.stop_reason = RequestStatus.FINISHED_STOPPED, tok
                 return
-        if n_out >= req.max_tokens:
+        if n_out >= req.max_tokens or (self.max_model_len is not None and req.num_tokens >= self.max_model_len):
             req.status = RequestStatus.FINISHED_LENGTH
 
     def _release(self, req: Request) -> None:

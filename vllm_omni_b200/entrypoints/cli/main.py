@@ -1,10 +1,13 @@
-"""Command line: ``vllm-omni-b200 serve MODEL [--omni] ...`` and ``vllm-omni-b200 bench ...``
+"""Command line: ``vllm-omni-b200 serve MODEL [--omni] ...``, ``vllm-omni-b200 bench ...`` and
+``vllm-omni-b200 trace ...`` (replay of a schedule of token ids)
 (vllm_omni/entrypoints/cli/main.py, cli/serve.py: the flag set of ``OmniServeCommand``)."""
 from __future__ import annotations
 
 import argparse
 import json
 import sys
+
+from ..trace import make_parser as make_trace_parser
 
 
 def make_serve_parser(sub=None) -> argparse.ArgumentParser:
@@ -72,6 +75,7 @@ def main(argv=None) -> int:
     ap = argparse.ArgumentParser("vllm-omni-b200")
     sub = ap.add_subparsers(dest="cmd", required=True)
     make_serve_parser(sub)
+    make_trace_parser(sub)
     b = sub.add_parser("bench", help="benchmarks")
     b.add_argument("what", choices=["serve", "image"])
     b.add_argument("rest", nargs=argparse.REMAINDER)
@@ -80,6 +84,9 @@ def main(argv=None) -> int:
         from ..openai.api_server import omni_run_server
         omni_run_server(args.model, host=args.host, port=args.port, **serve_kwargs(args))
         return 0
+    if args.cmd == "trace":
+        from ..trace import run
+        return run(args)
     if args.cmd == "bench":
         from ...benchmarks.serve_bench import main as bench_main
         return bench_main([args.what] + args.rest)

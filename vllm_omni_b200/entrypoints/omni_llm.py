@@ -17,7 +17,7 @@ from ..engine.llm_engine import LLMEngine
 from ..engine.tokenizer import get_tokenizer
 from ..inputs.data import SamplingParams
 from ..logger import init_logger
-from ..models.registry import build_stage_model
+from ..models.registry import arch_from_config, build_stage_model
 
 logger = init_logger(__name__)
 _BUILD_LOCK = threading.Lock()
@@ -69,6 +69,14 @@ class OmniEngineArgs:
         return a
 
 
+def resolve_scheduler(name):
+    """``scheduler_cls`` engine argument: None, a class, or the dotted path of one."""
+    if not isinstance(name, str):
+        return name
+    from .utils import resolve_callable
+    return resolve_callable(name) if "vllm_omni." not in name else None      # the reference's own names: the default
+
+
 _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float16": torch.float16, "float32": torch.float32,
            "fp32": torch.float32, "auto": torch.bfloat16}
 
@@ -98,7 +106,7 @@ class OmniLLM:
             with open(os.path.join(model, "config.json")) as f:
                 hf_cfg = json.load(f)
             hf_cfg.setdefault("_model_dir", model)          # for models that keep sub-configs in sub-folders
-        arch = a.model_arch or (hf_cfg.get("architectures") or ["Qwen3ForCausalLM"])[0]
+        arch = a.model_arch or arch_from_config(hf_cfg) or "Qwen3ForCausalLM"
         # stages that share a process are built on a thread pool and share torch's global generator:
         # seeding and random initialisation must not interleave, or the weights depend on thread timing
         with _BUILD_LOCK:
@@ -137,7 +145,8 @@ class OmniLLM:
                                 gpu_memory_utilization=a.gpu_memory_utilization, max_num_seqs=a.max_num_seqs,
                                 max_num_batched_tokens=a.max_num_batched_tokens, max_model_len=a.max_model_len,
                                 kv_transfer_criteria=crit, chunk_adapter=chunk_adapter, kv_transfer_manager=kv_mgr,
-                                stage_id=stage_id, engine_output_type=a.engine_output_type)
+                                stage_id=stage_id, engine_output_type=a.engine_output_type,
+                                scheduler_cls=resolve_scheduler(a.scheduler_cls))
         self.engine.stream_interval = int(a.stream_interval)
         self.engine.stream_mm_interval = int(a.stream_mm_interval)
         if a.stream_output_keys is not None:

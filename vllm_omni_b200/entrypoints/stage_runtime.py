@@ -24,7 +24,7 @@ from ..logger import init_logger
 from ..outputs import OmniRequestOutput
 from .stage_utils import OmniStageTaskType, set_stage_devices, to_host
 from .utils import (OmniPipelineConfig, StageConfig, inject_omni_kv_config, load_stage_configs_from_yaml,
-                    resolve_callable, resolve_model_config_path)
+                    resolve_callable, resolve_model_config_path, text_architecture)
 
 logger = init_logger(__name__)
 
@@ -499,6 +499,21 @@ def _default_diffusion_stage(kwargs: dict) -> dict:
             "final_output_type": "image"}
 
 
+def _default_text_stage(arch: str, kwargs: dict) -> dict:
+    """One AR stage for a causal-LM folder without a packaged stage configuration; engine arguments given to
+    ``Omni`` / ``serve`` reach the stage engine."""
+    args = {k: v for k, v in kwargs.items() if k not in ("max_batch_size", "parallel_config")}
+    if "max_batch_size" in kwargs:
+        args.setdefault("max_num_seqs", int(kwargs["max_batch_size"]))
+    tp = getattr(kwargs.get("parallel_config"), "tensor_parallel_size", 1) or 1
+    if tp > 1:
+        args["tensor_parallel_size"] = tp
+    return {"stage_id": 0, "stage_type": "llm",
+            "runtime": {"process": tp > 1, "devices": ",".join(str(i) for i in range(tp))},
+            "engine_args": {**args, "model_arch": arch, "worker_type": "ar", "engine_output_type": "text"},
+            "is_comprehension": True, "final_output": True, "final_output_type": "text"}
+
+
 def build_stages(model, stage_configs_path, kwargs: dict, stage_init_timeout=300, shm_threshold_bytes=65536,
                  worker_backend="mp", batch_timeout=10):
     """Returns (stages, connectors, pipeline_config).  ``batch_timeout`` is in milliseconds."""
@@ -514,7 +529,9 @@ def build_stages(model, stage_configs_path, kwargs: dict, stage_init_timeout=300
     else:
         from .utils import load_stage_configs_from_dict
         pcfg = load_stage_configs_from_dict({"stage_args": []})
-        pcfg.stages = [StageConfig.from_dict(_default_diffusion_stage(dict(kwargs)))]
+        arch = text_architecture(model)
+        pcfg.stages = [StageConfig.from_dict(_default_text_stage(arch, dict(kwargs)) if arch
+                                             else _default_diffusion_stage(dict(kwargs)))]
     inject_omni_kv_config(pcfg.stages)
     if worker_backend == "ray":
         placement_group = ray_utils.create_placement_group(pcfg.stages)

@@ -105,6 +105,18 @@ def get_model_type(model: str | None) -> str | None:
         return json.load(f).get("model_type")
 
 
+def text_architecture(model: str | None) -> str | None:
+    """Architecture of a local model folder that is one causal-LM stage: its ``config.json`` names a registered
+    AR model and no packaged stage configuration exists for it."""
+    p = os.path.join(model, "config.json") if model and os.path.isdir(model) else None
+    if p is None or not os.path.exists(p):
+        return None
+    from ..models.registry import arch_from_config, supported_archs
+    with open(p) as f:
+        arch = arch_from_config(json.load(f))
+    return arch if arch in supported_archs() else None
+
+
 _NAME_HINTS = (("qwen3-omni", "qwen3_omni_moe"), ("qwen3_omni", "qwen3_omni_moe"), ("qwen2.5-omni", "qwen2_5_omni"),
                ("qwen2_5_omni", "qwen2_5_omni"), ("qwen3-tts", "qwen3_tts"), ("qwen3_tts", "qwen3_tts"),
                ("bagel", "bagel"))

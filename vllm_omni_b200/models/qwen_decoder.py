@@ -48,6 +48,10 @@ class DecoderConfig:
     max_position_embeddings: int = 65536
     tie_word_embeddings: bool = False
 
+    def kv_layer_shapes(self) -> list[tuple[int, int, int]]:
+        """(KV heads, key channels, value channels) of every layer's pages."""
+        return [(self.num_key_value_heads, self.head_dim, self.head_dim)] * self.num_hidden_layers
+
     @classmethod
     def from_dict(cls, d: dict) -> "DecoderConfig":
         d = dict(d)
@@ -89,6 +93,7 @@ class ModelBatch:
     decode_seq_lens: torch.Tensor | None = None
     input_embeds: torch.Tensor | None = None   # [T, D] replaces the embedding lookup where mask is set
     embeds_mask: torch.Tensor | None = None    # bool [T]
+    seqs: object | None = None                 # SeqTable (models/seq_table.py) for decoders that take one
 
 
 class RotaryTable:

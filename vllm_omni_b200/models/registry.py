@@ -11,12 +11,24 @@ _MODELS: dict[str, tuple[str, str]] = {
     "Qwen3ForCausalLM": ("vllm_omni_b200.models.text", "build_text_model"),
     "Qwen2ForCausalLM": ("vllm_omni_b200.models.text", "build_text_model"),
     "Qwen3MoeForCausalLM": ("vllm_omni_b200.models.text", "build_text_model"),
+    "Tavulix": ("vllm_omni_b200.models.tavulix.model", "build_tavulix"),
     "BagelForConditionalGeneration": ("vllm_omni_b200.models.text", "build_text_model"),
 }
 
 
 def register_model(arch: str, module: str, factory: str) -> None:
     _MODELS[arch] = (module, factory)
+
+
+def native_libs(arch: str) -> tuple[str, ...] | None:
+    """Libraries under csrc/ that serving ``arch`` loads (the model module's ``NATIVE_LIBS``), None = not declared."""
+    return getattr(importlib.import_module(_MODELS[arch][0]), "NATIVE_LIBS", None)
+
+
+def arch_from_config(cfg: dict) -> str | None:
+    """Architecture name of a ``config.json``: first of ``architectures``, or ``architecture``."""
+    archs = cfg.get("architectures") or [cfg.get("architecture")]
+    return archs[0] if isinstance(archs, list) else archs
 
 
 def supported_archs() -> list[str]:

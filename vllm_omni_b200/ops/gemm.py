@@ -77,6 +77,9 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, a
             out.copy_(y.reshape(out.shape))
             return out
         return y
+    if x.dtype == torch.float32 and w.dtype == torch.float32:
+        assert act is None and residual is None and gate is None and scatter is None and row_scatter is None
+        return _linear_f32(x, w, bias, out)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16, "tcgen05 GEMM path is bf16"
     K = x.shape[-1]
     N = w.shape[0]
@@ -128,6 +131,23 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, a
         ctypes.byref(sync) if sync is not None else None, nv.ptr(st), nv.stream_ptr())
     nv.check_rc(rc, "omni_gemm_bf16")
     return None if to_peers else out
+
+
+def _linear_f32(x, w, bias, out):
+    """Exact mode: true fp32 products on the CUDA cores (csrc/gemm_f32.cu); plain ``x @ w.T (+ bias)`` only."""
+    K, N = x.shape[-1], w.shape[0]
+    x2 = x.reshape(-1, K)
+    if x2.stride(-1) != 1:
+        x2 = x2.contiguous()
+    if out is None:
+        out = torch.empty(*x.shape[:-1], N, dtype=x.dtype, device=x.device)
+    o2 = out.view(-1, N)
+    assert w.stride(-1) == 1 and o2.stride(-1) == 1
+    rc = nv.lib("gemm_f32").omni_gemm_f32(nv.ptr(x2), ctypes.c_long(x2.stride(0)), nv.ptr(w), ctypes.c_long(w.stride(0)),
+                                          nv.ptr(o2), ctypes.c_long(o2.stride(0)), ctypes.c_int(x2.shape[0]),
+                                          ctypes.c_int(N), ctypes.c_int(K), nv.ptr(bias), nv.stream_ptr())
+    nv.check_rc(rc, "omni_gemm_f32")
+    return out
 
 
 class _GemmDesc(ctypes.Structure):

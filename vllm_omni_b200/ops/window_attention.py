@@ -1,0 +1,152 @@
+"""Attention of a mixed batch (prompt portions and single decoded tokens) over the paged cache, with a
+sliding window that keeps the first tokens, bounded scores, a logarithmic distance bias, a softmax sink
+and a per-head output gate — each optional.  Kernels: csrc/attn_window_sm100.cu (tcgen05, portions of two
+tokens and more), csrc/attn_window.cu (single tokens; and one block per row for fp32 and head sizes the
+tensor-core kernels do not take)."""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+
+import torch
+
+from . import _native as nv
+
+c_int, c_long, c_float, c_void_p = ctypes.c_int, ctypes.c_long, ctypes.c_float, ctypes.c_void_p
+
+
+class _WinAttn(ctypes.Structure):
+    _fields_ = [("q", c_void_p), ("q_rs", c_long), ("k_cache", c_void_p), ("v_cache", c_void_p),
+                ("block_tables", c_void_p), ("bt_stride", c_int), ("q_start", c_void_p), ("context", c_void_p),
+                ("row_seq", c_void_p), ("seq_list", c_void_p), ("n_list", c_int), ("items", c_void_p), ("n_items", c_int),
+                ("out", c_void_p), ("o_rs", c_long), ("gate", c_void_p), ("g_rs", c_long), ("r1", c_void_p),
+                ("r2", c_void_p), ("sink", c_void_p), ("scale", c_float), ("cap", c_float), ("window", c_int),
+                ("keep_first", c_int), ("T", c_int), ("H", c_int), ("G", c_int), ("dp", c_int), ("vp", c_int),
+                ("num_seqs", c_int), ("num_blocks", c_int), ("block_size", c_int), ("splits", c_int),
+                ("part_o", c_void_p), ("part_ml", c_void_p), ("status", c_void_p)]
+
+
+@dataclass
+class ScoreRule:
+    """What turns q . k into an attention weight.  None / 0 switches a step off."""
+    scale: float
+    softcap: float | None = None
+    r1: torch.Tensor | None = None        # fp32 [H]: distance bias r1 ln(1 + r2 dist)
+    r2: torch.Tensor | None = None
+    sink: torch.Tensor | None = None      # fp32 [H]
+    window: int | None = None
+    keep_first: int = 0
+
+
+def prefill_rows_per_block(heads: int, kv_heads: int) -> int:
+    """Tokens one block of the tcgen05 kernel serves: two 128-row tiles of (token, head of the KV group) rows."""
+    return 2 * (128 // (heads // kv_heads))
+
+
+def prefill_kernel_ok(heads: int, kv_heads: int, dp: int, vp: int, block_size: int) -> bool:
+    return False and heads // kv_heads <= 128 and dp <= 256 and vp <= 128 and block_size >= 8 and block_size % 8 == 0 \
+        and 128 % block_size == 0
+
+
+def decode_splits(n: int, kv_heads: int, group: int, max_keys: int) -> int:
+    """Blocks that share one sequence's visible keys: enough for about two blocks per SM, at least 64 keys each."""
+    blocks = n * kv_heads * ((group + 15) // 16)
+    want = max(1, (2 * 148) // max(1, blocks))
+    return max(1, min(want, 32, (max_keys + 63) // 64))
+
+
+_scratch: dict = {}
+
+
+def _parts(device, n: int, vp: int):
+    """fp32 scratch of the split decode; grows, and is never freed: captured graphs hold its address."""
+    key = (device.index, n, vp)
+    t = _scratch.get(key)
+    if t is None:
+        t = (torch.empty(n * vp, dtype=torch.float32, device=device), torch.empty(n * 2, dtype=torch.float32, device=device))
+        _scratch[key] = t
+    return t
+
+
+def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None, impl: str | None = None):
+    """q [T, H, dp]; caches [num_blocks, block_size, G, dp | vp] that already hold this step's tokens;
+    ``seqs``: the batch's ``SeqTable``; ``out`` [T, H * vp]; ``gate`` [T, H] logits (a view is fine).
+
+    ``impl="rows"`` forces the row-per-block kernel for every row."""
+    T, H, dp = q.shape
+    nb, bs, G, _ = k_cache.shape
+    vp = v_cache.shape[3]
+    if not q.is_cuda:
+        return _cpu(q, k_cache, v_cache, seqs, rule, out, gate)
+    assert q.is_contiguous() and out.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert seqs.block_tables.dtype == torch.int32 and seqs.block_tables.stride(1) == 1
+    a = _WinAttn()
+    P = lambda t: 0 if t is None else t.data_ptr()
+    a.q, a.q_rs, a.k_cache, a.v_cache = P(q), q.stride(0), P(k_cache), P(v_cache)
+    a.block_tables, a.bt_stride = P(seqs.block_tables), seqs.block_tables.stride(0)
+    a.q_start, a.context, a.row_seq = P(seqs.q_start), P(seqs.context), P(seqs.row_seq)
+    a.out, a.o_rs = P(out), out.stride(0)
+    a.gate, a.g_rs = P(gate), 0 if gate is None else gate.stride(0)
+    a.r1, a.r2, a.sink = P(rule.r1), P(rule.r2), P(rule.sink)
+    a.scale, a.cap = rule.scale, rule.softcap or 0.0
+    a.window, a.keep_first = rule.window or 0, rule.keep_first
+    a.T, a.H, a.G, a.dp, a.vp, a.num_seqs, a.num_blocks, a.block_size = T, H, G, dp, vp, seqs.n_seqs, nb, bs
+    a.splits = 1
+    a.status = P(nv.status_word(q.device))
+    bf = q.dtype == torch.bfloat16
+    rows_only = impl == "rows" or not bf or dp > 256 or vp > 256 or not (
+        seqs.n_decode == seqs.n_seqs or prefill_kernel_ok(H, G, dp, vp, bs))
+    if rows_only:
+        rc = nv.lib("attn_window").omni_attn_window_rows(ctypes.byref(a), c_int(1 if bf else 0), nv.stream_ptr())
+        nv.check_rc(rc, "omni_attn_window_rows")
+        return out
+    if seqs.n_decode < seqs.n_seqs:
+        items, n = seqs.prefill_items(prefill_rows_per_block(H, G))
+        a.items, a.n_items = P(items), n
+        rc = nv.lib("attn_window_sm100").omni_attn_window_prefill(ctypes.byref(a), nv.stream_ptr())
+        nv.check_rc(rc, "omni_attn_window_prefill")
+    if seqs.n_decode:
+        a.seq_list, a.n_list = P(seqs.decode_list), seqs.n_decode
+        keys = seqs.max_context + 1
+        if rule.window:
+            keys = min(keys, rule.window + rule.keep_first)
+        a.splits = decode_splits(seqs.n_decode, G, H // G, keys)
+        if a.splits > 1:
+            po, pml = _parts(q.device, seqs.n_decode * H * a.splits, vp)
+            a.part_o, a.part_ml = P(po), P(pml)
+        nv.check_rc(nv.lib("attn_window").omni_attn_window_decode(ctypes.byref(a), nv.stream_ptr()),
+                    "omni_attn_window_decode")
+    return out
+
+
+def _cpu(q, k_cache, v_cache, seqs, rule, out, gate):
+    T, H, dp = q.shape
+    nb, bs, G, _ = k_cache.shape
+    vp = v_cache.shape[3]
+    kf, vf = k_cache.view(nb * bs, G, dp), v_cache.view(nb * bs, G, vp)
+    o = torch.empty(T, H, vp)
+    for s in range(seqs.n_seqs):
+        a, b, ctx = int(seqs.q_start[s]), int(seqs.q_start[s + 1]), int(seqs.context[s])
+        j = torch.arange(ctx + b - a)
+        i = torch.arange(ctx, ctx + b - a)[:, None]
+        slot = seqs.block_tables[s].long()[j // bs] * bs + j % bs
+        k = kf[slot].float().repeat_interleave(H // G, 1)
+        v = vf[slot].float().repeat_interleave(H // G, 1)
+        sc = torch.einsum("thd,jhd->htj", q[a:b].float(), k) * rule.scale
+        if rule.softcap:
+            sc = rule.softcap * torch.tanh(sc / rule.softcap)
+        dist = (i - j).float()
+        if rule.r1 is not None:
+            sc = sc - rule.r1[:, None, None] * torch.log1p(rule.r2[:, None, None] * dist.clamp_min(0))
+        see = dist >= 0
+        if rule.window:
+            see &= (dist < rule.window) | (j < rule.keep_first)
+        sc = sc.masked_fill(~see, float("-inf"))
+        if rule.sink is not None:
+            sc = torch.cat([sc, rule.sink.float()[:, None, None].expand(H, b - a, 1)], -1)
+        w = sc.softmax(-1)[..., : j.numel()]
+        o[a:b] = torch.einsum("htj,jhd->thd", w, v)
+    if gate is not None:
+        o = o * torch.sigmoid(gate.float())[:, :, None]
+    out.copy_(o.reshape(T, H * vp))
+    return out
