@@ -18,6 +18,7 @@ struct WinAttn {
   const int* row_seq;                  // [T] (row-per-block kernel)
   const int* seq_list; int n_list;     // decode kernel: sequences with exactly one row
   const int* items; int n_items;       // prefill kernel: (sequence, first token of the block) pairs
+  int block_tokens;                    // prefill kernel: tokens per block, one or two tiles' worth
   void* out; long o_rs;                // [T, H, vp]
   const void* gate; long g_rs;         // [T, H] logits or nullptr
   const float* r1; const float* r2;    // [H] or nullptr

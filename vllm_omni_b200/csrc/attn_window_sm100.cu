@@ -1,0 +1,480 @@
+// Windowed paged attention of prompt portions on tcgen05 tensor cores (attn_window.h says what is
+// computed).
+//
+// The query heads that share a KV head are packed: row r of a 128-row tile is (token r / R, head r % R) with
+// R = heads per KV head, so a K/V tile is fetched once for the whole group and a tile spans only 128 / R
+// tokens, which keeps the keys outside a row's window or its future few.  One block owns two such tiles (one where two do not fit)
+// of one (sequence, KV head) and visits the key tiles any of its rows sees: the tiles of the kept first tokens,
+// then those of the window.  Portions of all sequences of a batch are one launch.
+//   warp 0        TMA producer: Q (box {64 channels, R heads, 128 / R tokens}), then K / V pages
+//   warp 1        MMA issuer: S_t = Q_t K^T, O_t += P_t V (P read from TMEM)
+//   warps 2, 3    distance bias of the key tile: r1 log2(1 + r2 dist) depends on (head, distance) only, so a
+//                 tile needs R (127 + 2 * 128 / R) logarithms instead of 2 * 128 * 128; double-buffered table
+//                 in shared memory
+//   warps 4-11    softmax, one thread per row; scores are bounded, biased and exponentiated in fp32
+// TMEM columns: S0 [0,128) S1 [128,256) O0 [256,384) O1 [384,512); P_t over the first 64 columns of S_t.
+// Every wait is bounded.
+#include "attn_window.h"
+#include "host_util.h"
+#include "ptx_sm100.cuh"
+
+namespace omni {
+
+constexpr int WP_BM = 128, WP_BN = 128;
+constexpr int WP_THREADS = 384;
+constexpr int WP_BOX = WP_BM * 64 * 2;          // 64 channels of 128 rows: 16 KiB
+constexpr int WP_MAX_STAGES = 4;
+constexpr float WP_LOG2E = 1.4426950408889634f;
+
+struct WinPrefill {
+  WinAttn a;
+  int R, TT;            // heads per KV head, tokens per tile
+  int nq;               // query tiles per block (2; 1 where two of the widest heads would not fit)
+  int kb, vb;           // 64-channel boxes per key / value row
+  int stages;           // depth of the K and V rings
+  int tab_stride;       // floats between the bias rows of two heads
+};
+
+__device__ __forceinline__ float wp_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float wp_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float wp_lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// bits [a, b) of a 32-bit word, both clamped to [0, 32]
+__device__ __forceinline__ uint32_t bit_range(int a, int b) {
+  a = min(max(a, 0), 32);
+  b = min(max(b, 0), 32);
+  const uint32_t hi = b == 32 ? 0xffffffffu : (1u << b) - 1u;
+  const uint32_t lo = a == 32 ? 0xffffffffu : (1u << a) - 1u;
+  return hi & ~lo;
+}
+
+template <bool CAP, bool BIAS>
+__global__ void __launch_bounds__(WP_THREADS, 1)
+attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                           const __grid_constant__ CUtensorMap tmV, const __grid_constant__ WinPrefill w) {
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ __align__(8) uint64_t q_full, k_full[WP_MAX_STAGES], k_empty[WP_MAX_STAGES], v_full[WP_MAX_STAGES],
+      v_empty[WP_MAX_STAGES];
+  __shared__ __align__(8) uint64_t s_full[2], p_full[2][4], o_done[2], tab_full[2], tab_empty[2];
+  __shared__ uint32_t tmem_base_s;
+  __shared__ int s_abort;
+
+  const WinAttn& p = w.a;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int g = blockIdx.y;
+  const int seq = p.items[2 * blockIdx.x], off = p.items[2 * blockIdx.x + 1];
+  const int row0 = p.q_start[seq] + off;                     // first batch row of the block
+  const int n_seq = p.q_start[seq + 1] - p.q_start[seq];
+  const int ctx = p.context[seq];
+  const int nt = min(w.nq * w.TT, n_seq - off);               // tokens of the block
+  const int n_qt = nt > w.TT ? 2 : 1;
+  const int p_first = ctx + off, p_last = p_first + nt - 1;
+  const int lo_tile = p.window > 0 ? max(0, p_first - p.window + 1) / WP_BN : 0;
+  const int first_tiles = min(lo_tile, (p.keep_first + WP_BN - 1) / WP_BN);
+  const int n_kv = first_tiles + p_last / WP_BN - lo_tile + 1;
+  auto tile_of = [&](int j) { return j < first_tiles ? j : lo_tile + j - first_tiles; };
+
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  const uint32_t q_tile = w.kb * WP_BOX, k_tile = q_tile, v_tile = w.vb * WP_BOX;
+  const uint32_t sQ = base, sK = base + w.nq * q_tile, sV = sK + w.stages * k_tile;
+  float* tab = reinterpret_cast<float*>(smem_raw + (sV + w.stages * v_tile - smem_u32(smem_raw)));
+  const int tab_floats = w.R * w.tab_stride;
+
+  if (threadIdx.x == 0) {
+    s_abort = 0;
+    mbar_init(smem_u32(&q_full), 1);
+    for (int i = 0; i < w.stages; ++i) {
+      mbar_init(smem_u32(&k_full[i]), 1);
+      mbar_init(smem_u32(&k_empty[i]), 1);
+      mbar_init(smem_u32(&v_full[i]), 1);
+      mbar_init(smem_u32(&v_empty[i]), 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(smem_u32(&s_full[i]), 1);
+      for (int c = 0; c < 4; ++c) mbar_init(smem_u32(&p_full[i][c]), 4);
+      mbar_init(smem_u32(&o_done[i]), 1);
+      mbar_init(smem_u32(&tab_full[i]), 2);                  // the two bias warps
+      mbar_init(smem_u32(&tab_empty[i]), 4 * n_qt);          // the softmax warps of the tiles in use
+    }
+    fence_mbar_init();
+    tma_prefetch_desc(&tmQ);
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmV);
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_s), 512);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = tmem_base_s;
+  int* status = p.status;
+
+  if (warp == 0) {
+    // ------------------------------------------------------------------ TMA producer
+    if (elect_one()) {
+      const uint32_t qb = smem_u32(&q_full);
+      mbar_expect_tx(qb, (uint32_t)(n_qt * w.kb * w.R * w.TT * 128));
+      for (int t = 0; t < n_qt; ++t)
+        for (int x = 0; x < w.kb; ++x)
+          tma_load_4d(sQ + t * q_tile + x * WP_BOX, &tmQ, qb, 64 * x, 0, row0 + t * w.TT, g);
+      const int* bt = p.block_tables + (long)seq * p.bt_stride;
+      const int last_page = (ctx + n_seq - 1) / p.block_size;
+      const int ppt = WP_BN / p.block_size;
+      const uint32_t page_bytes = (uint32_t)p.block_size * 128u;
+      for (int j = 0; j < n_kv; ++j) {
+        const int st = j % w.stages;
+        const uint32_t ph = (j / w.stages) & 1;
+        const int pg0 = tile_of(j) * ppt;
+        // pages past the sequence's last one re-read it: finite data that the mask discards
+        mbar_wait(smem_u32(&k_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+        const uint32_t kb = smem_u32(&k_full[st]);
+        mbar_expect_tx(kb, k_tile);
+        for (int i = 0; i < ppt; ++i) {
+          const int page = min(max(bt[min(pg0 + i, last_page)], 0), p.num_blocks - 1);
+          for (int x = 0; x < w.kb; ++x)
+            tma_load_3d(sK + st * k_tile + x * WP_BOX + i * page_bytes, &tmK, kb, 64 * x, page * p.block_size, g);
+        }
+        mbar_wait(smem_u32(&v_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+        const uint32_t vbar = smem_u32(&v_full[st]);
+        mbar_expect_tx(vbar, v_tile);
+        for (int i = 0; i < ppt; ++i) {
+          const int page = min(max(bt[min(pg0 + i, last_page)], 0), p.num_blocks - 1);
+          for (int x = 0; x < w.vb; ++x)
+            tma_load_3d(sV + st * v_tile + x * WP_BOX + i * page_bytes, &tmV, vbar, 64 * x, page * p.block_size, g);
+        }
+      }
+    }
+  } else if (warp == 1) {
+    // -------------------------------------------------------------------- MMA issuer
+    if (elect_one()) {
+      const uint32_t idesc_qk = umma_idesc(WP_BM, WP_BN, 1, 1, 0, 0);
+      const uint32_t idesc_pv = w.vb == 1 ? umma_idesc(WP_BM, 64, 1, 1, 0, 1) : umma_idesc(WP_BM, 128, 1, 1, 0, 1);
+      const uint64_t box16 = WP_BOX >> 4, q16 = q_tile >> 4, k16 = k_tile >> 4, v16 = v_tile >> 4;
+      const uint64_t dQ = umma_desc_kmajor_sw128(sQ), dK = umma_desc_kmajor_sw128(sK);
+      const uint64_t dV = umma_desc_sw128(sV, WP_BOX, 1024);
+      const int ks = p.dp >> 4;
+      auto issue_s = [&](int t, int st) {
+        const uint64_t a0 = dQ + (uint64_t)t * q16, b0 = dK + (uint64_t)st * k16;
+        for (int k = 0; k < ks; ++k) {
+          const uint64_t o = (uint64_t)(k >> 2) * box16 + (uint64_t)((k & 3) * 2);   // 16 channels = 32 bytes of a row
+          mma_f16_ss(tmem_base + t * 128, a0 + o, b0 + o, idesc_qk, k == 0 ? 0u : 1u);
+        }
+      };
+      mbar_wait(smem_u32(&q_full), 0, &s_abort, status, ERR_WAIT_FULL);
+      mbar_wait(smem_u32(&k_full[0]), 0, &s_abort, status, ERR_WAIT_FULL);
+      tc_fence_after_sync();
+      for (int t = 0; t < n_qt; ++t) {
+        issue_s(t, 0);
+        tc_commit(smem_u32(&s_full[t]));
+      }
+      tc_commit(smem_u32(&k_empty[0]));
+      for (int j = 0; j < n_kv; ++j) {
+        const int st = j % w.stages, st1 = (j + 1) % w.stages;
+        const bool more = j + 1 < n_kv;
+        mbar_wait(smem_u32(&v_full[st]), (j / w.stages) & 1, &s_abort, status, ERR_WAIT_FULL);
+        if (more) mbar_wait(smem_u32(&k_full[st1]), ((j + 1) / w.stages) & 1, &s_abort, status, ERR_WAIT_FULL);
+        const uint64_t v0 = dV + (uint64_t)st * v16;
+        for (int t = 0; t < n_qt; ++t) {
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            // 32 keys of P as the softmax warps hand them over
+            mbar_wait(smem_u32(&p_full[t][c]), j & 1, &s_abort, status, ERR_WAIT_SOFTMAX);
+            tc_fence_after_sync();
+#pragma unroll
+            for (int kk = 0; kk < 2; ++kk) {
+              const int k = 2 * c + kk;
+              mma_f16_ts(tmem_base + 256 + t * 128, tmem_base + t * 128 + k * 8, v0 + (uint64_t)(k * 128), idesc_pv,
+                         (k == 0 && j == 0) ? 0u : 1u);
+            }
+          }
+          if (more) {
+            issue_s(t, st1);
+            tc_commit(smem_u32(&s_full[t]));
+          } else {
+            tc_commit(smem_u32(&o_done[t]));
+          }
+        }
+        tc_commit(smem_u32(&v_empty[st]));
+        if (more) tc_commit(smem_u32(&k_empty[st1]));
+      }
+    }
+  } else if (warp < 4) {
+    // ------------------------------------------------------------ bias of the key tiles
+    // entry i of head r: distance p_first - key tile base - 127 + i
+    if (BIAS) {
+      const float top = CAP ? p.cap * WP_LOG2E : 0.f;
+      const int width = 127 + 2 * w.TT;
+      for (int j = 0; j < n_kv; ++j) {
+        const int b = j & 1;
+        mbar_wait(smem_u32(&tab_empty[b]), ((j >> 1) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+        const int d0 = p_first - tile_of(j) * WP_BN - 127;
+        for (int r = 0; r < w.R; ++r) {
+          const float r1 = p.r1[g * w.R + r], r2 = p.r2[g * w.R + r];
+          float* dst = tab + b * tab_floats + r * w.tab_stride;
+          for (int i = threadIdx.x - 64; i < width; i += 64)
+            dst[i] = fmaf(-r1, wp_lg2(fmaf(r2, (float)max(d0 + i, 0), 1.0f)), top);
+        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&tab_full[b]));
+      }
+    }
+  } else {
+    // -------------------------------------------------------------- softmax + epilogue
+    const int t = (warp - 4) >> 2, q = warp & 3;
+    const int row = q * 32 + lane;
+    const int tok = row / w.R, r = row - tok * w.R;
+    const bool tile_used = t < n_qt;
+    const bool row_ok = tile_used && tok < w.TT && t * w.TT + tok < nt;
+    const bool rows_used = __any_sync(0xffffffffu, row_ok);
+    const int pos = p_first + t * w.TT + tok;
+    const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
+    const uint32_t tS = tmem_base + lane_addr + t * 128, tO = tmem_base + lane_addr + 256 + t * 128;
+    const int h = g * w.R + min(r, w.R - 1);
+    const float C = p.cap * WP_LOG2E;
+    const float mul = CAP ? p.scale * 2.0f * WP_LOG2E / p.cap : p.scale * WP_LOG2E;
+    float m = -INFINITY, l0 = 0.f, l1 = 0.f;     // reference exponent (log2 units) and two partial row sums
+    if (p.sink) {                                // the sink is a key without a value, seen before all others
+      m = p.sink[h] * WP_LOG2E;
+      l0 = 1.f;
+    }
+    const float* my_tab = tab + min(r, w.R - 1) * w.tab_stride + min(t * w.TT + tok, 2 * w.TT - 1) + 127;
+    for (int j = 0; tile_used && j < n_kv; ++j) {
+      mbar_wait(smem_u32(&s_full[t]), j & 1, &s_abort, status, ERR_WAIT_FULL);
+      if (!rows_used) {
+        if (lane == 0) {
+          for (int c = 0; c < 4; ++c) mbar_arrive(smem_u32(&p_full[t][c]));
+          if (BIAS) mbar_arrive(smem_u32(&tab_empty[j & 1]));
+        }
+        continue;
+      }
+      tc_fence_after_sync();
+      const int kbase = tile_of(j) * WP_BN;
+      const int hi = pos - kbase + 1;                                  // keys e < hi are not in the future
+      const int lo = p.window > 0 ? pos - p.window + 1 - kbase : 0;     // keys e >= lo are in the window
+      const bool masked = __any_sync(0xffffffffu, hi < WP_BN || lo > 0);
+      if (BIAS) mbar_wait(smem_u32(&tab_full[j & 1]), (j >> 1) & 1, &s_abort, status, ERR_WAIT_FULL);
+      const float* tb = my_tab + (j & 1) * tab_floats;
+      uint32_t v0[32], v1[32], v2[32], v3[32];
+      tmem_ld_32x32(tS, v0);
+      tmem_ld_32x32(tS + 32, v1);
+      tmem_ld_32x32(tS + 64, v2);
+      tmem_ld_32x32(tS + 96, v3);
+      tmem_wait_ld();
+      float mx = -INFINITY;
+      auto score = [&](uint32_t (&v)[32], int c) {
+#pragma unroll
+        for (int e = 0; e < 32; e += 2) {
+          float y0 = __uint_as_float(v[e]) * mul, y1 = __uint_as_float(v[e + 1]) * mul;
+          float b0 = CAP ? C : 0.f, b1 = b0;
+          if (BIAS) {
+            b0 = tb[-(c * 32 + e)];
+            b1 = tb[-(c * 32 + e + 1)];
+          }
+          if (CAP) {
+            // cap tanh(s / cap) = C - 2C / (1 + 2^y); the pair shares one reciprocal, y <= 60 keeps its
+            // product finite (there the bound is reached to the last bit)
+            const float a0 = wp_ex2(fminf(y0, 60.f)) + 1.0f, a1 = wp_ex2(fminf(y1, 60.f)) + 1.0f;
+            const float k = -2.0f * C * wp_rcp(a0 * a1);
+            y0 = fmaf(k, a1, b0);
+            y1 = fmaf(k, a0, b1);
+          } else if (BIAS) {
+            y0 += b0;
+            y1 += b1;
+          }
+          v[e] = __float_as_uint(y0);
+          v[e + 1] = __float_as_uint(y1);
+        }
+        if (masked) {
+          const uint32_t mk = bit_range(lo - 32 * c, hi - 32 * c) | bit_range(0, min(p.keep_first - kbase, hi) - 32 * c);
+#pragma unroll
+          for (int e = 0; e < 32; ++e)
+            if (!(mk & (1u << e))) v[e] = 0xff800000u;
+        }
+#pragma unroll
+        for (int e = 0; e < 32; ++e) mx = fmaxf(mx, __uint_as_float(v[e]));
+      };
+      score(v0, 0);
+      score(v1, 1);
+      score(v2, 2);
+      score(v3, 3);
+      if (BIAS) {
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&tab_empty[j & 1]));
+      }
+      const float m_new = fmaxf(m, mx);
+      if (j == 0) {
+        if (m != -INFINITY) l0 *= wp_ex2(m - m_new);
+        m = m_new;
+      } else if (__any_sync(0xffffffffu, m_new > m + 8.0f)) {
+        // rare: O follows the new reference; the scores wait in their own TMEM columns meanwhile
+        const float alpha = m_new == -INFINITY ? 1.f : wp_ex2(m - m_new);
+        l0 *= alpha;
+        l1 *= alpha;
+        tmem_st_32x32(tS, v0);
+        tmem_st_32x32(tS + 32, v1);
+        tmem_st_32x32(tS + 64, v2);
+        tmem_st_32x32(tS + 96, v3);
+        tmem_wait_st();
+#pragma unroll 1
+        for (int c = 0; c < 2 * w.vb; ++c) {
+          uint32_t v[32];
+          tmem_ld_32x32(tO + c * 32, v);
+          tmem_wait_ld();
+#pragma unroll
+          for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(__uint_as_float(v[e]) * alpha);
+          tmem_st_32x32(tO + c * 32, v);
+        }
+        tmem_wait_st();
+        m = m_new;
+        tmem_ld_32x32(tS, v0);
+        tmem_ld_32x32(tS + 32, v1);
+        tmem_ld_32x32(tS + 64, v2);
+        tmem_ld_32x32(tS + 96, v3);
+        tmem_wait_ld();
+      }
+      const float m_use = m == -INFINITY ? 0.f : m;
+      auto weights = [&](uint32_t (&v)[32], int c) {
+        uint32_t pk[16];
+#pragma unroll
+        for (int e = 0; e < 32; e += 2) {
+          const float e0 = wp_ex2(__uint_as_float(v[e]) - m_use), e1 = wp_ex2(__uint_as_float(v[e + 1]) - m_use);
+          l0 += e0;
+          l1 += e1;
+          pk[e >> 1] = pack_bf16(e0, e1);
+        }
+        tmem_st_32x16(tS + c * 16, pk);
+        tmem_wait_st();
+        tc_fence_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&p_full[t][c]));
+      };
+      weights(v0, 0);
+      weights(v1, 1);
+      weights(v2, 2);
+      weights(v3, 3);
+    }
+    if (rows_used) {
+      mbar_wait(smem_u32(&o_done[t]), 0, &s_abort, status, ERR_WAIT_PV);
+      tc_fence_after_sync();
+      const long orow = row0 + t * w.TT + tok;
+      float f = 1.0f / (l0 + l1);
+      if (p.gate && row_ok) {
+        const float z = (float)static_cast<const __nv_bfloat16*>(p.gate)[orow * p.g_rs + h];
+        f *= 1.0f / (1.0f + __expf(-z));
+      }
+      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + orow * p.o_rs + (long)h * p.vp;
+#pragma unroll 1
+      for (int c = 0; c < p.vp; c += 16) {
+        uint32_t v[16];
+        tmem_ld_32x16(tO + c, v);
+        tmem_wait_ld();
+        if (row_ok) {
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            uint4 o;
+            o.x = pack_bf16(__uint_as_float(v[x * 8 + 0]) * f, __uint_as_float(v[x * 8 + 1]) * f);
+            o.y = pack_bf16(__uint_as_float(v[x * 8 + 2]) * f, __uint_as_float(v[x * 8 + 3]) * f);
+            o.z = pack_bf16(__uint_as_float(v[x * 8 + 4]) * f, __uint_as_float(v[x * 8 + 5]) * f);
+            o.w = pack_bf16(__uint_as_float(v[x * 8 + 6]) * f, __uint_as_float(v[x * 8 + 7]) * f);
+            *reinterpret_cast<uint4*>(dst + c + x * 8) = o;
+          }
+        }
+      }
+    }
+  }
+
+  tc_fence_before_sync();
+  __syncthreads();
+  if (s_abort) {
+    // a wait ran out: give copies and products in flight time to finish before their memory goes
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) {
+    }
+  }
+  if (warp == 1) tmem_dealloc(tmem_base, 512);
+}
+
+// Q as (channel, head of the group, token, KV head)
+static int make_q_tmap(CUtensorMap* tm, const WinAttn& p, int R, int TT) {
+  EncodeTiledFn enc = get_encode_tiled();
+  if (!enc) return RC_NO_DRIVER;
+  if ((reinterpret_cast<uintptr_t>(p.q) & 15) || (p.q_rs & 7)) return RC_BAD_ARG;
+  cuuint64_t gdim[4] = {(cuuint64_t)p.dp, (cuuint64_t)R, (cuuint64_t)p.T, (cuuint64_t)p.G};
+  cuuint64_t gstr[3] = {(cuuint64_t)p.dp * 2, (cuuint64_t)p.q_rs * 2, (cuuint64_t)R * p.dp * 2};
+  cuuint32_t box[4] = {64, (cuuint32_t)R, (cuuint32_t)TT, 1};
+  cuuint32_t estr[4] = {1, 1, 1, 1};
+  CUresult r = enc(tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(p.q), gdim, gstr, box, estr,
+                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? RC_OK : RC_TMAP;
+}
+
+template <bool CAP, bool BIAS>
+static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const WinPrefill& w,
+                          int smem, cudaStream_t st) {
+  static unsigned long long prep = 0;
+  if (int e = ensure_dynamic_smem((const void*)attn_window_prefill_kernel<CAP, BIAS>, 227 * 1024 - 512, prep)) return e;
+  attn_window_prefill_kernel<CAP, BIAS><<<dim3(w.a.n_items, w.a.G), WP_THREADS, smem, st>>>(tq, tk, tv, w);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace omni
+
+using namespace omni;
+
+// items: int32 [n_items, 2] (sequence, first row within its portion; blocks of block_tokens rows).
+extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
+  WinPrefill w;
+  w.a = *args;
+  const WinAttn& p = w.a;
+  if (p.n_items <= 0) return RC_OK;
+  if (p.H <= 0 || p.G <= 0 || p.H % p.G || (p.dp & 15) || (p.vp & 15) || p.dp <= 0 || p.vp <= 0 || p.dp > 256 ||
+      p.vp > 128 || p.items == nullptr || p.num_seqs <= 0 || p.num_blocks <= 0 || p.keep_first < 0)
+    return RC_BAD_ARG;
+  if (p.block_size < 8 || (p.block_size & 7) || 128 % p.block_size || p.G > 65535) return RC_BAD_ARG;
+  if ((p.r1 == nullptr) != (p.r2 == nullptr) || (p.o_rs & 7) || (reinterpret_cast<uintptr_t>(p.out) & 15)) return RC_BAD_ARG;
+  w.R = p.H / p.G;
+  if (w.R > 128) return RC_BAD_ARG;
+  w.TT = 128 / w.R;
+  if (p.block_tokens != w.TT && p.block_tokens != 2 * w.TT) return RC_BAD_ARG;
+  w.nq = p.block_tokens / w.TT;
+  w.kb = (p.dp + 63) / 64;
+  w.vb = (p.vp + 63) / 64;
+  // rows of the bias table: a warp's 32 rows are 32 / R tokens of R heads; this pitch spreads them over all banks
+  const int width = 127 + 2 * w.TT;
+  const bool pow2 = (w.R & (w.R - 1)) == 0 && w.R <= 32;
+  const int want = pow2 ? (32 / w.R) % 32 : 1;
+  w.tab_stride = width;
+  while (w.tab_stride % 32 != want) ++w.tab_stride;
+  const int tab_bytes = p.r1 ? 2 * w.R * w.tab_stride * 4 : 0;
+  const int limit = 227 * 1024 - 1024 - 512;                 // less the alignment slack and the static barriers
+  const int q_bytes = w.nq * w.kb * WP_BOX, stage = (w.kb + w.vb) * WP_BOX;
+  w.stages = (limit - q_bytes - tab_bytes) / stage;
+  if (w.stages > WP_MAX_STAGES) w.stages = WP_MAX_STAGES;
+  if (w.stages < 1) return RC_TOO_LARGE;
+  const int smem = q_bytes + w.stages * stage + tab_bytes + 1024;
+  CUtensorMap tq, tk, tv;
+  const uint64_t slots = (uint64_t)p.num_blocks * p.block_size;
+  int rc = make_q_tmap(&tq, p, w.R, w.TT);
+  if (!rc) rc = make_tmap_3d(&tk, p.k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dp, slots, p.G, (uint64_t)p.G * p.dp * 2,
+                             (uint64_t)p.dp * 2, 64, p.block_size);
+  if (!rc) rc = make_tmap_3d(&tv, p.v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.vp, slots, p.G, (uint64_t)p.G * p.vp * 2,
+                             (uint64_t)p.vp * 2, 64, p.block_size);
+  if (rc) return rc;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (p.cap > 0.f) return p.r1 ? launch_prefill<true, true>(tq, tk, tv, w, smem, st) : launch_prefill<true, false>(tq, tk, tv, w, smem, st);
+  return p.r1 ? launch_prefill<false, true>(tq, tk, tv, w, smem, st) : launch_prefill<false, false>(tq, tk, tv, w, smem, st);
+}

@@ -8,7 +8,7 @@ from .config import TavulixConfig, tiny_config_dict
 from .decoder import TavulixDecoder
 
 # libraries under csrc/ that serving this model loads on a GPU
-NATIVE_LIBS = ("gemm_sm100", "gemm_f32", "lm_ops", "attn_window", "sampler", "rt_host", "io_host")
+NATIVE_LIBS = ("gemm_sm100", "gemm_f32", "lm_ops", "attn_window", "attn_window_sm100", "sampler", "rt_host", "io_host")
 
 
 class TavulixForCausalLM(StageModel):

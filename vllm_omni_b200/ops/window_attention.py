@@ -19,6 +19,7 @@ class _WinAttn(ctypes.Structure):
     _fields_ = [("q", c_void_p), ("q_rs", c_long), ("k_cache", c_void_p), ("v_cache", c_void_p),
                 ("block_tables", c_void_p), ("bt_stride", c_int), ("q_start", c_void_p), ("context", c_void_p),
                 ("row_seq", c_void_p), ("seq_list", c_void_p), ("n_list", c_int), ("items", c_void_p), ("n_items", c_int),
+                ("block_tokens", c_int),
                 ("out", c_void_p), ("o_rs", c_long), ("gate", c_void_p), ("g_rs", c_long), ("r1", c_void_p),
                 ("r2", c_void_p), ("sink", c_void_p), ("scale", c_float), ("cap", c_float), ("window", c_int),
                 ("keep_first", c_int), ("T", c_int), ("H", c_int), ("G", c_int), ("dp", c_int), ("vp", c_int),
@@ -38,13 +39,14 @@ class ScoreRule:
     keep_first: int = 0
 
 
-def prefill_rows_per_block(heads: int, kv_heads: int) -> int:
-    """Tokens one block of the tcgen05 kernel serves: two 128-row tiles of (token, head of the KV group) rows."""
-    return 2 * (128 // (heads // kv_heads))
+def prefill_rows_per_block(heads: int, kv_heads: int, dp: int) -> int:
+    """Tokens one block of the tcgen05 kernel serves: two 128-row tiles of (token, head of the KV group) rows,
+    one when two tiles of the widest heads do not fit in shared memory."""
+    return (1 if dp > 192 else 2) * (128 // (heads // kv_heads))
 
 
 def prefill_kernel_ok(heads: int, kv_heads: int, dp: int, vp: int, block_size: int) -> bool:
-    return False and heads // kv_heads <= 128 and dp <= 256 and vp <= 128 and block_size >= 8 and block_size % 8 == 0 \
+    return heads // kv_heads <= 128 and dp <= 256 and vp <= 128 and block_size >= 8 and block_size % 8 == 0 \
         and 128 % block_size == 0
 
 
@@ -101,8 +103,9 @@ def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None,
         nv.check_rc(rc, "omni_attn_window_rows")
         return out
     if seqs.n_decode < seqs.n_seqs:
-        items, n = seqs.prefill_items(prefill_rows_per_block(H, G))
-        a.items, a.n_items = P(items), n
+        a.block_tokens = prefill_rows_per_block(H, G, dp)
+        items, a.n_items = seqs.prefill_items(a.block_tokens)
+        a.items = P(items)
         rc = nv.lib("attn_window_sm100").omni_attn_window_prefill(ctypes.byref(a), nv.stream_ptr())
         nv.check_rc(rc, "omni_attn_window_prefill")
     if seqs.n_decode:
