@@ -41,6 +41,10 @@ def parse_args():
     ap.add_argument("--layers", type=int, default=60, help="60 = the 20B config; anything else is a smoke run")
     ap.add_argument("--parallelism", default=None, help="e.g. sp8, cfg2xsp4, tp8 (default: cfg2 at N=2, cfg2 x sp(N/2) above)")
     ap.add_argument("--no-e2e", action="store_true")
+    ap.add_argument("--workload", default="image", choices=["image", "lm"],
+                    help="image: the headline (default); lm: decoder layers of the causal-LM models")
+    ap.add_argument("--lm-sizes", default="2048,4096", help="lm workload: widths to run")
+    ap.add_argument("--lm-parts", default="steps,kernels", help="lm workload: which tables to fill")
     ap.add_argument("--ref-eager", action="store_true", help="reference arm: skip its regional torch.compile")
     return ap.parse_args()
 
@@ -135,10 +139,25 @@ def parse_parallelism(spec: str | None, n: int) -> dict:
     return out
 
 
+def lm_workload(args):
+    """Decoder layers of the causal-LM models, one GPU (vllm_omni_b200/benchmarks/lm_layers.py)."""
+    import torch
+    from vllm_omni_b200.benchmarks import lm_layers
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    rec = lm_layers.run(max(args.steps, 7), args.warmup, [int(w) for w in args.lm_sizes.split(",")], args.lm_parts.split(","))
+    rec["clocks"] = sampler.stop()
+    print(json.dumps(rec), flush=True)
+    return 0
+
+
 def main():
     args = parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.workload == "lm":
+        return lm_workload(args)
     import torch
     import torch.distributed as dist
     from vllm_omni_b200.diffusion.data import DiffusionParallelConfig

@@ -85,7 +85,7 @@ def _check(case, got, tol):
 
 MIXED = [(0, 70), (130, 1), (40, 33), (0, 1), (300, 2), (17, 1)]
 CASES = {
-    "grouped": dict(shape=(8, 2, 48, 64), portions=MIXED, window=40, keep=6, cap=9.0),
+    "grouped": dict(shape=(12, 3, 80, 48), portions=MIXED, window=40, keep=7, cap=9.0),
     "odd_sizes": dict(shape=(6, 2, 40, 24), portions=MIXED, window=33, keep=5, cap=9.0),
     "one_head_per_group": dict(shape=(4, 4, 64, 32), portions=MIXED, window=20, keep=3, cap=4.0),
     "three_per_group": dict(shape=(3, 1, 16, 16), portions=[(5, 100), (200, 1)], window=50, keep=0, cap=5.0),
@@ -98,8 +98,8 @@ CASES = {
     "cap_only": dict(shape=(8, 2, 64, 64), portions=MIXED, window=64, keep=4, cap=2.0, bias=False, sink=False),
     "wide_group": dict(shape=(20, 1, 64, 80), portions=MIXED, window=45, keep=6, cap=9.0),
     "very_wide_group": dict(shape=(24, 1, 32, 16), portions=[(0, 50), (120, 1), (64, 1)], window=45, keep=6, cap=9.0),
-    "page_of_8": dict(shape=(8, 2, 48, 64), portions=MIXED, window=40, keep=6, cap=9.0, block=8),
-    "page_of_64": dict(shape=(8, 2, 48, 64), portions=MIXED, window=40, keep=6, cap=9.0, block=64),
+    "page_of_8": dict(shape=(12, 3, 80, 48), portions=MIXED, window=40, keep=7, cap=9.0, block=8),
+    "page_of_64": dict(shape=(12, 3, 80, 48), portions=MIXED, window=40, keep=7, cap=9.0, block=64),
 }
 
 

@@ -47,10 +47,10 @@ def prepare(model: str) -> None:
 
 
 class TraceReplay:
-    def __init__(self, model: str, dtype: str, max_tokens: int):
+    def __init__(self, model: str, dtype: str, max_tokens: int, device: str | None = None):
         from ..engine.portion_scheduler import PortionScheduler
         from .omni_llm import OmniLLM
-        self.llm = OmniLLM(model, dtype=dtype, block_size=BLOCK, num_gpu_blocks=max(1, -(-max_tokens // BLOCK)),
+        self.llm = OmniLLM(model, dtype=dtype, device=device, block_size=BLOCK, num_gpu_blocks=max(1, -(-max_tokens // BLOCK)),
                            max_num_seqs=LIVE, scheduler_cls=PortionScheduler)
         self.engine = self.llm.engine
         self.live: dict = {}

@@ -57,7 +57,7 @@ def save_safetensors(tensors: dict[str, torch.Tensor], path: str, metadata: dict
     header, off, blobs = {}, 0, []
     for name, t in tensors.items():
         t = t.detach().contiguous().cpu()
-        raw = t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": _NAMES[t.dtype], "shape": list(t.shape), "data_offsets": [off, off + len(raw)]}
         off += len(raw)
         blobs.append(raw)
