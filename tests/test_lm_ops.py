@@ -221,6 +221,22 @@ def test_conv_heads_sizes_and_value_mixing(device, dtype, shape):
 
 
 @pytest.mark.parametrize("device,dtype", DEVICES)
+@pytest.mark.parametrize("taps", [1, 2, 3, 4, 5])
+def test_conv_heads_long_batches(device, dtype, taps):
+    """Batches long enough for the sliding-window kernel; sequences of one to many rows meet inside its runs."""
+    c = ConvCase((3, 1, 40, 24), taps, dtype, device, seed=20 + taps)
+    lens = [300, 1, 2, 5, 129, 3]
+    us = c.inputs(lens)
+    vf = [c.rnd(u.shape[0], 1, 24).to(dtype) for u in us]
+    cuts = [[290, 3, 7], [1, 0, 0], [2, 0, 0], [1, 4, 0], [3, 125, 1], [0, 2, 1]]
+    for mode, first in (("plain", None), ("mix", vf)):
+        for u, f, (q, k, v, _) in zip(us, vf, c.run(us, cuts, mode, first)):
+            eq, ek, _, ev = c.expected(u, f if mode == "mix" else None)
+            for got, want in ((q, eq), (k, ek), (v, ev)):
+                _close(got, want, dtype, scale=4)
+
+
+@pytest.mark.parametrize("device,dtype", DEVICES)
 def test_conv_heads_without_norms(device, dtype):
     c = ConvCase((2, 1, 32, 16), 2, dtype, device, norms=False)
     us = c.inputs([6])

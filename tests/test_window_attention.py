@@ -5,7 +5,7 @@ import torch
 
 import tavulix_oracle as O
 from vllm_omni_b200.models.seq_table import SeqTable
-from vllm_omni_b200.ops.window_attention import ScoreRule, decode_splits, window_attention
+from vllm_omni_b200.ops.window_attention import ScoreRule, bounded_scores, decode_splits, window_attention
 
 BS = 16
 
@@ -44,7 +44,7 @@ class Case:
             out.append(o[c:])
         return torch.cat(out)
 
-    def run(self, device, dtype, impl=None, spare=3):
+    def run(self, device, dtype, impl=None, spare=3, bounded=None):
         dp, vp, bs = _up(self.d, 16), _up(self.dv, 16), self.block
         need = [(c + n + bs - 1) // bs for c, n in self.portions]
         total = sum(need) + spare
@@ -68,7 +68,8 @@ class Case:
         qp[:, :, :self.d] = q
         seqs = SeqTable.build([n for _, n in self.portions], [c for c, _ in self.portions], tables, None, device)
         mv = lambda t: None if t is None else t.float().to(device)
-        rule = ScoreRule(self.scale, self.cap, mv(self.r1), mv(self.r2), mv(self.sink), self.window, self.keep)
+        rule = ScoreRule(self.scale, self.cap, mv(self.r1), mv(self.r2), mv(self.sink), self.window, self.keep,
+                         bounded=bounded_scores(self.cap, self.r1, self.r2) if bounded is None else bounded)
         out = torch.full((T, self.H * vp), float("nan"), dtype=dtype, device=device)
         gate = torch.cat(rows_g).to(device, dtype) if self.gate is not None else None
         window_attention(qp.to(device, dtype), kc.to(device, dtype), vc.to(device, dtype), seqs, rule, out, gate=gate, impl=impl)
@@ -142,6 +143,35 @@ LARGE = {
 def test_large_heads_bf16_gpu(name):
     c = Case(**LARGE[name])
     _check(c, c.run("cuda", torch.bfloat16), 0.02)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("name", [n for n in sorted(CASES) if CASES[n].get("cap")])
+def test_bounded_and_running_maximum_agree(name):
+    c = Case(**CASES[name])
+    assert bounded_scores(c.cap, c.r1, c.r2)
+    for bounded in (True, False):
+        _check(c, c.run("cuda", torch.bfloat16, bounded=bounded), 0.02)
+
+
+def test_when_the_cap_may_be_the_reference():
+    one = torch.ones(3)
+    assert bounded_scores(20.0) and not bounded_scores(None) and not bounded_scores(40.0)
+    assert bounded_scores(20.0, one, one) and not bounded_scores(20.0, -one, one) and not bounded_scores(20.0, one, -one)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("cap", [31.0, 60.0])
+def test_far_apart_scores(cap):
+    """Rows whose visible scores all sit near -cap or near +cap, with large biases: both references give the rows."""
+    for sign in (-1.0, 1.0):
+        c = Case((4, 2, 64, 32), [(500, 90), (800, 1)], 300, 4, cap=cap, scale=1.0, seed=8)
+        c.r1 = torch.full((4,), 6.0)
+        for s in range(2):
+            c.q[s] = c.q[s].abs()
+            c.k[s] = (sign * c.k[s].float().abs()).bfloat16()
+        c.sink = torch.full((4,), -200.0)
+        _check(c, c.run("cuda", torch.bfloat16), 0.02)
 
 
 @pytest.mark.gpu

@@ -157,7 +157,7 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
     seqs = SeqTable.build([T], [0], [list(range(nb))], [(0, 1)], dev)
     vecs = dict(r1=torch.rand(H, device=dev), r2=0.2 * torch.rand(H, device=dev), sink=torch.randn(H, device=dev))
     gate = rnd(T, H)
-    rule = lambda w: ScoreRule(DIM ** -0.5, 20.0, window=w, keep_first=4, **vecs)
+    rule = lambda w: ScoreRule(DIM ** -0.5, 20.0, window=w, keep_first=4, bounded=True, **vecs)
     row("attention prompt", "tavulix full", lambda: window_attention(q[0], kc, vc, seqs, rule(FULL), o, gate=gate), flops=full)
     row("attention prompt", f"tavulix w{WINDOW}", lambda: window_attention(q[0], kc, vc, seqs, rule(WINDOW), o, gate=gate),
         flops=4.0 * H * DIM * nwin)

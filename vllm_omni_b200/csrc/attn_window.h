@@ -24,6 +24,7 @@ struct WinAttn {
   const float* r1; const float* r2;    // [H] or nullptr
   const float* sink;                   // [H] or nullptr
   float scale, cap;                    // cap <= 0: no bound
+  int bounded;                         // the cap may serve as softmax reference (see attn_window_sm100.cu)
   int window, keep_first;              // window <= 0: unbounded
   int T, H, G, dp, vp, num_seqs, num_blocks, block_size;
   int splits; float* part_o; float* part_ml;    // decode: shares of the visible keys, merged by a second kernel

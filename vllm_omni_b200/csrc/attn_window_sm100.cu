@@ -3,18 +3,29 @@
 //
 // The query heads that share a KV head are packed: row r of a 128-row tile is (token r / R, head r % R) with
 // R = heads per KV head, so a K/V tile is fetched once for the whole group and a tile spans only 128 / R
-// tokens, which keeps the keys outside a row's window or its future few.  One block owns two such tiles (one where two do not fit)
-// of one (sequence, KV head) and visits the key tiles any of its rows sees: the tiles of the kept first tokens,
+// tokens, which keeps the keys outside a row's window or its future few.  One block owns two such tiles (one
+// where two do not fit) of one (sequence, KV head) and visits the key tiles any of its rows sees: the tiles of the kept first tokens,
 // then those of the window.  Portions of all sequences of a batch are one launch.
 //   warp 0        TMA producer: Q (box {64 channels, R heads, 128 / R tokens}), then K / V pages
 //   warp 1        MMA issuer: S_t = Q_t K^T, O_t += P_t V (P read from TMEM)
 //   warps 2, 3    distance bias of the key tile: r1 log2(1 + r2 dist) depends on (head, distance) only, so a
 //                 tile needs R (127 + 2 * 128 / R) logarithms instead of 2 * 128 * 128; double-buffered table
 //                 in shared memory
-//   warps 4-11    softmax, one thread per row; scores are bounded, biased and exponentiated in fp32
+//   warps 4-11    softmax, one thread per row; scores are bounded, biased and exponentiated in fp32.  The two
+//                 exponentials and the reciprocal of a bounded score make the MUFU unit, not the tensor pipe, the
+//                 limit; a pair of scores shares one reciprocal.  (Polynomial exponentials on the FMA pipe for 1/8 to
+//                 all of them were slower: the issue slots they take are not free.)
+// Bounded scores (cap > 0, `bounded` set) never exceed the cap, so max(cap, sink) serves as every row's softmax
+// reference: no running maximum, no rescaling, and each chunk of scores goes from tensor memory to weights in one pass.
+// The caller sets `bounded` when the smallest weight a row's own key can have, 2^-(2 cap log2 e), is well inside
+// fp32's range and the bias never raises a score.
+// The keys a block visits are a list of 32-key chunks, those of the kept first tokens followed by those of the
+// window; four chunks make a tile, so the kept tokens cost one chunk and the window's ends are cut to 32 keys.
+// The one tile that holds chunks of both parts has two bias tables.
 // TMEM columns: S0 [0,128) S1 [128,256) O0 [256,384) O1 [384,512); P_t over the first 64 columns of S_t.
 // Every wait is bounded.
 #include "attn_window.h"
+#include "f32x2.cuh"
 #include "host_util.h"
 #include "ptx_sm100.cuh"
 
@@ -59,7 +70,7 @@ __device__ __forceinline__ uint32_t bit_range(int a, int b) {
   return hi & ~lo;
 }
 
-template <bool CAP, bool BIAS>
+template <bool CAP, bool BIAS, bool BOUNDED>
 __global__ void __launch_bounds__(WP_THREADS, 1)
 attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                            const __grid_constant__ CUtensorMap tmV, const __grid_constant__ WinPrefill w) {
@@ -80,10 +91,10 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   const int nt = min(w.nq * w.TT, n_seq - off);               // tokens of the block
   const int n_qt = nt > w.TT ? 2 : 1;
   const int p_first = ctx + off, p_last = p_first + nt - 1;
-  const int lo_tile = p.window > 0 ? max(0, p_first - p.window + 1) / WP_BN : 0;
-  const int first_tiles = min(lo_tile, (p.keep_first + WP_BN - 1) / WP_BN);
-  const int n_kv = first_tiles + p_last / WP_BN - lo_tile + 1;
-  auto tile_of = [&](int j) { return j < first_tiles ? j : lo_tile + j - first_tiles; };
+  const int lo_chunk = p.window > 0 ? max(0, p_first - p.window + 1) / 32 : 0;
+  const int kept = min(lo_chunk, (p.keep_first + 31) / 32);       // chunks of the kept first tokens
+  const int n_kv = (kept + p_last / 32 - lo_chunk + 1 + 3) / 4;    // key tiles
+  auto chunk_of = [&](int u) { return u < kept ? u : lo_chunk + u - kept; };
 
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t q_tile = w.kb * WP_BOX, k_tile = q_tile, v_tile = w.vb * WP_BOX;
@@ -124,38 +135,47 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
+    // A key tile is 4 * (32 / rows) boxes of `rows` tokens times the 64-channel slices: one lane per copy, so that
+    // page lookups and address arithmetic of a tile run side by side, and a tile ahead of the ring.
     if (elect_one()) {
       const uint32_t qb = smem_u32(&q_full);
       mbar_expect_tx(qb, (uint32_t)(n_qt * w.kb * w.R * w.TT * 128));
       for (int t = 0; t < n_qt; ++t)
         for (int x = 0; x < w.kb; ++x)
           tma_load_4d(sQ + t * q_tile + x * WP_BOX, &tmQ, qb, 64 * x, 0, row0 + t * w.TT, g);
-      const int* bt = p.block_tables + (long)seq * p.bt_stride;
-      const int last_page = (ctx + n_seq - 1) / p.block_size;
-      const int ppt = WP_BN / p.block_size;
-      const uint32_t page_bytes = (uint32_t)p.block_size * 128u;
-      for (int j = 0; j < n_kv; ++j) {
-        const int st = j % w.stages;
-        const uint32_t ph = (j / w.stages) & 1;
-        const int pg0 = tile_of(j) * ppt;
-        // pages past the sequence's last one re-read it: finite data that the mask discards
-        mbar_wait(smem_u32(&k_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
-        const uint32_t kb = smem_u32(&k_full[st]);
-        mbar_expect_tx(kb, k_tile);
-        for (int i = 0; i < ppt; ++i) {
-          const int page = min(max(bt[min(pg0 + i, last_page)], 0), p.num_blocks - 1);
-          for (int x = 0; x < w.kb; ++x)
-            tma_load_3d(sK + st * k_tile + x * WP_BOX + i * page_bytes, &tmK, kb, 64 * x, page * p.block_size, g);
-        }
-        mbar_wait(smem_u32(&v_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
-        const uint32_t vbar = smem_u32(&v_full[st]);
-        mbar_expect_tx(vbar, v_tile);
-        for (int i = 0; i < ppt; ++i) {
-          const int page = min(max(bt[min(pg0 + i, last_page)], 0), p.num_blocks - 1);
-          for (int x = 0; x < w.vb; ++x)
-            tma_load_3d(sV + st * v_tile + x * WP_BOX + i * page_bytes, &tmV, vbar, 64 * x, page * p.block_size, g);
-        }
-      }
+    }
+    const int* bt = p.block_tables + (long)seq * p.bt_stride;
+    const int bs = p.block_size, last_page = (ctx + n_seq - 1) / bs;
+    const int rows = min(bs, 32), boxes = 32 / rows;                       // tokens per box, boxes per chunk (1, 2, 4)
+    const int n_box = 4 * boxes, box_log2 = boxes == 1 ? 2 : (boxes == 2 ? 3 : 4);
+    const uint32_t box_bytes = (uint32_t)rows * 128u;
+    const int my_box = lane & (n_box - 1), x_first = lane >> box_log2, x_step = 32 >> box_log2;
+    const int in_chunk = (my_box & (boxes - 1)) * rows, my_chunk = my_box / boxes;
+    // first cache row of this lane's box of key tile j; boxes past the sequence's last page re-read it: finite
+    // data that the mask discards
+    auto box_row = [&](int j) {
+      const int pos = chunk_of(4 * j + my_chunk) * 32 + in_chunk;
+      const int page = pos / bs;
+      const int id = min(max(bt[min(page, last_page)], 0), p.num_blocks - 1);
+      return id * bs + min(pos - page * bs, bs - rows);
+    };
+    int next = box_row(0);
+    for (int j = 0; j < n_kv; ++j) {
+      const int st = j % w.stages;
+      const uint32_t ph = (j / w.stages) & 1;
+      const int r = next;
+      if (j + 1 < n_kv) next = box_row(j + 1);
+      const uint32_t kbar = smem_u32(&k_full[st]), vbar = smem_u32(&v_full[st]);
+      mbar_wait(smem_u32(&k_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+      if (lane == 0) mbar_expect_tx(kbar, k_tile);
+      __syncwarp();
+      for (int x = x_first; x < w.kb; x += x_step)
+        tma_load_3d(sK + st * k_tile + x * WP_BOX + my_box * box_bytes, &tmK, kbar, 64 * x, r, g);
+      mbar_wait(smem_u32(&v_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+      if (lane == 0) mbar_expect_tx(vbar, v_tile);
+      __syncwarp();
+      for (int x = x_first; x < w.vb; x += x_step)
+        tma_load_3d(sV + st * v_tile + x * WP_BOX + my_box * box_bytes, &tmV, vbar, 64 * x, r, g);
     }
   } else if (warp == 1) {
     // -------------------------------------------------------------------- MMA issuer
@@ -168,9 +188,15 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       const int ks = p.dp >> 4;
       auto issue_s = [&](int t, int st) {
         const uint64_t a0 = dQ + (uint64_t)t * q16, b0 = dK + (uint64_t)st * k16;
-        for (int k = 0; k < ks; ++k) {
+        auto step = [&](int k) {
           const uint64_t o = (uint64_t)(k >> 2) * box16 + (uint64_t)((k & 3) * 2);   // 16 channels = 32 bytes of a row
           mma_f16_ss(tmem_base + t * 128, a0 + o, b0 + o, idesc_qk, k == 0 ? 0u : 1u);
+        };
+        if (ks == 8) {
+#pragma unroll
+          for (int k = 0; k < 8; ++k) step(k);
+        } else {
+          for (int k = 0; k < ks; ++k) step(k);
         }
       };
       mbar_wait(smem_u32(&q_full), 0, &s_abort, status, ERR_WAIT_FULL);
@@ -213,20 +239,26 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     }
   } else if (warp < 4) {
     // ------------------------------------------------------------ bias of the key tiles
-    // entry i of head r: distance p_first - key tile base - 127 + i
+    // Entry i of head r is for distance d0 + i, where d0 = p_first - (position of the tile's key 0) - 127.  A tile's
+    // keys are consecutive except where the kept part ends: that tile's kept chunks use the third table.
     if (BIAS) {
-      const float top = CAP ? p.cap * WP_LOG2E : 0.f;
       const int width = 127 + 2 * w.TT;
-      for (int j = 0; j < n_kv; ++j) {
-        const int b = j & 1;
-        mbar_wait(smem_u32(&tab_empty[b]), ((j >> 1) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
-        const int d0 = p_first - tile_of(j) * WP_BN - 127;
+      auto fill = [&](float* dst0, int d0) {
         for (int r = 0; r < w.R; ++r) {
           const float r1 = p.r1[g * w.R + r], r2 = p.r2[g * w.R + r];
-          float* dst = tab + b * tab_floats + r * w.tab_stride;
+          float top = CAP ? p.cap * WP_LOG2E : 0.f;
+          if (BOUNDED) top = p.sink ? fminf(0.f, top - p.sink[g * w.R + r] * WP_LOG2E) : 0.f;   // less the reference
+          float* dst = dst0 + r * w.tab_stride;
           for (int i = threadIdx.x - 64; i < width; i += 64)
             dst[i] = fmaf(-r1, wp_lg2(fmaf(r2, (float)max(d0 + i, 0), 1.0f)), top);
         }
+      };
+      for (int j = 0; j < n_kv; ++j) {
+        const int b = j & 1;
+        mbar_wait(smem_u32(&tab_empty[b]), ((j >> 1) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+        const bool both = 4 * j < kept && 4 * j + 4 > kept;
+        if (4 * j < kept) fill(tab + (both ? 2 : b) * tab_floats, p_first - 128 * j - 127);
+        if (4 * j + 4 > kept) fill(tab + b * tab_floats, p_first - 32 * (lo_chunk + 4 * j - kept) - 127);
         __syncwarp();
         if (lane == 0) mbar_arrive(smem_u32(&tab_full[b]));
       }
@@ -245,10 +277,20 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     const int h = g * w.R + min(r, w.R - 1);
     const float C = p.cap * WP_LOG2E;
     const float mul = CAP ? p.scale * 2.0f * WP_LOG2E / p.cap : p.scale * WP_LOG2E;
-    float m = -INFINITY, l0 = 0.f, l1 = 0.f;     // reference exponent (log2 units) and two partial row sums
+    const float neg2C = -2.0f * C;
+    const uint64_t mul_2 = pack2(mul, mul);
+    float m = -INFINITY;                         // reference exponent (log2 units)
+    uint64_t l2a = 0ull, l2b = 0ull;             // four partial row sums
     if (p.sink) {                                // the sink is a key without a value, seen before all others
       m = p.sink[h] * WP_LOG2E;
-      l0 = 1.f;
+      l2a = pack2(1.f, 0.f);
+    }
+    float b_const = CAP ? C : 0.f;               // what a score without bias is relative to
+    if (BOUNDED) {
+      const float ref = fmaxf(C, m);
+      l2a = p.sink ? pack2(wp_ex2(m - ref), 0.f) : 0ull;
+      m = ref;
+      b_const = C - ref;
     }
     const float* my_tab = tab + min(r, w.R - 1) * w.tab_stride + min(t * w.TT + tok, 2 * w.TT - 1) + 127;
     for (int j = 0; tile_used && j < n_kv; ++j) {
@@ -261,33 +303,36 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         continue;
       }
       tc_fence_after_sync();
-      const int kbase = tile_of(j) * WP_BN;
-      const int hi = pos - kbase + 1;                                  // keys e < hi are not in the future
-      const int lo = p.window > 0 ? pos - p.window + 1 - kbase : 0;     // keys e >= lo are in the window
-      const bool masked = __any_sync(0xffffffffu, hi < WP_BN || lo > 0);
       if (BIAS) mbar_wait(smem_u32(&tab_full[j & 1]), (j >> 1) & 1, &s_abort, status, ERR_WAIT_FULL);
       const float* tb = my_tab + (j & 1) * tab_floats;
+      const float* tb_kept = 4 * j + 4 > kept ? my_tab + 2 * tab_floats : tb;
       uint32_t v0[32], v1[32], v2[32], v3[32];
       tmem_ld_32x32(tS, v0);
       tmem_ld_32x32(tS + 32, v1);
       tmem_ld_32x32(tS + 64, v2);
       tmem_ld_32x32(tS + 96, v3);
       tmem_wait_ld();
-      float mx = -INFINITY;
+      float ma = -INFINITY, mb = -INFINITY, mc = -INFINITY, md = -INFINITY;
       auto score = [&](uint32_t (&v)[32], int c) {
+        const int u = 4 * j + c;
+        const float* tc = (u < kept ? tb_kept : tb) - c * 32;
 #pragma unroll
         for (int e = 0; e < 32; e += 2) {
-          float y0 = __uint_as_float(v[e]) * mul, y1 = __uint_as_float(v[e + 1]) * mul;
-          float b0 = CAP ? C : 0.f, b1 = b0;
+          uint64_t y2 = mul2(pack2(__uint_as_float(v[e]), __uint_as_float(v[e + 1])), mul_2);
+          float y0, y1;
+          float b0 = b_const, b1 = b_const;
           if (BIAS) {
-            b0 = tb[-(c * 32 + e)];
-            b1 = tb[-(c * 32 + e + 1)];
+            b0 = tc[-e];
+            b1 = tc[-e - 1];
           }
+          unpack2(y2, y0, y1);
           if (CAP) {
-            // cap tanh(s / cap) = C - 2C / (1 + 2^y); the pair shares one reciprocal, y <= 60 keeps its
-            // product finite (there the bound is reached to the last bit)
-            const float a0 = wp_ex2(fminf(y0, 60.f)) + 1.0f, a1 = wp_ex2(fminf(y1, 60.f)) + 1.0f;
-            const float k = -2.0f * C * wp_rcp(a0 * a1);
+            // cap tanh(s / cap) = C - 2C / (1 + 2^y); the pair shares one reciprocal, and |y| <= 60 keeps the
+            // product of the two denominators finite (there the bound is reached to the last bit)
+            const uint64_t e2 = pack2(wp_ex2(fminf(y0, 60.f)), wp_ex2(fminf(y1, 60.f)));
+            float a0, a1;
+            unpack2(add2(e2, pack2(1.f, 1.f)), a0, a1);
+            const float k = neg2C * wp_rcp(a0 * a1);
             y0 = fmaf(k, a1, b0);
             y1 = fmaf(k, a0, b1);
           } else if (BIAS) {
@@ -297,32 +342,78 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
           v[e] = __float_as_uint(y0);
           v[e + 1] = __float_as_uint(y1);
         }
-        if (masked) {
-          const uint32_t mk = bit_range(lo - 32 * c, hi - 32 * c) | bit_range(0, min(p.keep_first - kbase, hi) - 32 * c);
+        const int kbase = chunk_of(u) * 32;
+        const int hi = pos - kbase + 1;                                   // keys e < hi are not in the future
+        const int lo = p.window > 0 ? pos - p.window + 1 - kbase : 0;      // keys e >= lo are in the window
+        if (__any_sync(0xffffffffu, hi < 32 || lo > 0)) {
+          const uint32_t mk = bit_range(lo, hi) | bit_range(0, min(p.keep_first - kbase, hi));
 #pragma unroll
           for (int e = 0; e < 32; ++e)
             if (!(mk & (1u << e))) v[e] = 0xff800000u;
         }
+        if constexpr (!BOUNDED) {
 #pragma unroll
-        for (int e = 0; e < 32; ++e) mx = fmaxf(mx, __uint_as_float(v[e]));
+          for (int e = 0; e < 32; e += 8) {
+            ma = max3(ma, __uint_as_float(v[e]), __uint_as_float(v[e + 1]));
+            mb = max3(mb, __uint_as_float(v[e + 2]), __uint_as_float(v[e + 3]));
+            mc = max3(mc, __uint_as_float(v[e + 4]), __uint_as_float(v[e + 5]));
+            md = max3(md, __uint_as_float(v[e + 6]), __uint_as_float(v[e + 7]));
+          }
+        }
       };
+      // exponents x (already relative to the reference) -> weights, bf16 pairs over the chunk's first score columns
+      auto weights = [&](uint32_t (&v)[32], int c, uint64_t negm2) {
+        uint32_t pk[16];
+#pragma unroll
+        for (int e = 0; e < 32; e += 2) {
+          uint64_t x2 = pack2(__uint_as_float(v[e]), __uint_as_float(v[e + 1]));
+          if (!BOUNDED) x2 = add2(x2, negm2);
+          float e0, e1;
+          unpack2(x2, e0, e1);
+          e0 = wp_ex2(e0);
+          e1 = wp_ex2(e1);
+          const uint64_t p2 = pack2(e0, e1);
+          if (e & 2) l2b = add2(l2b, p2); else l2a = add2(l2a, p2);
+          pk[e >> 1] = pack_bf16(e0, e1);
+        }
+        tmem_st_32x16(tS + c * 16, pk);
+        tmem_wait_st();
+        tc_fence_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&p_full[t][c]));
+      };
+      auto table_done = [&]() {
+        if (BIAS) {
+          __syncwarp();
+          if (lane == 0) mbar_arrive(smem_u32(&tab_empty[j & 1]));
+        }
+      };
+      if (BOUNDED) {
+        score(v0, 0);
+        weights(v0, 0, 0ull);
+        score(v1, 1);
+        weights(v1, 1, 0ull);
+        score(v2, 2);
+        weights(v2, 2, 0ull);
+        score(v3, 3);
+        table_done();
+        weights(v3, 3, 0ull);
+        continue;
+      }
       score(v0, 0);
       score(v1, 1);
       score(v2, 2);
       score(v3, 3);
-      if (BIAS) {
-        __syncwarp();
-        if (lane == 0) mbar_arrive(smem_u32(&tab_empty[j & 1]));
-      }
-      const float m_new = fmaxf(m, mx);
+      table_done();
+      const float m_new = fmaxf(m, fmaxf(fmaxf(ma, mb), fmaxf(mc, md)));
       if (j == 0) {
-        if (m != -INFINITY) l0 *= wp_ex2(m - m_new);
+        if (m != -INFINITY) l2a = pack2(wp_ex2(m - m_new), 0.f);          // the sink's share so far
         m = m_new;
       } else if (__any_sync(0xffffffffu, m_new > m + 8.0f)) {
         // rare: O follows the new reference; the scores wait in their own TMEM columns meanwhile
         const float alpha = m_new == -INFINITY ? 1.f : wp_ex2(m - m_new);
-        l0 *= alpha;
-        l1 *= alpha;
+        l2a = mul2(l2a, pack2(alpha, alpha));
+        l2b = mul2(l2b, pack2(alpha, alpha));
         tmem_st_32x32(tS, v0);
         tmem_st_32x32(tS + 32, v1);
         tmem_st_32x32(tS + 64, v2);
@@ -346,31 +437,20 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         tmem_wait_ld();
       }
       const float m_use = m == -INFINITY ? 0.f : m;
-      auto weights = [&](uint32_t (&v)[32], int c) {
-        uint32_t pk[16];
-#pragma unroll
-        for (int e = 0; e < 32; e += 2) {
-          const float e0 = wp_ex2(__uint_as_float(v[e]) - m_use), e1 = wp_ex2(__uint_as_float(v[e + 1]) - m_use);
-          l0 += e0;
-          l1 += e1;
-          pk[e >> 1] = pack_bf16(e0, e1);
-        }
-        tmem_st_32x16(tS + c * 16, pk);
-        tmem_wait_st();
-        tc_fence_before_sync();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(smem_u32(&p_full[t][c]));
-      };
-      weights(v0, 0);
-      weights(v1, 1);
-      weights(v2, 2);
-      weights(v3, 3);
+      const uint64_t negm2 = pack2(-m_use, -m_use);
+      weights(v0, 0, negm2);
+      weights(v1, 1, negm2);
+      weights(v2, 2, negm2);
+      weights(v3, 3, negm2);
     }
     if (rows_used) {
       mbar_wait(smem_u32(&o_done[t]), 0, &s_abort, status, ERR_WAIT_PV);
       tc_fence_after_sync();
       const long orow = row0 + t * w.TT + tok;
-      float f = 1.0f / (l0 + l1);
+      float s0, s1, s2, s3;
+      unpack2(l2a, s0, s1);
+      unpack2(l2b, s2, s3);
+      float f = 1.0f / ((s0 + s1) + (s2 + s3));
       if (p.gate && row_ok) {
         const float z = (float)static_cast<const __nv_bfloat16*>(p.gate)[orow * p.g_rs + h];
         f *= 1.0f / (1.0f + __expf(-z));
@@ -422,12 +502,12 @@ static int make_q_tmap(CUtensorMap* tm, const WinAttn& p, int R, int TT) {
   return r == CUDA_SUCCESS ? RC_OK : RC_TMAP;
 }
 
-template <bool CAP, bool BIAS>
+template <bool CAP, bool BIAS, bool BOUNDED>
 static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const WinPrefill& w,
                           int smem, cudaStream_t st) {
   static unsigned long long prep = 0;
-  if (int e = ensure_dynamic_smem((const void*)attn_window_prefill_kernel<CAP, BIAS>, 227 * 1024 - 512, prep)) return e;
-  attn_window_prefill_kernel<CAP, BIAS><<<dim3(w.a.n_items, w.a.G), WP_THREADS, smem, st>>>(tq, tk, tv, w);
+  if (int e = ensure_dynamic_smem((const void*)attn_window_prefill_kernel<CAP, BIAS, BOUNDED>, 227 * 1024 - 512, prep)) return e;
+  attn_window_prefill_kernel<CAP, BIAS, BOUNDED><<<dim3(w.a.n_items, w.a.G), WP_THREADS, smem, st>>>(tq, tk, tv, w);
   return (int)cudaGetLastError();
 }
 
@@ -459,7 +539,7 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   const int want = pow2 ? (32 / w.R) % 32 : 1;
   w.tab_stride = width;
   while (w.tab_stride % 32 != want) ++w.tab_stride;
-  const int tab_bytes = p.r1 ? 2 * w.R * w.tab_stride * 4 : 0;
+  const int tab_bytes = p.r1 ? 3 * w.R * w.tab_stride * 4 : 0;
   const int limit = 227 * 1024 - 1024 - 512;                 // less the alignment slack and the static barriers
   const int q_bytes = w.nq * w.kb * WP_BOX, stage = (w.kb + w.vb) * WP_BOX;
   w.stages = (limit - q_bytes - tab_bytes) / stage;
@@ -470,11 +550,14 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   const uint64_t slots = (uint64_t)p.num_blocks * p.block_size;
   int rc = make_q_tmap(&tq, p, w.R, w.TT);
   if (!rc) rc = make_tmap_3d(&tk, p.k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dp, slots, p.G, (uint64_t)p.G * p.dp * 2,
-                             (uint64_t)p.dp * 2, 64, p.block_size);
+                             (uint64_t)p.dp * 2, 64, p.block_size < 32 ? p.block_size : 32);
   if (!rc) rc = make_tmap_3d(&tv, p.v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.vp, slots, p.G, (uint64_t)p.G * p.vp * 2,
-                             (uint64_t)p.vp * 2, 64, p.block_size);
+                             (uint64_t)p.vp * 2, 64, p.block_size < 32 ? p.block_size : 32);
   if (rc) return rc;
   cudaStream_t st = (cudaStream_t)stream;
-  if (p.cap > 0.f) return p.r1 ? launch_prefill<true, true>(tq, tk, tv, w, smem, st) : launch_prefill<true, false>(tq, tk, tv, w, smem, st);
-  return p.r1 ? launch_prefill<false, true>(tq, tk, tv, w, smem, st) : launch_prefill<false, false>(tq, tk, tv, w, smem, st);
+  if (p.cap > 0.f && p.bounded)
+    return p.r1 ? launch_prefill<true, true, true>(tq, tk, tv, w, smem, st) : launch_prefill<true, false, true>(tq, tk, tv, w, smem, st);
+  if (p.cap > 0.f)
+    return p.r1 ? launch_prefill<true, true, false>(tq, tk, tv, w, smem, st) : launch_prefill<true, false, false>(tq, tk, tv, w, smem, st);
+  return p.r1 ? launch_prefill<false, true, false>(tq, tk, tv, w, smem, st) : launch_prefill<false, false, false>(tq, tk, tv, w, smem, st);
 }

@@ -176,22 +176,37 @@ add_norm_kernel(float* __restrict__ x, const T* __restrict__ y, int ldy, const f
 }
 
 // --------------------------------------------------------------------------------- PolyNorm
+// The row stays in registers as it was loaded (bf16 rows: half the registers of fp32 ones), so that blocks are small
+// and several rows are in flight per SM.
+template <typename T> struct Raw8;
+template <> struct Raw8<__nv_bfloat16> { uint4 a; };
+template <> struct Raw8<float> { uint4 a, b; };
+template <typename T> __device__ __forceinline__ void unraw8(const Raw8<T>& r, float (&v)[8]) {
+  load8<T>(reinterpret_cast<const T*>(&r), v);
+}
+
 template <typename T, int NV>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(NV == 8 ? 1024 : 320)
 poly_norm_kernel(const T* __restrict__ z, int ldz, T* __restrict__ out, int ldo, const float* __restrict__ coef, int F,
                  int Fp, float eps) {
   __shared__ float sh[96];
   const long r = blockIdx.x;
-  float v[NV][8];
+  Raw8<T> raw[NV];
   float ss[3] = {0.f, 0.f, 0.f};
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c < Fp) raw[i] = *reinterpret_cast<const Raw8<T>*>(z + r * ldz + c);
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
     if (c < Fp) {
-      load8<T>(z + r * ldz + c, v[i]);
+      float v[8];
+      unraw8<T>(raw[i], v);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        const float q = v[i][e] * v[i][e];
+        const float q = v[e] * v[e];
         ss[0] += q;
         ss[1] = fmaf(q, q, ss[1]);
         ss[2] = fmaf(q * q, q, ss[2]);
@@ -205,9 +220,11 @@ poly_norm_kernel(const T* __restrict__ z, int ldz, T* __restrict__ out, int ldo,
   for (int i = 0; i < NV; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * 8;
     if (c < Fp) {
+      float v[8];
+      unraw8<T>(raw[i], v);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[i][e] = fmaf(v[i][e], fmaf(v[i][e], fmaf(v[i][e], k3, k2), k1), k0);
-      store8<T>(out + r * ldo + c, v[i]);
+      for (int e = 0; e < 8; ++e) v[e] = fmaf(v[e], fmaf(v[e], fmaf(v[e], k3, k2), k1), k0);
+      store8<T>(out + r * ldo + c, v);
     }
   }
 }
@@ -356,6 +373,121 @@ conv_heads_kernel(ConvHeads p) {
   }
 }
 
+// The same for long batches: a group owns RUN consecutive rows of one head, holds the taps of its eight channels
+// in registers and slides a window of projected rows along, so every projected value is loaded once (plus
+// TAPS - 1 per run) and the weights once per run.
+template <int TAPS, int RUN>
+__global__ void __launch_bounds__(256)
+conv_heads_run_kernel(ConvHeads p) {
+  typedef __nv_bfloat16 T;
+  constexpr int HIST = TAPS - 1;
+  const int lane = threadIdx.x & (p.lph - 1);
+  const int t0 = (blockIdx.x * (blockDim.x / p.lph) + threadIdx.x / p.lph) * RUN;
+  const int head = blockIdx.y;
+  const int kind = head < p.H ? 0 : (head < p.H + p.G ? 1 : 2);
+  const int width = kind == 2 ? p.vp : p.dp;
+  const int hk = kind == 0 ? head : (kind == 1 ? head - p.H : head - p.H - p.G);
+  const int C = (p.H + p.G) * p.dp + p.G * p.vp;
+  const int c = lane * 8;
+  const int col = (kind == 0 ? hk * p.dp : (kind == 1 ? (p.H + hk) * p.dp : (p.H + p.G) * p.dp + hk * p.vp)) + c;
+  const bool in = c < width;
+  const T* proj = static_cast<const T*>(p.proj) + col;
+  T* state = static_cast<T*>(p.state) + col;
+  uint4 raw[RUN];                                          // all loads of the run in flight at once
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    raw[i] = make_uint4(0u, 0u, 0u, 0u);
+    if (in && t0 + i < p.T) raw[i] = *reinterpret_cast<const uint4*>(proj + (long)(t0 + i) * p.ldp);
+  }
+  float w[TAPS][8];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) w[j][e] = 0.f;
+    if (in) load8<float>(p.conv + (long)j * C + col, w[j]);
+  }
+  const float* nw = kind == 0 ? p.q_norm : (kind == 1 ? p.k_norm : nullptr);
+  const float lam = p.v_mode == 2 ? p.lambda[0] : 0.f;
+  uint4 win[HIST > 0 ? HIST : 1];                          // the rows before the current one
+  int prev_seq = -1, q0 = 0, ctx = 0, q1 = 0, sin = 0, sout = -1;
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    const int row = t0 + i;
+    const bool live = row < p.T;
+    const int seq = live ? min(max(p.row_seq[row], 0), p.num_seqs - 1) : prev_seq;
+    if (live && seq != prev_seq) {                         // first row of the run or of a sequence: fetch its history
+      prev_seq = seq;
+      q0 = p.q_start[seq];
+      q1 = p.q_start[seq + 1];
+      ctx = p.context[seq];
+      if (HIST > 0) {
+        sin = p.state_in[seq];
+        sout = p.state_out[seq];
+        if (sin < 0 || sin >= p.num_state || sout >= p.num_state) {
+          if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+          sin = 0;
+          sout = -1;
+        }
+#pragma unroll
+        for (int m = 0; m < HIST; ++m) {
+          const int b = row - q0 - HIST + m;               // row of the portion; negative: history
+          win[m] = make_uint4(0u, 0u, 0u, 0u);
+          if (in && b >= 0) win[m] = *reinterpret_cast<const uint4*>(proj + (long)(q0 + b) * p.ldp);
+          else if (in && ctx + b >= 0) win[m] = *reinterpret_cast<const uint4*>(state + ((long)sin * HIST + HIST + b) * C);
+        }
+      }
+    }
+    float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      float u[8];
+      load8<T>(reinterpret_cast<const T*>(j < HIST ? &win[j] : &raw[i]), u);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = fmaf(w[j][e], u[e], v[e]);
+    }
+    if (HIST > 0) {
+#pragma unroll
+      for (int m = 0; m + 1 < HIST; ++m) win[m] = win[m + 1];
+      win[HIST > 0 ? HIST - 1 : 0] = raw[i];
+      // after its last row the window is the sequence's new history
+      if (live && in && sout >= 0 && row == q1 - 1) {
+#pragma unroll
+        for (int m = 0; m < HIST; ++m) *reinterpret_cast<uint4*>(state + ((long)sout * HIST + m) * C) = win[m];
+      }
+    }
+    if (nw != nullptr) {                                   // uniform over the block
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+      for (int o = p.lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (in) scale_gain8(v, rms_scale(ss, p.d, p.eps), nw, 1, c);
+    }
+    if (!live || !in) continue;
+    if (kind == 0) {
+      store8<T>(static_cast<T*>(p.q_out) + (long)row * p.H * p.dp + col, v);
+      continue;
+    }
+    int slot = p.slots[row];
+    if (slot >= p.num_slots) {
+      if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+      slot = -1;
+    }
+    if (kind == 1) {
+      if (slot >= 0) store8<T>(static_cast<T*>(p.k_cache) + ((long)slot * p.G + hk) * p.dp + c, v);
+    } else {
+      T* vf = static_cast<T*>(p.v_first) + (long)row * p.G * p.vp + hk * p.vp + c;
+      if (p.v_mode == 1) store8<T>(vf, v);
+      if (p.v_mode == 2) {
+        float f[8];
+        load8<T>(vf, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = (1.f - lam) * v[e] + lam * f[e];
+      }
+      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + ((long)slot * p.G + hk) * p.vp + c, v);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------ logit cap
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -426,8 +558,22 @@ extern "C" int omni_poly_norm(const void* z, int ldz, void* out, int ldo, const 
                               float eps, int is_bf16, void* stream) {
   if (rows <= 0) return RC_OK;
   int threads, nv;
-  if ((Fp & 7) || (ldz & 7) || (ldo & 7) || F > Fp || !row_shape(Fp, threads, nv)) return RC_BAD_ARG;
-  OMNI_ROW_DISPATCH(poly_norm_kernel, rows, (const T*)z, ldz, (T*)out, ldo, coef, F, Fp, eps);
+  if (Fp <= 0 || (Fp & 7) || (ldz & 7) || (ldo & 7) || F > Fp || Fp > 65536) return RC_BAD_ARG;
+  const int vec = Fp / 8;
+  nv = vec <= 128 ? 1 : (vec <= 512 ? 2 : (vec <= 1280 ? 4 : 8));
+  threads = ((vec + nv - 1) / nv + 31) / 32 * 32;
+  cudaStream_t st = (cudaStream_t)stream;
+#define OMNI_POLY(T, NV) poly_norm_kernel<T, NV><<<rows, threads, 0, st>>>((const T*)z, ldz, (T*)out, ldo, coef, F, Fp, eps)
+#define OMNI_POLY_NV(T)           \
+  do {                            \
+    if (nv == 1) OMNI_POLY(T, 1); \
+    else if (nv == 2) OMNI_POLY(T, 2); \
+    else if (nv == 4) OMNI_POLY(T, 4); \
+    else OMNI_POLY(T, 8);         \
+  } while (0)
+  if (is_bf16) OMNI_POLY_NV(bf16); else OMNI_POLY_NV(float);
+#undef OMNI_POLY_NV
+#undef OMNI_POLY
   return (int)cudaGetLastError();
 }
 
@@ -445,6 +591,18 @@ extern "C" int omni_conv_heads(const ConvHeads* args, int is_bf16, void* stream)
   const int rows_per_cta = 256 / p.lph;
   dim3 grid((p.T + rows_per_cta - 1) / rows_per_cta, p.H + 2 * p.G);
   cudaStream_t st = (cudaStream_t)stream;
+  constexpr int RUN = 8;
+  if (is_bf16 && lanes <= 32 && p.T >= 256 && p.taps <= 4 && p.conv != nullptr) {
+    const int rows = rows_per_cta * RUN;
+    dim3 rgrid((p.T + rows - 1) / rows, p.H + 2 * p.G);
+    switch (p.taps) {
+      case 1: conv_heads_run_kernel<1, RUN><<<rgrid, 256, 0, st>>>(p); break;
+      case 2: conv_heads_run_kernel<2, RUN><<<rgrid, 256, 0, st>>>(p); break;
+      case 3: conv_heads_run_kernel<3, RUN><<<rgrid, 256, 0, st>>>(p); break;
+      default: conv_heads_run_kernel<4, RUN><<<rgrid, 256, 0, st>>>(p); break;
+    }
+    return (int)cudaGetLastError();
+  }
   if (is_bf16) {
     if (lanes <= 32) conv_heads_kernel<bf16, 1><<<grid, 256, 0, st>>>(p);
     else conv_heads_kernel<bf16, 4><<<grid, 256, 0, st>>>(p);

@@ -20,7 +20,7 @@ from torch import nn
 
 from ...diffusion.layers.linear import FusedLinear
 from ...ops import lm
-from ...ops.window_attention import ScoreRule, window_attention
+from ...ops.window_attention import ScoreRule, bounded_scores, window_attention
 from ..qwen_decoder import ModelBatch
 from .config import LayerConfig, TavulixConfig, _up
 
@@ -42,6 +42,7 @@ class TavulixLayer(nn.Module):
         f32 = lambda *s: _zeros(*s, dtype=torch.float32, device=device)
         D, m = cfg.hidden_size, lc.mixer
         self.lc, self.hs = lc, lc.mixer.head_shape
+        self.bounded = False         # whether the score bound may serve as softmax reference; set with the weights
         hs = self.hs
         self.norm1, self.norm1b = f32(1), f32(1)
         self.qkvg = _linear(D, hs.channels + m.heads, dtype, device)
@@ -57,7 +58,7 @@ class TavulixLayer(nn.Module):
 
     def rule(self) -> ScoreRule:
         m = self.lc.mixer
-        return ScoreRule(m.scale, m.softcap, self.r1, self.r2, self.sink, m.window, m.keep_first)
+        return ScoreRule(m.scale, m.softcap, self.r1, self.r2, self.sink, m.window, m.keep_first, self.bounded)
 
 
 class TavulixDecoder(nn.Module):
@@ -175,6 +176,8 @@ class TavulixDecoder(nn.Module):
             for dst, sel in targets[name]:
                 dst.copy_(w[sel].to(dst.dtype))
             loaded.add(name)
+        for layer in self.layers:
+            layer.bounded = bounded_scores(layer.lc.mixer.softcap, layer.r1, layer.r2)
         missing = sorted(set(targets) - loaded)
         if missing:
             raise ValueError(f"checkpoint lacks {len(missing)} tensors: {', '.join(missing[:8])}")

@@ -6,6 +6,7 @@ tensor-core kernels do not take)."""
 from __future__ import annotations
 
 import ctypes
+import math
 from dataclasses import dataclass
 
 import torch
@@ -21,7 +22,7 @@ class _WinAttn(ctypes.Structure):
                 ("row_seq", c_void_p), ("seq_list", c_void_p), ("n_list", c_int), ("items", c_void_p), ("n_items", c_int),
                 ("block_tokens", c_int),
                 ("out", c_void_p), ("o_rs", c_long), ("gate", c_void_p), ("g_rs", c_long), ("r1", c_void_p),
-                ("r2", c_void_p), ("sink", c_void_p), ("scale", c_float), ("cap", c_float), ("window", c_int),
+                ("r2", c_void_p), ("sink", c_void_p), ("scale", c_float), ("cap", c_float), ("bounded", c_int), ("window", c_int),
                 ("keep_first", c_int), ("T", c_int), ("H", c_int), ("G", c_int), ("dp", c_int), ("vp", c_int),
                 ("num_seqs", c_int), ("num_blocks", c_int), ("block_size", c_int), ("splits", c_int),
                 ("part_o", c_void_p), ("part_ml", c_void_p), ("status", c_void_p)]
@@ -37,6 +38,19 @@ class ScoreRule:
     sink: torch.Tensor | None = None      # fp32 [H]
     window: int | None = None
     keep_first: int = 0
+    bounded: bool = False                 # see ``bounded_scores``
+
+
+def bounded_scores(softcap, r1=None, r2=None) -> bool:
+    """May the cap stand in for the row maximum?  A row always sees its own position, where the bias is zero and the
+    score at least -cap: relative to the cap its weight is at least 2^-(2 cap log2 e), and what lies far below that
+    does not count.  True when this is well inside fp32's range and the bias never raises a score.  Reads r1 / r2
+    on the host."""
+    if not softcap:
+        return False
+    if r1 is not None and (bool((r1 < 0).any()) or bool((r2 < 0).any())):
+        return False
+    return 2.0 * softcap * math.log2(math.e) <= 90.0
 
 
 def prefill_rows_per_block(heads: int, kv_heads: int, dp: int) -> int:
@@ -91,7 +105,7 @@ def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None,
     a.gate, a.g_rs = P(gate), 0 if gate is None else gate.stride(0)
     a.r1, a.r2, a.sink = P(rule.r1), P(rule.r2), P(rule.sink)
     a.scale, a.cap = rule.scale, rule.softcap or 0.0
-    a.window, a.keep_first = rule.window or 0, rule.keep_first
+    a.bounded, a.window, a.keep_first = int(rule.bounded), rule.window or 0, rule.keep_first
     a.T, a.H, a.G, a.dp, a.vp, a.num_seqs, a.num_blocks, a.block_size = T, H, G, dp, vp, seqs.n_seqs, nb, bs
     a.splits = 1
     a.status = P(nv.status_word(q.device))
