@@ -14,6 +14,7 @@ from __future__ import annotations
 
 import torch
 
+from ..models.seq_table import layer_caches
 from .kernel_cases import _peaks
 
 LAYERS = 4
@@ -67,11 +68,7 @@ def _decoders(width: int, dev):
 
 
 def _caches(model, blocks: int, dev, seqs: int):
-    z = lambda *s: torch.randn(*s, dtype=torch.bfloat16, device=dev)
-    kv = [(z(blocks, BS, h, dk), z(blocks, BS, h, dv)) for h, dk, dv in model.cfg.kv_layer_shapes()]
-    if hasattr(model.cfg, "state_shapes"):
-        kv = [c if s is None else c + (z(2 * seqs, *s),) for c, s in zip(kv, model.cfg.state_shapes())]
-    return kv
+    return layer_caches(model.cfg, blocks, BS, 2 * seqs, torch.bfloat16, dev, fill=torch.randn)
 
 
 def _batch(lens, contexts, dev):

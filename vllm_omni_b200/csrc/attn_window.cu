@@ -65,7 +65,7 @@ attn_window_rows_kernel(WinAttn p) {
   for (int v = warp; v < n; v += 4) {
     const int j = v < nf ? v : lo + v - nf;
     const long slot = (long)wa_page(p, seq, j) * p.block_size + j % p.block_size;
-    const T* k = static_cast<const T*>(p.k_cache) + (slot * p.G + g) * p.dp;
+    const T* k = static_cast<const T*>(p.k_cache) + slot * p.k_ts + (long)g * p.dp;
     float d = 0.f;
     for (int c = lane; c < p.dp; c += 32) d = fmaf(sq[c], (float)k[c], d);
 #pragma unroll
@@ -77,7 +77,7 @@ attn_window_rows_kernel(WinAttn p) {
     const float a = expf(m - mn), e = expf(s - mn);
     l = l * a + e;
     m = mn;
-    const T* vv = static_cast<const T*>(p.v_cache) + (slot * p.G + g) * p.vp;
+    const T* vv = static_cast<const T*>(p.v_cache) + slot * p.v_ts + (long)g * p.vp;
 #pragma unroll
     for (int i = 0; i < NACC; ++i) {
       const int c = lane + 32 * i;
@@ -171,8 +171,8 @@ attn_window_decode_kernel(WinAttn p) {
       const int v = min(t * WD_KEYS + r, n_vis - 1);          // past the end: a valid key, masked below
       const int j = v < nf ? v : lo + v - nf;
       const long slot = (long)wa_page(p, seq, j) * p.block_size + j % p.block_size;
-      const __nv_bfloat16* ks = kc + (slot * p.G + g) * p.dp;
-      const __nv_bfloat16* vs = vc + (slot * p.G + g) * p.vp;
+      const __nv_bfloat16* ks = kc + slot * p.k_ts + (long)g * p.dp;
+      const __nv_bfloat16* vs = vc + slot * p.v_ts + (long)g * p.vp;
       for (int c = l8 * 8; c < p.dp; c += 64) cp_async16(kd + r * kpitch + c * 2, ks + c);
       for (int c = l8 * 8; c < p.vp; c += 64) cp_async16(vd + r * vpitch + c * 2, vs + c);
     }
@@ -371,7 +371,8 @@ attn_window_merge_kernel(WinAttn p) {
 
 static bool win_args_ok(const WinAttn& p) {
   return p.H > 0 && p.G > 0 && p.H % p.G == 0 && (p.dp & 15) == 0 && (p.vp & 15) == 0 && p.dp > 0 && p.vp > 0 &&
-         p.num_seqs > 0 && p.num_blocks > 0 && p.block_size > 0 && p.keep_first >= 0 && (p.r1 == nullptr) == (p.r2 == nullptr);
+         p.num_seqs > 0 && p.num_blocks > 0 && p.block_size > 0 && p.keep_first >= 0 && p.k_ts > 0 && p.v_ts > 0 && p.dp_u == p.dp &&
+         p.key_start == nullptr && (p.r1 == nullptr) == (p.r2 == nullptr);
 }
 
 template <int KS, int VS>
@@ -418,7 +419,7 @@ extern "C" int omni_attn_window_decode(const WinAttn* args, void* stream) {
   const WinAttn& p = *args;
   if (p.n_list <= 0) return RC_OK;
   if (!win_args_ok(p) || p.dp > 256 || p.vp > 256 || p.splits < 1 || p.seq_list == nullptr) return RC_BAD_ARG;
-  if ((p.q_rs & 1) || (p.splits > 1 && (p.part_o == nullptr || p.part_ml == nullptr))) return RC_BAD_ARG;
+  if ((p.q_rs & 1) || (p.k_ts & 7) || (p.v_ts & 7) || (p.splits > 1 && (p.part_o == nullptr || p.part_ml == nullptr))) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
   const int mx = p.dp > p.vp ? p.dp : p.vp;
   int rc = mx <= 64 ? launch_decode<4, 4>(p, st) : (mx <= 128 ? launch_decode<8, 8>(p, st) : launch_decode<16, 16>(p, st));

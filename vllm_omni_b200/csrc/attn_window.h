@@ -29,6 +29,12 @@ struct WinAttn {
   int T, H, G, dp, vp, num_seqs, num_blocks, block_size;
   int splits; float* part_o; float* part_ml;    // decode: shares of the visible keys, merged by a second kernel
   int* status;
+  long k_ts, v_ts;                     // elements from one cached token to the next in k_cache / v_cache
+  // Keys in two parts (prefill kernel): the first dp_u channels of a key are the head's own (k_cache), the other
+  // dp - dp_u are one vector per token shared by all heads (k_shared, pitch ks_ts).  dp_u = dp: one part.
+  const void* k_shared; long ks_ts; int dp_u;
+  // Keys back to back instead of in pages (prefill kernel): key j of sequence s is row key_start[s] + j of key_rows.
+  const int* key_start; long key_rows;
 };
 
 }  // namespace omni

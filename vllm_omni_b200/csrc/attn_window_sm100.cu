@@ -42,7 +42,8 @@ struct WinPrefill {
   int R, TT;            // heads per KV head, tokens per tile
   int nq;               // query tiles per block (2; 1 where two of the widest heads would not fit)
   int kb, vb;           // 64-channel boxes per key / value row
-  int stages;           // depth of the K and V rings
+  int kbu;              // key boxes of the head's own part; the others hold the part shared by all heads
+  int k_stages, v_stages;       // depth of the K and V rings
   int tab_stride;       // floats between the bias rows of two heads
 };
 
@@ -73,7 +74,8 @@ __device__ __forceinline__ uint32_t bit_range(int a, int b) {
 template <bool CAP, bool BIAS, bool BOUNDED>
 __global__ void __launch_bounds__(WP_THREADS, 1)
 attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                           const __grid_constant__ CUtensorMap tmV, const __grid_constant__ WinPrefill w) {
+                           const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmS,
+                           const __grid_constant__ WinPrefill w) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t q_full, k_full[WP_MAX_STAGES], k_empty[WP_MAX_STAGES], v_full[WP_MAX_STAGES],
       v_empty[WP_MAX_STAGES];
@@ -98,16 +100,18 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
 
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t q_tile = w.kb * WP_BOX, k_tile = q_tile, v_tile = w.vb * WP_BOX;
-  const uint32_t sQ = base, sK = base + w.nq * q_tile, sV = sK + w.stages * k_tile;
-  float* tab = reinterpret_cast<float*>(smem_raw + (sV + w.stages * v_tile - smem_u32(smem_raw)));
+  const uint32_t sQ = base, sK = base + w.nq * q_tile, sV = sK + w.k_stages * k_tile;
+  float* tab = reinterpret_cast<float*>(smem_raw + (sV + w.v_stages * v_tile - smem_u32(smem_raw)));
   const int tab_floats = w.R * w.tab_stride;
 
   if (threadIdx.x == 0) {
     s_abort = 0;
     mbar_init(smem_u32(&q_full), 1);
-    for (int i = 0; i < w.stages; ++i) {
+    for (int i = 0; i < w.k_stages; ++i) {
       mbar_init(smem_u32(&k_full[i]), 1);
       mbar_init(smem_u32(&k_empty[i]), 1);
+    }
+    for (int i = 0; i < w.v_stages; ++i) {
       mbar_init(smem_u32(&v_full[i]), 1);
       mbar_init(smem_u32(&v_empty[i]), 1);
     }
@@ -122,6 +126,7 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmV);
+    if (w.kbu < w.kb) tma_prefetch_desc(&tmS);
   }
   if (warp == 1) {
     tmem_alloc(smem_u32(&tmem_base_s), 512);
@@ -142,10 +147,12 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       mbar_expect_tx(qb, (uint32_t)(n_qt * w.kb * w.R * w.TT * 128));
       for (int t = 0; t < n_qt; ++t)
         for (int x = 0; x < w.kb; ++x)
-          tma_load_4d(sQ + t * q_tile + x * WP_BOX, &tmQ, qb, 64 * x, 0, row0 + t * w.TT, g);
+          tma_load_4d(sQ + t * q_tile + x * WP_BOX, &tmQ, qb, x < w.kbu ? 64 * x : p.dp_u + 64 * (x - w.kbu), 0,
+                      row0 + t * w.TT, g);
     }
     const int* bt = p.block_tables + (long)seq * p.bt_stride;
-    const int bs = p.block_size, last_page = (ctx + n_seq - 1) / bs;
+    const int bs = p.key_start ? 32 : p.block_size, last_page = (ctx + n_seq - 1) / bs;
+    const int key0 = p.key_start ? p.key_start[seq] : 0;
     const int rows = min(bs, 32), boxes = 32 / rows;                       // tokens per box, boxes per chunk (1, 2, 4)
     const int n_box = 4 * boxes, box_log2 = boxes == 1 ? 2 : (boxes == 2 ? 3 : 4);
     const uint32_t box_bytes = (uint32_t)rows * 128u;
@@ -155,27 +162,31 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     // data that the mask discards
     auto box_row = [&](int j) {
       const int pos = chunk_of(4 * j + my_chunk) * 32 + in_chunk;
+      // back to back: rows past the sequence's last belong to another one or are zero fill, and are masked either way
+      if (p.key_start) return key0 + pos;
       const int page = pos / bs;
       const int id = min(max(bt[min(page, last_page)], 0), p.num_blocks - 1);
       return id * bs + min(pos - page * bs, bs - rows);
     };
     int next = box_row(0);
     for (int j = 0; j < n_kv; ++j) {
-      const int st = j % w.stages;
-      const uint32_t ph = (j / w.stages) & 1;
+      const int ks = j % w.k_stages, vs = j % w.v_stages;
       const int r = next;
       if (j + 1 < n_kv) next = box_row(j + 1);
-      const uint32_t kbar = smem_u32(&k_full[st]), vbar = smem_u32(&v_full[st]);
-      mbar_wait(smem_u32(&k_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+      const uint32_t kbar = smem_u32(&k_full[ks]), vbar = smem_u32(&v_full[vs]);
+      mbar_wait(smem_u32(&k_empty[ks]), ((j / w.k_stages) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
       if (lane == 0) mbar_expect_tx(kbar, k_tile);
       __syncwarp();
-      for (int x = x_first; x < w.kb; x += x_step)
-        tma_load_3d(sK + st * k_tile + x * WP_BOX + my_box * box_bytes, &tmK, kbar, 64 * x, r, g);
-      mbar_wait(smem_u32(&v_empty[st]), ph ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+      for (int x = x_first; x < w.kb; x += x_step) {
+        const uint32_t dst = sK + ks * k_tile + x * WP_BOX + my_box * box_bytes;
+        if (x < w.kbu) tma_load_3d(dst, &tmK, kbar, 64 * x, r, g);
+        else tma_load_3d(dst, &tmS, kbar, 64 * (x - w.kbu), r, 0);
+      }
+      mbar_wait(smem_u32(&v_empty[vs]), ((j / w.v_stages) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
       if (lane == 0) mbar_expect_tx(vbar, v_tile);
       __syncwarp();
       for (int x = x_first; x < w.vb; x += x_step)
-        tma_load_3d(sV + st * v_tile + x * WP_BOX + my_box * box_bytes, &tmV, vbar, 64 * x, r, g);
+        tma_load_3d(sV + vs * v_tile + x * WP_BOX + my_box * box_bytes, &tmV, vbar, 64 * x, r, g);
     }
   } else if (warp == 1) {
     // -------------------------------------------------------------------- MMA issuer
@@ -185,14 +196,15 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       const uint64_t box16 = WP_BOX >> 4, q16 = q_tile >> 4, k16 = k_tile >> 4, v16 = v_tile >> 4;
       const uint64_t dQ = umma_desc_kmajor_sw128(sQ), dK = umma_desc_kmajor_sw128(sK);
       const uint64_t dV = umma_desc_sw128(sV, WP_BOX, 1024);
-      const int ks = p.dp >> 4;
+      const int ks = p.dp >> 4, ksu = p.dp_u >> 4;
       auto issue_s = [&](int t, int st) {
         const uint64_t a0 = dQ + (uint64_t)t * q16, b0 = dK + (uint64_t)st * k16;
-        auto step = [&](int k) {
+        auto step = [&](int k0) {
+          const int k = k0 < ksu ? k0 : 4 * w.kbu + k0 - ksu;       // the shared part starts a box of its own
           const uint64_t o = (uint64_t)(k >> 2) * box16 + (uint64_t)((k & 3) * 2);   // 16 channels = 32 bytes of a row
-          mma_f16_ss(tmem_base + t * 128, a0 + o, b0 + o, idesc_qk, k == 0 ? 0u : 1u);
+          mma_f16_ss(tmem_base + t * 128, a0 + o, b0 + o, idesc_qk, k0 == 0 ? 0u : 1u);
         };
-        if (ks == 8) {
+        if (ks == 8 && ksu == 8) {
 #pragma unroll
           for (int k = 0; k < 8; ++k) step(k);
         } else {
@@ -208,10 +220,10 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       }
       tc_commit(smem_u32(&k_empty[0]));
       for (int j = 0; j < n_kv; ++j) {
-        const int st = j % w.stages, st1 = (j + 1) % w.stages;
+        const int st = j % w.v_stages, st1 = (j + 1) % w.k_stages;
         const bool more = j + 1 < n_kv;
-        mbar_wait(smem_u32(&v_full[st]), (j / w.stages) & 1, &s_abort, status, ERR_WAIT_FULL);
-        if (more) mbar_wait(smem_u32(&k_full[st1]), ((j + 1) / w.stages) & 1, &s_abort, status, ERR_WAIT_FULL);
+        mbar_wait(smem_u32(&v_full[st]), (j / w.v_stages) & 1, &s_abort, status, ERR_WAIT_FULL);
+        if (more) mbar_wait(smem_u32(&k_full[st1]), ((j + 1) / w.k_stages) & 1, &s_abort, status, ERR_WAIT_FULL);
         const uint64_t v0 = dV + (uint64_t)st * v16;
         for (int t = 0; t < n_qt; ++t) {
 #pragma unroll
@@ -503,11 +515,11 @@ static int make_q_tmap(CUtensorMap* tm, const WinAttn& p, int R, int TT) {
 }
 
 template <bool CAP, bool BIAS, bool BOUNDED>
-static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const WinPrefill& w,
+static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const WinPrefill& w,
                           int smem, cudaStream_t st) {
   static unsigned long long prep = 0;
   if (int e = ensure_dynamic_smem((const void*)attn_window_prefill_kernel<CAP, BIAS, BOUNDED>, 227 * 1024 - 512, prep)) return e;
-  attn_window_prefill_kernel<CAP, BIAS, BOUNDED><<<dim3(w.a.n_items, w.a.G), WP_THREADS, smem, st>>>(tq, tk, tv, w);
+  attn_window_prefill_kernel<CAP, BIAS, BOUNDED><<<dim3(w.a.n_items, w.a.G), WP_THREADS, smem, st>>>(tq, tk, tv, ts, w);
   return (int)cudaGetLastError();
 }
 
@@ -524,14 +536,18 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   if (p.H <= 0 || p.G <= 0 || p.H % p.G || (p.dp & 15) || (p.vp & 15) || p.dp <= 0 || p.vp <= 0 || p.dp > 256 ||
       p.vp > 128 || p.items == nullptr || p.num_seqs <= 0 || p.num_blocks <= 0 || p.keep_first < 0)
     return RC_BAD_ARG;
-  if (p.block_size < 8 || (p.block_size & 7) || 128 % p.block_size || p.G > 65535) return RC_BAD_ARG;
+  if (p.key_start == nullptr && (p.block_size < 8 || (p.block_size & 7) || 128 % p.block_size)) return RC_BAD_ARG;
+  if (p.G > 65535 || (p.k_ts & 7) || (p.v_ts & 7) || p.dp_u <= 0 || (p.dp_u & 15) || p.dp_u > p.dp) return RC_BAD_ARG;
+  if (p.dp_u < p.dp && (p.k_shared == nullptr || (p.ks_ts & 7))) return RC_BAD_ARG;
+  if (p.key_start && (p.key_rows <= 0 || p.key_rows > 0x7fffffffl)) return RC_BAD_ARG;
   if ((p.r1 == nullptr) != (p.r2 == nullptr) || (p.o_rs & 7) || (reinterpret_cast<uintptr_t>(p.out) & 15)) return RC_BAD_ARG;
   w.R = p.H / p.G;
   if (w.R > 128) return RC_BAD_ARG;
   w.TT = 128 / w.R;
   if (p.block_tokens != w.TT && p.block_tokens != 2 * w.TT) return RC_BAD_ARG;
   w.nq = p.block_tokens / w.TT;
-  w.kb = (p.dp + 63) / 64;
+  w.kbu = (p.dp_u + 63) / 64;
+  w.kb = w.kbu + (p.dp - p.dp_u + 63) / 64;
   w.vb = (p.vp + 63) / 64;
   // rows of the bias table: a warp's 32 rows are 32 / R tokens of R heads; this pitch spreads them over all banks
   const int width = 127 + 2 * w.TT;
@@ -541,23 +557,34 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   while (w.tab_stride % 32 != want) ++w.tab_stride;
   const int tab_bytes = p.r1 ? 3 * w.R * w.tab_stride * 4 : 0;
   const int limit = 227 * 1024 - 1024 - 512;                 // less the alignment slack and the static barriers
-  const int q_bytes = w.nq * w.kb * WP_BOX, stage = (w.kb + w.vb) * WP_BOX;
-  w.stages = (limit - q_bytes - tab_bytes) / stage;
-  if (w.stages > WP_MAX_STAGES) w.stages = WP_MAX_STAGES;
-  if (w.stages < 1) return RC_TOO_LARGE;
-  const int smem = q_bytes + w.stages * stage + tab_bytes + 1024;
-  CUtensorMap tq, tk, tv;
-  const uint64_t slots = (uint64_t)p.num_blocks * p.block_size;
+  const int q_bytes = w.nq * w.kb * WP_BOX, k_bytes = w.kb * WP_BOX, v_bytes = w.vb * WP_BOX;
+  w.k_stages = w.v_stages = 1;
+  int used = q_bytes + tab_bytes + k_bytes + v_bytes;
+  if (used > limit) return RC_TOO_LARGE;
+  // the key ring grows first: the next tile's scores are issued before the current tile's values are done with
+  for (bool grew = true; grew;) {
+    grew = false;
+    if (w.k_stages < WP_MAX_STAGES && used + k_bytes <= limit) { ++w.k_stages; used += k_bytes; grew = true; }
+    if (w.v_stages < WP_MAX_STAGES && used + v_bytes <= limit) { ++w.v_stages; used += v_bytes; grew = true; }
+  }
+  const int smem = used + 1024;
+  CUtensorMap tq, tk, tv, ts;
+  const uint64_t slots = p.key_start ? (uint64_t)p.key_rows : (uint64_t)p.num_blocks * p.block_size;
+  const uint32_t box_rows = p.key_start ? 32 : (p.block_size < 32 ? p.block_size : 32);
   int rc = make_q_tmap(&tq, p, w.R, w.TT);
-  if (!rc) rc = make_tmap_3d(&tk, p.k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dp, slots, p.G, (uint64_t)p.G * p.dp * 2,
-                             (uint64_t)p.dp * 2, 64, p.block_size < 32 ? p.block_size : 32);
-  if (!rc) rc = make_tmap_3d(&tv, p.v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.vp, slots, p.G, (uint64_t)p.G * p.vp * 2,
-                             (uint64_t)p.vp * 2, 64, p.block_size < 32 ? p.block_size : 32);
+  if (!rc) rc = make_tmap_3d(&tk, p.k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dp_u, slots, p.G, (uint64_t)p.k_ts * 2,
+                             (uint64_t)p.dp_u * 2, 64, box_rows);
+  if (!rc) rc = make_tmap_3d(&tv, p.v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.vp, slots, p.G, (uint64_t)p.v_ts * 2,
+                             (uint64_t)p.vp * 2, 64, box_rows);
+  ts = tk;
+  if (!rc && w.kbu < w.kb)
+    rc = make_tmap_3d(&ts, p.k_shared, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dp - p.dp_u, slots, 1, (uint64_t)p.ks_ts * 2,
+                      (uint64_t)p.ks_ts * 2, 64, box_rows);
   if (rc) return rc;
   cudaStream_t st = (cudaStream_t)stream;
   if (p.cap > 0.f && p.bounded)
-    return p.r1 ? launch_prefill<true, true, true>(tq, tk, tv, w, smem, st) : launch_prefill<true, false, true>(tq, tk, tv, w, smem, st);
+    return p.r1 ? launch_prefill<true, true, true>(tq, tk, tv, ts, w, smem, st) : launch_prefill<true, false, true>(tq, tk, tv, ts, w, smem, st);
   if (p.cap > 0.f)
-    return p.r1 ? launch_prefill<true, true, false>(tq, tk, tv, w, smem, st) : launch_prefill<true, false, false>(tq, tk, tv, w, smem, st);
-  return p.r1 ? launch_prefill<false, true, false>(tq, tk, tv, w, smem, st) : launch_prefill<false, false, false>(tq, tk, tv, w, smem, st);
+    return p.r1 ? launch_prefill<true, true, false>(tq, tk, tv, ts, w, smem, st) : launch_prefill<true, false, false>(tq, tk, tv, ts, w, smem, st);
+  return p.r1 ? launch_prefill<false, true, false>(tq, tk, tv, ts, w, smem, st) : launch_prefill<false, false, false>(tq, tk, tv, ts, w, smem, st);
 }

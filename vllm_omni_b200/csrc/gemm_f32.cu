@@ -8,9 +8,18 @@ namespace omni {
 
 constexpr int FB = 64, FK = 16;
 
+// element strides between the problems of a batch (one per grid layer)
+struct GemmF32Batch {
+  long a, w, c, bias;
+};
+
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ A, long lda, const float* __restrict__ W, long ldw, float* __restrict__ C,
-                long ldc, int M, int N, int K, const float* __restrict__ bias) {
+                long ldc, int M, int N, int K, const float* __restrict__ bias, int act, GemmF32Batch b) {
+  A += blockIdx.z * b.a;
+  W += blockIdx.z * b.w;
+  C += blockIdx.z * b.c;
+  if (bias) bias += blockIdx.z * b.bias;
   __shared__ float sA[FK][FB + 4], sW[FK][FB + 4];
   const int m0 = blockIdx.y * FB, n0 = blockIdx.x * FB;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -43,17 +52,32 @@ gemm_f32_kernel(const float* __restrict__ A, long lda, const float* __restrict__
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (m < M && n < N) C[(long)m * ldc + n] = acc[i][j] + (bias ? bias[n] : 0.f);
+      if (m < M && n < N) {
+        float v = acc[i][j] + (bias ? bias[n] : 0.f);
+        if (act == 3) {                                    // squared ReLU
+          v = fmaxf(v, 0.f);
+          v *= v;
+        }
+        C[(long)m * ldc + n] = v;
+      }
     }
 }
 
 }  // namespace omni
 
+// `batch` problems of one shape whose operands lie the given strides apart; act: 0 none, 3 squared ReLU.
+extern "C" int omni_gemm_f32_batched(const float* A, long lda, const float* W, long ldw, float* C, long ldc, int M, int N, int K,
+                                     const float* bias, int act, int batch, long a_stride, long w_stride, long c_stride,
+                                     long bias_stride, void* stream) {
+  if (M <= 0 || N <= 0 || batch <= 0) return omni::RC_OK;
+  if (K <= 0 || (M + omni::FB - 1) / omni::FB > 65535 || batch > 65535 || (act != 0 && act != 3)) return omni::RC_BAD_ARG;
+  dim3 grid((N + omni::FB - 1) / omni::FB, (M + omni::FB - 1) / omni::FB, batch);
+  const omni::GemmF32Batch b = {a_stride, w_stride, c_stride, bias_stride};
+  omni::gemm_f32_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(A, lda, W, ldw, C, ldc, M, N, K, bias, act, b);
+  return (int)cudaGetLastError();
+}
+
 extern "C" int omni_gemm_f32(const float* A, long lda, const float* W, long ldw, float* C, long ldc, int M, int N, int K,
                              const float* bias, void* stream) {
-  if (M <= 0 || N <= 0) return omni::RC_OK;
-  if (K <= 0 || (M + omni::FB - 1) / omni::FB > 65535) return omni::RC_BAD_ARG;
-  dim3 grid((N + omni::FB - 1) / omni::FB, (M + omni::FB - 1) / omni::FB);
-  omni::gemm_f32_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(A, lda, W, ldw, C, ldc, M, N, K, bias);
-  return (int)cudaGetLastError();
+  return omni_gemm_f32_batched(A, lda, W, ldw, C, ldc, M, N, K, bias, 0, 1, 0, 0, 0, 0, stream);
 }

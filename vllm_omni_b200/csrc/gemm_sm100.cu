@@ -41,7 +41,7 @@ constexpr int BM = 128;
 constexpr int BK = 64;  // 64 bf16 = one 128-byte swizzle row
 constexpr int GEMM_THREADS = 320;  // warp 0 TMA, warp 1 MMA, warps 2-9 epilogue
 
-enum Act : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_SILU = 2 };
+enum Act : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU2 = 3 };
 
 struct GemmEpilogue {
   const __nv_bfloat16* bias;      // [N] or nullptr
@@ -172,6 +172,12 @@ __device__ __forceinline__ void epilogue_math32(const uint32_t (&v)[32], int row
       } else if (epi.act == ACT_SILU) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) x[e] = silu(x[e]);
+      } else if (epi.act == ACT_RELU2) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float r = fmaxf(x[e], 0.f);
+          x[e] = r * r;
+        }
       }
       if (gate_row) {
         uint4 g = *reinterpret_cast<const uint4*>(gate_row + col0 + j * 8);

@@ -1,0 +1,534 @@
+// Attention over a cache of latents.  A token leaves one row in the pages, shared by all heads: its latent c (rank_p
+// channels, normed) and a rotated key part (rot_p channels).  Head h has keys [W_uk[h] c, rotated part] and values
+// W_uv[h] c; queries are [dim_p unrotated | rot_p rotated] channels per head.  All sizes are multiples of 16 with
+// zero padding.
+//
+//   omni_latent_rows     rotates the queries in place, norms and rotates a token's row, writes it to its page
+//   omni_latent_gather   rows of several sequences from their pages to one buffer (prompts expand them to keys and
+//                        values with one GEMM and run on attn_window_sm100.cu)
+//   omni_head_gemm       one small product per head: queries into the latent space (W_uk^T q) and attention results
+//                        out of it (W_uv o, times the output gate); weights are read once per 64 rows
+//   omni_latent_decode   decoded tokens (and rows of short portions): scores and weighted sums directly on the
+//                        latent rows, so a row is read once for all heads.  A block owns 16 or 32 heads of one token
+//                        and a share of its keys; 64-key tiles go through a two-deep cp.async ring, eight warps share
+//                        the score product by (keys, channel half) and the weighted sum by channels
+//
+// A decode step reads every latent once per group of heads and does little arithmetic on it, so the warp-level
+// products (no operand staging through tensor memory) suffice.
+#include "host_util.h"
+#include "row_ops.cuh"
+
+namespace omni {
+
+typedef __nv_bfloat16 bf16;
+
+// ------------------------------------------------------------------------------- rows and pages
+struct LatentRows {
+  void* proj; long ldp;            // [T, ldp]: q (H heads of dim_p + rot_p) | latent rank_p | rot_p
+  int T, H, dim_p, rot, rot_p;
+  int rank, rank_p;
+  const float* turns;              // [T, rot / 2, 2] cos, sin
+  const int* slots;                // [T], < 0: not written
+  void* pages; long num_slots;     // [num_slots, rank_p + rot_p]
+  const float* norm;               // [rank_p]; nullptr: the layer writes no row
+  float eps;
+  int* status;
+};
+
+template <typename T> struct Pair;
+template <> struct Pair<float> {
+  static __device__ __forceinline__ float2 ld(const float* p) { return *reinterpret_cast<const float2*>(p); }
+  static __device__ __forceinline__ void st(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+};
+template <> struct Pair<bf16> {
+  static __device__ __forceinline__ float2 ld(const bf16* p) { return unpack_bf16(*reinterpret_cast<const uint32_t*>(p)); }
+  static __device__ __forceinline__ void st(bf16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(a, b); }
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_rows_kernel(const LatentRows p) {
+  __shared__ float sh[32];
+  const long t = blockIdx.x;
+  T* row = static_cast<T*>(p.proj) + t * p.ldp;
+  const float2* turn = reinterpret_cast<const float2*>(p.turns) + t * (p.rot / 2);
+  const int half = p.rot / 2, hc = p.dim_p + p.rot_p;
+  for (int i = threadIdx.x; i < p.H * half; i += 128) {
+    const int h = i / half, c = i - h * half;
+    T* q = row + h * hc + p.dim_p + 2 * c;
+    const float2 v = Pair<T>::ld(q), a = turn[c];
+    Pair<T>::st(q, v.x * a.x - v.y * a.y, v.y * a.x + v.x * a.y);
+  }
+  if (p.norm == nullptr) return;
+  const T* z = row + p.H * hc;
+  float ss[1] = {0.f};
+  for (int i = threadIdx.x; i < p.rank_p / 2; i += 128) {
+    const float2 v = Pair<T>::ld(z + 2 * i);
+    ss[0] = fmaf(v.x, v.x, fmaf(v.y, v.y, ss[0]));
+  }
+  block_sum<1>(ss, sh);
+  const float s = rms_scale(ss[0], p.rank, p.eps);
+  const long slot = p.slots[t];
+  if (slot >= p.num_slots && p.status && threadIdx.x == 0) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+  if (slot < 0 || slot >= p.num_slots) return;
+  T* page = static_cast<T*>(p.pages) + slot * (p.rank_p + p.rot_p);
+  for (int i = threadIdx.x; i < p.rank_p / 2; i += 128) {
+    const float2 v = Pair<T>::ld(z + 2 * i), g = *reinterpret_cast<const float2*>(p.norm + 2 * i);
+    Pair<T>::st(page + 2 * i, v.x * s * g.x, v.y * s * g.y);
+  }
+  for (int i = threadIdx.x; i < p.rot_p / 2; i += 128) {
+    float2 o = make_float2(0.f, 0.f);
+    if (i < half) {
+      const float2 v = Pair<T>::ld(z + p.rank_p + 2 * i), a = turn[i];
+      o = make_float2(v.x * a.x - v.y * a.y, v.y * a.x + v.x * a.y);
+    }
+    Pair<T>::st(page + p.rank_p + 2 * i, o.x, o.y);
+  }
+}
+
+// members: (sequence, first row of the output) pairs closed by (-1, rows); 16-byte pieces.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ pages, int row16, const int* __restrict__ tables, int bt_stride, int block_size,
+                     int num_blocks, const int* __restrict__ members, int n_members, uint4* __restrict__ out, long rows) {
+  const long total = rows * row16;
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
+    const int r = (int)(i / row16), c = (int)(i - (long)r * row16);
+    int lo = 0, hi = n_members - 1;                          // the last member that starts at or before r
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (members[2 * mid + 1] <= r) lo = mid; else hi = mid - 1;
+    }
+    const int pos = r - members[2 * lo + 1];
+    int pg = tables[(long)members[2 * lo] * bt_stride + pos / block_size];
+    pg = min(max(pg, 0), num_blocks - 1);
+    out[i] = pages[((long)pg * block_size + pos % block_size) * row16 + c];
+  }
+}
+
+// -------------------------------------------------------------------------- one product per head
+struct HeadGemm {
+  const bf16* A; long a_row, a_head; const int* a_rows;     // A[(a_rows[m] or m) * a_row + h * a_head + k]
+  const bf16* W;                                            // [H, N, K]
+  bf16* C; long c_row, c_head; const int* c_rows;
+  const bf16* gate; long g_row;                             // logits at the row of C and head, or nullptr
+  int M, N, K, H, rows_a, rows_c;
+};
+
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                         uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+               "{%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+// A block: 16 MT rows of one head, 64 outputs (16 per warp).  Lane group j of a quad owns channels 8 j .. 8 j + 7 of
+// every 32-channel chunk in both operands (the contraction is permuted alike), so all loads are 16 bytes.
+template <int MT>
+__global__ void __launch_bounds__(128)
+head_gemm_kernel(const HeadGemm p) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+  const int h = blockIdx.y, n0 = blockIdx.x * 64 + warp * 16, m0 = blockIdx.z * (16 * MT);
+  if (n0 >= p.N) return;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  const bf16* a[MT][2];
+  bool live[MT][2];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int r = m0 + m * 16 + u * 8 + g;
+      live[m][u] = r < p.M;
+      int row = live[m][u] ? (p.a_rows ? p.a_rows[r] : r) : 0;
+      row = min(max(row, 0), p.rows_a - 1);
+      a[m][u] = p.A + row * p.a_row + h * p.a_head + j * 8;
+    }
+  const bf16* w0 = p.W + ((long)h * p.N + n0 + g) * p.K + j * 8;
+  const bf16* w1 = w0 + 8l * p.K;
+  float acc[MT][2][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
+#pragma unroll 4
+  for (int k = 0; k < p.K; k += 32) {
+    const bool in = k + j * 8 < p.K;                        // K is a multiple of 16
+    const uint4 b0 = in ? *reinterpret_cast<const uint4*>(w0 + k) : zero;
+    const uint4 b1 = in ? *reinterpret_cast<const uint4*>(w1 + k) : zero;
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const uint4 x = in && live[m][0] ? *reinterpret_cast<const uint4*>(a[m][0] + k) : zero;
+      const uint4 y = in && live[m][1] ? *reinterpret_cast<const uint4*>(a[m][1] + k) : zero;
+      mma_bf16(acc[m][0], x.x, y.x, x.y, y.y, b0.x, b0.y);
+      mma_bf16(acc[m][0], x.z, y.z, x.w, y.w, b0.z, b0.w);
+      mma_bf16(acc[m][1], x.x, y.x, x.y, y.y, b1.x, b1.y);
+      mma_bf16(acc[m][1], x.z, y.z, x.w, y.w, b1.z, b1.w);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int r = m0 + m * 16 + u * 8 + g;
+      if (r >= p.M) continue;
+      int row = p.c_rows ? p.c_rows[r] : r;
+      row = min(max(row, 0), p.rows_c - 1);
+      float f = 1.f;
+      if (p.gate) f = 1.0f / (1.0f + __expf(-(float)p.gate[row * p.g_row + h]));
+      bf16* c = p.C + row * p.c_row + h * p.c_head + n0 + j * 2;
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+        *reinterpret_cast<uint32_t*>(c + n * 8) = pack_bf16(acc[m][n][2 * u] * f, acc[m][n][2 * u + 1] * f);
+    }
+}
+
+// ---------------------------------------------------------------------------------- decode
+struct LatentDecode {
+  const bf16* q_lat;                   // [n, H, rank_p]
+  const bf16* proj; long ldp; int head_cols, dim_p;         // rotated query part: proj[row * ldp + h * head_cols + dim_p]
+  const bf16* pages; int rank_p, rot_p;
+  const int* block_tables; int bt_stride, block_size, num_blocks;
+  const int* rows; int n;              // batch rows served
+  const int* row_seq; const int* q_start; const int* context; int num_seqs, T;
+  float scale;
+  bf16* out;                           // [n, H, rank_p]
+  int H, splits;
+  float* part_o; float* part_ml;       // [n, H, splits, rank_p], [n, H, splits, 2]
+};
+
+constexpr int LD_KEYS = 64;
+constexpr float LD_LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ float ld_ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void ld_cp16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void ld_m4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ld_m4t(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+
+// shared memory of one block: two key tiles, the queries, weights (bf16) and two partial score tiles (fp32)
+inline int latent_decode_smem(int row_ch, int mt) {
+  const int pitch = row_ch * 2 + 16;
+  return 2 * LD_KEYS * pitch + 16 * mt * pitch + 16 * mt * (LD_KEYS * 2 + 16) + 2 * 16 * mt * (LD_KEYS + 4) * 4;
+}
+
+// MT: 16-head tiles of the block; CPW: 16-channel slices of the weighted sum per warp (rank_p <= 128 CPW).
+template <int MT, int CPW>
+__global__ void __launch_bounds__(256)
+latent_decode_kernel(const LatentDecode p) {
+  constexpr int ROWS = 16 * MT, PER = 256 / ROWS, KPT = LD_KEYS / PER;      // threads per row, keys per thread
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ float s_alpha[ROWS], s_m[ROWS], s_l[ROWS];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h0 = blockIdx.y * ROWS, nh = min(ROWS, p.H - h0), split = blockIdx.z;
+  const int row = min(max(p.rows[blockIdx.x], 0), p.T - 1);
+  const int seq = min(max(p.row_seq[row], 0), p.num_seqs - 1);
+  const int n_vis = p.context[seq] + row - p.q_start[seq] + 1;
+  const int tiles_all = (n_vis + LD_KEYS - 1) / LD_KEYS;
+  const int per = (tiles_all + p.splits - 1) / p.splits;
+  const int t0 = min(tiles_all, split * per), t1 = min(tiles_all, t0 + per);
+  const int ch = p.rank_p + p.rot_p, pitch = ch * 2 + 16, pp = LD_KEYS * 2 + 16;
+  const uint32_t sK = smem_u32(smem), sQ = sK + 2 * LD_KEYS * pitch, sP = sQ + ROWS * pitch;
+  float* sS = reinterpret_cast<float*>(smem + 2 * LD_KEYS * pitch + ROWS * pitch + ROWS * pp);   // [2][ROWS][LD_KEYS + 4]
+  constexpr int SP = LD_KEYS + 4;
+
+  auto fetch = [&](int t, int buf) {
+    // four threads per key row, 16 bytes each
+    const int r = tid >> 2;
+    const int pos = min(t * LD_KEYS + r, n_vis - 1);        // past the end: a valid key, masked below
+    int pg = p.block_tables[(long)seq * p.bt_stride + pos / p.block_size];
+    pg = min(max(pg, 0), p.num_blocks - 1);
+    const bf16* src = p.pages + ((long)pg * p.block_size + pos % p.block_size) * ch;
+    const uint32_t dst = sK + (buf * LD_KEYS + r) * pitch;
+    for (int c = (tid & 3) * 8; c < ch; c += 32) ld_cp16(dst + c * 2, src + c);
+  };
+  if (t0 < t1) fetch(t0, 0);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  // queries: latent part, rotated part; rows past the last head are zero
+  for (int i = tid; i < ROWS * (ch / 8); i += 256) {
+    const int r = i / (ch / 8), c = (i - r * (ch / 8)) * 8;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (r < nh) {
+      const bf16* src = c < p.rank_p ? p.q_lat + ((long)blockIdx.x * p.H + h0 + r) * p.rank_p + c
+                                     : p.proj + (long)row * p.ldp + (long)(h0 + r) * p.head_cols + p.dim_p + (c - p.rank_p);
+      v = *reinterpret_cast<const uint4*>(src);
+    }
+    st_shared_v4(sQ + r * pitch + c * 2, v);
+  }
+
+  const int half = warp >> 2, kg = warp & 3;                // score product: channel half, group of 16 keys
+  const int steps = ch / 16, k_lo = half ? (steps + 1) / 2 : 0, k_hi = half ? steps : (steps + 1) / 2;
+  const int srow = tid / PER, sk0 = (tid % PER) * KPT;      // softmax: row and first key of this thread
+  float m_run = -INFINITY, l_run = 0.f;
+  const float mul = p.scale * LD_LOG2E;
+  float acc[MT][CPW][2][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int c = 0; c < CPW; ++c)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[m][c][n][i] = 0.f;
+
+  for (int t = t0; t < t1; ++t) {
+    const int buf = (t - t0) & 1;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                        // tile t is here; everyone is done with the other buffer
+    if (t + 1 < t1) fetch(t + 1, buf ^ 1);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const uint32_t kt = sK + buf * LD_KEYS * pitch;
+    {
+      float s[MT][2][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) s[m][n][i] = 0.f;
+      // K matrices: keys 0-7 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 0-7 | keys 8-15 ch 8-15
+      const uint32_t ka = kt + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
+      // Q matrices: rows 0-7 ch 0-7 | rows 8-15 ch 0-7 | rows 0-7 ch 8-15 | rows 8-15 ch 8-15
+      const uint32_t qa = sQ + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
+#pragma unroll 4
+      for (int k = k_lo; k < k_hi; ++k) {
+        uint32_t b[4];
+        ld_m4(ka + k * 32, b);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          uint32_t a[4];
+          ld_m4(qa + m * 16 * pitch + k * 32, a);
+          mma_bf16(s[m][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+          mma_bf16(s[m][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int u = 0; u < 2; ++u)
+            *reinterpret_cast<float2*>(sS + (half * ROWS + m * 16 + u * 8 + (lane >> 2)) * SP + kg * 16 + n * 8 + (lane & 3) * 2) =
+                make_float2(s[m][n][2 * u], s[m][n][2 * u + 1]);
+    }
+    __syncthreads();
+    {
+      float y[KPT], mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < KPT; i += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(sS + srow * SP + sk0 + i);
+        const float4 b = *reinterpret_cast<const float4*>(sS + (ROWS + srow) * SP + sk0 + i);
+        y[i] = (a.x + b.x) * mul; y[i + 1] = (a.y + b.y) * mul; y[i + 2] = (a.z + b.z) * mul; y[i + 3] = (a.w + b.w) * mul;
+      }
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) {
+        if (t * LD_KEYS + sk0 + i >= n_vis) y[i] = -INFINITY;
+        mx = fmaxf(mx, y[i]);
+      }
+#pragma unroll
+      for (int o = PER / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float m_new = fmaxf(m_run, mx);                 // finite: a tile holds at least one visible key
+      const float alpha = ld_ex2(m_run - m_new);
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) {
+        y[i] = ld_ex2(y[i] - m_new);
+        sum += y[i];
+      }
+      l_run = fmaf(l_run, alpha, sum);                      // this thread's keys only; summed at the end
+      m_run = m_new;
+      if (tid % PER == 0) s_alpha[srow] = alpha;
+      const uint32_t pd = sP + srow * pp + sk0 * 2;
+#pragma unroll
+      for (int i = 0; i < KPT; i += 2)
+        asm volatile("st.shared.b32 [%0], %1;" ::"r"(pd + i * 2), "r"(pack_bf16(y[i], y[i + 1])) : "memory");
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float a0 = s_alpha[m * 16 + (lane >> 2)], a1 = s_alpha[m * 16 + 8 + (lane >> 2)];
+#pragma unroll
+      for (int c = 0; c < CPW; ++c)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          acc[m][c][n][0] *= a0; acc[m][c][n][1] *= a0;
+          acc[m][c][n][2] *= a1; acc[m][c][n][3] *= a1;
+        }
+    }
+    const uint32_t pa = sP + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pp + (lane >> 4) * 16;
+    // V matrices, transposed: keys 0-7 ch 0-7 | keys 8-15 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 8-15
+    const uint32_t va = kt + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
+#pragma unroll
+    for (int k = 0; k < LD_KEYS / 16; ++k) {
+      uint32_t a[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) ld_m4(pa + m * 16 * pp + k * 32, a[m]);
+#pragma unroll
+      for (int c = 0; c < CPW; ++c) {
+        const int sl = c * 8 + warp;
+        if (sl * 16 < p.rank_p) {
+          uint32_t b[4];
+          ld_m4t(va + k * 16 * pitch + sl * 32, b);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            mma_bf16(acc[m][c][0], a[m][0], a[m][1], a[m][2], a[m][3], b[0], b[1]);
+            mma_bf16(acc[m][c][1], a[m][0], a[m][1], a[m][2], a[m][3], b[2], b[3]);
+          }
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int o = PER / 2; o > 0; o >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, o);
+  if (tid % PER == 0) {
+    s_m[srow] = m_run;
+    s_l[srow] = l_run;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int r = m * 16 + u * 8 + (lane >> 2);
+      if (r >= nh) continue;
+      const long hi = (long)blockIdx.x * p.H + h0 + r;
+#pragma unroll
+      for (int c = 0; c < CPW; ++c) {
+        const int sl = c * 8 + warp;
+        if (sl * 16 >= p.rank_p) continue;
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          const int col = sl * 16 + n * 8 + (lane & 3) * 2;
+          const float x = acc[m][c][n][2 * u], y = acc[m][c][n][2 * u + 1];
+          if (p.splits == 1) {
+            const float f = 1.0f / s_l[r];
+            *reinterpret_cast<uint32_t*>(p.out + hi * p.rank_p + col) = pack_bf16(x * f, y * f);
+          } else {
+            *reinterpret_cast<float2*>(p.part_o + (hi * p.splits + split) * p.rank_p + col) = make_float2(x, y);
+          }
+        }
+      }
+      if (p.splits > 1 && warp == 0 && (lane & 3) == 0) {
+        p.part_ml[2 * (hi * p.splits + split)] = s_m[r];
+        p.part_ml[2 * (hi * p.splits + split) + 1] = s_l[r];
+      }
+    }
+}
+
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const LatentDecode p) {
+  const long base = (long)blockIdx.x * p.splits;            // blockIdx.x: (row, head)
+  float top = -INFINITY;
+  for (int s = 0; s < p.splits; ++s) top = fmaxf(top, p.part_ml[2 * (base + s)]);
+  float den = 0.f;
+  for (int s = 0; s < p.splits; ++s) {
+    const float ms = p.part_ml[2 * (base + s)];
+    den += ms == -INFINITY ? 0.f : p.part_ml[2 * (base + s) + 1] * ld_ex2(ms - top);
+  }
+  const float f = 1.0f / den;
+  for (int c = threadIdx.x * 4; c < p.rank_p; c += 512) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < p.splits; ++s) {
+      const float ms = p.part_ml[2 * (base + s)];
+      if (ms == -INFINITY) continue;
+      const float a = ld_ex2(ms - top) * f;
+      const float4 v = *reinterpret_cast<const float4*>(p.part_o + (base + s) * p.rank_p + c);
+      o.x = fmaf(v.x, a, o.x); o.y = fmaf(v.y, a, o.y); o.z = fmaf(v.z, a, o.z); o.w = fmaf(v.w, a, o.w);
+    }
+    *reinterpret_cast<uint2*>(p.out + (long)blockIdx.x * p.rank_p + c) = make_uint2(pack_bf16(o.x, o.y), pack_bf16(o.z, o.w));
+  }
+}
+
+template <int MT, int CPW>
+static int launch_latent_decode(const LatentDecode& p, int smem, cudaStream_t st) {
+  static unsigned long long prep = 0;
+  if (int e = ensure_dynamic_smem((const void*)latent_decode_kernel<MT, CPW>, 227 * 1024 - 1024, prep)) return e;
+  dim3 grid(p.n, (p.H + 16 * MT - 1) / (16 * MT), p.splits);
+  latent_decode_kernel<MT, CPW><<<grid, 256, smem, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
+template <int MT>
+static int pick_latent_decode(const LatentDecode& p, int smem, cudaStream_t st) {
+  if (p.rank_p <= 128) return launch_latent_decode<MT, 1>(p, smem, st);
+  if (p.rank_p <= 256) return launch_latent_decode<MT, 2>(p, smem, st);
+  return launch_latent_decode<MT, 4>(p, smem, st);
+}
+
+}  // namespace omni
+
+using namespace omni;
+
+extern "C" int omni_latent_rows(const LatentRows* args, int is_bf16, void* stream) {
+  const LatentRows& p = *args;
+  if (p.T <= 0) return RC_OK;
+  if (p.H < 0 || p.rot < 0 || (p.rot & 1) || p.rot > p.rot_p || (p.dim_p & 15) || (p.rot_p & 15) || (p.rank_p & 15) || (p.ldp & 7))
+    return RC_BAD_ARG;
+  if (p.norm && (p.pages == nullptr || p.rank <= 0 || p.rank > p.rank_p || p.num_slots <= 0)) return RC_BAD_ARG;
+  if (is_bf16) latent_rows_kernel<bf16><<<p.T, 128, 0, (cudaStream_t)stream>>>(p);
+  else latent_rows_kernel<float><<<p.T, 128, 0, (cudaStream_t)stream>>>(p);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_latent_gather(const void* pages, int row_bytes, const int* tables, int bt_stride, int block_size, int num_blocks,
+                                  const int* members, int n_members, void* out, long rows, void* stream) {
+  if (rows <= 0) return RC_OK;
+  if ((row_bytes & 15) || row_bytes <= 0 || n_members <= 0 || block_size <= 0 || num_blocks <= 0) return RC_BAD_ARG;
+  long blocks = (rows * (row_bytes / 16) + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  latent_gather_kernel<<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>((const uint4*)pages, row_bytes / 16, tables, bt_stride,
+                                                                          block_size, num_blocks, members, n_members, (uint4*)out, rows);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_head_gemm(const HeadGemm* args, void* stream) {
+  const HeadGemm& p = *args;
+  if (p.M <= 0 || p.H <= 0) return RC_OK;
+  if ((p.N & 15) || (p.K & 15) || p.N <= 0 || p.K <= 0 || (p.a_row & 7) || (p.a_head & 7) || (p.c_row & 1) || (p.c_head & 1) ||
+      p.H > 65535 || p.rows_a <= 0 || p.rows_c <= 0)
+    return RC_BAD_ARG;
+  cudaStream_t st = (cudaStream_t)stream;
+  const unsigned nb = (p.N + 63) / 64;
+  if (p.M <= 16) head_gemm_kernel<1><<<dim3(nb, p.H, 1), 128, 0, st>>>(p);
+  else if (p.M <= 32) head_gemm_kernel<2><<<dim3(nb, p.H, 1), 128, 0, st>>>(p);
+  else {
+    if ((p.M + 63) / 64 > 65535) return RC_BAD_ARG;
+    head_gemm_kernel<4><<<dim3(nb, p.H, (p.M + 63) / 64), 128, 0, st>>>(p);
+  }
+  return (int)cudaGetLastError();
+}
+
+// 0: the sizes do not fit the decode kernel; otherwise the heads a block serves.
+extern "C" int omni_latent_decode_heads(int heads, int rank_p, int rot_p) {
+  if (rank_p > 512 || rank_p <= 0 || rot_p < 0) return 0;
+  if (heads > 16 && latent_decode_smem(rank_p + rot_p, 2) <= 227 * 1024 - 1024) return 32;
+  return latent_decode_smem(rank_p + rot_p, 1) <= 227 * 1024 - 1024 ? 16 : 0;
+}
+
+extern "C" int omni_latent_decode(const LatentDecode* args, void* stream) {
+  const LatentDecode& p = *args;
+  if (p.n <= 0) return RC_OK;
+  const int heads = omni_latent_decode_heads(p.H, p.rank_p, p.rot_p);
+  if (heads == 0 || p.H <= 0 || (p.rank_p & 15) || (p.rot_p & 15) || (p.ldp & 7) || (p.head_cols & 7) || (p.dim_p & 7) || p.splits < 1 ||
+      p.splits > 65535 || p.block_size <= 0 || p.num_blocks <= 0 || p.num_seqs <= 0 || p.T <= 0)
+    return RC_BAD_ARG;
+  if (p.splits > 1 && (!p.part_o || !p.part_ml)) return RC_BAD_ARG;
+  cudaStream_t st = (cudaStream_t)stream;
+  int rc = heads == 32 ? pick_latent_decode<2>(p, latent_decode_smem(p.rank_p + p.rot_p, 2), st)
+                       : pick_latent_decode<1>(p, latent_decode_smem(p.rank_p + p.rot_p, 1), st);
+  if (rc || p.splits == 1) return rc;
+  latent_merge_kernel<<<(unsigned)(p.n * p.H), 128, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}

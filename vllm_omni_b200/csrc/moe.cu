@@ -1,6 +1,10 @@
 // K10: mixture-of-experts routing, dispatch and combine around the grouped tcgen05 GEMM.
 //
 //   omni_moe_route     softmax over expert logits, top-k, optional renormalisation
+//   omni_moe_router    router product and choice in one launch: fp32 logits with a bias, the top-k largest, softmax
+//                      among them (bf16 rows)
+//   omni_moe_topk      the same choice from fp32 logits
+//   omni_moe_pairs_f32 y[p] = act(W[expert of pair p] x[p / per]) in true fp32 (exact mode)
 //   omni_moe_plan      per-expert counts -> segment offsets padded to 128 rows (the GEMM's M
 //                      tile), the expert of every M tile, and the row of every (token, k) pair
 //   omni_moe_dispatch  copy token rows into the expert-major padded buffer
@@ -72,6 +76,159 @@ moe_route_kernel(const __nv_bfloat16* __restrict__ logits, int ld, int T, int E,
     const float r = 1.0f / fmaxf(picked, 1e-20f);
     for (int j = 0; j < k; ++j) weights[(size_t)t * k + j] *= r;
   }
+}
+
+// Choice of one token by one warp: the k largest of v (lane + 32 i holds expert lane + 32 i), ties to the lower index;
+// weights are the softmax of the chosen logits.  E <= 256, k <= 16.
+__device__ __forceinline__ void topk_softmax(float (&v)[8], int E, int k, int lane, int* ids, float* weights) {
+  float top = 0.f, sum = 0.f, mine = 0.f;
+  int mine_id = 0;
+  for (int j = 0; j < k; ++j) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int e = lane + i * 32;
+      if (e < E && (v[i] > best || (v[i] == best && e < bi))) { best = v[i]; bi = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+    }
+    if (bi >= E) bi = j;                       // no finite logit left: any index inside the range
+    if (j == 0) top = best;
+    const float w = expf(best - top);
+    sum += w;
+    if (lane == j) { mine = w; mine_id = bi; }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (bi == lane + i * 32) v[i] = -INFINITY;
+  }
+  if (lane < k) {
+    ids[lane] = mine_id;
+    weights[lane] = mine / sum;
+  }
+}
+
+__global__ void __launch_bounds__(256)
+moe_topk_kernel(const float* __restrict__ logits, long ld, int T, int E, int k, int* __restrict__ ids,
+                float* __restrict__ weights) {
+  const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= T) return;
+  float v[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int e = lane + i * 32;
+    v[i] = e < E ? logits[t * ld + e] : -INFINITY;
+  }
+  topk_softmax(v, E, k, lane, ids + (long)t * k, weights + (long)t * k);
+}
+
+// Router of MT * 16 tokens per block: eight warps share the contraction (each takes every eighth 32-channel chunk),
+// 64 experts at a time; partial sums meet in shared memory in a fixed order.  A warp reads 16 bytes per row and
+// chunk: lane group j of a quad owns channels 8 j .. 8 j + 7 of the chunk for both operands, which permutes the
+// contraction alike on both sides.
+template <int MT>
+__global__ void __launch_bounds__(256)
+moe_router_kernel(const __nv_bfloat16* __restrict__ x, long ldx, const __nv_bfloat16* __restrict__ w, long ldw,
+                  const float* __restrict__ bias, int T, int D, int E, int Ep, int k, int* __restrict__ ids,
+                  float* __restrict__ weights) {
+  extern __shared__ float sm[];
+  float* part = sm;                            // [8 warps][MT * 16][64]
+  float* logit = sm + 8 * MT * 16 * 64;        // [MT * 16][256]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+  const int t0 = blockIdx.x * (MT * 16);
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  for (int e0 = 0; e0 < E; e0 += 64) {
+    float acc[MT][8][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
+    for (int c = warp * 32; c < D; c += 256) {
+      const int ch = c + j * 8;
+      const bool in = ch < D;                  // D is a multiple of 8
+      uint4 a[MT][2];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int t = t0 + m * 16 + h * 8 + g;
+          a[m][h] = in && t < T ? *reinterpret_cast<const uint4*>(x + (long)t * ldx + ch) : zero;
+        }
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {
+        const int e = e0 + n * 8 + g;
+        const uint4 b = in && e < Ep ? *reinterpret_cast<const uint4*>(w + (long)e * ldw + ch) : zero;
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+                       "{%0, %1, %2, %3};"
+                       : "+f"(acc[m][n][0]), "+f"(acc[m][n][1]), "+f"(acc[m][n][2]), "+f"(acc[m][n][3])
+                       : "r"(a[m][0].x), "r"(a[m][1].x), "r"(a[m][0].y), "r"(a[m][1].y), "r"(b.x), "r"(b.y));
+          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+                       "{%0, %1, %2, %3};"
+                       : "+f"(acc[m][n][0]), "+f"(acc[m][n][1]), "+f"(acc[m][n][2]), "+f"(acc[m][n][3])
+                       : "r"(a[m][0].z), "r"(a[m][1].z), "r"(a[m][0].w), "r"(a[m][1].w), "r"(b.z), "r"(b.w));
+        }
+      }
+    }
+    __syncthreads();                           // the previous group's sums are read
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+          *reinterpret_cast<float2*>(part + ((long)warp * MT * 16 + m * 16 + h * 8 + g) * 64 + n * 8 + j * 2) =
+              make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
+    __syncthreads();
+    for (int i = threadIdx.x; i < MT * 16 * 64; i += 256) {
+      const int e = e0 + (i & 63);
+      if (e < E) {
+        float s = bias ? bias[e] : 0.f;
+#pragma unroll
+        for (int q = 0; q < 8; ++q) s += part[q * MT * 16 * 64 + i];
+        logit[(i >> 6) * 256 + e] = s;
+      }
+    }
+  }
+  __syncthreads();
+  for (int r = warp; r < MT * 16; r += 8) {
+    const int t = t0 + r;
+    if (t >= T) break;
+    float v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = lane + i * 32 < E ? logit[r * 256 + lane + i * 32] : -INFINITY;
+    topk_softmax(v, E, k, lane, ids + (long)t * k, weights + (long)t * k);
+  }
+}
+
+// Exact mode: one warp per (pair, output); a result is one fixed-order chain plus a fixed-order sum over lanes.
+__global__ void __launch_bounds__(256)
+moe_pairs_f32_kernel(const float* __restrict__ x, long ldx, int per, const int* __restrict__ ids, const float* __restrict__ w,
+                     int E, float* __restrict__ y, long ldy, long pairs, int N, int K, int relu2) {
+  const long i = (long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (i >= pairs * N) return;
+  const long p = i / N;
+  const int n = (int)(i - p * N);
+  const int e = min(max(ids[p], 0), E - 1);
+  const float* a = x + (p / per) * ldx;
+  const float* b = w + ((long)e * N + n) * K;
+  float s = 0.f;
+  for (int c = lane; c < K; c += 32) s = fmaf(a[c], b[c], s);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+  if (relu2) {
+    s = fmaxf(s, 0.f);
+    s *= s;
+  }
+  if (lane == 0) y[p * ldy + n] = s;
 }
 
 // single CTA: histogram, padded prefix sum, tile->expert table, (token,k)->row map.
@@ -271,6 +428,7 @@ moe_combine_scatter_kernel(const __nv_bfloat16* __restrict__ y, const int* __res
 }  // namespace omni
 
 using namespace omni;
+typedef __nv_bfloat16 bf16;
 
 // 1 when this library was compiled with -DOMNI_BOUNDS_CHECK
 extern "C" int omni_moe_bounds_check_enabled(void) {
@@ -306,6 +464,45 @@ extern "C" int omni_moe_route(const void* logits, int ld, int T, int E, int k, i
   if (T <= 0) return RC_OK;
   if (E > 256 || k > 16 || k > E) return RC_BAD_ARG;
   moe_route_kernel<<<(T + 7) / 8, 256, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)logits, ld, T, E, k, renorm, ids, weights);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_moe_topk(const float* logits, long ld, int T, int E, int k, int* ids, float* weights, void* stream) {
+  if (T <= 0) return RC_OK;
+  if (E > 256 || k > 16 || k > E || k < 1) return RC_BAD_ARG;
+  moe_topk_kernel<<<(T + 7) / 8, 256, 0, (cudaStream_t)stream>>>(logits, ld, T, E, k, ids, weights);
+  return (int)cudaGetLastError();
+}
+
+// x [T, D] and w [Ep >= E, D] bf16 (D, pitches multiples of 8), bias [E] fp32 or null.
+extern "C" int omni_moe_router(const void* x, long ldx, const void* w, long ldw, const float* bias, int T, int D, int E, int Ep,
+                               int k, int* ids, float* weights, void* stream) {
+  if (T <= 0) return RC_OK;
+  if (E > 256 || k > 16 || k > E || k < 1 || D <= 0 || (D & 7) || (ldx & 7) || (ldw & 7)) return RC_BAD_ARG;
+  cudaStream_t st = (cudaStream_t)stream;
+  const bf16* xb = (const bf16*)x;
+  const bf16* wb = (const bf16*)w;
+  static unsigned long long prep[2] = {0, 0};
+  if (T > 148 * 16) {
+    const int smem = (8 * 32 * 64 + 32 * 256) * 4;
+    if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<2>, smem, prep[0])) return e;
+    moe_router_kernel<2><<<(T + 31) / 32, 256, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
+  } else {
+    const int smem = (8 * 16 * 64 + 16 * 256) * 4;
+    if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<1>, smem, prep[1])) return e;
+    moe_router_kernel<1><<<(T + 15) / 16, 256, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
+  }
+  return (int)cudaGetLastError();
+}
+
+// Pair p reads row p / per of x.
+extern "C" int omni_moe_pairs_f32(const float* x, long ldx, int per, const int* ids, const float* w, int E, float* y, long ldy,
+                                  long pairs, int N, int K, int relu2, void* stream) {
+  if (pairs <= 0 || N <= 0) return RC_OK;
+  if (per < 1 || E < 1 || K < 1) return RC_BAD_ARG;
+  const long blocks = (pairs * N + 7) / 8;
+  if (blocks > 0x7fffffffL) return RC_BAD_ARG;
+  moe_pairs_f32_kernel<<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>(x, ldx, per, ids, w, E, y, ldy, pairs, N, K, relu2);
   return (int)cudaGetLastError();
 }
 

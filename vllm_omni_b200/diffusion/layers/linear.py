@@ -59,6 +59,8 @@ def _epilogue(y, act, residual, gate, out):
         y = F.gelu(y.float(), approximate="tanh").to(y.dtype)
     elif act == "silu":
         y = F.silu(y)
+    elif act == "relu2":
+        y = F.relu(y).square()
     if gate is not None:
         B = gate.shape[0]
         y = (y.reshape(B, -1, y.shape[-1]) * gate.unsqueeze(1)).reshape(y.shape)

@@ -54,7 +54,7 @@ class LLMEngine:
                 num_gpu_blocks = self._profile_num_blocks(dec, block_size, gpu_memory_utilization, max_model_len,
                                                           max_num_seqs)
             # models that carry per-sequence state beside the pages have a slot for every running sequence
-            stateful = any(s is not None for s in dec.state_shapes()) if hasattr(dec, "state_shapes") else False
+            stateful = any(dec.state_shapes()) if hasattr(dec, "state_shapes") else False
             self.kv = KVCacheManager(num_gpu_blocks, block_size, max_num_seqs if stateful else 0)
             self.runner = ARModelRunner(model, self.device, dtype, num_gpu_blocks, block_size,
                                         self.kv.state.num_rows if stateful else 0)

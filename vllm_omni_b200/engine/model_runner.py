@@ -19,7 +19,7 @@ import zlib
 import torch
 
 from ..models.qwen_decoder import ModelBatch, PrefillSeg
-from ..models.seq_table import SeqTable
+from ..models.seq_table import SeqTable, layer_caches
 from ..ops import kv_cache as KC
 from ..ops.sampler import RowParams, sample
 from .scheduler import SchedulerOutput
@@ -35,13 +35,8 @@ class ARModelRunner:
         decoder = getattr(model, "decoder", None)
         local = getattr(decoder, "kv_heads_local", None)
         self.seq_table = bool(getattr(decoder, "uses_seq_table", False))
-        z = lambda *s: torch.zeros(*s, dtype=dtype, device=device)
-        self.kv_caches = [(z(num_blocks, block_size, local or h, dk), z(num_blocks, block_size, local or h, dv))
-                          for h, dk, dv in dec.kv_layer_shapes()]
-        if num_state_rows:
-            # a layer's cache entry is (k pages, v pages, state rows) where the layer carries state
-            self.kv_caches = [kv if s is None else kv + (z(num_state_rows, *s),)
-                              for kv, s in zip(self.kv_caches, dec.state_shapes())]
+        # a layer's cache entry is (key pages, value pages, *pools of its per-sequence state)
+        self.kv_caches = layer_caches(dec, num_blocks, block_size, num_state_rows, dtype, device, local)
         self.tp_group = None        # set by OmniLLM: sampled ids of every step come from rank 0
         # decode-only steps replay a captured graph per batch-size bucket (on by default on a GPU,
         # ``OMNI_AR_CUDA_GRAPH=0`` switches it off); contexts longer than ``OMNI_AR_GRAPH_MAX_TOKENS``
@@ -172,11 +167,14 @@ class ARModelRunner:
         layers = []
         for li, (kc, vc, *_) in enumerate(self.kv_caches):
             ok, ov = (out_buffers[li] if out_buffers is not None else (None, None))
+            if not vc.numel():                             # keys only, or a layer without pages
+                layers.append((KC.rows_gather(kc, bt, T), vc.new_empty(T, *vc.shape[2:])))
+                continue
             layers.append(KC.kv_gather(kc, vc, bt, T, ok, ov))
         out = {"num_tokens": T, "layers": layers}
         if request.state_slot is not None:
             row = 2 * request.state_slot + request.state_phase
-            out["state"] = [c[2][row].clone() if len(c) > 2 else None for c in self.kv_caches]
+            out["state"] = [tuple(t[row].clone() for t in c[2:]) for c in self.kv_caches]
         return out
 
 

@@ -12,6 +12,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "Qwen2ForCausalLM": ("vllm_omni_b200.models.text", "build_text_model"),
     "Qwen3MoeForCausalLM": ("vllm_omni_b200.models.text", "build_text_model"),
     "Tavulix": ("vllm_omni_b200.models.tavulix.model", "build_tavulix"),
+    "Nidilix": ("vllm_omni_b200.models.nidilix.model", "build_nidilix"),
     "BagelForConditionalGeneration": ("vllm_omni_b200.models.text", "build_text_model"),
 }
 

@@ -4,10 +4,8 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 
 from ...ops.lm import HeadShape
-
-
-def _up(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
+from ..packed_decoder import round_up as _up
+from ..seq_table import StateTensor
 
 
 @dataclass
@@ -102,10 +100,10 @@ class TavulixConfig:
         hs = [l.mixer.head_shape for l in self.layers]
         return [(h.kv_heads, h.dp, h.vp) for h in hs]
 
-    def state_shapes(self) -> list[tuple[int, ...] | None]:
-        """Per layer: shape of what one sequence carries besides its pages, None = nothing."""
+    def state_shapes(self) -> list[tuple[StateTensor, ...]]:
+        """Per layer: what one sequence carries besides its pages."""
         hs = [l.mixer.head_shape for l in self.layers]
-        return [(h.taps - 1, h.channels) if h.taps > 1 else None for h in hs]
+        return [(StateTensor((h.taps - 1, h.channels)),) if h.taps > 1 else () for h in hs]
 
     def tensor_shapes(self) -> dict[str, tuple[int, ...]]:
         """Checkpoint tensor names and shapes."""

@@ -18,22 +18,11 @@ import torch
 import torch.nn.functional as F
 from torch import nn
 
-from ...diffusion.layers.linear import FusedLinear
 from ...ops import lm
 from ...ops.window_attention import ScoreRule, bounded_scores, window_attention
+from ..packed_decoder import PackedDecoder, packed_linear as _linear, zeros_param as _zeros
 from ..qwen_decoder import ModelBatch
-from .config import LayerConfig, TavulixConfig, _up
-
-
-def _zeros(*shape, dtype, device):
-    return nn.Parameter(torch.zeros(*shape, dtype=dtype, device=device), requires_grad=False)
-
-
-def _linear(n_in: int, n_out: int, dtype, device) -> FusedLinear:
-    """Zero weights at sizes padded for the GEMM; checkpoint rows and columns are copied into place."""
-    m = FusedLinear(_up(n_in, 8), _up(n_out, 8), bias=False, dtype=dtype, device="meta")
-    m.weight = _zeros(_up(n_out, 8), _up(n_in, 8), dtype=dtype, device=device)
-    return m
+from .config import LayerConfig, TavulixConfig
 
 
 class TavulixLayer(nn.Module):
@@ -61,9 +50,7 @@ class TavulixLayer(nn.Module):
         return ScoreRule(m.scale, m.softcap, self.r1, self.r2, self.sink, m.window, m.keep_first, self.bounded)
 
 
-class TavulixDecoder(nn.Module):
-    uses_seq_table = True            # the runner hands a SeqTable with every batch
-
+class TavulixDecoder(PackedDecoder):
     def __init__(self, cfg: TavulixConfig, dtype=torch.bfloat16, device=None):
         super().__init__()
         self.cfg, self.dtype_ = cfg, dtype
@@ -126,8 +113,7 @@ class TavulixDecoder(nn.Module):
         return lm.logit_softcap(self.lm_head(hidden), self.cfg.logit_softcap, self.cfg.vocab_size)
 
     # ------------------------------------------------------------------ weights
-    def _targets(self) -> dict:
-        """Checkpoint name -> list of (destination view, selection of the checkpoint tensor that goes there)."""
+    def targets(self) -> dict:
         cfg, D = self.cfg, self.cfg.hidden_size
         whole = slice(None)
         t = {"embed": [(self.embed_tokens[:, :D], whole)], "pos": [(self.pos_table[:, :D], whole)],
@@ -161,27 +147,9 @@ class TavulixDecoder(nn.Module):
                 t[p + "mlp.act"] = [(layer.act, whole)]
         return t
 
-    @torch.no_grad()
-    def load_weights(self, weights) -> set:
-        """Copies (name, tensor) pairs into the packed layout; a missing or misshapen tensor is an error."""
-        targets, shapes, loaded = self._targets(), self.cfg.tensor_shapes(), set()
-        for name, w in weights:
-            if name not in targets:
-                continue
-            if tuple(w.shape) != shapes[name]:
-                raise ValueError(f"{name}: shape {tuple(w.shape)}, expected {shapes[name]}")
-            w = w.reshape(1) if w.dim() == 0 else w
-            if any(sel != slice(None) for _, sel in targets[name]):
-                w = w.to(targets[name][0][0].device)        # one transfer, then copies per head
-            for dst, sel in targets[name]:
-                dst.copy_(w[sel].to(dst.dtype))
-            loaded.add(name)
+    def weights_loaded(self) -> None:
         for layer in self.layers:
             layer.bounded = bounded_scores(layer.lc.mixer.softcap, layer.r1, layer.r2)
-        missing = sorted(set(targets) - loaded)
-        if missing:
-            raise ValueError(f"checkpoint lacks {len(missing)} tensors: {', '.join(missing[:8])}")
-        return loaded
 
     def random_weights(self, seed: int | None = None):
         """(name, tensor) pairs of a random checkpoint (runs without weights)."""

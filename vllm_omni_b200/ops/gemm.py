@@ -15,7 +15,7 @@ import torch.nn.functional as F
 
 from . import _native as nv
 
-ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2}
+ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3}
 
 PAIR_BN = 512   # force_bn value that selects the CTA-pair (cta_group::2, 256 x 256 tile) kernel
 
@@ -36,6 +36,8 @@ def linear_reference(x, w, bias=None, act=None, residual=None, gate=None):
         y = F.gelu(y, approximate="tanh")
     elif act == "silu":
         y = F.silu(y)
+    elif act == "relu2":
+        y = F.relu(y).square()
     if gate is not None:
         B = gate.shape[0]
         shp = y.shape
@@ -78,8 +80,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, a
             return out
         return y
     if x.dtype == torch.float32 and w.dtype == torch.float32:
-        assert act is None and residual is None and gate is None and scatter is None and row_scatter is None
-        return _linear_f32(x, w, bias, out)
+        assert act in (None, "relu2") and residual is None and gate is None and scatter is None and row_scatter is None
+        return _linear_f32(x, w, bias, out, act)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16, "tcgen05 GEMM path is bf16"
     K = x.shape[-1]
     N = w.shape[0]
@@ -133,8 +135,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, a
     return None if to_peers else out
 
 
-def _linear_f32(x, w, bias, out):
-    """Exact mode: true fp32 products on the CUDA cores (csrc/gemm_f32.cu); plain ``x @ w.T (+ bias)`` only."""
+def _linear_f32(x, w, bias, out, act=None):
+    """Exact mode: true fp32 products on the CUDA cores (csrc/gemm_f32.cu); ``act(x @ w.T (+ bias))`` only."""
     K, N = x.shape[-1], w.shape[0]
     x2 = x.reshape(-1, K)
     if x2.stride(-1) != 1:
@@ -143,10 +145,19 @@ def _linear_f32(x, w, bias, out):
         out = torch.empty(*x.shape[:-1], N, dtype=x.dtype, device=x.device)
     o2 = out.view(-1, N)
     assert w.stride(-1) == 1 and o2.stride(-1) == 1
-    rc = nv.lib("gemm_f32").omni_gemm_f32(nv.ptr(x2), ctypes.c_long(x2.stride(0)), nv.ptr(w), ctypes.c_long(w.stride(0)),
-                                          nv.ptr(o2), ctypes.c_long(o2.stride(0)), ctypes.c_int(x2.shape[0]),
-                                          ctypes.c_int(N), ctypes.c_int(K), nv.ptr(bias), nv.stream_ptr())
-    nv.check_rc(rc, "omni_gemm_f32")
+    batched_f32(x2, w, o2, bias=bias, act=act)
+    return out
+
+
+def batched_f32(a, w, out, *, bias=None, act=None, batch: int = 1, a_stride: int = 0, w_stride: int = 0, c_stride: int = 0,
+                bias_stride: int = 0):
+    """out[b] = act(a[b] @ w[b].T + bias[b]) in true fp32: 2-D operands of batch 0, element strides between batches."""
+    rc = nv.lib("gemm_f32").omni_gemm_f32_batched(
+        nv.ptr(a), ctypes.c_long(a.stride(0)), nv.ptr(w), ctypes.c_long(w.stride(0)), nv.ptr(out), ctypes.c_long(out.stride(0)),
+        ctypes.c_int(a.shape[0]), ctypes.c_int(w.shape[0]), ctypes.c_int(w.shape[1]), nv.ptr(bias), ctypes.c_int(ACT[act]),
+        ctypes.c_int(batch), ctypes.c_long(a_stride), ctypes.c_long(w_stride), ctypes.c_long(c_stride), ctypes.c_long(bias_stride),
+        nv.stream_ptr())
+    nv.check_rc(rc, "omni_gemm_f32_batched")
     return out
 
 

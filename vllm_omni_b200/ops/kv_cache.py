@@ -60,6 +60,15 @@ def kv_gather(k_cache, v_cache, block_table, T, out_k=None, out_v=None):
     return out_k, out_v
 
 
+def rows_gather(k_cache, block_table, T):
+    """Pages of one sequence that hold one tensor (or none) -> contiguous [T, Hkv, D]."""
+    if not k_cache.numel():
+        return k_cache.new_empty(T, *k_cache.shape[2:])
+    bs = k_cache.shape[1]
+    j = torch.arange(T, device=k_cache.device)
+    return k_cache.view(-1, *k_cache.shape[2:])[block_table.long()[j // bs] * bs + j % bs]
+
+
 _scratch: dict = {}
 
 

@@ -10,12 +10,13 @@ semantics of vllm_omni/model_executor/models/qwen3_omni/qwen3_moe.py).
 from __future__ import annotations
 
 import ctypes
+from dataclasses import dataclass
 
 import torch
 import torch.nn.functional as F
 
 from . import _native as nv
-from . import fused
+from . import fused, gemm
 
 c_int, c_long = ctypes.c_int, ctypes.c_long
 
@@ -110,6 +111,93 @@ class MoEWorkspace:
         return self
 
 
+@dataclass
+class ExpertRows:
+    """Results of the chosen experts before their weighted sum: pair p (token p // k, choice p % k) is row
+    ``row_of_pair[p]`` of ``y`` (row p without it); weights fp32 [T, k]."""
+    y: torch.Tensor
+    row_of_pair: torch.Tensor | None
+    weights: torch.Tensor
+
+
+def _grouped(ws, a, lda, w, c, ldc, n, kk, tile_expert, act=0):
+    """c = act(a @ w[e].T) over the workspace's expert tiles."""
+    g, st, status = nv.lib("gemm_sm100"), nv.stream_ptr(), nv.status_word(a.device)
+    if ws.padded:
+        nv.check_rc(g.omni_gemm_bf16_grouped(nv.ptr(a), c_int(lda), nv.ptr(w), c_int(w.shape[0]), nv.ptr(c), c_int(ldc),
+                                             c_int(ws.max_rows), c_int(n), c_int(kk), nv.ptr(tile_expert), c_int(act), c_int(0),
+                                             nv.ptr(status), st), "omni_gemm_bf16_grouped")
+    else:
+        nv.check_rc(g.omni_gemm_bf16_grouped_compact(nv.ptr(a), c_int(lda), nv.ptr(w), c_int(w.shape[0]), nv.ptr(c), c_int(ldc),
+                                                     c_int(ws.max_rows), c_int(n), c_int(kk), nv.ptr(tile_expert),
+                                                     nv.ptr(ws.tile_row0), nv.ptr(ws.tile_rows), c_int(ws.max_tiles),
+                                                     c_int(act), c_int(0), nv.ptr(status), st),
+                    "omni_gemm_bf16_grouped_compact")
+
+
+def _plan_and_dispatch(ws, x, E, e_lo, e_hi, k):
+    """Rows of every expert side by side: ``ws.xp``, tile tables and ``ws.row_of_pair`` from ``ws.ids``."""
+    lib, st = nv.lib("moe"), nv.stream_ptr()
+    T, D = x.shape
+    if nv.bounds_check_enabled():
+        # checked build: expert ids outside [0, E) and rows outside the expert-major buffers are reported, not used
+        lib.omni_moe_set_bounds(c_long(ws.xp.shape[0]), nv.ptr(nv.status_word(x.device)))
+    if ws.padded:
+        nv.check_rc(lib.omni_moe_plan(nv.ptr(ws.ids), c_int(T * k), c_int(E), c_int(e_lo), c_int(e_hi),
+                                      c_int(ws.max_tiles), nv.ptr(ws.row_of_pair), nv.ptr(ws.tile_expert),
+                                      nv.ptr(ws.offsets), nv.ptr(ws.n_rows), st), "omni_moe_plan")
+    else:
+        nv.check_rc(lib.omni_moe_plan_compact(nv.ptr(ws.ids), c_int(T * k), c_int(E), c_int(e_lo), c_int(e_hi),
+                                              c_int(ws.max_tiles), nv.ptr(ws.row_of_pair), nv.ptr(ws.tile_expert),
+                                              nv.ptr(ws.tile_row0), nv.ptr(ws.tile_rows), nv.ptr(ws.n_rows), st),
+                    "omni_moe_plan_compact")
+    nv.check_rc(lib.omni_moe_dispatch(nv.ptr(x), c_long(x.stride(0)), nv.ptr(ws.row_of_pair), c_int(T * k), c_int(k),
+                                      c_int(D), nv.ptr(ws.xp), st), "omni_moe_dispatch")
+
+
+def expert_rows(x, router_w, router_b, experts: int, k: int, up, down, act: str, ws: MoEWorkspace | None = None) -> ExpertRows:
+    """Two-matrix experts behind a router with fp32 logits: the k largest of ``router_w x + router_b`` (rows past
+    ``experts`` are padding), weighted by the softmax among themselves; y = down[e] act(up[e] x) per choice.
+
+    x [T, D]; router_w [>= E, D]; router_b fp32; up [E, F, D]; down [E, D, F].  The weighted sum is the caller's
+    (ops/stream.py add_expert_rows_ fuses it with the residual add)."""
+    assert act == "relu2"
+    T, D = x.shape
+    Fd = down.shape[2]
+    if not x.is_cuda:
+        logits = F.linear(x.float(), router_w.float(), router_b)[:, :experts]
+        val, ids = torch.topk(logits, k, dim=-1)
+        y = torch.empty(T * k, D)
+        for e in range(experts):
+            hit = (ids.reshape(-1) == e).nonzero()[:, 0]
+            if hit.numel():
+                h = F.relu(F.linear(x[hit // k].float(), up[e].float())).square().to(x.dtype).float()
+                y[hit] = F.linear(h, down[e].float())
+        return ExpertRows(y.to(x.dtype), None, torch.softmax(val, -1))
+    assert x.stride(1) == 1 and router_b.dtype == torch.float32 and up.is_contiguous() and down.is_contiguous()
+    lib, st = nv.lib("moe"), nv.stream_ptr()
+    if x.dtype == torch.float32:
+        logits = gemm.linear(x, router_w, router_b)
+        ids = torch.empty(T, k, dtype=torch.int32, device=x.device)
+        w = torch.empty(T, k, dtype=torch.float32, device=x.device)
+        nv.check_rc(lib.omni_moe_topk(nv.ptr(logits), c_long(logits.stride(0)), c_int(T), c_int(experts), c_int(k), nv.ptr(ids),
+                                      nv.ptr(w), st), "omni_moe_topk")
+        h, y = (torch.empty(T * k, n, dtype=x.dtype, device=x.device) for n in (Fd, D))
+        for a, per, m, out, relu in ((x, k, up, h, 1), (h, 1, down, y, 0)):
+            nv.check_rc(lib.omni_moe_pairs_f32(nv.ptr(a), c_long(a.stride(0)), c_int(per), nv.ptr(ids), nv.ptr(m), c_int(experts),
+                                               nv.ptr(out), c_long(out.stride(0)), c_long(T * k), c_int(m.shape[1]),
+                                               c_int(m.shape[2]), c_int(relu), st), "omni_moe_pairs_f32")
+        return ExpertRows(y, None, w)
+    ws = (ws or MoEWorkspace()).get(T, k, experts, D, Fd, x.device, x.dtype)
+    nv.check_rc(lib.omni_moe_router(nv.ptr(x), c_long(x.stride(0)), nv.ptr(router_w), c_long(router_w.stride(0)), nv.ptr(router_b),
+                                    c_int(T), c_int(D), c_int(experts), c_int(router_w.shape[0]), c_int(k), nv.ptr(ws.ids),
+                                    nv.ptr(ws.weights), st), "omni_moe_router")
+    _plan_and_dispatch(ws, x, experts, 0, experts, k)
+    _grouped(ws, ws.xp, D, up, ws.h, Fd, Fd, D, ws.tile_expert, gemm.ACT[act])
+    _grouped(ws, ws.h, Fd, down, ws.y, D, D, Fd, ws.tile_expert)
+    return ExpertRows(ws.y, ws.row_of_pair, ws.weights)
+
+
 def moe_forward(x, router_logits, w13, w2, k, renorm=True, e_lo=0, e_hi=None, ws: MoEWorkspace | None = None,
                 residual=None, out=None, scatter=None):
     """x [T, D] bf16, router_logits [T, E] bf16, w13 [E_local, 2F, D], w2 [E_local, D, F] (the
@@ -145,42 +233,15 @@ def moe_forward(x, router_logits, w13, w2, k, renorm=True, e_lo=0, e_hi=None, ws
     assert router_logits.dtype == torch.bfloat16 and router_logits.stride(1) == 1
     nv.check_rc(lib.omni_moe_route(nv.ptr(router_logits), c_int(router_logits.stride(0)), c_int(T), c_int(E), c_int(k),
                                    c_int(1 if renorm else 0), nv.ptr(ws.ids), nv.ptr(ws.weights), st), "omni_moe_route")
-    g = nv.lib("gemm_sm100")
-    status = nv.status_word(x.device)
-    El = w13.shape[0]
-    if nv.bounds_check_enabled():
-        # checked build: expert ids outside [0, E) and rows outside the expert-major buffers are reported, not used
-        lib.omni_moe_set_bounds(c_long(ws.xp.shape[0]), nv.ptr(status))
-    if ws.padded:
-        nv.check_rc(lib.omni_moe_plan(nv.ptr(ws.ids), c_int(T * k), c_int(E), c_int(e_lo), c_int(e_hi),
-                                      c_int(ws.max_tiles), nv.ptr(ws.row_of_pair), nv.ptr(ws.tile_expert),
-                                      nv.ptr(ws.offsets), nv.ptr(ws.n_rows), st), "omni_moe_plan")
-    else:
-        nv.check_rc(lib.omni_moe_plan_compact(nv.ptr(ws.ids), c_int(T * k), c_int(E), c_int(e_lo), c_int(e_hi),
-                                              c_int(ws.max_tiles), nv.ptr(ws.row_of_pair), nv.ptr(ws.tile_expert),
-                                              nv.ptr(ws.tile_row0), nv.ptr(ws.tile_rows), nv.ptr(ws.n_rows), st),
-                    "omni_moe_plan_compact")
-    nv.check_rc(lib.omni_moe_dispatch(nv.ptr(x), c_long(x.stride(0)), nv.ptr(ws.row_of_pair), c_int(T * k), c_int(k),
-                                      c_int(D), nv.ptr(ws.xp), st), "omni_moe_dispatch")
+    _plan_and_dispatch(ws, x, E, e_lo, e_hi, k)
     # tile_expert holds GLOBAL expert ids; the local weight tensors start at e_lo
     te = ws.tile_expert
     if e_lo:
         te = torch.where(te >= 0, te - e_lo, te)
 
-    def grouped(a, lda, w, c, ldc, n, kk):
-        if ws.padded:
-            nv.check_rc(g.omni_gemm_bf16_grouped(nv.ptr(a), c_int(lda), nv.ptr(w), c_int(El), nv.ptr(c), c_int(ldc),
-                                                 c_int(ws.max_rows), c_int(n), c_int(kk), nv.ptr(te), c_int(0), c_int(0),
-                                                 nv.ptr(status), st), "omni_gemm_bf16_grouped")
-        else:
-            nv.check_rc(g.omni_gemm_bf16_grouped_compact(nv.ptr(a), c_int(lda), nv.ptr(w), c_int(El), nv.ptr(c), c_int(ldc),
-                                                         c_int(ws.max_rows), c_int(n), c_int(kk), nv.ptr(te),
-                                                         nv.ptr(ws.tile_row0), nv.ptr(ws.tile_rows), c_int(ws.max_tiles),
-                                                         c_int(0), c_int(0), nv.ptr(status), st),
-                        "omni_gemm_bf16_grouped_compact")
-    grouped(ws.xp, D, w13, ws.h13, 2 * Fd, 2 * Fd, D)
+    _grouped(ws, ws.xp, D, w13, ws.h13, 2 * Fd, 2 * Fd, D, te)
     fused.silu_mul(ws.h13, out=ws.h)
-    grouped(ws.h, Fd, w2, ws.y, D, D, Fd)
+    _grouped(ws, ws.h, Fd, w2, ws.y, D, D, Fd, te)
     if scatter is not None:
         per, ptrs = scatter
         arr = (ctypes.c_void_p * len(ptrs))(*ptrs)

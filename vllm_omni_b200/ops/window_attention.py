@@ -25,7 +25,8 @@ class _WinAttn(ctypes.Structure):
                 ("r2", c_void_p), ("sink", c_void_p), ("scale", c_float), ("cap", c_float), ("bounded", c_int), ("window", c_int),
                 ("keep_first", c_int), ("T", c_int), ("H", c_int), ("G", c_int), ("dp", c_int), ("vp", c_int),
                 ("num_seqs", c_int), ("num_blocks", c_int), ("block_size", c_int), ("splits", c_int),
-                ("part_o", c_void_p), ("part_ml", c_void_p), ("status", c_void_p)]
+                ("part_o", c_void_p), ("part_ml", c_void_p), ("status", c_void_p), ("k_ts", c_long), ("v_ts", c_long),
+                ("k_shared", c_void_p), ("ks_ts", c_long), ("dp_u", c_int), ("key_start", c_void_p), ("key_rows", c_long)]
 
 
 @dataclass
@@ -107,6 +108,7 @@ def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None,
     a.scale, a.cap = rule.scale, rule.softcap or 0.0
     a.bounded, a.window, a.keep_first = int(rule.bounded), rule.window or 0, rule.keep_first
     a.T, a.H, a.G, a.dp, a.vp, a.num_seqs, a.num_blocks, a.block_size = T, H, G, dp, vp, seqs.n_seqs, nb, bs
+    a.k_ts, a.v_ts, a.dp_u = G * dp, G * vp, dp
     a.splits = 1
     a.status = P(nv.status_word(q.device))
     bf = q.dtype == torch.bfloat16
