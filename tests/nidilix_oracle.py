@@ -56,21 +56,26 @@ def causal_softmax(s):
     return e / e.sum(-1, keepdim=True)
 
 
+def attend_latent(q_u, q_r, c, kr, uk, uv, scale):
+    """q_u [T, H, d], q_r [T, H, r] (rotated), c [T, rank], kr [T, r] (rotated), uk [H, d, rank], uv [H, dv, rank]
+    -> [T, H, dv], one head at a time."""
+    outs = []
+    for n in range(q_u.shape[1]):
+        s = (q_u[:, n] @ (c @ uk[n].T).T + q_r[:, n] @ kr.T) * scale
+        outs.append(causal_softmax(s) @ (c @ uv[n].T))
+    return torch.stack(outs, dim=1)
+
+
 def latent_attention(h, latent, W, p, m):
     """h [T, D]; latent: pair from ``latent_of`` (the layer's own or another layer's); m: the mixer's entry."""
     c, kr = latent
     T, H, d, r, dv = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"]
     pos = torch.arange(T, dtype=h.dtype)
     q = (h @ W[p + "q"].T).reshape(T, H, d + r)
+    q_r = rotate_pairs(q[:, :, d:], pos, m["rot"]["base"])
+    o = attend_latent(q[:, :, :d], q_r, c, kr, W[p + "uk"].reshape(H, d, -1), W[p + "uv"].reshape(H, dv, -1), m["scale"])
     gate = torch.sigmoid(h @ W[p + "g"].T)
-    outs = []
-    for n in range(H):
-        k_n = c @ W[p + "uk"][n * d:(n + 1) * d].T
-        v_n = c @ W[p + "uv"][n * dv:(n + 1) * dv].T
-        q_rot = rotate_pairs(q[:, n, d:], pos, m["rot"]["base"])
-        s = (q[:, n, :d] @ k_n.T + q_rot @ kr.T) * m["scale"]
-        outs.append((causal_softmax(s) @ v_n) * gate[:, n:n + 1])
-    return torch.cat(outs, dim=1) @ W[p + "o"].T
+    return (o * gate[:, :, None]).reshape(T, H * dv) @ W[p + "o"].T
 
 
 def causal_conv(u, w, b):

@@ -8,15 +8,13 @@ import pytest
 import torch
 
 import tavulix_oracle as O
+from lm_harness import check, folder_fixture, modes, replay, tokens
 from vllm_omni_b200.entrypoints.omni_llm import OmniLLM
 from vllm_omni_b200.entrypoints.trace import TraceReplay
 from vllm_omni_b200.inputs.data import SamplingParams
 from vllm_omni_b200.models.tavulix import TavulixConfig, tiny_config_dict
-from vllm_omni_b200.utils.safetensors_reader import save_safetensors
 
-MODES = [pytest.param(("cpu", "float32", 1e-4), id="cpu"),
-         pytest.param(("cuda", "float32", 1e-4), id="fp32", marks=pytest.mark.gpu),
-         pytest.param(("cuda", "bfloat16", 0.04), id="bf16", marks=pytest.mark.gpu)]
+MODES = modes(0.04)
 
 
 def mixer(heads=6, kv=2, dim=40, vdim=24, conv=3, size=30, keep=4, cap=9.0, mix=True, scale=0.3):
@@ -68,62 +66,7 @@ def weights(cfg, seed=0):
     return out
 
 
-_folders: dict = {}
-
-
-@pytest.fixture(scope="module")
-def folder(tmp_path_factory):
-    def make(name):
-        if name not in _folders:
-            d = tmp_path_factory.mktemp(name)
-            cfg = CONFIGS[name]
-            (d / "config.json").write_text(json.dumps(cfg))
-            W = weights(cfg)
-            save_safetensors(W, str(d / "model.safetensors"))
-            _folders[name] = (str(d), cfg, W, {})
-        return _folders[name]
-    yield make
-    _folders.clear()
-
-
-def tokens(cfg, n, seed=1):
-    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-def expected(f, ids):
-    d, cfg, W, memo = f
-    key = tuple(ids)
-    if key not in memo:
-        memo[key] = O.forward(cfg, W, ids)
-    return memo[key]
-
-
-def check(got, want, tol):
-    got, want = got.double(), want.double()
-    err = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-    assert torch.isfinite(got).all() and got.shape == want.shape
-    assert err.max() < tol, f"row {int(err.argmax())}: {float(err.max()):.4g}"
-
-
-def replay(f, mode, seqs, rounds, max_tokens=None):
-    """Runs ``rounds`` (lists of {request: tokens of this step}); returns every row's logits per request."""
-    dev, dtype, _ = mode
-    room = max_tokens or sum((len(s) + 63) // 64 * 64 for s in seqs.values())
-    rp = TraceReplay(f[0], dtype, room, device=dev)
-    at, out = {r: 0 for r in seqs}, {r: [] for r in seqs}
-    for step in rounds:
-        entries = [{"id": r, "tokens": seqs[r][at[r]:at[r] + n], "want": list(range(n))} for r, n in step.items()]
-        for r, n in step.items():
-            at[r] += n
-        end = [r for r in step if at[r] == len(seqs[r])]
-        lg, o = rp.step(entries, end), 0
-        for r, n in step.items():
-            out[r].append(lg[o:o + n])
-            o += n
-    kv = rp.engine.kv
-    assert kv.pool.num_free == kv.pool.num_blocks and not rp.engine.scheduler.running
-    assert kv.state is None or kv.state.num_free == kv.state.num_slots
-    return {r: torch.cat(v) for r, v in out.items()}
+folder = folder_fixture(CONFIGS, weights, O.forward)
 
 
 # ----------------------------------------------------------------------------- prompts and portions
@@ -131,16 +74,16 @@ def replay(f, mode, seqs, rounds, max_tokens=None):
 @pytest.mark.parametrize("name", sorted(CONFIGS))
 def test_whole_prompt(folder, mode, name):
     f = folder(name)
-    ids = tokens(f[1], 150)
-    check(replay(f, mode, {"a": ids}, [{"a": 150}])["a"], expected(f, ids), mode[2])
+    ids = tokens(f.cfg, 150)
+    check(replay(f, mode, {"a": ids}, [{"a": 150}])["a"], f.expected(ids), mode[2])
 
 
 @pytest.mark.parametrize("mode", MODES)
 @pytest.mark.parametrize("name", sorted(CONFIGS))
 def test_token_by_token(folder, mode, name):
     f = folder(name)
-    ids = tokens(f[1], 90)
-    check(replay(f, mode, {"a": ids}, [{"a": 1}] * 90)["a"], expected(f, ids), mode[2])
+    ids = tokens(f.cfg, 90)
+    check(replay(f, mode, {"a": ids}, [{"a": 1}] * 90)["a"], f.expected(ids), mode[2])
 
 
 CUTS = {"pairs": [2] * 75, "threes": [3] * 50, "page_and_more": [16, 17, 15, 1, 31, 33, 37], "growing": [2, 3, 5, 8, 13, 21, 34, 64],
@@ -151,9 +94,9 @@ CUTS = {"pairs": [2] * 75, "threes": [3] * 50, "page_and_more": [16, 17, 15, 1, 
 @pytest.mark.parametrize("cut", sorted(CUTS))
 def test_portions(folder, mode, cut):
     f = folder("base")
-    ids = tokens(f[1], 150)
+    ids = tokens(f.cfg, 150)
     assert sum(CUTS[cut]) == 150
-    check(replay(f, mode, {"a": ids}, [{"a": n} for n in CUTS[cut]])["a"], expected(f, ids), mode[2])
+    check(replay(f, mode, {"a": ids}, [{"a": n} for n in CUTS[cut]])["a"], f.expected(ids), mode[2])
 
 
 @pytest.mark.parametrize("mode", MODES)
@@ -162,77 +105,70 @@ def test_mixed_batches_reuse_pages_and_slots(folder, mode):
     requests that sit out steps, pages and slots handed on with stale contents in them."""
     f = folder("base")
     lens = {"a": 130, "b": 1, "c": 70, "d": 33, "e": 64, "f": 97, "g": 2}
-    seqs = {r: tokens(f[1], n, seed=10 + i) for i, (r, n) in enumerate(lens.items())}
+    seqs = {r: tokens(f.cfg, n, seed=10 + i) for i, (r, n) in enumerate(lens.items())}
     rounds = [{"a": 40, "b": 1, "c": 2}, {"c": 17, "a": 1}, {"d": 2, "a": 1, "c": 1, "e": 30}, {"d": 3, "e": 1}, {"a": 50, "d": 28, "e": 1},
               {"c": 50, "e": 32}, {"f": 64, "a": 1, "g": 2}, {"a": 37, "f": 31}, {"f": 1}, {"f": 1}]
     got = replay(f, mode, seqs, rounds, max_tokens=192 + 128 + 64 + 64)
     for r, ids in seqs.items():
-        check(got[r], expected(f, ids), mode[2])
+        check(got[r], f.expected(ids), mode[2])
 
 
 @pytest.mark.parametrize("mode", MODES)
 def test_long_decode(folder, mode):
     """Windows of 30, 50 and 17 tokens pass several times over decoded tokens."""
     f = folder("base")
-    ids = tokens(f[1], 260, seed=4)
-    check(replay(f, mode, {"a": ids}, [{"a": 3}] + [{"a": 1}] * 257)["a"], expected(f, ids), mode[2])
+    ids = tokens(f.cfg, 260, seed=4)
+    check(replay(f, mode, {"a": ids}, [{"a": 3}] + [{"a": 1}] * 257)["a"], f.expected(ids), mode[2])
 
 
 @pytest.mark.parametrize("mode", MODES)
 def test_first_tokens(folder, mode):
     f = folder("base")
-    ids = tokens(f[1], 6, seed=5)
+    ids = tokens(f.cfg, 6, seed=5)
     for rounds in ([{"a": 6}], [{"a": 1}] * 6, [{"a": 2}] * 3, [{"a": 1}, {"a": 5}]):
-        check(replay(f, mode, {"a": ids}, rounds)["a"], expected(f, ids), mode[2])
+        check(replay(f, mode, {"a": ids}, rounds)["a"], f.expected(ids), mode[2])
 
 
 @pytest.mark.parametrize("mode", MODES)
 def test_stream_after_every_layer(folder, mode):
     dev, dtype, tol = mode
     f = folder("layers_differ")
-    ids = tokens(f[1], 40)
+    ids = tokens(f.cfg, 40)
     trace = []
-    O.forward(f[1], f[2], ids, trace=trace)
-    rp = TraceReplay(f[0], dtype, 64, device=dev)
+    O.forward(f.cfg, f.weights, ids, trace=trace)
+    rp = TraceReplay(f.path, dtype, 64, device=dev)
     dec, got = rp.llm.model.decoder, {}
     plain = dec.forward
     dec.forward = lambda b, kv, **kw: got.update(r=plain(b, kv, capture_layers=range(9))) or got["r"]
     rp.step([{"id": "a", "tokens": ids, "want": [0]}])
     for i, want in enumerate(trace):
-        x = got["r"][1][i + 1][:, :f[1]["width"]]
+        x = got["r"][1][i + 1][:, :f.cfg["width"]]
         assert x.dtype == torch.float32
         check(x.cpu(), want, tol)
 
 
 # --------------------------------------------------------------------------------- generation
-def greedy(f, prompt, n):
-    ids = list(prompt)
-    for _ in range(n):
-        ids.append(int(O.forward(f[1], f[2], ids)[-1].argmax()))
-    return ids[len(prompt):]
-
-
 @pytest.mark.parametrize("mode", MODES[:2])
 def test_greedy_generation_matches(folder, mode):
     """Through the engine's own scheduler: a prompt longer than the step budget, short ones beside it."""
     f = folder("base")
-    prompts = [tokens(f[1], n, seed=20 + n) for n in (45, 7, 1)]
-    llm = OmniLLM(f[0], dtype=mode[1], device=mode[0], num_gpu_blocks=40, max_num_seqs=3, max_num_batched_tokens=16)
+    prompts = [tokens(f.cfg, n, seed=20 + n) for n in (45, 7, 1)]
+    llm = OmniLLM(f.path, dtype=mode[1], device=mode[0], num_gpu_blocks=40, max_num_seqs=3, max_num_batched_tokens=16)
     outs = llm.generate([{"prompt_token_ids": p} for p in prompts],
                         SamplingParams(temperature=0.0, max_tokens=24, ignore_eos=True, detokenize=False))
     for p, o in zip(prompts, outs):
-        assert list(o.outputs[0].token_ids) == greedy(f, p, 24)
+        assert list(o.outputs[0].token_ids) == f.greedy(p, 24)
     assert llm.engine.kv.state.num_free == 3
 
 
 def test_preemption_recomputes_the_state(folder):
     """A pool that forces preemption, and fewer state slots than requests: the same tokens."""
     f = folder("base")
-    prompts = [{"prompt_token_ids": tokens(f[1], n, seed=40 + n)} for n in (20, 9, 14, 5)]
+    prompts = [{"prompt_token_ids": tokens(f.cfg, n, seed=40 + n)} for n in (20, 9, 14, 5)]
     sp = SamplingParams(temperature=0.0, max_tokens=30, ignore_eos=True, detokenize=False)
 
     def run(blocks, seqs):
-        llm = OmniLLM(f[0], dtype="float32", device="cpu", num_gpu_blocks=blocks, block_size=8, max_num_seqs=seqs)
+        llm = OmniLLM(f.path, dtype="float32", device="cpu", num_gpu_blocks=blocks, block_size=8, max_num_seqs=seqs)
         out = [list(o.outputs[0].token_ids) for o in llm.generate(prompts, sp)]
         assert llm.engine.kv.pool.num_free == blocks and llm.engine.kv.state.num_free == seqs
         return out
@@ -244,12 +180,12 @@ def test_preemption_recomputes_the_state(folder):
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
 def test_decode_graph_equals_eager(folder, dtype, monkeypatch):
     f = folder("base")
-    prompts = [{"prompt_token_ids": tokens(f[1], n, seed=60 + n)} for n in (50, 3, 30)]
+    prompts = [{"prompt_token_ids": tokens(f.cfg, n, seed=60 + n)} for n in (50, 3, 30)]
     sp = SamplingParams(temperature=0.0, max_tokens=40, ignore_eos=True, detokenize=False)
 
     def run(graph):
         monkeypatch.setenv("OMNI_AR_CUDA_GRAPH", graph)
-        llm = OmniLLM(f[0], dtype=dtype, num_gpu_blocks=64, max_num_seqs=3)
+        llm = OmniLLM(f.path, dtype=dtype, num_gpu_blocks=64, max_num_seqs=3)
         out = [list(o.outputs[0].token_ids) for o in llm.generate(prompts, sp)]
         assert (llm.engine.runner.graph_runner.replays > 30) if graph == "1" else llm.engine.runner.graph_runner is None
         return out
@@ -264,10 +200,10 @@ def test_decode_buckets_on_cpu(folder, monkeypatch):
     """The static-buffer step a graph replays, with padding rows that write neither pages nor state."""
     f = folder("base")
     monkeypatch.setenv("OMNI_AR_CUDA_GRAPH", "1")
-    ids = {r: tokens(f[1], 30, seed=i) for i, r in enumerate("abc")}
+    ids = {r: tokens(f.cfg, 30, seed=i) for i, r in enumerate("abc")}
     got = replay(f, ("cpu", "float32", 0), ids, [{"a": 10, "b": 12, "c": 11}] + [{"a": 1, "b": 1, "c": 1}] * 18 + [{"a": 2, "c": 1}])
     for r in "ac":
-        check(got[r], expected(f, ids[r]), 1e-4)
+        check(got[r], f.expected(ids[r]), 1e-4)
 
 
 def test_length_limit(folder):
@@ -285,41 +221,41 @@ def test_omni_serves_the_folder(folder):
     """The public entry point picks the model by its config.json and runs it as one text stage."""
     from vllm_omni_b200.entrypoints.omni import Omni
     f = folder("base")
-    p = tokens(f[1], 12, seed=3)
-    with Omni(f[0], dtype="float32", device="cpu", num_gpu_blocks=32) as omni:
+    p = tokens(f.cfg, 12, seed=3)
+    with Omni(f.path, dtype="float32", device="cpu", num_gpu_blocks=32) as omni:
         out = omni.generate({"prompt_token_ids": p}, SamplingParams(temperature=0.0, max_tokens=8, ignore_eos=True, detokenize=False))[0]
     assert list(out.request_output[0].outputs[0].token_ids if isinstance(out.request_output, list)
-                else out.request_output.outputs[0].token_ids) == greedy(f, p, 8)
+                else out.request_output.outputs[0].token_ids) == f.greedy(p, 8)
 
 
 # ------------------------------------------------------------------------------------- replay
 def test_replay_program(folder, tmp_path):
     from vllm_omni_b200.entrypoints import trace
     f = folder("base")
-    ids = tokens(f[1], 20)
+    ids = tokens(f.cfg, 20)
     steps = [{"step": 0, "entries": [{"id": "a", "tokens": ids[:9], "want": []}], "end": []},
              {"step": 1, "entries": [{"id": "a", "tokens": ids[9:], "want": [0, 10]}, {"id": "b", "tokens": ids[:1], "want": [0]}],
               "end": ["a"]},
              {"step": 2, "entries": [], "end": ["b"]}]
-    args = trace.make_parser().parse_args(["--model", f[0], "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "128"])
+    args = trace.make_parser().parse_args(["--model", f.path, "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "128"])
     out = io.StringIO()
     assert trace.run(args, io.StringIO("\n".join(map(json.dumps, steps)) + "\n"), out) == 0
     assert out.getvalue().split("\n")[:3] == ["done 0", "done 1", "done 2"]
     assert sorted(p.name for p in tmp_path.iterdir()) == ["1.f32"]
     raw = (tmp_path / "1.f32").read_bytes()
     got = torch.tensor(struct.unpack(f"<{len(raw) // 4}f", raw)).view(3, -1)
-    want = expected(f, ids)
+    want = f.expected(ids)
     check(got, want[[9, 19, 0]], 1e-4)
 
 
 def test_replay_refuses_what_does_not_fit(folder):
     f = folder("base")
-    rp = TraceReplay(f[0], "float32", 64, device="cpu")
+    rp = TraceReplay(f.path, "float32", 64, device="cpu")
     with pytest.raises(RuntimeError):
-        rp.step([{"id": "a", "tokens": tokens(f[1], 65), "want": []}])
-    rp = TraceReplay(f[0], "float32", 1024, device="cpu")
+        rp.step([{"id": "a", "tokens": tokens(f.cfg, 65), "want": []}])
+    rp = TraceReplay(f.path, "float32", 1024, device="cpu")
     with pytest.raises(ValueError):
-        rp.step([{"id": "a", "tokens": tokens(f[1], 513), "want": []}])
+        rp.step([{"id": "a", "tokens": tokens(f.cfg, 513), "want": []}])
     with pytest.raises(ValueError):
         rp.step([{"id": "b", "tokens": [1, 2], "want": [2]}])
     with pytest.raises(RuntimeError):

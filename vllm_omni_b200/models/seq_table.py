@@ -140,7 +140,7 @@ class SeqTable:
         buf = torch.tensor(flat, dtype=torch.int32).to(self.q_start.device)
         o1 = round_up4(len(start))
         o2 = o1 + round_up4(len(members))
-        return KeyGroup(buf[:len(start)], buf[o1:o1 + len(members)], len(seqs), at, buf[o2:o2 + 2 * len(items)], len(items),
+        return KeyGroup(buf[:len(start)], buf[o1:o1 + len(members)], len(seqs), at, buf[o2:o2 + 2 * len(items)].view(-1, 2), len(items),
                         rows_per_block)
 
     def time_chunks(self, pick):
