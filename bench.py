@@ -44,6 +44,7 @@ def parse_args():
     ap.add_argument("--workload", default="image", choices=["image", "lm"],
                     help="image: the headline (default); lm: decoder layers of the causal-LM models")
     ap.add_argument("--lm-sizes", default="2048,4096", help="lm workload: widths to run")
+    ap.add_argument("--lm-design", default="tavulix", choices=["tavulix", "nidilix"], help="lm workload: decoder to measure")
     ap.add_argument("--lm-parts", default="steps,kernels", help="lm workload: which tables to fill")
     ap.add_argument("--ref-eager", action="store_true", help="reference arm: skip its regional torch.compile")
     return ap.parse_args()
@@ -146,7 +147,8 @@ def lm_workload(args):
     torch.cuda.set_device(0)
     sampler = ClockSampler(0)
     sampler.start()
-    rec = lm_layers.run(max(args.steps, 7), args.warmup, [int(w) for w in args.lm_sizes.split(",")], args.lm_parts.split(","))
+    rec = lm_layers.run(max(args.steps, 7), args.warmup, [int(w) for w in args.lm_sizes.split(",")], args.lm_parts.split(","),
+                        args.lm_design)
     rec["clocks"] = sampler.stop()
     print(json.dumps(rec), flush=True)
     return 0

@@ -53,11 +53,14 @@ def folder_fixture(configs, weights, oracle):
     return folder
 
 
-def check(got, want, tol):
+def check(got, want, tol, tail: float = 0.0):
+    """Every row's error (relative to the size of all logits) is below ``tol``; with ``tail``, one row in ten (or one) may
+    reach that instead: where a near tie of a router is decided by rounding."""
     got, want = got.double(), want.double()
     err = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
     assert torch.isfinite(got).all() and got.shape == want.shape
-    assert err.max() < tol, f"row {int(err.argmax())}: {float(err.max()):.4g}"
+    assert err.max() < (tail or tol), f"row {int(err.argmax())}: {float(err.max()):.4g}"
+    assert not tail or (err > tol).sum() <= max(1, 0.1 * err.numel()), f"{int((err > tol).sum())} of {err.numel()} rows over {tol}"
 
 
 def replay(f, mode, seqs, rounds, max_tokens=None):

@@ -131,10 +131,9 @@ def route(logits, top):
 def mixture(h, W, p, m):
     ids, wt = route(h @ W[p + "router"].T + W[p + "router.b"], m["router"]["top"])
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for j in range(ids.shape[1]):
-            e = f"{p}e{int(ids[t, j])}"
-            out[t] += wt[t, j] * expert(h[t], W[e + ".up"], W[e + ".down"])
+    for e in range(m["router"]["experts"]):
+        w_e = (wt * (ids == e)).sum(-1, keepdim=True)                 # 0 where the expert is not chosen
+        out += w_e * expert(h, W[f"{p}e{e}.up"], W[f"{p}e{e}.down"])
     if m.get("shared"):
         out = out + expert(h, W[p + "shared.up"], W[p + "shared.down"])
     return out

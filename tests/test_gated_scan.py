@@ -91,7 +91,7 @@ def test_portions_beside_single_tokens(mode, name):
 @pytest.mark.parametrize("mode", MODES)
 @pytest.mark.parametrize("cut", ["whole", "tokens", "runs"])
 def test_several_runs(mode, cut):
-    """Portions of several runs (128 tokens each) that hand their state on, and the same tokens cut otherwise."""
+    """Portions of several runs that hand their state on, and the same tokens cut otherwise."""
     layer = Layer(SIZES["base"], mode[1], mode[0], lam=-6.0)
     d = rows(layer, 700, 3)
     cuts = {"whole": [700], "tokens": [5] + [1] * 20 + [675], "runs": [128, 129, 2, 255, 31, 33, 122]}[cut]
@@ -120,7 +120,7 @@ def test_long_memory(mode):
 def test_many_tokens_and_plain_kernels():
     mode = ("cuda", torch.bfloat16, 0.02)
     layer = Layer((160, 2, 4), mode[1], mode[0])
-    d = rows(layer, 4200, 6)                              # 34 runs of 128
+    d = rows(layer, 4200, 6)                              # many runs
     want = reference(layer, *d)
     compare(run(layer, [d], [{0: 4199}, {0: 1}], mode)[0], want, mode[2])
     compare(run(layer, [d], [{0: 700}, {0: 3500}], mode, impl="plain")[0], want, mode[2])
@@ -151,6 +151,10 @@ def test_padding_rows_write_no_state(mode):
 
 
 def test_run_lengths():
-    for n in (2, 31, 128, 129, 4096, 4097, 9000, 100000):
-        L = R.run_length(n)
-        assert L % 32 == 0 and L >= 128 and -(-n // L) <= 32
+    for lens in ([2], [31], [64], [65, 2], [4096], [4097], [9000], [100000], [1024] * 8, [300000, 5]):
+        for tiles in (1, 16, 40, 200):
+            L = R.run_length(lens, tiles)
+            assert L % 64 == 0 and L >= 64 and -(-max(lens) // L) <= 64
+    t = SeqTable.build([5, 1, 70], [0, 4, 9], [[0]] * 3, None, "cpu")
+    runs, n, several = t.time_runs(0, lambda lens: 64)
+    assert n == 3 and several and runs.tolist() == [[0, 0, 5, 0], [2, 0, 64, 1], [2, 64, 6, 1]]

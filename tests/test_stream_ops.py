@@ -34,7 +34,7 @@ def near(got, want, tol):
 def test_branch_and_next_rows(mode, D, n, kind):
     dev, dtype, tol = mode
     T, eps, mult = 5, 1e-3, 0.37
-    x, y, gain = rnd(T, D, seed=1), 3 * rnd(T, D, seed=2), rnd(D, seed=3)
+    x, y, gain = rnd(T, D, seed=1), 4 * rnd(T, D, seed=2), rnd(D, seed=3)
     for t in (x, y):
         t[:, n:] = 0
     gain[n:] = 0

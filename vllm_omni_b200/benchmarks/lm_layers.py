@@ -98,12 +98,17 @@ def _batch(lens, contexts, dev):
     return b, nxt
 
 
-@torch.no_grad()
 def step_rows(width: int, timer: Timer) -> list[dict]:
+    return step_table(width, timer, _decoders)
+
+
+@torch.no_grad()
+def step_table(width: int, timer: Timer, decoders) -> list[dict]:
+    """Prompt and decode steps of every (name, model) that ``decoders`` yields."""
     from ..engine.graph_runner import DecodeGraphRunner
     dev = torch.device("cuda")
     rows = []
-    for name, model in _decoders(width, dev):
+    for name, model in decoders(width, dev):
         r = {"width": width, "decoder": name}
         for label, lens in (("prefill_1x8192", [8192]), ("prefill_8x1024", [1024] * 8)):
             b, nb = _batch(lens, [0] * len(lens), dev)
@@ -214,16 +219,18 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
     return out
 
 
-def run(steps: int, warmup: int, widths, parts=("steps", "kernels")) -> dict:
+def run(steps: int, warmup: int, widths, parts=("steps", "kernels"), design: str = "tavulix") -> dict:
+    import importlib
     from ..ops import _native as nv
+    tables = importlib.import_module(".lm_nidilix" if design == "nidilix" else ".lm_layers", __package__)
     timer = Timer(steps, warmup)
     n0 = nv.launch_count
-    rec = {"metric": "lm_layers", "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16", "data": "synthetic (random weights)",
+    rec = {"metric": "lm_layers", "design": design, "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16", "data": "synthetic (random weights)",
            "l2": "flushed (256 MB written) before every timed launch", "peaks": dict(zip(("bf16_tflops", "hbm_gbs", "source"), _peaks()))}
     if "kernels" in parts:
-        rec["kernels"] = [r for w in widths for r in kernel_rows(w, timer)]
+        rec["kernels"] = [r for w in widths for r in tables.kernel_rows(w, timer)]
     if "steps" in parts:
-        rec["steps"] = [r for w in widths for r in step_rows(w, timer)]
+        rec["steps"] = [r for w in widths for r in tables.step_rows(w, timer)]
     rec["gpu_launches"] = nv.launch_count - n0
     nv.check_status()
     return rec

@@ -85,8 +85,8 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
 
   const WinAttn& p = w.a;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int g = blockIdx.y;
-  const int seq = p.items[2 * blockIdx.x], off = p.items[2 * blockIdx.x + 1];
+  const int g = blockIdx.x;                                  // heads vary fastest: the items with the most keys start first
+  const int seq = p.items[2 * blockIdx.y], off = p.items[2 * blockIdx.y + 1];
   const int row0 = p.q_start[seq] + off;                     // first batch row of the block
   const int n_seq = p.q_start[seq + 1] - p.q_start[seq];
   const int ctx = p.context[seq];
@@ -519,7 +519,7 @@ static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CU
                           int smem, cudaStream_t st) {
   static unsigned long long prep = 0;
   if (int e = ensure_dynamic_smem((const void*)attn_window_prefill_kernel<CAP, BIAS, BOUNDED>, 227 * 1024 - 512, prep)) return e;
-  attn_window_prefill_kernel<CAP, BIAS, BOUNDED><<<dim3(w.a.n_items, w.a.G), WP_THREADS, smem, st>>>(tq, tk, tv, ts, w);
+  attn_window_prefill_kernel<CAP, BIAS, BOUNDED><<<dim3(w.a.G, w.a.n_items), WP_THREADS, smem, st>>>(tq, tk, tv, ts, w);
   return (int)cudaGetLastError();
 }
 
@@ -537,7 +537,7 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
       p.vp > 128 || p.items == nullptr || p.num_seqs <= 0 || p.num_blocks <= 0 || p.keep_first < 0)
     return RC_BAD_ARG;
   if (p.key_start == nullptr && (p.block_size < 8 || (p.block_size & 7) || 128 % p.block_size)) return RC_BAD_ARG;
-  if (p.G > 65535 || (p.k_ts & 7) || (p.v_ts & 7) || p.dp_u <= 0 || (p.dp_u & 15) || p.dp_u > p.dp) return RC_BAD_ARG;
+  if (p.n_items > 65535 || (p.k_ts & 7) || (p.v_ts & 7) || p.dp_u <= 0 || (p.dp_u & 15) || p.dp_u > p.dp) return RC_BAD_ARG;
   if (p.dp_u < p.dp && (p.k_shared == nullptr || (p.ks_ts & 7))) return RC_BAD_ARG;
   if (p.key_start && (p.key_rows <= 0 || p.key_rows > 0x7fffffffl)) return RC_BAD_ARG;
   if ((p.r1 == nullptr) != (p.r2 == nullptr) || (p.o_rs & 7) || (reinterpret_cast<uintptr_t>(p.out) & 15)) return RC_BAD_ARG;

@@ -25,7 +25,7 @@ struct GatedScan {
   const int* seq_list; int n_list;              // sequences with exactly one row
   const int* runs; int n_runs;                  // (sequence, first row of the portion, rows, first run of the sequence)
   float* sums;                                  // [n_runs, 2, C]: product of a, state from zero
-  float* u; float* z;                           // [T, C], [2, T, C] (plain kernels)
+  void* u; float* z;                            // [T, C] fp32 (plain kernels) or bf16; [2, T, C] (plain kernels)
   void* out;                                    // [T, C]
   int* status;
 };

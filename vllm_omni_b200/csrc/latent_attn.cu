@@ -7,11 +7,11 @@
 //   omni_latent_gather   rows of several sequences from their pages to one buffer (prompts expand them to keys and
 //                        values with one GEMM and run on attn_window_sm100.cu)
 //   omni_head_gemm       one small product per head: queries into the latent space (W_uk^T q) and attention results
-//                        out of it (W_uv o, times the output gate); weights are read once per 64 rows
+//                        out of it (W_uv o, times the output gate); weights are read once per 16 rows
 //   omni_latent_decode   decoded tokens (and rows of short portions): scores and weighted sums directly on the
-//                        latent rows, so a row is read once for all heads.  A block owns 16 or 32 heads of one token
-//                        and a share of its keys; 64-key tiles go through a two-deep cp.async ring, eight warps share
-//                        the score product by (keys, channel half) and the weighted sum by channels
+//                        latent rows, so a row is read once per 16 heads.  A block owns 16 heads of one token and
+//                        a share of its keys; 32-key tiles go through a two-deep cp.async ring, eight warps share the
+//                        score product by (keys, channel quarter) and the weighted sum by channels; two blocks per SM
 //
 // A decode step reads every latent once per group of heads and does little arithmetic on it, so the warp-level
 // products (no operand staging through tensor memory) suffice.
@@ -35,15 +35,18 @@ struct LatentRows {
   int* status;
 };
 
-template <typename T> struct Pair;
-template <> struct Pair<float> {
-  static __device__ __forceinline__ float2 ld(const float* p) { return *reinterpret_cast<const float2*>(p); }
-  static __device__ __forceinline__ void st(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
-};
-template <> struct Pair<bf16> {
-  static __device__ __forceinline__ float2 ld(const bf16* p) { return unpack_bf16(*reinterpret_cast<const uint32_t*>(p)); }
-  static __device__ __forceinline__ void st(bf16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16(a, b); }
-};
+// four rotated pairs: channels 8 i .. 8 i + 7 of a part of 2 `half` rotated channels (padding passes unchanged)
+__device__ __forceinline__ void turn8(float (&v)[8], const float2* turn, int i, int half) {
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    if (i * 4 + e < half) {
+      const float2 a = turn[i * 4 + e];
+      const float x = v[2 * e], y = v[2 * e + 1];
+      v[2 * e] = x * a.x - y * a.y;
+      v[2 * e + 1] = y * a.x + x * a.y;
+    }
+  }
+}
 
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -52,19 +55,23 @@ latent_rows_kernel(const LatentRows p) {
   const long t = blockIdx.x;
   T* row = static_cast<T*>(p.proj) + t * p.ldp;
   const float2* turn = reinterpret_cast<const float2*>(p.turns) + t * (p.rot / 2);
-  const int half = p.rot / 2, hc = p.dim_p + p.rot_p;
-  for (int i = threadIdx.x; i < p.H * half; i += 128) {
-    const int h = i / half, c = i - h * half;
-    T* q = row + h * hc + p.dim_p + 2 * c;
-    const float2 v = Pair<T>::ld(q), a = turn[c];
-    Pair<T>::st(q, v.x * a.x - v.y * a.y, v.y * a.x + v.x * a.y);
+  const int half = p.rot / 2, hc = p.dim_p + p.rot_p, rv = (p.rot + 7) / 8;
+  for (int i = threadIdx.x; i < p.H * rv; i += 128) {
+    const int h = i / rv, c = i - h * rv;
+    T* q = row + h * hc + p.dim_p + 8 * c;
+    float v[8];
+    load8<T>(q, v);
+    turn8(v, turn, c, half);
+    store8<T>(q, v);
   }
   if (p.norm == nullptr) return;
   const T* z = row + p.H * hc;
   float ss[1] = {0.f};
-  for (int i = threadIdx.x; i < p.rank_p / 2; i += 128) {
-    const float2 v = Pair<T>::ld(z + 2 * i);
-    ss[0] = fmaf(v.x, v.x, fmaf(v.y, v.y, ss[0]));
+  for (int i = threadIdx.x; i < p.rank_p / 8; i += 128) {
+    float v[8];
+    load8<T>(z + 8 * i, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss[0] = fmaf(v[e], v[e], ss[0]);
   }
   block_sum<1>(ss, sh);
   const float s = rms_scale(ss[0], p.rank, p.eps);
@@ -72,17 +79,12 @@ latent_rows_kernel(const LatentRows p) {
   if (slot >= p.num_slots && p.status && threadIdx.x == 0) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
   if (slot < 0 || slot >= p.num_slots) return;
   T* page = static_cast<T*>(p.pages) + slot * (p.rank_p + p.rot_p);
-  for (int i = threadIdx.x; i < p.rank_p / 2; i += 128) {
-    const float2 v = Pair<T>::ld(z + 2 * i), g = *reinterpret_cast<const float2*>(p.norm + 2 * i);
-    Pair<T>::st(page + 2 * i, v.x * s * g.x, v.y * s * g.y);
-  }
-  for (int i = threadIdx.x; i < p.rot_p / 2; i += 128) {
-    float2 o = make_float2(0.f, 0.f);
-    if (i < half) {
-      const float2 v = Pair<T>::ld(z + p.rank_p + 2 * i), a = turn[i];
-      o = make_float2(v.x * a.x - v.y * a.y, v.y * a.x + v.x * a.y);
-    }
-    Pair<T>::st(page + p.rank_p + 2 * i, o.x, o.y);
+  for (int i = threadIdx.x; i < (p.rank_p + p.rot_p) / 8; i += 128) {
+    float v[8];
+    load8<T>(z + 8 * i, v);
+    if (8 * i < p.rank_p) scale_gain8(v, s, p.norm, 1, 8 * i);
+    else turn8(v, turn, i - p.rank_p / 8, half);
+    store8<T>(page + 8 * i, v);
   }
 }
 
@@ -122,66 +124,58 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-// A block: 16 MT rows of one head, 64 outputs (16 per warp).  Lane group j of a quad owns channels 8 j .. 8 j + 7 of
-// every 32-channel chunk in both operands (the contraction is permuted alike), so all loads are 16 bytes.
-template <int MT>
+// A block: 16 rows of one head, 32 outputs; its four warps take every fourth 32-channel chunk of the contraction, so
+// that the loads of a short contraction are all in flight at once.  Lane group j of a quad owns channels 8 j .. 8 j + 7
+// of a chunk in both operands (the contraction is permuted alike), so all loads are 16 bytes.
 __global__ void __launch_bounds__(128)
 head_gemm_kernel(const HeadGemm p) {
+  __shared__ __align__(16) float part[4][16][36];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
-  const int h = blockIdx.y, n0 = blockIdx.x * 64 + warp * 16, m0 = blockIdx.z * (16 * MT);
-  if (n0 >= p.N) return;
+  const int h = blockIdx.y, n0 = blockIdx.x * 32, m0 = blockIdx.z * 16;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-  const bf16* a[MT][2];
-  bool live[MT][2];
+  const bf16* a[2];
+  bool live[2];
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      const int r = m0 + m * 16 + u * 8 + g;
-      live[m][u] = r < p.M;
-      int row = live[m][u] ? (p.a_rows ? p.a_rows[r] : r) : 0;
-      row = min(max(row, 0), p.rows_a - 1);
-      a[m][u] = p.A + row * p.a_row + h * p.a_head + j * 8;
-    }
-  const bf16* w0 = p.W + ((long)h * p.N + n0 + g) * p.K + j * 8;
-  const bf16* w1 = w0 + 8l * p.K;
-  float acc[MT][2][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
+  for (int u = 0; u < 2; ++u) {
+    const int r = m0 + u * 8 + g;
+    live[u] = r < p.M;
+    int row = live[u] ? (p.a_rows ? p.a_rows[r] : r) : 0;
+    row = min(max(row, 0), p.rows_a - 1);
+    a[u] = p.A + row * p.a_row + h * p.a_head + j * 8;
+  }
+  const bf16* w = p.W + ((long)h * p.N + n0 + g) * p.K + j * 8;
+  float acc[4][4] = {};
 #pragma unroll 4
-  for (int k = 0; k < p.K; k += 32) {
+  for (int k = warp * 32; k < p.K; k += 128) {
     const bool in = k + j * 8 < p.K;                        // K is a multiple of 16
-    const uint4 b0 = in ? *reinterpret_cast<const uint4*>(w0 + k) : zero;
-    const uint4 b1 = in ? *reinterpret_cast<const uint4*>(w1 + k) : zero;
+    const uint4 x = in && live[0] ? *reinterpret_cast<const uint4*>(a[0] + k) : zero;
+    const uint4 y = in && live[1] ? *reinterpret_cast<const uint4*>(a[1] + k) : zero;
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const uint4 x = in && live[m][0] ? *reinterpret_cast<const uint4*>(a[m][0] + k) : zero;
-      const uint4 y = in && live[m][1] ? *reinterpret_cast<const uint4*>(a[m][1] + k) : zero;
-      mma_bf16(acc[m][0], x.x, y.x, x.y, y.y, b0.x, b0.y);
-      mma_bf16(acc[m][0], x.z, y.z, x.w, y.w, b0.z, b0.w);
-      mma_bf16(acc[m][1], x.x, y.x, x.y, y.y, b1.x, b1.y);
-      mma_bf16(acc[m][1], x.z, y.z, x.w, y.w, b1.z, b1.w);
+    for (int n = 0; n < 4; ++n) {
+      const uint4 b = in && n0 + n * 8 < p.N ? *reinterpret_cast<const uint4*>(w + (long)n * 8 * p.K + k) : zero;
+      mma_bf16(acc[n], x.x, y.x, x.y, y.y, b.x, b.y);
+      mma_bf16(acc[n], x.z, y.z, x.w, y.w, b.z, b.w);
     }
   }
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int n = 0; n < 4; ++n)
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      const int r = m0 + m * 16 + u * 8 + g;
-      if (r >= p.M) continue;
-      int row = p.c_rows ? p.c_rows[r] : r;
-      row = min(max(row, 0), p.rows_c - 1);
-      float f = 1.f;
-      if (p.gate) f = 1.0f / (1.0f + __expf(-(float)p.gate[row * p.g_row + h]));
-      bf16* c = p.C + row * p.c_row + h * p.c_head + n0 + j * 2;
+    for (int u = 0; u < 2; ++u)
+      *reinterpret_cast<float2*>(&part[warp][u * 8 + g][n * 8 + j * 2]) = make_float2(acc[n][2 * u], acc[n][2 * u + 1]);
+  __syncthreads();
+  const int r = threadIdx.x >> 3, c = (threadIdx.x & 7) * 4;
+  if (m0 + r >= p.M || n0 + c >= p.N) return;
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
-        *reinterpret_cast<uint32_t*>(c + n * 8) = pack_bf16(acc[m][n][2 * u] * f, acc[m][n][2 * u + 1] * f);
-    }
+  for (int q = 0; q < 4; ++q) {
+    const float4 v = *reinterpret_cast<const float4*>(&part[q][r][c]);
+    o.x += v.x; o.y += v.y; o.z += v.z; o.w += v.w;
+  }
+  int row = p.c_rows ? p.c_rows[m0 + r] : m0 + r;
+  row = min(max(row, 0), p.rows_c - 1);
+  float f = 1.f;
+  if (p.gate) f = 1.0f / (1.0f + __expf(-(float)p.gate[row * p.g_row + h]));
+  *reinterpret_cast<uint2*>(p.C + row * p.c_row + h * p.c_head + n0 + c) = make_uint2(pack_bf16(o.x * f, o.y * f), pack_bf16(o.z * f, o.w * f));
 }
 
 // ---------------------------------------------------------------------------------- decode
@@ -198,7 +192,7 @@ struct LatentDecode {
   float* part_o; float* part_ml;       // [n, H, splits, rank_p], [n, H, splits, 2]
 };
 
-constexpr int LD_KEYS = 64;
+constexpr int LD_KEYS = 32, LD_ROWS = 16;
 constexpr float LD_LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ float ld_ex2(float x) {
@@ -218,46 +212,52 @@ __device__ __forceinline__ void ld_m4t(uint32_t addr, uint32_t (&r)[4]) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-// shared memory of one block: two key tiles, the queries, weights (bf16) and two partial score tiles (fp32)
-inline int latent_decode_smem(int row_ch, int mt) {
+// shared memory of one block: two key tiles, the queries, weights (bf16) and four partial score tiles (fp32)
+inline int latent_decode_smem(int row_ch) {
   const int pitch = row_ch * 2 + 16;
-  return 2 * LD_KEYS * pitch + 16 * mt * pitch + 16 * mt * (LD_KEYS * 2 + 16) + 2 * 16 * mt * (LD_KEYS + 4) * 4;
+  return 2 * LD_KEYS * pitch + LD_ROWS * pitch + LD_ROWS * (LD_KEYS * 2 + 16) + 4 * LD_ROWS * (LD_KEYS + 4) * 4;
 }
 
-// MT: 16-head tiles of the block; CPW: 16-channel slices of the weighted sum per warp (rank_p <= 128 CPW).
-template <int MT, int CPW>
-__global__ void __launch_bounds__(256)
+// CPW: 16-channel slices of the weighted sum per warp (rank_p <= 128 CPW).
+template <int CPW>
+__global__ void __launch_bounds__(256, 2)
 latent_decode_kernel(const LatentDecode p) {
-  constexpr int ROWS = 16 * MT, PER = 256 / ROWS, KPT = LD_KEYS / PER;      // threads per row, keys per thread
+  constexpr int SP = LD_KEYS + 4, pp = LD_KEYS * 2 + 16;
   extern __shared__ __align__(16) uint8_t smem[];
-  __shared__ float s_alpha[ROWS], s_m[ROWS], s_l[ROWS];
+  __shared__ float s_alpha[LD_ROWS], s_m[LD_ROWS], s_l[LD_ROWS];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h0 = blockIdx.y * ROWS, nh = min(ROWS, p.H - h0), split = blockIdx.z;
+  const int h0 = blockIdx.y * LD_ROWS, nh = min(LD_ROWS, p.H - h0), split = blockIdx.z;
   const int row = min(max(p.rows[blockIdx.x], 0), p.T - 1);
   const int seq = min(max(p.row_seq[row], 0), p.num_seqs - 1);
   const int n_vis = p.context[seq] + row - p.q_start[seq] + 1;
   const int tiles_all = (n_vis + LD_KEYS - 1) / LD_KEYS;
   const int per = (tiles_all + p.splits - 1) / p.splits;
   const int t0 = min(tiles_all, split * per), t1 = min(tiles_all, t0 + per);
-  const int ch = p.rank_p + p.rot_p, pitch = ch * 2 + 16, pp = LD_KEYS * 2 + 16;
-  const uint32_t sK = smem_u32(smem), sQ = sK + 2 * LD_KEYS * pitch, sP = sQ + ROWS * pitch;
-  float* sS = reinterpret_cast<float*>(smem + 2 * LD_KEYS * pitch + ROWS * pitch + ROWS * pp);   // [2][ROWS][LD_KEYS + 4]
-  constexpr int SP = LD_KEYS + 4;
+  const int ch = p.rank_p + p.rot_p, pitch = ch * 2 + 16;
+  const uint32_t sK = smem_u32(smem), sQ = sK + 2 * LD_KEYS * pitch, sP = sQ + LD_ROWS * pitch;
+  float* sS = reinterpret_cast<float*>(smem + (2 * LD_KEYS + LD_ROWS) * pitch + LD_ROWS * pp);   // [4][LD_ROWS][SP]
 
-  auto fetch = [&](int t, int buf) {
-    // four threads per key row, 16 bytes each
-    const int r = tid >> 2;
-    const int pos = min(t * LD_KEYS + r, n_vis - 1);        // past the end: a valid key, masked below
-    int pg = p.block_tables[(long)seq * p.bt_stride + pos / p.block_size];
+  // eight threads per key row, 16 bytes each; page numbers are looked up a tile ahead
+  const int* bt = p.block_tables + (long)seq * p.bt_stride;
+  const int fr = tid >> 3, fc = (tid & 7) * 8;
+  auto lookup = [&](int t) { return bt[min(t * LD_KEYS + fr, n_vis - 1) / p.block_size]; };
+  auto fetch = [&](int t, int buf, int pg) {
+    const int pos = min(t * LD_KEYS + fr, n_vis - 1);       // past the end: a valid key, masked below
     pg = min(max(pg, 0), p.num_blocks - 1);
     const bf16* src = p.pages + ((long)pg * p.block_size + pos % p.block_size) * ch;
-    const uint32_t dst = sK + (buf * LD_KEYS + r) * pitch;
-    for (int c = (tid & 3) * 8; c < ch; c += 32) ld_cp16(dst + c * 2, src + c);
+    const uint32_t dst = sK + (buf * LD_KEYS + fr) * pitch;
+#pragma unroll 3
+    for (int c = fc; c < ch; c += 64) ld_cp16(dst + c * 2, src + c);
   };
-  if (t0 < t1) fetch(t0, 0);
+  int page = 0;
+  if (t0 < t1) {
+    page = lookup(t0);
+    fetch(t0, 0, page);
+    if (t0 + 1 < t1) page = lookup(t0 + 1);
+  }
   asm volatile("cp.async.commit_group;" ::: "memory");
   // queries: latent part, rotated part; rows past the last head are zero
-  for (int i = tid; i < ROWS * (ch / 8); i += 256) {
+  for (int i = tid; i < LD_ROWS * (ch / 8); i += 256) {
     const int r = i / (ch / 8), c = (i - r * (ch / 8)) * 8;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
     if (r < nh) {
@@ -268,163 +268,135 @@ latent_decode_kernel(const LatentDecode p) {
     st_shared_v4(sQ + r * pitch + c * 2, v);
   }
 
-  const int half = warp >> 2, kg = warp & 3;                // score product: channel half, group of 16 keys
-  const int steps = ch / 16, k_lo = half ? (steps + 1) / 2 : 0, k_hi = half ? steps : (steps + 1) / 2;
-  const int srow = tid / PER, sk0 = (tid % PER) * KPT;      // softmax: row and first key of this thread
+  const int quarter = warp >> 1, kg = warp & 1;             // score product: channel quarter, group of 16 keys
+  const int steps = ch / 16, k_lo = steps * quarter / 4, k_hi = steps * (quarter + 1) / 4;
+  const int srow = tid >> 4, sk0 = (tid & 15) * 2;          // softmax: row and first of two keys of this thread
   float m_run = -INFINITY, l_run = 0.f;
   const float mul = p.scale * LD_LOG2E;
-  float acc[MT][CPW][2][4];
+  float acc[CPW][2][4];
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int c = 0; c < CPW; ++c)
 #pragma unroll
-    for (int c = 0; c < CPW; ++c)
+    for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) acc[m][c][n][i] = 0.f;
+      for (int i = 0; i < 4; ++i) acc[c][n][i] = 0.f;
 
   for (int t = t0; t < t1; ++t) {
     const int buf = (t - t0) & 1;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                        // tile t is here; everyone is done with the other buffer
-    if (t + 1 < t1) fetch(t + 1, buf ^ 1);
+    if (t + 1 < t1) {
+      fetch(t + 1, buf ^ 1, page);
+      if (t + 2 < t1) page = lookup(t + 2);
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
     const uint32_t kt = sK + buf * LD_KEYS * pitch;
     {
-      float s[MT][2][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int i = 0; i < 4; ++i) s[m][n][i] = 0.f;
+      float s[2][4] = {};
       // K matrices: keys 0-7 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 0-7 | keys 8-15 ch 8-15
       const uint32_t ka = kt + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
       // Q matrices: rows 0-7 ch 0-7 | rows 8-15 ch 0-7 | rows 0-7 ch 8-15 | rows 8-15 ch 8-15
       const uint32_t qa = sQ + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
-#pragma unroll 4
+#pragma unroll 5
       for (int k = k_lo; k < k_hi; ++k) {
-        uint32_t b[4];
+        uint32_t a[4], b[4];
         ld_m4(ka + k * 32, b);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t a[4];
-          ld_m4(qa + m * 16 * pitch + k * 32, a);
-          mma_bf16(s[m][0], a[0], a[1], a[2], a[3], b[0], b[1]);
-          mma_bf16(s[m][1], a[0], a[1], a[2], a[3], b[2], b[3]);
-        }
+        ld_m4(qa + k * 32, a);
+        mma_bf16(s[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+        mma_bf16(s[1], a[0], a[1], a[2], a[3], b[2], b[3]);
       }
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+      for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int u = 0; u < 2; ++u)
-            *reinterpret_cast<float2*>(sS + (half * ROWS + m * 16 + u * 8 + (lane >> 2)) * SP + kg * 16 + n * 8 + (lane & 3) * 2) =
-                make_float2(s[m][n][2 * u], s[m][n][2 * u + 1]);
+        for (int u = 0; u < 2; ++u)
+          *reinterpret_cast<float2*>(sS + (quarter * LD_ROWS + u * 8 + (lane >> 2)) * SP + kg * 16 + n * 8 + (lane & 3) * 2) =
+              make_float2(s[n][2 * u], s[n][2 * u + 1]);
     }
     __syncthreads();
     {
-      float y[KPT], mx = -INFINITY;
+      float2 y = make_float2(0.f, 0.f);
 #pragma unroll
-      for (int i = 0; i < KPT; i += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(sS + srow * SP + sk0 + i);
-        const float4 b = *reinterpret_cast<const float4*>(sS + (ROWS + srow) * SP + sk0 + i);
-        y[i] = (a.x + b.x) * mul; y[i + 1] = (a.y + b.y) * mul; y[i + 2] = (a.z + b.z) * mul; y[i + 3] = (a.w + b.w) * mul;
+      for (int q = 0; q < 4; ++q) {
+        const float2 v = *reinterpret_cast<const float2*>(sS + (q * LD_ROWS + srow) * SP + sk0);
+        y.x += v.x;
+        y.y += v.y;
       }
+      const int left = n_vis - t * LD_KEYS - sk0;           // keys of this thread that are visible
+      y.x = left > 0 ? y.x * mul : -INFINITY;
+      y.y = left > 1 ? y.y * mul : -INFINITY;
+      float mx = fmaxf(y.x, y.y);
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        if (t * LD_KEYS + sk0 + i >= n_vis) y[i] = -INFINITY;
-        mx = fmaxf(mx, y[i]);
-      }
-#pragma unroll
-      for (int o = PER / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       const float m_new = fmaxf(m_run, mx);                 // finite: a tile holds at least one visible key
       const float alpha = ld_ex2(m_run - m_new);
-      float sum = 0.f;
-#pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        y[i] = ld_ex2(y[i] - m_new);
-        sum += y[i];
-      }
-      l_run = fmaf(l_run, alpha, sum);                      // this thread's keys only; summed at the end
+      y.x = ld_ex2(y.x - m_new);
+      y.y = ld_ex2(y.y - m_new);
+      l_run = fmaf(l_run, alpha, y.x + y.y);                // this thread's keys only; summed at the end
       m_run = m_new;
-      if (tid % PER == 0) s_alpha[srow] = alpha;
-      const uint32_t pd = sP + srow * pp + sk0 * 2;
-#pragma unroll
-      for (int i = 0; i < KPT; i += 2)
-        asm volatile("st.shared.b32 [%0], %1;" ::"r"(pd + i * 2), "r"(pack_bf16(y[i], y[i + 1])) : "memory");
+      if ((tid & 15) == 0) s_alpha[srow] = alpha;
+      asm volatile("st.shared.b32 [%0], %1;" ::"r"(sP + srow * pp + sk0 * 2), "r"(pack_bf16(y.x, y.y)) : "memory");
     }
     __syncthreads();
+    const float a0 = s_alpha[lane >> 2], a1 = s_alpha[8 + (lane >> 2)];
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const float a0 = s_alpha[m * 16 + (lane >> 2)], a1 = s_alpha[m * 16 + 8 + (lane >> 2)];
+    for (int c = 0; c < CPW; ++c)
 #pragma unroll
-      for (int c = 0; c < CPW; ++c)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          acc[m][c][n][0] *= a0; acc[m][c][n][1] *= a0;
-          acc[m][c][n][2] *= a1; acc[m][c][n][3] *= a1;
-        }
-    }
+      for (int n = 0; n < 2; ++n) {
+        acc[c][n][0] *= a0; acc[c][n][1] *= a0;
+        acc[c][n][2] *= a1; acc[c][n][3] *= a1;
+      }
     const uint32_t pa = sP + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pp + (lane >> 4) * 16;
     // V matrices, transposed: keys 0-7 ch 0-7 | keys 8-15 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 8-15
     const uint32_t va = kt + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
 #pragma unroll
     for (int k = 0; k < LD_KEYS / 16; ++k) {
-      uint32_t a[MT][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) ld_m4(pa + m * 16 * pp + k * 32, a[m]);
+      uint32_t a[4];
+      ld_m4(pa + k * 32, a);
 #pragma unroll
       for (int c = 0; c < CPW; ++c) {
         const int sl = c * 8 + warp;
         if (sl * 16 < p.rank_p) {
           uint32_t b[4];
           ld_m4t(va + k * 16 * pitch + sl * 32, b);
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            mma_bf16(acc[m][c][0], a[m][0], a[m][1], a[m][2], a[m][3], b[0], b[1]);
-            mma_bf16(acc[m][c][1], a[m][0], a[m][1], a[m][2], a[m][3], b[2], b[3]);
-          }
+          mma_bf16(acc[c][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+          mma_bf16(acc[c][1], a[0], a[1], a[2], a[3], b[2], b[3]);
         }
       }
     }
   }
 #pragma unroll
-  for (int o = PER / 2; o > 0; o >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, o);
-  if (tid % PER == 0) {
+  for (int o = 8; o > 0; o >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, o);
+  if ((tid & 15) == 0) {
     s_m[srow] = m_run;
     s_l[srow] = l_run;
   }
   __syncthreads();
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int u = 0; u < 2; ++u) {
+    const int r = u * 8 + (lane >> 2);
+    if (r >= nh) continue;
+    const long hi = (long)blockIdx.x * p.H + h0 + r;
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      const int r = m * 16 + u * 8 + (lane >> 2);
-      if (r >= nh) continue;
-      const long hi = (long)blockIdx.x * p.H + h0 + r;
+    for (int c = 0; c < CPW; ++c) {
+      const int sl = c * 8 + warp;
+      if (sl * 16 >= p.rank_p) continue;
 #pragma unroll
-      for (int c = 0; c < CPW; ++c) {
-        const int sl = c * 8 + warp;
-        if (sl * 16 >= p.rank_p) continue;
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          const int col = sl * 16 + n * 8 + (lane & 3) * 2;
-          const float x = acc[m][c][n][2 * u], y = acc[m][c][n][2 * u + 1];
-          if (p.splits == 1) {
-            const float f = 1.0f / s_l[r];
-            *reinterpret_cast<uint32_t*>(p.out + hi * p.rank_p + col) = pack_bf16(x * f, y * f);
-          } else {
-            *reinterpret_cast<float2*>(p.part_o + (hi * p.splits + split) * p.rank_p + col) = make_float2(x, y);
-          }
+      for (int n = 0; n < 2; ++n) {
+        const int col = sl * 16 + n * 8 + (lane & 3) * 2;
+        const float x = acc[c][n][2 * u], y = acc[c][n][2 * u + 1];
+        if (p.splits == 1) {
+          const float f = 1.0f / s_l[r];
+          *reinterpret_cast<uint32_t*>(p.out + hi * p.rank_p + col) = pack_bf16(x * f, y * f);
+        } else {
+          *reinterpret_cast<float2*>(p.part_o + (hi * p.splits + split) * p.rank_p + col) = make_float2(x, y);
         }
       }
-      if (p.splits > 1 && warp == 0 && (lane & 3) == 0) {
-        p.part_ml[2 * (hi * p.splits + split)] = s_m[r];
-        p.part_ml[2 * (hi * p.splits + split) + 1] = s_l[r];
-      }
     }
+    if (p.splits > 1 && warp == 0 && (lane & 3) == 0) {
+      p.part_ml[2 * (hi * p.splits + split)] = s_m[r];
+      p.part_ml[2 * (hi * p.splits + split) + 1] = s_l[r];
+    }
+  }
 }
 
 __global__ void __launch_bounds__(128)
@@ -451,20 +423,13 @@ latent_merge_kernel(const LatentDecode p) {
   }
 }
 
-template <int MT, int CPW>
-static int launch_latent_decode(const LatentDecode& p, int smem, cudaStream_t st) {
+template <int CPW>
+static int launch_latent_decode(const LatentDecode& p, cudaStream_t st) {
   static unsigned long long prep = 0;
-  if (int e = ensure_dynamic_smem((const void*)latent_decode_kernel<MT, CPW>, 227 * 1024 - 1024, prep)) return e;
-  dim3 grid(p.n, (p.H + 16 * MT - 1) / (16 * MT), p.splits);
-  latent_decode_kernel<MT, CPW><<<grid, 256, smem, st>>>(p);
+  if (int e = ensure_dynamic_smem((const void*)latent_decode_kernel<CPW>, 227 * 1024 - 1024, prep)) return e;
+  dim3 grid(p.n, (p.H + LD_ROWS - 1) / LD_ROWS, p.splits);
+  latent_decode_kernel<CPW><<<grid, 256, latent_decode_smem(p.rank_p + p.rot_p), st>>>(p);
   return (int)cudaGetLastError();
-}
-
-template <int MT>
-static int pick_latent_decode(const LatentDecode& p, int smem, cudaStream_t st) {
-  if (p.rank_p <= 128) return launch_latent_decode<MT, 1>(p, smem, st);
-  if (p.rank_p <= 256) return launch_latent_decode<MT, 2>(p, smem, st);
-  return launch_latent_decode<MT, 4>(p, smem, st);
 }
 
 }  // namespace omni
@@ -496,38 +461,30 @@ extern "C" int omni_latent_gather(const void* pages, int row_bytes, const int* t
 extern "C" int omni_head_gemm(const HeadGemm* args, void* stream) {
   const HeadGemm& p = *args;
   if (p.M <= 0 || p.H <= 0) return RC_OK;
-  if ((p.N & 15) || (p.K & 15) || p.N <= 0 || p.K <= 0 || (p.a_row & 7) || (p.a_head & 7) || (p.c_row & 1) || (p.c_head & 1) ||
+  if ((p.N & 15) || (p.K & 15) || p.N <= 0 || p.K <= 0 || (p.a_row & 7) || (p.a_head & 7) || (p.c_row & 3) || (p.c_head & 3) ||
       p.H > 65535 || p.rows_a <= 0 || p.rows_c <= 0)
     return RC_BAD_ARG;
-  cudaStream_t st = (cudaStream_t)stream;
-  const unsigned nb = (p.N + 63) / 64;
-  if (p.M <= 16) head_gemm_kernel<1><<<dim3(nb, p.H, 1), 128, 0, st>>>(p);
-  else if (p.M <= 32) head_gemm_kernel<2><<<dim3(nb, p.H, 1), 128, 0, st>>>(p);
-  else {
-    if ((p.M + 63) / 64 > 65535) return RC_BAD_ARG;
-    head_gemm_kernel<4><<<dim3(nb, p.H, (p.M + 63) / 64), 128, 0, st>>>(p);
-  }
+  if ((p.M + 15) / 16 > 65535) return RC_BAD_ARG;
+  head_gemm_kernel<<<dim3((p.N + 31) / 32, p.H, (p.M + 15) / 16), 128, 0, (cudaStream_t)stream>>>(p);
   return (int)cudaGetLastError();
 }
 
 // 0: the sizes do not fit the decode kernel; otherwise the heads a block serves.
-extern "C" int omni_latent_decode_heads(int heads, int rank_p, int rot_p) {
+extern "C" int omni_latent_decode_heads(int rank_p, int rot_p) {
   if (rank_p > 512 || rank_p <= 0 || rot_p < 0) return 0;
-  if (heads > 16 && latent_decode_smem(rank_p + rot_p, 2) <= 227 * 1024 - 1024) return 32;
-  return latent_decode_smem(rank_p + rot_p, 1) <= 227 * 1024 - 1024 ? 16 : 0;
+  return latent_decode_smem(rank_p + rot_p) <= 227 * 1024 - 1024 ? LD_ROWS : 0;
 }
 
 extern "C" int omni_latent_decode(const LatentDecode* args, void* stream) {
   const LatentDecode& p = *args;
   if (p.n <= 0) return RC_OK;
-  const int heads = omni_latent_decode_heads(p.H, p.rank_p, p.rot_p);
-  if (heads == 0 || p.H <= 0 || (p.rank_p & 15) || (p.rot_p & 15) || (p.ldp & 7) || (p.head_cols & 7) || (p.dim_p & 7) || p.splits < 1 ||
+  if (omni_latent_decode_heads(p.rank_p, p.rot_p) == 0 || p.H <= 0 || (p.rank_p & 15) || (p.rot_p & 15) || (p.ldp & 7) || (p.head_cols & 7) || (p.dim_p & 7) || p.splits < 1 ||
       p.splits > 65535 || p.block_size <= 0 || p.num_blocks <= 0 || p.num_seqs <= 0 || p.T <= 0)
     return RC_BAD_ARG;
   if (p.splits > 1 && (!p.part_o || !p.part_ml)) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
-  int rc = heads == 32 ? pick_latent_decode<2>(p, latent_decode_smem(p.rank_p + p.rot_p, 2), st)
-                       : pick_latent_decode<1>(p, latent_decode_smem(p.rank_p + p.rot_p, 1), st);
+  const int rc = p.rank_p <= 128 ? launch_latent_decode<1>(p, st)
+                                 : (p.rank_p <= 256 ? launch_latent_decode<2>(p, st) : launch_latent_decode<4>(p, st));
   if (rc || p.splits == 1) return rc;
   latent_merge_kernel<<<(unsigned)(p.n * p.H), 128, 0, st>>>(p);
   return (int)cudaGetLastError();

@@ -17,20 +17,6 @@
 
 namespace omni {
 
-// multiply eight values by `s` and the gains of their channels
-__device__ __forceinline__ void scale_gain8(float (&v)[8], float s, const float* g, int gs, int c) {
-  if (gs == 0) {
-    const float k = s * g[0];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] *= k;
-  } else {
-    float w[8];
-    load8<float>(g + c, w);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] *= s * w[e];
-  }
-}
-
 // ------------------------------------------------------------------ embedding + first norm
 template <typename T, int NV>
 __global__ void __launch_bounds__(1024)

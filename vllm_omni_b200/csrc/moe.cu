@@ -126,18 +126,17 @@ moe_topk_kernel(const float* __restrict__ logits, long ld, int T, int E, int k, 
   topk_softmax(v, E, k, lane, ids + (long)t * k, weights + (long)t * k);
 }
 
-// Router of MT * 16 tokens per block: eight warps share the contraction (each takes every eighth 32-channel chunk),
-// 64 experts at a time; partial sums meet in shared memory in a fixed order.  A warp reads 16 bytes per row and
+// Router of MT * 16 tokens per block: NW warps share the contraction (each takes every NW-th 32-channel chunk), 64 experts at a time; partial sums meet in shared memory in a fixed order.  A warp reads 16 bytes per row and
 // chunk: lane group j of a quad owns channels 8 j .. 8 j + 7 of the chunk for both operands, which permutes the
 // contraction alike on both sides.
-template <int MT>
-__global__ void __launch_bounds__(256)
+template <int MT, int NW>
+__global__ void __launch_bounds__(32 * NW)
 moe_router_kernel(const __nv_bfloat16* __restrict__ x, long ldx, const __nv_bfloat16* __restrict__ w, long ldw,
                   const float* __restrict__ bias, int T, int D, int E, int Ep, int k, int* __restrict__ ids,
                   float* __restrict__ weights) {
   extern __shared__ float sm[];
-  float* part = sm;                            // [8 warps][MT * 16][64]
-  float* logit = sm + 8 * MT * 16 * 64;        // [MT * 16][256]
+  float* part = sm;                            // [NW][MT * 16][64]
+  float* logit = sm + NW * MT * 16 * 64;        // [MT * 16][256]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
   const int t0 = blockIdx.x * (MT * 16);
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
@@ -149,7 +148,8 @@ moe_router_kernel(const __nv_bfloat16* __restrict__ x, long ldx, const __nv_bflo
       for (int n = 0; n < 8; ++n)
 #pragma unroll
         for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
-    for (int c = warp * 32; c < D; c += 256) {
+#pragma unroll(MT == 1 ? 2 : 1)
+    for (int c = warp * 32; c < D; c += 32 * NW) {
       const int ch = c + j * 8;
       const bool in = ch < D;                  // D is a multiple of 8
       uint4 a[MT][2];
@@ -187,18 +187,18 @@ moe_router_kernel(const __nv_bfloat16* __restrict__ x, long ldx, const __nv_bflo
           *reinterpret_cast<float2*>(part + ((long)warp * MT * 16 + m * 16 + h * 8 + g) * 64 + n * 8 + j * 2) =
               make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
     __syncthreads();
-    for (int i = threadIdx.x; i < MT * 16 * 64; i += 256) {
+    for (int i = threadIdx.x; i < MT * 16 * 64; i += 32 * NW) {
       const int e = e0 + (i & 63);
       if (e < E) {
         float s = bias ? bias[e] : 0.f;
 #pragma unroll
-        for (int q = 0; q < 8; ++q) s += part[q * MT * 16 * 64 + i];
+        for (int q = 0; q < NW; ++q) s += part[q * MT * 16 * 64 + i];
         logit[(i >> 6) * 256 + e] = s;
       }
     }
   }
   __syncthreads();
-  for (int r = warp; r < MT * 16; r += 8) {
+  for (int r = warp; r < MT * 16; r += NW) {
     const int t = t0 + r;
     if (t >= T) break;
     float v[8];
@@ -485,12 +485,12 @@ extern "C" int omni_moe_router(const void* x, long ldx, const void* w, long ldw,
   static unsigned long long prep[2] = {0, 0};
   if (T > 148 * 16) {
     const int smem = (8 * 32 * 64 + 32 * 256) * 4;
-    if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<2>, smem, prep[0])) return e;
-    moe_router_kernel<2><<<(T + 31) / 32, 256, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
+    if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<2, 8>, smem, prep[0])) return e;
+    moe_router_kernel<2, 8><<<(T + 31) / 32, 256, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
   } else {
-    const int smem = (8 * 16 * 64 + 16 * 256) * 4;
-    if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<1>, smem, prep[1])) return e;
-    moe_router_kernel<1><<<(T + 15) / 16, 256, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
+    const int smem = (16 * 16 * 64 + 16 * 256) * 4;
+    if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<1, 16>, smem, prep[1])) return e;
+    moe_router_kernel<1, 16><<<(T + 15) / 16, 512, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
   }
   return (int)cudaGetLastError();
 }

@@ -56,6 +56,20 @@ __device__ __forceinline__ float rms_scale(float sumsq, int n, float eps) {
   return 1.0f / sqrtf(sumsq / (float)n + eps);
 }
 
+// multiply eight values by `s` and the gains of their channels
+__device__ __forceinline__ void scale_gain8(float (&v)[8], float s, const float* g, int gs, int c) {
+  if (gs == 0) {
+    const float k = s * g[0];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= k;
+  } else {
+    float w[8];
+    load8<float>(g + c, w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= s * w[e];
+  }
+}
+
 // threads and vectors per thread for a row of n channels (n <= 32768)
 inline bool row_shape(int n, int& threads, int& nv) {
   const int vec = n / 8;

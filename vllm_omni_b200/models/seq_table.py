@@ -143,20 +143,21 @@ class SeqTable:
         return KeyGroup(buf[:len(start)], buf[o1:o1 + len(members)], len(seqs), at, buf[o2:o2 + 2 * len(items)].view(-1, 2), len(items),
                         rows_per_block)
 
-    def time_chunks(self, pick):
-        """Runs of consecutive rows of the sequences with more than one row, for scans over time: ``pick(n)`` gives the
-        run length of a sequence with n rows.  int32 [m, 4] of (sequence, first row in the portion, rows, index of the
-        sequence's first run), m, and whether any sequence has several runs."""
-        got = self._items.get("time")
+    def time_runs(self, key, pick):
+        """Runs of consecutive rows of the sequences with more than one row, for scans over time: ``pick(lens)`` gives the
+        run length for portions of ``lens`` rows (asked once per ``key``).  int32 [m, 4] of (sequence, first row in the
+        portion, rows, index of the sequence's first run), m, and whether any sequence has several runs."""
+        got = self._items.get(("time", key))
         if got is None:
             runs, several = [], False
+            step = pick([n for n in self.lens if n > 1])
             for s, n in enumerate(self.lens):
                 if n > 1:
-                    step, first = pick(n), len(runs)
+                    first = len(runs)
                     runs += [(s, o, min(step, n - o), first) for o in range(0, n, step)]
                     several |= len(runs) - first > 1
-            got = (torch.tensor(runs or [(0, 0, 0, 0)], dtype=torch.int32).to(self.q_start.device), len(runs), several)
-            self._items["time"] = got
+            got = (torch.tensor(runs, dtype=torch.int32).to(self.q_start.device), len(runs), several)
+            self._items[("time", key)] = got
         return got
 
     def prefill_items(self, rows_per_block: int):

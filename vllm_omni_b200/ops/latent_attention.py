@@ -133,7 +133,7 @@ def latent_attention(proj, s: LatentShape, pages, seqs, uk_t, kv_up, scale: floa
         return _cpu(proj, s, pages, seqs, kv_up, scale, out, gate)
     assert proj.stride(1) == 1 and out.is_contiguous() and uk_t.is_contiguous() and kv_up.is_contiguous()
     bf = proj.dtype == torch.bfloat16
-    if impl == "rows" or not bf or not nv.lib("latent_attn").omni_latent_decode_heads(s.heads, s.rank_p, s.rot_p):
+    if impl == "rows" or not bf or not nv.lib("latent_attn").omni_latent_decode_heads(s.rank_p, s.rot_p):
         return _rows(proj, s, pages, seqs, uk_t, kv_up, scale, out, gate)
     short = 1 << 30 if impl == "latent" or not _expands(s) else SHORT
     rows, n, keys = seqs.short_rows(short)
@@ -165,7 +165,12 @@ def _expanded(proj, s, pages, seqs, kv_up, scale, out, gate, group):
         nv.ptr(pages), c_int(s.row * pages.element_size()), nv.ptr(seqs.block_tables), c_int(seqs.block_tables.stride(0)), c_int(bs),
         c_int(nb), nv.ptr(group.members), c_int(group.n_members), nv.ptr(rows), c_long(group.keys), nv.stream_ptr()),
         "omni_latent_gather")
-    kv = gemm.linear(rows[:, :s.rank_p], kv_up)
+    expanded_attention(proj, s, rows, gemm.linear(rows[:, :s.rank_p], kv_up), seqs, scale, out, gate, group)
+
+
+def expanded_attention(proj, s, rows, kv, seqs, scale, out, gate, group):
+    """Attention of a group's portions over expanded keys and values ``kv`` [keys, H dim_p | H vdim_p]; the shared key
+    parts are the last channels of ``rows`` [keys, row]."""
     nk = s.heads * s.dim_p
     a = WA._WinAttn()
     a.q, a.q_rs, a.k_cache, a.v_cache = _P(proj), proj.stride(0), _P(kv), _P(kv[:, nk:])
@@ -174,7 +179,7 @@ def _expanded(proj, s, pages, seqs, kv_up, scale, out, gate, group):
     a.items, a.n_items, a.block_tokens = _P(group.items), group.n_items, group.rows_per_block
     a.out, a.o_rs, a.gate, a.g_rs = _P(out), out.stride(0), _P(gate), 0 if gate is None else gate.stride(0)
     a.scale, a.T, a.H, a.G, a.dp, a.vp = scale, proj.shape[0], s.heads, s.heads, s.head_cols, s.vdim_p
-    a.num_seqs, a.num_blocks, a.block_size, a.splits, a.status = seqs.n_seqs, nb, bs, 1, _P(nv.status_word(proj.device))
+    a.num_seqs, a.num_blocks, a.block_size, a.splits, a.status = seqs.n_seqs, 1, 32, 1, _P(nv.status_word(proj.device))
     a.k_ts = a.v_ts = kv.stride(0)
     a.dp_u, a.k_shared, a.ks_ts = s.dim_p, _P(rows[:, s.rank_p:]), rows.stride(0)
     a.key_start, a.key_rows = _P(group.key_start), group.keys
@@ -182,12 +187,12 @@ def _expanded(proj, s, pages, seqs, kv_up, scale, out, gate, group):
                 "omni_attn_window_prefill")
 
 
-def decode_splits(blocks: int, keys: int, sms: int = 148) -> int:
-    """Blocks that share one row's keys: fills the SMs evenly, at least 256 keys each."""
+def decode_splits(blocks: int, keys: int, slots: int = 2 * 148) -> int:
+    """Blocks that share one row's keys: fills the block slots of the GPU evenly, about 256 keys each at least."""
     best, best_cost = 1, None
     for n in range(1, max(1, min(64, (keys + 255) // 256)) + 1):
-        waves = -(-blocks * n // sms)
-        cost = waves * (-(-keys // (64 * n)) + 3)           # key tiles of a block and its start-up, per wave
+        waves = -(-blocks * n // slots)
+        cost = waves * (-(-keys // (32 * n)) + 4)           # key tiles of a block and its start-up, per wave
         if best_cost is None or cost < best_cost:
             best, best_cost = n, cost
     return best
@@ -204,12 +209,20 @@ def head_gemm(a, a_row: int, a_head: int, w, c, c_row: int, c_head: int, M: int,
 
 
 def _latent_space(proj, s, pages, seqs, uk_t, kv_up, scale, out, gate, rows, n, keys):
-    H, dev = s.heads, proj.device
-    q_lat = torch.empty(n, H, s.rank_p, dtype=proj.dtype, device=dev)
+    H = s.heads
+    q_lat = torch.empty(n, H, s.rank_p, dtype=proj.dtype, device=proj.device)
     head_gemm(proj, proj.stride(0), s.head_cols, uk_t, q_lat, H * s.rank_p, s.rank_p, n, H, a_rows=rows)
+    o_lat = latent_decode(q_lat, proj, s, pages, seqs, rows, n, keys, scale)
+    head_gemm(o_lat, H * s.rank_p, s.rank_p, kv_up[H * s.dim_p:].view(H, s.vdim_p, s.rank_p), out, out.stride(0), s.vdim_p, n, H,
+              c_rows=rows, gate=gate)
+
+
+def latent_decode(q_lat, proj, s, pages, seqs, rows, n, keys, scale):
+    """Weighted sums of latent rows [n, H, rank_p] for ``n`` batch ``rows`` that see ``keys`` keys at most."""
+    H, dev = s.heads, proj.device
     o_lat = torch.empty_like(q_lat)
     lib = nv.lib("latent_attn")
-    hb = lib.omni_latent_decode_heads(H, s.rank_p, s.rot_p)
+    hb = lib.omni_latent_decode_heads(s.rank_p, s.rot_p)
     a = _LatentDecode()
     a.q_lat, a.proj, a.ldp, a.head_cols, a.dim_p = _P(q_lat), _P(proj), proj.stride(0), s.head_cols, s.dim_p
     a.pages, a.rank_p, a.rot_p = _P(pages), s.rank_p, s.rot_p
@@ -222,8 +235,7 @@ def _latent_space(proj, s, pages, seqs, uk_t, kv_up, scale, out, gate, rows, n, 
         po, pml = WA._parts(dev, n * H * a.splits, s.rank_p)
         a.part_o, a.part_ml = _P(po), _P(pml)
     nv.check_rc(lib.omni_latent_decode(ctypes.byref(a), nv.stream_ptr()), "omni_latent_decode")
-    head_gemm(o_lat, H * s.rank_p, s.rank_p, kv_up[H * s.dim_p:].view(H, s.vdim_p, s.rank_p), out, out.stride(0), s.vdim_p, n, H,
-              c_rows=rows, gate=gate)
+    return o_lat
 
 
 def _rows(proj, s, pages, seqs, uk_t, kv_up, scale, out, gate):

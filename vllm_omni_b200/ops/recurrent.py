@@ -46,10 +46,24 @@ class _Scan(ctypes.Structure):
                 ("out", c_void_p), ("status", c_void_p)]
 
 
-def run_length(n: int) -> int:
-    """Tokens of one run of a portion with n tokens: at most 32 runs read each other's sums, long ones keep the gate
-    weights busy."""
-    return max(128, (n + 31) // 32 + 31 & ~31)
+_STREAMS = 4             # runs a block of the prompt kernel walks side by side
+
+
+def run_length(lens, channel_tiles: int, sms: int = 148) -> int:
+    """Tokens of a run for portions of ``lens`` tokens: fills the SMs evenly, 64 runs per portion at most."""
+    most = max(lens)
+    best, best_cost = None, None
+    for n in range(64, 4096 + 1, 64):
+        if n * 64 < most and n < 4096:
+            continue
+        runs = sum(-(-k // n) for k in lens)
+        waves = -(-channel_tiles * -(-runs // _STREAMS) // sms)
+        cost = waves * (min(n, -(-most // 64) * 64) + 64) * (1 if most <= n else 2)       # several runs: two passes
+        if best_cost is None or cost < best_cost:
+            best, best_cost = n, cost
+        if n >= most:
+            break
+    return best if best * 64 >= most else -(-most // 4096) * 64
 
 
 def gated_scan(proj, s: GatedScanShape, seqs, conv, conv_b, gates, gates_b, decay, hist, state, impl: str | None = None):
@@ -74,7 +88,7 @@ def gated_scan(proj, s: GatedScanShape, seqs, conv, conv_b, gates, gates_b, deca
     a.num_state, a.num_seqs, a.out, a.status = state.shape[0], seqs.n_seqs, P(out), P(nv.status_word(proj.device))
     bf = proj.dtype == torch.bfloat16
     lib = nv.lib("gated_scan")
-    if impl == "plain" or not bf or s.part_p > 256 or s.taps > 8:
+    if impl == "plain" or not bf or s.part_p > 256:
         u = torch.empty(T, C, dtype=torch.float32, device=proj.device)
         z = torch.empty(2, T, C, dtype=torch.float32, device=proj.device)
         a.u, a.z = P(u), P(z)
@@ -89,7 +103,11 @@ def gated_scan(proj, s: GatedScanShape, seqs, conv, conv_b, gates, gates_b, deca
         a.seq_list, a.n_list = P(seqs.decode_list), seqs.n_decode
         nv.check_rc(lib.omni_scan_step(ctypes.byref(a), nv.stream_ptr()), "omni_scan_step")
     if seqs.n_decode < seqs.n_seqs:
-        runs, a.n_runs, several = seqs.time_chunks(run_length)
+        u = torch.empty(T, C, dtype=proj.dtype, device=proj.device)
+        a.u = P(u)
+        nv.check_rc(lib.omni_scan_conv_bf16(ctypes.byref(a), nv.stream_ptr()), "omni_scan_conv_bf16")
+        tiles = s.blocks * ((s.part_p + 127) // 128)
+        runs, a.n_runs, several = seqs.time_runs(tiles, lambda lens: run_length(lens, tiles))
         a.runs = P(runs)
         sums = torch.empty(a.n_runs, 2, C, dtype=torch.float32, device=proj.device) if several else None
         a.sums = P(sums)
