@@ -561,11 +561,11 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   w.k_stages = w.v_stages = 1;
   int used = q_bytes + tab_bytes + k_bytes + v_bytes;
   if (used > limit) return RC_TOO_LARGE;
-  // the key ring grows first: the next tile's scores are issued before the current tile's values are done with
+  // the value ring grows first: a key slot is free as soon as its scores are issued, a value slot only after the softmax
   for (bool grew = true; grew;) {
     grew = false;
-    if (w.k_stages < WP_MAX_STAGES && used + k_bytes <= limit) { ++w.k_stages; used += k_bytes; grew = true; }
     if (w.v_stages < WP_MAX_STAGES && used + v_bytes <= limit) { ++w.v_stages; used += v_bytes; grew = true; }
+    if (w.k_stages < WP_MAX_STAGES && used + k_bytes <= limit) { ++w.k_stages; used += k_bytes; grew = true; }
   }
   const int smem = used + 1024;
   CUtensorMap tq, tk, tv, ts;

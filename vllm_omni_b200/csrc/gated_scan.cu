@@ -239,9 +239,9 @@ scan_step_kernel(const GatedScan p) {
     float2 S = make_float2(0.f, 0.f);
     if (s_ctx[t] > 0) S = *reinterpret_cast<const float2*>(p.state + (long)s_in[t] * p.C + c);
     float la, a, add;
-    gate_step(acc[0][2 * u] + b0.x, acc[1][2 * u] + b1.x, x.x, dec.x * GS_LOG2E, la, a, add);
+    gate_step(acc[0][2 * u], acc[1][2 * u], -GS_LOG2E * b0.x, -GS_LOG2E * b1.x, x.x, dec.x * GS_LOG2E, la, a, add);
     S.x = fmaf(a, S.x, add);
-    gate_step(acc[0][2 * u + 1] + b0.y, acc[1][2 * u + 1] + b1.y, x.y, dec.y * GS_LOG2E, la, a, add);
+    gate_step(acc[0][2 * u + 1], acc[1][2 * u + 1], -GS_LOG2E * b0.y, -GS_LOG2E * b1.y, x.y, dec.y * GS_LOG2E, la, a, add);
     S.y = fmaf(a, S.y, add);
     if (s_out[t] >= 0) *reinterpret_cast<float2*>(p.state + (long)s_out[t] * p.C + c) = S;
     *reinterpret_cast<uint32_t*>(static_cast<bf16*>(p.out) + row * p.C + c) = pack_bf16(S.x * gelu_short(y.x), S.y * gelu_short(y.y));

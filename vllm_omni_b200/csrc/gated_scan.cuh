@@ -48,24 +48,26 @@ __device__ __forceinline__ float gs_sqrt(float x) {
 
 constexpr float GS_LOG2E = 1.4426950408889634f, GS_LN2 = 0.6931471805599453f;
 
-// One token of one channel for bf16 rows: la2 = log2 a, a, and the input term.  decay2 = decay log2 e.
-__device__ __forceinline__ void gate_step(float zr, float zi, float u, float decay2, float& la2, float& a, float& add) {
+// One token of one channel for bf16 rows: la2 = log2 a, a, and the input term.  nbr, nbi: gate biases times -log2 e;
+// decay2 = decay log2 e.
+__device__ __forceinline__ void gate_step(float zr, float zi, float nbr, float nbi, float u, float decay2, float& la2, float& a,
+                                          float& add) {
   // both sigmoids from one reciprocal; the clamp keeps the product of the denominators finite
-  const float er = 1.0f + gs_ex2(fminf(-zr * GS_LOG2E, 60.f)), ei = 1.0f + gs_ex2(fminf(-zi * GS_LOG2E, 60.f));
+  const float er = 1.0f + gs_ex2(fminf(fmaf(zr, -GS_LOG2E, nbr), 60.f)), ei = 1.0f + gs_ex2(fminf(fmaf(zi, -GS_LOG2E, nbi), 60.f));
   const float k = gs_rcp(er * ei);
   la2 = decay2 * (k * ei);
   a = gs_ex2(la2);
   // 1 - e^x for x = 2 ln a <= 0: the series near zero, where 1 - a^2 would cancel
   const float x = 2.0f * GS_LN2 * la2;
-  const float series = -x * fmaf(x * 0.5f, fmaf(x * (1.f / 3.f), fmaf(x * 0.25f, fmaf(x * 0.2f, fmaf(x, 1.f / 6.f, 1.f), 1.f), 1.f), 1.f), 1.f);
-  const float d = x > -0.5f ? series : fmaf(-a, a, 1.0f);
+  const float series = -x * fmaf(0.5f * x, fmaf(x, 1.f / 3.f, 1.f), 1.f);
+  const float d = x > -0.03f ? series : fmaf(-a, a, 1.0f);
   add = gs_sqrt(d) * (k * er) * u;
 }
 
-// gelu with the tanh form, as z * sigmoid
+// gelu with the tanh form, as z * sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))
 __device__ __forceinline__ float gelu_short(float z) {
-  const float t = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
-  return z * gs_rcp(1.0f + gs_ex2(fminf(-t * GS_LOG2E, 126.f)));
+  constexpr float A = -1.5957691216057308f * GS_LOG2E, B = A * 0.044715f;
+  return z * gs_rcp(1.0f + gs_ex2(fminf(z * fmaf(B, z * z, A), 126.f)));
 }
 
 // pool rows of a sequence, checked; a bad index is reported and not used

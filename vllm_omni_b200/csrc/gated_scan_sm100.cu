@@ -2,35 +2,49 @@
 // convolution's rows come from gated_scan.cu).
 //
 // A portion is cut into runs of consecutive tokens.  One block owns 128 channels of one part and four runs (streams),
-// and keeps the gate weights of its channels in shared memory; a run is walked in tiles of 64 tokens.  The gates are
+// and keeps the gate weights of its channels in shared memory; a run is walked in tiles of 32 tokens.  The gates are
 // computed transposed, D[channel, token] = W[channel, k] u[token, k]^T, so that a thread of the epilogue owns one
 // channel (a TMEM lane) and meets its tokens in order: the scan is a register recurrence.
-//   warps 0-15   epilogue, four warps per stream: both gates from tensor memory, decay, input term, scan; output
-//   warp 16      TMA: gate weights, then tiles of u in turn for every stream
+//   warps 0-15   epilogue, four warps per stream: both gates from tensor memory, decay, input term, scan; the output
+//                takes the place of the gelu branch's tile in shared memory and leaves in 16-byte stores
+//   warp 16      TMA: gate weights, then tiles of u and of the gelu branch in turn for every stream
 //   warp 17      MMA issue in the same order
-// The epilogue is bound by its exponentials, reciprocals and roots; four streams hide each other's waits.
+// The epilogue is bound by instruction issue and its exponentials, reciprocals and roots: it reads its operands from
+// shared memory at constant offsets (no address arithmetic), and four streams hide each other's waits.
 // A run starts from what its sequence's earlier runs leave.  When a portion has several runs the kernel runs twice:
 // first for every run but the last the product of its decays and its state from zero go to `sums`, then every run
 // folds the sums before it and writes its results.  (Computing the gates twice moves less memory than storing decays
 // and input terms in fp32.)
-// TMEM columns: 64 per (stream, gate), 512 in all.  Every wait is bounded.
+// TMEM columns: 32 per (stream, slot, gate), 512 in all.  Every wait is bounded.
+#include <type_traits>
+
 #include "gated_scan.cuh"
 
 namespace omni {
 
 typedef __nv_bfloat16 bf16;
 
-constexpr int SR_STREAMS = 4, SR_TOK = 64, SR_MAX_BUF = 8;
+constexpr int SR_STREAMS = 4, SR_TOK = 32, SR_SLOTS = 2;
 constexpr int SR_THREADS = (4 * SR_STREAMS + 2) * 32;
 constexpr int SR_WBOX = 128 * 128;               // 64 channels (128 bytes) of 128 gate rows
 constexpr int SR_UBOX = SR_TOK * 128;            // 64 channels of a tile's tokens
 
+__device__ __forceinline__ float sr_ld(uint32_t addr) {
+  unsigned short v;
+  asm volatile("ld.shared.u16 %0, [%1];" : "=h"(v) : "r"(addr));
+  return __bfloat162float(__ushort_as_bfloat16(v));
+}
+__device__ __forceinline__ void sr_st(uint32_t addr, float x) {
+  asm volatile("st.shared.u16 [%0], %1;" ::"r"(addr), "h"(__bfloat16_as_ushort(__float2bfloat16(x))) : "memory");
+}
+
+// n_slots: tiles of a stream in flight (1 where shared memory allows no more)
 template <bool SUMS>
 __global__ void __launch_bounds__(SR_THREADS, 1)
 scan_runs_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmU,
-                 const __grid_constant__ GatedScan p, const int n_buf) {
+                 const __grid_constant__ CUtensorMap tmY, const __grid_constant__ GatedScan p, const int n_slots) {
   extern __shared__ uint8_t smem_raw[];
-  __shared__ __align__(8) uint64_t w_full, u_full[SR_MAX_BUF], u_empty[SR_MAX_BUF], t_full[SR_STREAMS], t_empty[SR_STREAMS];
+  __shared__ __align__(8) uint64_t w_full, full[SR_STREAMS][SR_SLOTS], t_full[SR_STREAMS][SR_SLOTS], done[SR_STREAMS][SR_SLOTS];
   __shared__ uint32_t tmem_base_s;
   __shared__ int s_abort;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -38,7 +52,8 @@ scan_runs_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
   const int ctiles = (p.part + 127) / 128;
   const int blk = blockIdx.x / ctiles, ct = blockIdx.x % ctiles;
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  const uint32_t sW = base, sU = base + 2 * kb * SR_WBOX;                  // u: [buffer][box]
+  const uint32_t sW = base, sT = base + 2 * kb * SR_WBOX;                  // tiles: [stream][slot]{u boxes, two y boxes}
+  const uint32_t t_bytes = (kb + 2) * SR_UBOX;
   int* status = p.status;
 
   // the runs of the block: sequence, first row, tokens, first run of the sequence
@@ -58,17 +73,16 @@ scan_runs_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
   if (threadIdx.x == 0) {
     s_abort = 0;
     mbar_init(smem_u32(&w_full), 1);
-    for (int i = 0; i < n_buf; ++i) {
-      mbar_init(smem_u32(&u_full[i]), 1);
-      mbar_init(smem_u32(&u_empty[i]), 1);
-    }
-    for (int s = 0; s < SR_STREAMS; ++s) {
-      mbar_init(smem_u32(&t_full[s]), 1);
-      mbar_init(smem_u32(&t_empty[s]), 4);                   // epilogue warps
-    }
+    for (int s = 0; s < SR_STREAMS; ++s)
+      for (int d = 0; d < SR_SLOTS; ++d) {
+        mbar_init(smem_u32(&full[s][d]), 1);
+        mbar_init(smem_u32(&t_full[s][d]), 1);
+        mbar_init(smem_u32(&done[s][d]), 4);                 // epilogue warps
+      }
     fence_mbar_init();
     tma_prefetch_desc(&tmW);
     tma_prefetch_desc(&tmU);
+    tma_prefetch_desc(&tmY);
   }
   if (warp == 17) {
     tmem_alloc(smem_u32(&tmem_base_s), 512);
@@ -90,7 +104,6 @@ scan_runs_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
         most = max(most, tiles[s]);
       }
       const uint32_t wb = smem_u32(&w_full);
-      int i = 0;                                             // tile count: buffer i % n_buf
       if (warp == 16) {
         mbar_expect_tx(wb, (uint32_t)(2 * kb * SR_WBOX));
         for (int g = 0; g < 2; ++g)
@@ -99,38 +112,37 @@ scan_runs_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
         for (int it = 0; it < most; ++it)
           for (int s = 0; s < SR_STREAMS; ++s) {
             if (it >= tiles[s]) continue;
-            const int b = i % n_buf;
-            mbar_wait(smem_u32(&u_empty[b]), ((i / n_buf) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
-            mbar_expect_tx(smem_u32(&u_full[b]), (uint32_t)(kb * SR_UBOX));
-            for (int x = 0; x < kb; ++x)
-              tma_load_3d(sU + (b * kb + x) * SR_UBOX, &tmU, smem_u32(&u_full[b]), 64 * x, row0[s] + it * SR_TOK, blk);
-            ++i;
+            const int d = it % n_slots;
+            const uint32_t fb = smem_u32(&full[s][d]), dst = sT + (s * n_slots + d) * t_bytes;
+            const int row = row0[s] + it * SR_TOK;
+            mbar_wait(smem_u32(&done[s][d]), ((it / n_slots) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
+            mbar_expect_tx(fb, SUMS ? (uint32_t)(kb * SR_UBOX) : t_bytes);
+            for (int x = 0; x < kb; ++x) tma_load_3d(dst + x * SR_UBOX, &tmU, fb, 64 * x, row, blk);
+            if (!SUMS)
+              for (int x = 0; x < 2; ++x) tma_load_3d(dst + (kb + x) * SR_UBOX, &tmY, fb, ct * 128 + 64 * x, row, blk);
           }
       } else {
         const uint32_t idesc = umma_idesc(128, SR_TOK, 1, 1, 0, 0);
-        const uint64_t dW = umma_desc_kmajor_sw128(sW), dU = umma_desc_kmajor_sw128(sU);
+        const uint64_t dW = umma_desc_kmajor_sw128(sW), dT = umma_desc_kmajor_sw128(sT);
         const uint64_t wbox = SR_WBOX >> 4, ubox = SR_UBOX >> 4;
         const int steps = p.part >> 4;
         mbar_wait(wb, 0, &s_abort, status, ERR_WAIT_FULL);
         for (int it = 0; it < most; ++it)
           for (int s = 0; s < SR_STREAMS; ++s) {
             if (it >= tiles[s]) continue;
-            const int b = i % n_buf;
-            mbar_wait(smem_u32(&t_empty[s]), (it & 1) ^ 1, &s_abort, status, ERR_WAIT_TMEM_EMPTY);
-            mbar_wait(smem_u32(&u_full[b]), (i / n_buf) & 1, &s_abort, status, ERR_WAIT_FULL);
+            const int d = it % n_slots;
+            mbar_wait(smem_u32(&full[s][d]), (it / n_slots) & 1, &s_abort, status, ERR_WAIT_FULL);
             tc_fence_after_sync();
-            const uint64_t u0 = dU + (uint64_t)(b * kb) * ubox;
+            const uint64_t u0 = dT + (uint64_t)((s * n_slots + d) * (t_bytes >> 4));
             for (int g = 0; g < 2; ++g) {
               const uint64_t w0 = dW + (uint64_t)(g * kb) * wbox;
-              const uint32_t d = tmem + (s * 2 + g) * SR_TOK;
+              const uint32_t acc = tmem + ((s * SR_SLOTS + d) * 2 + g) * SR_TOK;
               for (int k = 0; k < steps; ++k) {
                 const uint64_t in = (uint64_t)((k & 3) * 2);             // 16 channels = 32 bytes of a row
-                mma_f16_ss(d, w0 + (uint64_t)(k >> 2) * wbox + in, u0 + (uint64_t)(k >> 2) * ubox + in, idesc, k == 0 ? 0u : 1u);
+                mma_f16_ss(acc, w0 + (uint64_t)(k >> 2) * wbox + in, u0 + (uint64_t)(k >> 2) * ubox + in, idesc, k == 0 ? 0u : 1u);
               }
             }
-            tc_commit(smem_u32(&u_empty[b]));
-            tc_commit(smem_u32(&t_full[s]));
-            ++i;
+            tc_commit(smem_u32(&t_full[s][d]));
           }
       }
     }
@@ -157,44 +169,62 @@ scan_runs_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
         for (int i = first; i < run; ++i) S = fmaf(p.sums[(long)i * 2 * p.C + c], S, p.sums[((long)i * 2 + 1) * p.C + c]);
       }
     }
-    const float br = p.gates_b[c], bi = p.gates_b[p.C + c], decay2 = p.decay[c] * GS_LOG2E;
-    const bf16* y = static_cast<const bf16*>(p.proj) + (long)(q0 + off) * p.ldp + c;
-    const bf16* u = static_cast<const bf16*>(p.u) + (long)(q0 + off) * p.C + c;
-    bf16* out = static_cast<bf16*>(p.out) + (long)(q0 + off) * p.C + c;
-    for (int it = 0; it < tiles; ++it) {
-      const uint32_t ta = tmem + ((uint32_t)(q * 32) << 16) + s * 2 * SR_TOK;
+    const float nbr = -GS_LOG2E * p.gates_b[c], nbi = -GS_LOG2E * p.gates_b[p.C + c], decay2 = p.decay[c] * GS_LOG2E;
+    // a thread's channel in a row of a swizzled box: 16-byte piece `vec` ^ (row & 7)
+    const int vec = (q & 1) * 4 + (lane >> 3);
+    const uint32_t lane_off = (uint32_t)(vec << 4) + (lane & 7) * 2;
+    const uint32_t u_box = min((uint32_t)(2 * ct + (q >> 1)), (uint32_t)kb - 1) * SR_UBOX, y_box = (uint32_t)(kb + (q >> 1)) * SR_UBOX;
+    // 16-byte pieces of the warp's 32 channels that a lane stores: piece of the row, rows lane / 4 + 8 i
+    const int sv = (q & 1) * 4 + (lane & 3), sc = ct * 128 + q * 32 + (lane & 3) * 8;
+    bf16* out = static_cast<bf16*>(p.out) + (long)(q0 + off) * p.C + blk * p.part + sc;
+
+    auto walk = [&](auto whole, uint32_t ua, uint32_t ya, uint32_t ta, int nt) {
+      constexpr bool WHOLE = decltype(whole)::value;         // all 32 tokens exist
 #pragma unroll 1
       for (int k = 0; k < SR_TOK; k += 16) {
-        const int t0 = it * SR_TOK + k, left = n - t0;       // tokens of this chunk that exist
-        if (left <= 0 && k > 0) break;
-        bf16 uv[16], yv[16];
-#pragma unroll
-        for (int e = 0; e < 16; ++e) {
-          uv[e] = e < left ? u[(long)(t0 + e) * p.C] : __float2bfloat16(0.f);
-          if (!SUMS) yv[e] = e < left ? y[(long)(t0 + e) * p.ldp] : __float2bfloat16(0.f);
-        }
-        if (k == 0) {
-          mbar_wait(smem_u32(&t_full[s]), it & 1, &s_abort, status, ERR_WAIT_TMEM_FULL);
-          tc_fence_after_sync();
-        }
+        if (!WHOLE && k >= nt) break;
         uint32_t zr[16], zi[16];
         tmem_ld_32x16(ta + k, zr);
         tmem_ld_32x16(ta + SR_TOK + k, zi);
         tmem_wait_ld();
 #pragma unroll
         for (int e = 0; e < 16; ++e) {
+          const uint32_t at = (uint32_t)((e & 7) << 4), to = (uint32_t)(e * 128);
           float la2, a, add;
-          gate_step(__uint_as_float(zr[e]) + br, __uint_as_float(zi[e]) + bi, __bfloat162float(uv[e]), decay2, la2, a, add);
-          if (e < left) {
+          gate_step(__uint_as_float(zr[e]), __uint_as_float(zi[e]), nbr, nbi, sr_ld((ua ^ at) + to), decay2, la2, a, add);
+          if (WHOLE || k + e < nt) {
             S = fmaf(a, S, add);
             if (SUMS) la_sum += la2;
-            else if (ok) out[(long)(t0 + e) * p.C] = __float2bfloat16(S * gelu_short(__bfloat162float(yv[e])));
           }
+          if (!SUMS) sr_st((ya ^ at) + to, S * gelu_short(sr_ld((ya ^ at) + to)));
         }
+        ua += 16 * 128;
+        ya += 16 * 128;
+      }
+    };
+    for (int it = 0; it < tiles; ++it) {
+      const int d = it % n_slots, t0 = it * SR_TOK, nt = min(SR_TOK, n - t0);
+      const uint32_t tile = sT + (s * n_slots + d) * t_bytes;
+      const uint32_t ph = (it / n_slots) & 1;
+      mbar_wait(smem_u32(&full[s][d]), ph, &s_abort, status, ERR_WAIT_FULL);
+      mbar_wait(smem_u32(&t_full[s][d]), ph, &s_abort, status, ERR_WAIT_TMEM_FULL);
+      tc_fence_after_sync();
+      const uint32_t ta = tmem + ((uint32_t)(q * 32) << 16) + (s * SR_SLOTS + d) * 2 * SR_TOK;
+      if (nt == SR_TOK) walk(std::true_type{}, tile + u_box + lane_off, tile + y_box + lane_off, ta, nt);
+      else walk(std::false_type{}, tile + u_box + lane_off, tile + y_box + lane_off, ta, nt);
+      if (!SUMS) {
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < SR_TOK / 8; ++i) {
+          const int tk = i * 8 + (lane >> 2);
+          const uint4 v = ld_shared_v4(tile + y_box + tk * 128 + ((sv ^ (tk & 7)) << 4));
+          if (tk < nt && sc < p.part) *reinterpret_cast<uint4*>(out + (long)(t0 + tk) * p.C) = v;
+        }
+        fence_proxy_async_smem();
       }
       tc_fence_before_sync();
       __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(&t_empty[s]));
+      if (lane == 0) mbar_arrive(smem_u32(&done[s][d]));
     }
     if (n > 0 && ok) {
       if (SUMS) {
@@ -226,26 +256,28 @@ extern "C" int omni_scan_runs(const GatedScan* args, void* stream) {
   const GatedScan& p = *args;
   if (p.n_runs <= 0) return RC_OK;
   if (!scan_args_ok(p) || !p.runs || !p.u || p.part > 256 || (p.n_runs + SR_STREAMS - 1) / SR_STREAMS > 65535) return RC_BAD_ARG;
-  CUtensorMap tw, tu;
+  CUtensorMap tw, tu, ty;
   int rc = make_tmap_3d(&tw, p.gates, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.part, p.part, 2 * p.blocks, (uint64_t)p.part * 2,
                         (uint64_t)p.part * p.part * 2, 64, 128);
-  // u as (channel of a part, row, part)
+  // u and the gelu branch as (channel of a part, row, part)
   if (!rc) rc = make_tmap_3d(&tu, p.u, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.part, p.T, p.blocks, (uint64_t)p.C * 2,
+                             (uint64_t)p.part * 2, 64, SR_TOK);
+  if (!rc) rc = make_tmap_3d(&ty, p.proj, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.part, p.T, p.blocks, (uint64_t)p.ldp * 2,
                              (uint64_t)p.part * 2, 64, SR_TOK);
   if (rc) return rc;
   const int kb = (p.part + 63) / 64, limit = 226 * 1024;
-  int n_buf = (limit - 1024 - 2 * kb * SR_WBOX) / (kb * SR_UBOX);
-  if (n_buf > SR_MAX_BUF) n_buf = SR_MAX_BUF;
-  const int smem = 2 * kb * SR_WBOX + n_buf * kb * SR_UBOX + 1024;
+  const int tiles = SR_STREAMS * (kb + 2) * SR_UBOX;                        // one slot of every stream
+  const int n_slots = 2 * kb * SR_WBOX + 2 * tiles + 1024 <= limit ? 2 : 1;
+  const int smem = 2 * kb * SR_WBOX + n_slots * tiles + 1024;
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid(p.blocks * ((p.part + 127) / 128), (p.n_runs + SR_STREAMS - 1) / SR_STREAMS);
   static unsigned long long prep[2] = {0, 0};
   if (p.sums) {
     if (int e = ensure_dynamic_smem((const void*)scan_runs_kernel<true>, limit, prep[0])) return e;
-    scan_runs_kernel<true><<<grid, SR_THREADS, smem, st>>>(tw, tu, p, n_buf);
+    scan_runs_kernel<true><<<grid, SR_THREADS, smem, st>>>(tw, tu, ty, p, n_slots);
     if (int e = (int)cudaGetLastError()) return e;
   }
   if (int e = ensure_dynamic_smem((const void*)scan_runs_kernel<false>, limit, prep[1])) return e;
-  scan_runs_kernel<false><<<grid, SR_THREADS, smem, st>>>(tw, tu, p, n_buf);
+  scan_runs_kernel<false><<<grid, SR_THREADS, smem, st>>>(tw, tu, ty, p, n_slots);
   return (int)cudaGetLastError();
 }

@@ -10,8 +10,8 @@
 //                        out of it (W_uv o, times the output gate); weights are read once per 16 rows
 //   omni_latent_decode   decoded tokens (and rows of short portions): scores and weighted sums directly on the
 //                        latent rows, so a row is read once per 16 heads.  A block owns 16 heads of one token and
-//                        a share of its keys; 32-key tiles go through a two-deep cp.async ring, eight warps share the
-//                        score product by (keys, channel quarter) and the weighted sum by channels; two blocks per SM
+//                        a share of its keys; 16-key tiles go through a four-deep cp.async ring, eight warps share
+//                        the score product and the weighted sum by channels; two blocks per SM
 //
 // A decode step reads every latent once per group of heads and does little arithmetic on it, so the warp-level
 // products (no operand staging through tensor memory) suffice.
@@ -192,7 +192,7 @@ struct LatentDecode {
   float* part_o; float* part_ml;       // [n, H, splits, rank_p], [n, H, splits, 2]
 };
 
-constexpr int LD_KEYS = 32, LD_ROWS = 16;
+constexpr int LD_KEYS = 16, LD_ROWS = 16, LD_STAGES = 4;
 constexpr float LD_LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ float ld_ex2(float x) {
@@ -212,10 +212,10 @@ __device__ __forceinline__ void ld_m4t(uint32_t addr, uint32_t (&r)[4]) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-// shared memory of one block: two key tiles, the queries, weights (bf16) and four partial score tiles (fp32)
+// shared memory of one block: the key ring, the queries, weights (bf16) and eight partial score tiles (fp32)
 inline int latent_decode_smem(int row_ch) {
   const int pitch = row_ch * 2 + 16;
-  return 2 * LD_KEYS * pitch + LD_ROWS * pitch + LD_ROWS * (LD_KEYS * 2 + 16) + 4 * LD_ROWS * (LD_KEYS + 4) * 4;
+  return (LD_STAGES * LD_KEYS + LD_ROWS) * pitch + LD_ROWS * (LD_KEYS * 2 + 16) + 8 * LD_ROWS * (LD_KEYS + 4) * 4;
 }
 
 // CPW: 16-channel slices of the weighted sum per warp (rank_p <= 128 CPW).
@@ -234,28 +234,29 @@ latent_decode_kernel(const LatentDecode p) {
   const int per = (tiles_all + p.splits - 1) / p.splits;
   const int t0 = min(tiles_all, split * per), t1 = min(tiles_all, t0 + per);
   const int ch = p.rank_p + p.rot_p, pitch = ch * 2 + 16;
-  const uint32_t sK = smem_u32(smem), sQ = sK + 2 * LD_KEYS * pitch, sP = sQ + LD_ROWS * pitch;
-  float* sS = reinterpret_cast<float*>(smem + (2 * LD_KEYS + LD_ROWS) * pitch + LD_ROWS * pp);   // [4][LD_ROWS][SP]
+  const uint32_t sK = smem_u32(smem), sQ = sK + LD_STAGES * LD_KEYS * pitch, sP = sQ + LD_ROWS * pitch;
+  float* sS = reinterpret_cast<float*>(smem + (LD_STAGES * LD_KEYS + LD_ROWS) * pitch + LD_ROWS * pp);   // [8][LD_ROWS][SP]
 
-  // eight threads per key row, 16 bytes each; page numbers are looked up a tile ahead
+  // sixteen threads per key row, 16 bytes each; page numbers are looked up a tile ahead
   const int* bt = p.block_tables + (long)seq * p.bt_stride;
-  const int fr = tid >> 3, fc = (tid & 7) * 8;
+  const int fr = tid >> 4, fc = (tid & 15) * 8;
   auto lookup = [&](int t) { return bt[min(t * LD_KEYS + fr, n_vis - 1) / p.block_size]; };
-  auto fetch = [&](int t, int buf, int pg) {
+  auto fetch = [&](int t, int pg) {
     const int pos = min(t * LD_KEYS + fr, n_vis - 1);       // past the end: a valid key, masked below
     pg = min(max(pg, 0), p.num_blocks - 1);
     const bf16* src = p.pages + ((long)pg * p.block_size + pos % p.block_size) * ch;
-    const uint32_t dst = sK + (buf * LD_KEYS + fr) * pitch;
-#pragma unroll 3
-    for (int c = fc; c < ch; c += 64) ld_cp16(dst + c * 2, src + c);
+    const uint32_t dst = sK + (((t - t0) & (LD_STAGES - 1)) * LD_KEYS + fr) * pitch;
+    for (int c = fc; c < ch; c += 128) ld_cp16(dst + c * 2, src + c);
   };
-  int page = 0;
-  if (t0 < t1) {
-    page = lookup(t0);
-    fetch(t0, 0, page);
-    if (t0 + 1 < t1) page = lookup(t0 + 1);
+  int page = t0 < t1 ? lookup(t0) : 0;
+#pragma unroll
+  for (int i = 0; i < LD_STAGES - 1; ++i) {
+    if (t0 + i < t1) {
+      fetch(t0 + i, page);
+      if (t0 + i + 1 < t1) page = lookup(t0 + i + 1);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
   }
-  asm volatile("cp.async.commit_group;" ::: "memory");
   // queries: latent part, rotated part; rows past the last head are zero
   for (int i = tid; i < LD_ROWS * (ch / 8); i += 256) {
     const int r = i / (ch / 8), c = (i - r * (ch / 8)) * 8;
@@ -268,9 +269,8 @@ latent_decode_kernel(const LatentDecode p) {
     st_shared_v4(sQ + r * pitch + c * 2, v);
   }
 
-  const int quarter = warp >> 1, kg = warp & 1;             // score product: channel quarter, group of 16 keys
-  const int steps = ch / 16, k_lo = steps * quarter / 4, k_hi = steps * (quarter + 1) / 4;
-  const int srow = tid >> 4, sk0 = (tid & 15) * 2;          // softmax: row and first of two keys of this thread
+  const int steps = ch / 16, k_lo = steps * warp / 8, k_hi = steps * (warp + 1) / 8;   // score product: this warp's channels
+  const int srow = tid >> 4, skey = tid & 15;               // softmax: row and key of this thread
   float m_run = -INFINITY, l_run = 0.f;
   const float mul = p.scale * LD_LOG2E;
   float acc[CPW][2][4];
@@ -282,19 +282,18 @@ latent_decode_kernel(const LatentDecode p) {
       for (int i = 0; i < 4; ++i) acc[c][n][i] = 0.f;
 
   for (int t = t0; t < t1; ++t) {
-    const int buf = (t - t0) & 1;
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                        // tile t is here; everyone is done with the other buffer
-    if (t + 1 < t1) {
-      fetch(t + 1, buf ^ 1, page);
-      if (t + 2 < t1) page = lookup(t + 2);
+    asm volatile("cp.async.wait_group %0;" ::"n"(LD_STAGES - 2) : "memory");
+    __syncthreads();                                        // tile t is here; everyone is done with tile t - 1
+    if (t + LD_STAGES - 1 < t1) {
+      fetch(t + LD_STAGES - 1, page);
+      if (t + LD_STAGES < t1) page = lookup(t + LD_STAGES);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
-    const uint32_t kt = sK + buf * LD_KEYS * pitch;
+    const uint32_t kt = sK + ((t - t0) & (LD_STAGES - 1)) * LD_KEYS * pitch;
     {
       float s[2][4] = {};
       // K matrices: keys 0-7 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 0-7 | keys 8-15 ch 8-15
-      const uint32_t ka = kt + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
+      const uint32_t ka = kt + ((lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
       // Q matrices: rows 0-7 ch 0-7 | rows 8-15 ch 0-7 | rows 0-7 ch 8-15 | rows 8-15 ch 8-15
       const uint32_t qa = sQ + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
 #pragma unroll 5
@@ -309,32 +308,25 @@ latent_decode_kernel(const LatentDecode p) {
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int u = 0; u < 2; ++u)
-          *reinterpret_cast<float2*>(sS + (quarter * LD_ROWS + u * 8 + (lane >> 2)) * SP + kg * 16 + n * 8 + (lane & 3) * 2) =
+          *reinterpret_cast<float2*>(sS + (warp * LD_ROWS + u * 8 + (lane >> 2)) * SP + n * 8 + (lane & 3) * 2) =
               make_float2(s[n][2 * u], s[n][2 * u + 1]);
     }
     __syncthreads();
     {
-      float2 y = make_float2(0.f, 0.f);
+      float y = 0.f;
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
-        const float2 v = *reinterpret_cast<const float2*>(sS + (q * LD_ROWS + srow) * SP + sk0);
-        y.x += v.x;
-        y.y += v.y;
-      }
-      const int left = n_vis - t * LD_KEYS - sk0;           // keys of this thread that are visible
-      y.x = left > 0 ? y.x * mul : -INFINITY;
-      y.y = left > 1 ? y.y * mul : -INFINITY;
-      float mx = fmaxf(y.x, y.y);
+      for (int q = 0; q < 8; ++q) y += sS[(q * LD_ROWS + srow) * SP + skey];
+      y = t * LD_KEYS + skey < n_vis ? y * mul : -INFINITY;
+      float mx = y;
 #pragma unroll
       for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       const float m_new = fmaxf(m_run, mx);                 // finite: a tile holds at least one visible key
       const float alpha = ld_ex2(m_run - m_new);
-      y.x = ld_ex2(y.x - m_new);
-      y.y = ld_ex2(y.y - m_new);
-      l_run = fmaf(l_run, alpha, y.x + y.y);                // this thread's keys only; summed at the end
+      y = ld_ex2(y - m_new);
+      l_run = fmaf(l_run, alpha, y);                        // this thread's keys only; summed at the end
       m_run = m_new;
-      if ((tid & 15) == 0) s_alpha[srow] = alpha;
-      asm volatile("st.shared.b32 [%0], %1;" ::"r"(sP + srow * pp + sk0 * 2), "r"(pack_bf16(y.x, y.y)) : "memory");
+      if (skey == 0) s_alpha[srow] = alpha;
+      asm volatile("st.shared.b16 [%0], %1;" ::"r"(sP + srow * pp + skey * 2), "h"(__bfloat16_as_ushort(__float2bfloat16(y))) : "memory");
     }
     __syncthreads();
     const float a0 = s_alpha[lane >> 2], a1 = s_alpha[8 + (lane >> 2)];

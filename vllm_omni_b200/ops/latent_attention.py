@@ -192,7 +192,7 @@ def decode_splits(blocks: int, keys: int, slots: int = 2 * 148) -> int:
     best, best_cost = 1, None
     for n in range(1, max(1, min(64, (keys + 255) // 256)) + 1):
         waves = -(-blocks * n // slots)
-        cost = waves * (-(-keys // (32 * n)) + 4)           # key tiles of a block and its start-up, per wave
+        cost = waves * (-(-keys // (16 * n)) + 8)           # key tiles of a block and its start-up, per wave
         if best_cost is None or cost < best_cost:
             best, best_cost = n, cost
     return best
