@@ -64,6 +64,8 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
                     "bound": "tensor" if a >= b else "memory", "of_measured": round(max(a, b) / ms, 3)})
 
     rnd = lambda *sh, dt=bf: torch.randn(*sh, dtype=dt, device=dev)
+    one, tiny = torch.zeros(1, dtype=torch.int64, device=dev), torch.zeros(1, 8, dtype=bf, device=dev)
+    row("timing floor", "an 8-channel lookup", lambda: stream.gelu_lookup_(tiny, tiny, one, 0, 8), bytes_=48.0)
     # ---- attention of a prompt
     q, k, v = rnd(1, T, H, DIM), rnd(1, T, G, DIM), rnd(1, T, G, DIM)
     o = rnd(T, H * DIM)
@@ -152,14 +154,17 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
             ci(width), ci(E), ci(E), ci(k2), P(idb), P(wtb), nv.stream_ptr()), bytes_=rbytes, flops=2.0 * rows_ * E * width)
         up, down = rnd(E, F2, width) * 0.02, rnd(E, width, F2) * 0.02
         er = moe.expert_rows(xr, rw, rb, E, k2, up, down, act="relu2")
-        ws = moe.MoEWorkspace()
-        n_used = min(E, rows_ * k2)
+        ws, ws_q = moe.MoEWorkspace(), moe.MoEWorkspace()
+        moe.expert_rows(xr, rw, rb, E, k2, up, down, act="relu2", ws=ws)
+        n_used = ws.ids.unique().numel()                            # experts whose weights are read
         row(f"experts, {tag}", "nidilix (router to expert rows)", lambda: moe.expert_rows(xr, rw, rb, E, k2, up, down, act="relu2", ws=ws),
             flops=4.0 * rows_ * k2 * width * F2, bytes_=4.0 * n_used * width * F2)
         w13, w2 = rnd(E, 2 * F_, width) * 0.02, rnd(E, width, F_) * 0.02
         lg = gemm.linear(xr, rw)
-        row(f"experts, {tag}", "qwen3_moe (route to combined rows)", lambda: moe.moe_forward(xr, lg, w13, w2, s["top"], ws=ws, residual=xr, out=xr),
-            flops=6.0 * rows_ * s["top"] * width * F_, bytes_=6.0 * min(E, rows_ * s["top"]) * width * F_)
+        moe.moe_forward(xr, lg, w13, w2, s["top"], ws=ws_q)
+        n_used_q = ws_q.ids.unique().numel()
+        row(f"experts, {tag}", "qwen3_moe (route to combined rows)", lambda: moe.moe_forward(xr, lg, w13, w2, s["top"], ws=ws_q, residual=xr, out=torch.empty_like(xr)),
+            flops=6.0 * rows_ * s["top"] * width * F_, bytes_=6.0 * n_used_q * width * F_)
         if rows_ == T:
             sh = rnd(T, width)
             row("experts' sum", "nidilix (sum + shared + add + cast)", lambda: stream.add_expert_rows_(x, er, sh, 0.5, xn, stream.CAST),

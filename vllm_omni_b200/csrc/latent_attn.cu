@@ -9,9 +9,11 @@
 //   omni_head_gemm       one small product per head: queries into the latent space (W_uk^T q) and attention results
 //                        out of it (W_uv o, times the output gate); weights are read once per 16 rows
 //   omni_latent_decode   decoded tokens (and rows of short portions): scores and weighted sums directly on the
-//                        latent rows, so a row is read once per 16 heads.  A block owns 16 heads of one token and
-//                        a share of its keys; 16-key tiles go through a four-deep cp.async ring, eight warps share
-//                        the score product and the weighted sum by channels; two blocks per SM
+//                        latent rows, so a row is read once per 16 or 32 heads.  A block owns one token's heads and a
+//                        share of its keys; a producer warp copies 32-key tiles into a ring (bulk copies), two groups of
+//                        eight warps take tiles in turn (or, with more than 16 heads, the same tile for 16 heads each);
+//                        a group's warps share the score product by (keys, channel quarter) and the weighted sum by
+//                        channels.  Every wait is bounded
 //
 // A decode step reads every latent once per group of heads and does little arithmetic on it, so the warp-level
 // products (no operand staging through tensor memory) suffice.
@@ -190,9 +192,10 @@ struct LatentDecode {
   bf16* out;                           // [n, H, rank_p]
   int H, splits;
   float* part_o; float* part_ml;       // [n, H, splits, rank_p], [n, H, splits, 2]
+  int* status;
 };
 
-constexpr int LD_KEYS = 16, LD_ROWS = 16, LD_STAGES = 4;
+constexpr int LD_KEYS = 32, LD_ROWS = 16, LD_MAX_STAGES = 8;
 constexpr float LD_LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ float ld_ex2(float x) {
@@ -200,8 +203,11 @@ __device__ __forceinline__ float ld_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ void ld_cp16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+// contiguous bytes to shared memory, counted on an mbarrier (both addresses and the size: multiples of 16)
+__device__ __forceinline__ void ld_bulk(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes),
+               "r"(bar)
+               : "memory");
 }
 __device__ __forceinline__ void ld_m4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -212,67 +218,60 @@ __device__ __forceinline__ void ld_m4t(uint32_t addr, uint32_t (&r)[4]) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 
-// shared memory of one block: the key ring, the queries, weights (bf16) and eight partial score tiles (fp32)
-inline int latent_decode_smem(int row_ch) {
+// shared memory of one block: the key ring, the queries, and per group of warps the weights (bf16) and four partial
+// score tiles (fp32)
+constexpr int LD_GROUP_BYTES = LD_ROWS * (LD_KEYS * 2 + 16) + 4 * LD_ROWS * (LD_KEYS + 4) * 4;
+constexpr int LD_LIMIT = 226 * 1024;
+
+inline int latent_decode_stages(int row_ch, bool wide) {
   const int pitch = row_ch * 2 + 16;
-  return (LD_STAGES * LD_KEYS + LD_ROWS) * pitch + LD_ROWS * (LD_KEYS * 2 + 16) + 8 * LD_ROWS * (LD_KEYS + 4) * 4;
+  const int n = (LD_LIMIT - 2 * LD_GROUP_BYTES - (wide ? 2 : 1) * LD_ROWS * pitch) / (LD_KEYS * pitch);
+  return n < LD_MAX_STAGES ? n : LD_MAX_STAGES;
 }
 
-// CPW: 16-channel slices of the weighted sum per warp (rank_p <= 128 CPW).
-template <int CPW>
-__global__ void __launch_bounds__(256, 2)
-latent_decode_kernel(const LatentDecode p) {
-  constexpr int SP = LD_KEYS + 4, pp = LD_KEYS * 2 + 16;
+// CPW: 16-channel slices of the weighted sum per warp (rank_p <= 128 CPW).  WIDE: more than 16 heads, the two groups of
+// warps own 16 heads each and share every tile; otherwise they own the same heads and take tiles in turn.
+template <int CPW, bool WIDE>
+__global__ void __launch_bounds__(544, 1)
+latent_decode_kernel(const LatentDecode p, const int stages) {
+  constexpr int SP = LD_KEYS + 4, pp = LD_KEYS * 2 + 16, QROWS = WIDE ? 2 * LD_ROWS : LD_ROWS;
   extern __shared__ __align__(16) uint8_t smem[];
-  __shared__ float s_alpha[LD_ROWS], s_m[LD_ROWS], s_l[LD_ROWS];
+  __shared__ __align__(8) uint64_t k_full[LD_MAX_STAGES], k_empty[LD_MAX_STAGES];
+  __shared__ float s_alpha[2][LD_ROWS], s_m[2][LD_ROWS], s_l[2][LD_ROWS];
+  __shared__ int s_abort;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h0 = blockIdx.y * LD_ROWS, nh = min(LD_ROWS, p.H - h0), split = blockIdx.z;
+  const int h0 = blockIdx.y * QROWS, split = blockIdx.z;
   const int row = min(max(p.rows[blockIdx.x], 0), p.T - 1);
   const int seq = min(max(p.row_seq[row], 0), p.num_seqs - 1);
   const int n_vis = p.context[seq] + row - p.q_start[seq] + 1;
   const int tiles_all = (n_vis + LD_KEYS - 1) / LD_KEYS;
   const int per = (tiles_all + p.splits - 1) / p.splits;
-  const int t0 = min(tiles_all, split * per), t1 = min(tiles_all, t0 + per);
+  const int t0 = min(tiles_all, split * per), n_tiles = min(tiles_all, t0 + per) - t0;
   const int ch = p.rank_p + p.rot_p, pitch = ch * 2 + 16;
-  const uint32_t sK = smem_u32(smem), sQ = sK + LD_STAGES * LD_KEYS * pitch, sP = sQ + LD_ROWS * pitch;
-  float* sS = reinterpret_cast<float*>(smem + (LD_STAGES * LD_KEYS + LD_ROWS) * pitch + LD_ROWS * pp);   // [8][LD_ROWS][SP]
+  const uint32_t sK = smem_u32(smem), sQ = sK + stages * LD_KEYS * pitch, sG = sQ + QROWS * pitch;
 
-  // sixteen threads per key row, 16 bytes each; page numbers are looked up a tile ahead
-  const int* bt = p.block_tables + (long)seq * p.bt_stride;
-  const int fr = tid >> 4, fc = (tid & 15) * 8;
-  auto lookup = [&](int t) { return bt[min(t * LD_KEYS + fr, n_vis - 1) / p.block_size]; };
-  auto fetch = [&](int t, int pg) {
-    const int pos = min(t * LD_KEYS + fr, n_vis - 1);       // past the end: a valid key, masked below
-    pg = min(max(pg, 0), p.num_blocks - 1);
-    const bf16* src = p.pages + ((long)pg * p.block_size + pos % p.block_size) * ch;
-    const uint32_t dst = sK + (((t - t0) & (LD_STAGES - 1)) * LD_KEYS + fr) * pitch;
-    for (int c = fc; c < ch; c += 128) ld_cp16(dst + c * 2, src + c);
-  };
-  int page = t0 < t1 ? lookup(t0) : 0;
-#pragma unroll
-  for (int i = 0; i < LD_STAGES - 1; ++i) {
-    if (t0 + i < t1) {
-      fetch(t0 + i, page);
-      if (t0 + i + 1 < t1) page = lookup(t0 + i + 1);
+  if (tid == 0) {
+    s_abort = 0;
+    for (int i = 0; i < stages; ++i) {
+      mbar_init(smem_u32(&k_full[i]), 1);
+      mbar_init(smem_u32(&k_empty[i]), WIDE ? 16 : 8);       // warps that read a tile
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    fence_mbar_init();
   }
   // queries: latent part, rotated part; rows past the last head are zero
-  for (int i = tid; i < LD_ROWS * (ch / 8); i += 256) {
+  for (int i = tid; i < QROWS * (ch / 8); i += 544) {
     const int r = i / (ch / 8), c = (i - r * (ch / 8)) * 8;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < nh) {
+    if (h0 + r < p.H) {
       const bf16* src = c < p.rank_p ? p.q_lat + ((long)blockIdx.x * p.H + h0 + r) * p.rank_p + c
                                      : p.proj + (long)row * p.ldp + (long)(h0 + r) * p.head_cols + p.dim_p + (c - p.rank_p);
       v = *reinterpret_cast<const uint4*>(src);
     }
     st_shared_v4(sQ + r * pitch + c * 2, v);
   }
+  __syncthreads();
 
-  const int steps = ch / 16, k_lo = steps * warp / 8, k_hi = steps * (warp + 1) / 8;   // score product: this warp's channels
-  const int srow = tid >> 4, skey = tid & 15;               // softmax: row and key of this thread
-  float m_run = -INFINITY, l_run = 0.f;
-  const float mul = p.scale * LD_LOG2E;
+  const int grp = (warp >> 3) & 1, gw = warp & 7, gt = tid & 255;
   float acc[CPW][2][4];
 #pragma unroll
   for (int c = 0; c < CPW; ++c)
@@ -281,112 +280,191 @@ latent_decode_kernel(const LatentDecode p) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[c][n][i] = 0.f;
 
-  for (int t = t0; t < t1; ++t) {
-    asm volatile("cp.async.wait_group %0;" ::"n"(LD_STAGES - 2) : "memory");
-    __syncthreads();                                        // tile t is here; everyone is done with tile t - 1
-    if (t + LD_STAGES - 1 < t1) {
-      fetch(t + LD_STAGES - 1, page);
-      if (t + LD_STAGES < t1) page = lookup(t + LD_STAGES);
+  if (warp == 16) {
+    // ------------------------------------------- producer: a lane copies one key row, pages are looked up a tile ahead
+    const int* bt = p.block_tables + (long)seq * p.bt_stride;
+    auto src_row = [&](int t) {
+      const int pos = min((t0 + t) * LD_KEYS + lane, n_vis - 1);           // past the end: a valid key, masked below
+      const int pg = min(max(bt[pos / p.block_size], 0), p.num_blocks - 1);
+      return p.pages + ((long)pg * p.block_size + pos % p.block_size) * ch;
+    };
+    const bf16* next = n_tiles > 0 ? src_row(0) : nullptr;
+    int st = 0;
+    uint32_t ph = 1;
+    for (int t = 0; t < n_tiles; ++t) {
+      const bf16* src = next;
+      if (t + 1 < n_tiles) next = src_row(t + 1);
+      const uint32_t bar = smem_u32(&k_full[st]);
+      mbar_wait(smem_u32(&k_empty[st]), ph, &s_abort, p.status, ERR_WAIT_EMPTY);
+      if (lane == 0) mbar_expect_tx(bar, (uint32_t)(LD_KEYS * ch * 2));
+      __syncwarp();
+      ld_bulk(sK + (st * LD_KEYS + lane) * pitch, src, (uint32_t)(ch * 2), bar);
+      if (++st == stages) {
+        st = 0;
+        ph ^= 1;
+      }
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-    const uint32_t kt = sK + ((t - t0) & (LD_STAGES - 1)) * LD_KEYS * pitch;
-    {
-      float s[2][4] = {};
-      // K matrices: keys 0-7 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 0-7 | keys 8-15 ch 8-15
-      const uint32_t ka = kt + ((lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
-      // Q matrices: rows 0-7 ch 0-7 | rows 8-15 ch 0-7 | rows 0-7 ch 8-15 | rows 8-15 ch 8-15
-      const uint32_t qa = sQ + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
+  } else {
+    const uint32_t sP = sG + grp * LD_GROUP_BYTES;
+    float* sS = reinterpret_cast<float*>(smem + (sP - sK) + LD_ROWS * pp);                 // [4][LD_ROWS][SP]
+    const uint32_t q0 = sQ + (WIDE ? grp * LD_ROWS * pitch : 0);
+    const int quarter = gw >> 1, kg = gw & 1;                // score product: channel quarter, group of 16 keys
+    const int steps = ch / 16, k_lo = steps * quarter / 4, k_hi = steps * (quarter + 1) / 4;
+    const int srow = gt >> 4, sk0 = (gt & 15) * 2;           // softmax: row and first of two keys of this thread
+    float m_run = -INFINITY, l_run = 0.f;
+    const float mul = p.scale * LD_LOG2E;
+    auto group_sync = [&]() { asm volatile("bar.sync %0, 256;" ::"r"(1 + grp) : "memory"); };
+    for (int t = WIDE ? 0 : grp; t < n_tiles; t += WIDE ? 1 : 2) {
+      const int st = t % stages;
+      mbar_wait(smem_u32(&k_full[st]), (t / stages) & 1, &s_abort, p.status, ERR_WAIT_FULL);
+      const uint32_t kt = sK + st * LD_KEYS * pitch;
+      {
+        float s[2][4] = {};
+        // K matrices: keys 0-7 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 0-7 | keys 8-15 ch 8-15
+        const uint32_t ka = kt + (kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * pitch + ((lane >> 3) & 1) * 16;
+        // Q matrices: rows 0-7 ch 0-7 | rows 8-15 ch 0-7 | rows 0-7 ch 8-15 | rows 8-15 ch 8-15
+        const uint32_t qa = q0 + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
 #pragma unroll 5
-      for (int k = k_lo; k < k_hi; ++k) {
-        uint32_t a[4], b[4];
-        ld_m4(ka + k * 32, b);
-        ld_m4(qa + k * 32, a);
-        mma_bf16(s[0], a[0], a[1], a[2], a[3], b[0], b[1]);
-        mma_bf16(s[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        for (int k = k_lo; k < k_hi; ++k) {
+          uint32_t a[4], b[4];
+          ld_m4(ka + k * 32, b);
+          ld_m4(qa + k * 32, a);
+          mma_bf16(s[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+          mma_bf16(s[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int u = 0; u < 2; ++u)
+            *reinterpret_cast<float2*>(sS + (quarter * LD_ROWS + u * 8 + (lane >> 2)) * SP + kg * 16 + n * 8 + (lane & 3) * 2) =
+                make_float2(s[n][2 * u], s[n][2 * u + 1]);
       }
+      group_sync();
+      {
+        float2 y = make_float2(0.f, 0.f);
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
+        for (int q = 0; q < 4; ++q) {
+          const float2 v = *reinterpret_cast<const float2*>(sS + (q * LD_ROWS + srow) * SP + sk0);
+          y.x += v.x;
+          y.y += v.y;
+        }
+        const int left = n_vis - (t0 + t) * LD_KEYS - sk0;   // keys of this thread that are visible
+        y.x = left > 0 ? y.x * mul : -INFINITY;
+        y.y = left > 1 ? y.y * mul : -INFINITY;
+        float mx = fmaxf(y.x, y.y);
 #pragma unroll
-        for (int u = 0; u < 2; ++u)
-          *reinterpret_cast<float2*>(sS + (warp * LD_ROWS + u * 8 + (lane >> 2)) * SP + n * 8 + (lane & 3) * 2) =
-              make_float2(s[n][2 * u], s[n][2 * u + 1]);
-    }
-    __syncthreads();
-    {
-      float y = 0.f;
-#pragma unroll
-      for (int q = 0; q < 8; ++q) y += sS[(q * LD_ROWS + srow) * SP + skey];
-      y = t * LD_KEYS + skey < n_vis ? y * mul : -INFINITY;
-      float mx = y;
-#pragma unroll
-      for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float m_new = fmaxf(m_run, mx);                 // finite: a tile holds at least one visible key
-      const float alpha = ld_ex2(m_run - m_new);
-      y = ld_ex2(y - m_new);
-      l_run = fmaf(l_run, alpha, y);                        // this thread's keys only; summed at the end
-      m_run = m_new;
-      if (skey == 0) s_alpha[srow] = alpha;
-      asm volatile("st.shared.b16 [%0], %1;" ::"r"(sP + srow * pp + skey * 2), "h"(__bfloat16_as_ushort(__float2bfloat16(y))) : "memory");
-    }
-    __syncthreads();
-    const float a0 = s_alpha[lane >> 2], a1 = s_alpha[8 + (lane >> 2)];
-#pragma unroll
-    for (int c = 0; c < CPW; ++c)
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        acc[c][n][0] *= a0; acc[c][n][1] *= a0;
-        acc[c][n][2] *= a1; acc[c][n][3] *= a1;
+        for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float m_new = fmaxf(m_run, mx);                // finite: a tile holds at least one visible key
+        const float alpha = ld_ex2(m_run - m_new);
+        y.x = ld_ex2(y.x - m_new);
+        y.y = ld_ex2(y.y - m_new);
+        l_run = fmaf(l_run, alpha, y.x + y.y);               // this thread's keys only; summed at the end
+        m_run = m_new;
+        if ((gt & 15) == 0) s_alpha[grp][srow] = alpha;
+        asm volatile("st.shared.b32 [%0], %1;" ::"r"(sP + srow * pp + sk0 * 2), "r"(pack_bf16(y.x, y.y)) : "memory");
       }
-    const uint32_t pa = sP + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pp + (lane >> 4) * 16;
-    // V matrices, transposed: keys 0-7 ch 0-7 | keys 8-15 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 8-15
-    const uint32_t va = kt + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
+      group_sync();
+      const float a0 = s_alpha[grp][lane >> 2], a1 = s_alpha[grp][8 + (lane >> 2)];
+      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
-    for (int k = 0; k < LD_KEYS / 16; ++k) {
-      uint32_t a[4];
-      ld_m4(pa + k * 32, a);
+        for (int c = 0; c < CPW; ++c)
 #pragma unroll
-      for (int c = 0; c < CPW; ++c) {
-        const int sl = c * 8 + warp;
-        if (sl * 16 < p.rank_p) {
-          uint32_t b[4];
-          ld_m4t(va + k * 16 * pitch + sl * 32, b);
-          mma_bf16(acc[c][0], a[0], a[1], a[2], a[3], b[0], b[1]);
-          mma_bf16(acc[c][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+          for (int n = 0; n < 2; ++n) {
+            acc[c][n][0] *= a0; acc[c][n][1] *= a0;
+            acc[c][n][2] *= a1; acc[c][n][3] *= a1;
+          }
+      }
+      const uint32_t pa = sP + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pp + (lane >> 4) * 16;
+      // V matrices, transposed: keys 0-7 ch 0-7 | keys 8-15 ch 0-7 | keys 0-7 ch 8-15 | keys 8-15 ch 8-15
+      const uint32_t va = kt + ((lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + (lane >> 4) * 16;
+#pragma unroll
+      for (int k = 0; k < LD_KEYS / 16; ++k) {
+        uint32_t a[4];
+        ld_m4(pa + k * 32, a);
+#pragma unroll
+        for (int c = 0; c < CPW; ++c) {
+          const int sl = c * 8 + gw;
+          if (sl * 16 < p.rank_p) {
+            uint32_t b[4];
+            ld_m4t(va + k * 16 * pitch + sl * 32, b);
+            mma_bf16(acc[c][0], a[0], a[1], a[2], a[3], b[0], b[1]);
+            mma_bf16(acc[c][1], a[0], a[1], a[2], a[3], b[2], b[3]);
+          }
         }
       }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&k_empty[st]));
+    }
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, o);
+    if ((gt & 15) == 0) {
+      s_m[grp][srow] = m_run;
+      s_l[grp][srow] = l_run;
     }
   }
-#pragma unroll
-  for (int o = 8; o > 0; o >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, o);
-  if ((tid & 15) == 0) {
-    s_m[srow] = m_run;
-    s_l[srow] = l_run;
+  __syncthreads();                                           // every tile is read
+  if (s_abort) {
+    // a wait ran out: give copies in flight time to finish before their memory goes
+    const unsigned long long t_end = globaltimer_ns() + 200000ull;
+    while (globaltimer_ns() < t_end) {
+    }
   }
-  __syncthreads();
+  if (!WIDE) {
+    // the second group's sums join the first's through the ring's memory
+    float* other = reinterpret_cast<float*>(smem);           // [LD_ROWS][rank_p]
+    if (warp < 16 && grp == 1) {
+#pragma unroll
+      for (int c = 0; c < CPW; ++c)
+        if ((c * 8 + gw) * 16 < p.rank_p)
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+              *reinterpret_cast<float2*>(other + (u * 8 + (lane >> 2)) * p.rank_p + (c * 8 + gw) * 16 + n * 8 + (lane & 3) * 2) =
+                  make_float2(acc[c][n][2 * u], acc[c][n][2 * u + 1]);
+    }
+    __syncthreads();
+  }
+  if (warp == 16 || (!WIDE && grp == 1)) return;
+  const float* other = reinterpret_cast<const float*>(smem);
 #pragma unroll
   for (int u = 0; u < 2; ++u) {
-    const int r = u * 8 + (lane >> 2);
-    if (r >= nh) continue;
-    const long hi = (long)blockIdx.x * p.H + h0 + r;
+    const int r = u * 8 + (lane >> 2), h = h0 + (WIDE ? grp * LD_ROWS : 0) + r;
+    if (h >= p.H) continue;
+    const long hi = (long)blockIdx.x * p.H + h;
+    float m = s_m[grp][r], l = s_l[grp][r], f0 = 1.f, f1 = 0.f;
+    if (!WIDE) {                                             // group 0 has a tile wherever group 1 has one
+      const float m1 = s_m[1][r];
+      const float top = fmaxf(m, m1);
+      f0 = m == -INFINITY ? 0.f : ld_ex2(m - top);
+      f1 = m1 == -INFINITY ? 0.f : ld_ex2(m1 - top);
+      l = l * f0 + s_l[1][r] * f1;
+      m = top;
+    }
 #pragma unroll
     for (int c = 0; c < CPW; ++c) {
-      const int sl = c * 8 + warp;
+      const int sl = c * 8 + gw;
       if (sl * 16 >= p.rank_p) continue;
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
         const int col = sl * 16 + n * 8 + (lane & 3) * 2;
-        const float x = acc[c][n][2 * u], y = acc[c][n][2 * u + 1];
+        float x = acc[c][n][2 * u], y = acc[c][n][2 * u + 1];
+        if (!WIDE) {
+          const float2 o = *reinterpret_cast<const float2*>(other + r * p.rank_p + col);
+          x = x * f0 + o.x * f1;
+          y = y * f0 + o.y * f1;
+        }
         if (p.splits == 1) {
-          const float f = 1.0f / s_l[r];
+          const float f = 1.0f / l;
           *reinterpret_cast<uint32_t*>(p.out + hi * p.rank_p + col) = pack_bf16(x * f, y * f);
         } else {
           *reinterpret_cast<float2*>(p.part_o + (hi * p.splits + split) * p.rank_p + col) = make_float2(x, y);
         }
       }
     }
-    if (p.splits > 1 && warp == 0 && (lane & 3) == 0) {
-      p.part_ml[2 * (hi * p.splits + split)] = s_m[r];
-      p.part_ml[2 * (hi * p.splits + split) + 1] = s_l[r];
+    if (p.splits > 1 && gw == 0 && (lane & 3) == 0) {
+      p.part_ml[2 * (hi * p.splits + split)] = m;
+      p.part_ml[2 * (hi * p.splits + split) + 1] = l;
     }
   }
 }
@@ -415,13 +493,19 @@ latent_merge_kernel(const LatentDecode p) {
   }
 }
 
-template <int CPW>
+template <int CPW, bool WIDE>
 static int launch_latent_decode(const LatentDecode& p, cudaStream_t st) {
   static unsigned long long prep = 0;
-  if (int e = ensure_dynamic_smem((const void*)latent_decode_kernel<CPW>, 227 * 1024 - 1024, prep)) return e;
-  dim3 grid(p.n, (p.H + LD_ROWS - 1) / LD_ROWS, p.splits);
-  latent_decode_kernel<CPW><<<grid, 256, latent_decode_smem(p.rank_p + p.rot_p), st>>>(p);
+  if (int e = ensure_dynamic_smem((const void*)latent_decode_kernel<CPW, WIDE>, LD_LIMIT, prep)) return e;
+  const int heads = WIDE ? 2 * LD_ROWS : LD_ROWS, ch = p.rank_p + p.rot_p, stages = latent_decode_stages(ch, WIDE);
+  const int smem = (stages * LD_KEYS + heads) * (ch * 2 + 16) + 2 * LD_GROUP_BYTES;
+  latent_decode_kernel<CPW, WIDE><<<dim3(p.n, (p.H + heads - 1) / heads, p.splits), 544, smem, st>>>(p, stages);
   return (int)cudaGetLastError();
+}
+
+template <int CPW>
+static int pick_latent_decode(const LatentDecode& p, bool wide, cudaStream_t st) {
+  return wide ? launch_latent_decode<CPW, true>(p, st) : launch_latent_decode<CPW, false>(p, st);
 }
 
 }  // namespace omni
@@ -462,21 +546,24 @@ extern "C" int omni_head_gemm(const HeadGemm* args, void* stream) {
 }
 
 // 0: the sizes do not fit the decode kernel; otherwise the heads a block serves.
-extern "C" int omni_latent_decode_heads(int rank_p, int rot_p) {
+extern "C" int omni_latent_decode_heads(int heads, int rank_p, int rot_p) {
   if (rank_p > 512 || rank_p <= 0 || rot_p < 0) return 0;
-  return latent_decode_smem(rank_p + rot_p) <= 227 * 1024 - 1024 ? LD_ROWS : 0;
+  if (heads > LD_ROWS && latent_decode_stages(rank_p + rot_p, true) >= 2) return 2 * LD_ROWS;
+  return latent_decode_stages(rank_p + rot_p, false) >= 2 ? LD_ROWS : 0;
 }
 
 extern "C" int omni_latent_decode(const LatentDecode* args, void* stream) {
   const LatentDecode& p = *args;
   if (p.n <= 0) return RC_OK;
-  if (omni_latent_decode_heads(p.rank_p, p.rot_p) == 0 || p.H <= 0 || (p.rank_p & 15) || (p.rot_p & 15) || (p.ldp & 7) || (p.head_cols & 7) || (p.dim_p & 7) || p.splits < 1 ||
+  const int heads = p.H > 0 ? omni_latent_decode_heads(p.H, p.rank_p, p.rot_p) : 0;
+  if (heads == 0 || (p.rank_p & 15) || (p.rot_p & 15) || (p.ldp & 7) || (p.head_cols & 7) || (p.dim_p & 7) || p.splits < 1 ||
       p.splits > 65535 || p.block_size <= 0 || p.num_blocks <= 0 || p.num_seqs <= 0 || p.T <= 0)
     return RC_BAD_ARG;
   if (p.splits > 1 && (!p.part_o || !p.part_ml)) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
-  const int rc = p.rank_p <= 128 ? launch_latent_decode<1>(p, st)
-                                 : (p.rank_p <= 256 ? launch_latent_decode<2>(p, st) : launch_latent_decode<4>(p, st));
+  const bool wide = heads > LD_ROWS;
+  const int rc = p.rank_p <= 128 ? pick_latent_decode<1>(p, wide, st)
+                                 : (p.rank_p <= 256 ? pick_latent_decode<2>(p, wide, st) : pick_latent_decode<4>(p, wide, st));
   if (rc || p.splits == 1) return rc;
   latent_merge_kernel<<<(unsigned)(p.n * p.H), 128, 0, st>>>(p);
   return (int)cudaGetLastError();

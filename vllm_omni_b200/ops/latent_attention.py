@@ -82,7 +82,8 @@ class _LatentDecode(ctypes.Structure):
                 ("pages", c_void_p), ("rank_p", c_int), ("rot_p", c_int), ("block_tables", c_void_p), ("bt_stride", c_int),
                 ("block_size", c_int), ("num_blocks", c_int), ("rows", c_void_p), ("n", c_int), ("row_seq", c_void_p),
                 ("q_start", c_void_p), ("context", c_void_p), ("num_seqs", c_int), ("T", c_int), ("scale", c_float),
-                ("out", c_void_p), ("H", c_int), ("splits", c_int), ("part_o", c_void_p), ("part_ml", c_void_p)]
+                ("out", c_void_p), ("H", c_int), ("splits", c_int), ("part_o", c_void_p), ("part_ml", c_void_p),
+                ("status", c_void_p)]
 
 
 def _P(t):
@@ -133,7 +134,7 @@ def latent_attention(proj, s: LatentShape, pages, seqs, uk_t, kv_up, scale: floa
         return _cpu(proj, s, pages, seqs, kv_up, scale, out, gate)
     assert proj.stride(1) == 1 and out.is_contiguous() and uk_t.is_contiguous() and kv_up.is_contiguous()
     bf = proj.dtype == torch.bfloat16
-    if impl == "rows" or not bf or not nv.lib("latent_attn").omni_latent_decode_heads(s.rank_p, s.rot_p):
+    if impl == "rows" or not bf or not nv.lib("latent_attn").omni_latent_decode_heads(s.heads, s.rank_p, s.rot_p):
         return _rows(proj, s, pages, seqs, uk_t, kv_up, scale, out, gate)
     short = 1 << 30 if impl == "latent" or not _expands(s) else SHORT
     rows, n, keys = seqs.short_rows(short)
@@ -187,12 +188,12 @@ def expanded_attention(proj, s, rows, kv, seqs, scale, out, gate, group):
                 "omni_attn_window_prefill")
 
 
-def decode_splits(blocks: int, keys: int, slots: int = 2 * 148) -> int:
-    """Blocks that share one row's keys: fills the block slots of the GPU evenly, about 256 keys each at least."""
+def decode_splits(blocks: int, keys: int, sms: int = 148) -> int:
+    """Blocks that share one row's keys: fills the SMs evenly, about 256 keys each at least."""
     best, best_cost = 1, None
     for n in range(1, max(1, min(64, (keys + 255) // 256)) + 1):
-        waves = -(-blocks * n // slots)
-        cost = waves * (-(-keys // (16 * n)) + 8)           # key tiles of a block and its start-up, per wave
+        waves = -(-blocks * n // sms)
+        cost = waves * (-(-keys // (32 * n)) + 6)           # key tiles of a block and its start-up, per wave
         if best_cost is None or cost < best_cost:
             best, best_cost = n, cost
     return best
@@ -222,7 +223,7 @@ def latent_decode(q_lat, proj, s, pages, seqs, rows, n, keys, scale):
     H, dev = s.heads, proj.device
     o_lat = torch.empty_like(q_lat)
     lib = nv.lib("latent_attn")
-    hb = lib.omni_latent_decode_heads(s.rank_p, s.rot_p)
+    hb = lib.omni_latent_decode_heads(H, s.rank_p, s.rot_p)
     a = _LatentDecode()
     a.q_lat, a.proj, a.ldp, a.head_cols, a.dim_p = _P(q_lat), _P(proj), proj.stride(0), s.head_cols, s.dim_p
     a.pages, a.rank_p, a.rot_p = _P(pages), s.rank_p, s.rot_p
@@ -230,7 +231,7 @@ def latent_decode(q_lat, proj, s, pages, seqs, rows, n, keys, scale):
         pages.shape[0]
     a.rows, a.n, a.row_seq, a.q_start, a.context = _P(rows), n, _P(seqs.row_seq), _P(seqs.q_start), _P(seqs.context)
     a.num_seqs, a.T, a.scale, a.out, a.H = seqs.n_seqs, proj.shape[0], scale, _P(o_lat), H
-    a.splits = decode_splits(n * -(-H // hb), keys)
+    a.splits, a.status = decode_splits(n * -(-H // hb), keys), _P(nv.status_word(dev))
     if a.splits > 1:
         po, pml = WA._parts(dev, n * H * a.splits, s.rank_p)
         a.part_o, a.part_ml = _P(po), _P(pml)
