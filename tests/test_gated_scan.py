@@ -12,7 +12,7 @@ GPU = pytest.mark.gpu
 MODES = [pytest.param(("cpu", torch.float32, 1e-4), id="cpu"), pytest.param(("cuda", torch.float32, 1e-4), id="fp32", marks=GPU),
          pytest.param(("cuda", torch.bfloat16, 0.02), id="bf16", marks=GPU)]
 # width, blocks, taps
-SIZES = {"base": (144, 3, 4), "one_block": (80, 1, 3), "full_part": (512, 2, 2), "no_history": (320, 4, 1), "many_taps": (48, 3, 6),
+SIZES = {"base": (144, 3, 4), "one_block": (80, 1, 3), "full_part": (512, 2, 2), "no_history": (336, 4, 1), "many_taps": (48, 3, 6),
          "wide_part": (600, 2, 3), "padded_part": (36, 2, 3), "two_tiles": (340, 2, 4), "more_taps": (32, 2, 9)}
 
 

@@ -4,8 +4,8 @@
 // The query heads that share a KV head are packed: row r of a 128-row tile is (token r / R, head r % R) with
 // R = heads per KV head, so a K/V tile is fetched once for the whole group and a tile spans only 128 / R
 // tokens, which keeps the keys outside a row's window or its future few.  One block owns two such tiles (one
-// where two do not fit) of one (sequence, KV head) and visits the key tiles any of its rows sees: the tiles of the kept first tokens,
-// then those of the window.  Portions of all sequences of a batch are one launch.
+// where two do not fit) of one (sequence, KV head) and visits the key tiles any of its rows sees: the tiles of the kept
+// first tokens, then those of the window.  Portions of all sequences of a batch are one launch.
 //   warp 0        TMA producer: Q (box {64 channels, R heads, 128 / R tokens}), then K / V pages
 //   warp 1        MMA issuer: S_t = Q_t K^T, O_t += P_t V (P read from TMEM)
 //   warps 2, 3    distance bias of the key tile: r1 log2(1 + r2 dist) depends on (head, distance) only, so a

@@ -126,9 +126,10 @@ moe_topk_kernel(const float* __restrict__ logits, long ld, int T, int E, int k, 
   topk_softmax(v, E, k, lane, ids + (long)t * k, weights + (long)t * k);
 }
 
-// Router of MT * 16 tokens per block: NW warps share the contraction (each takes every NW-th 32-channel chunk), 64 experts at a time; partial sums meet in shared memory in a fixed order.  A warp reads 16 bytes per row and
-// chunk: lane group j of a quad owns channels 8 j .. 8 j + 7 of the chunk for both operands, which permutes the
-// contraction alike on both sides.
+// Router of MT * 16 tokens per block: NW warps share the contraction (each takes every NW-th 32-channel chunk), 64 experts
+// at a time; partial sums meet in shared memory in a fixed order.  A warp reads 16 bytes per row and chunk: lane group j
+// of a quad owns channels 8 j .. 8 j + 7 of the chunk for both operands, which permutes the contraction alike on both
+// sides.
 template <int MT, int NW>
 __global__ void __launch_bounds__(32 * NW)
 moe_router_kernel(const __nv_bfloat16* __restrict__ x, long ldx, const __nv_bfloat16* __restrict__ w, long ldw,
