@@ -104,7 +104,7 @@ def test_experts(mode, T, D, ff, E, k):
     Ep = (E + 7) // 8 * 8
     rw, rbp = torch.zeros(Ep, D), torch.zeros(Ep)
     rw[:E], rbp[:E] = router, rb
-    er = moe.expert_rows(x.to(dev, dtype), rw.to(dev, dtype), rbp.to(dev), E, k, up.to(dev, dtype), down.to(dev, dtype), act="relu2")
+    er = moe.expert_rows(x.to(dev, dtype), rw.to(dev, dtype), rbp.to(dev), moe.Router(E, k), up.to(dev, dtype), down.to(dev, dtype), act="relu2")
     near(er.weights.sort(-1).values, w.sort(-1).values, 2e-5)
     for sh in (None, shared):
         s = torch.zeros(T, D, device=dev)
@@ -126,7 +126,7 @@ def test_router_keeps_fp32_logits(T):
     w[7, 0] = w[21, 0] = 8.0
     b = torch.zeros(E)
     b[21] = 0.0009765625                                    # logits 128 and 128.00098
-    er = moe.expert_rows(x.cuda().bfloat16(), w.cuda().bfloat16(), b.cuda(), E, 1, torch.ones(E, 8, D).cuda().bfloat16(),
+    er = moe.expert_rows(x.cuda().bfloat16(), w.cuda().bfloat16(), b.cuda(), moe.Router(E, 1), torch.ones(E, 8, D).cuda().bfloat16(),
                          (torch.arange(E).float()[:, None, None] * torch.ones(E, D, 8)).cuda().bfloat16(), act="relu2")
     s, out = torch.zeros(T, D, device="cuda"), torch.empty(T, D, dtype=torch.bfloat16, device="cuda")
     stream.add_expert_rows_(s, er, None, 1.0, out, stream.CAST)

@@ -8,6 +8,8 @@ same number of weights and use the same number per token.  Of the four Nidilix l
 second reads the first one's latents) and two are recurrences as wide as the stream, in parts of 256 channels."""
 from __future__ import annotations
 
+import ctypes
+
 import torch
 
 from .kernel_cases import _peaks
@@ -55,6 +57,7 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
     s = SIZES[width]
     H, G, T, E, F_ = s["heads"], s["kv"], 8192, s["experts"], s["ff"]
     F2, k2 = F_ * 3 // 2, s["top"] - 1
+    router = moe.Router(E, k2)
     out = []
 
     def row(name, like, fn, flops=0.0, bytes_=0.0):
@@ -151,13 +154,13 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
         rbytes = 2.0 * xr.numel() + 2.0 * rw.numel()
         row(f"router, {tag}", "qwen3_moe (two kernels)", dense_router, bytes_=rbytes, flops=2.0 * rows_ * E * width)
         row(f"router, {tag}", "nidilix", lambda: lib.omni_moe_router(P(xr), LA.c_long(width), P(rw), LA.c_long(width), P(rb), ci(rows_),
-            ci(width), ci(E), ci(E), ci(k2), P(idb), P(wtb), nv.stream_ptr()), bytes_=rbytes, flops=2.0 * rows_ * E * width)
+            ci(width), ci(E), ci(E), ci(k2), ctypes.byref(router.rule), P(idb), P(wtb), nv.stream_ptr()), bytes_=rbytes, flops=2.0 * rows_ * E * width)
         up, down = rnd(E, F2, width) * 0.02, rnd(E, width, F2) * 0.02
-        er = moe.expert_rows(xr, rw, rb, E, k2, up, down, act="relu2")
+        er = moe.expert_rows(xr, rw, rb, router, up, down, act="relu2")
         ws, ws_q = moe.MoEWorkspace(), moe.MoEWorkspace()
-        moe.expert_rows(xr, rw, rb, E, k2, up, down, act="relu2", ws=ws)
+        moe.expert_rows(xr, rw, rb, router, up, down, act="relu2", ws=ws)
         n_used = ws.ids.unique().numel()                            # experts whose weights are read
-        row(f"experts, {tag}", "nidilix (router to expert rows)", lambda: moe.expert_rows(xr, rw, rb, E, k2, up, down, act="relu2", ws=ws),
+        row(f"experts, {tag}", "nidilix (router to expert rows)", lambda: moe.expert_rows(xr, rw, rb, router, up, down, act="relu2", ws=ws),
             flops=4.0 * rows_ * k2 * width * F2, bytes_=4.0 * n_used * width * F2)
         w13, w2 = rnd(E, 2 * F_, width) * 0.02, rnd(E, width, F_) * 0.02
         lg = gemm.linear(xr, rw)

@@ -22,6 +22,9 @@
 // The keys a block visits are a list of 32-key chunks, those of the kept first tokens followed by those of the
 // window; four chunks make a tile, so the kept tokens cost one chunk and the window's ends are cut to 32 keys.
 // The one tile that holds chunks of both parts has two bias tables.
+// Two maps (differential attention, PAIR): the block's two tiles are the maps of the SAME tokens.  A key tile holds both
+// maps' keys, the value tile is shared, and the epilogue combines the two accumulators row by row: warps t = 0 and 1 of a
+// quarter share its rows, take every other 16 channels, and exchange denominators and sums of squares in shared memory.
 // TMEM columns: S0 [0,128) S1 [128,256) O0 [256,384) O1 [384,512); P_t over the first 64 columns of S_t.
 // Every wait is bounded.
 #include "attn_window.h"
@@ -41,7 +44,7 @@ struct WinPrefill {
   WinAttn a;
   int R, TT;            // heads per KV head, tokens per tile
   int nq;               // query tiles per block (2; 1 where two of the widest heads would not fit)
-  int kb, vb;           // 64-channel boxes per key / value row
+  int kb, vb;           // 64-channel boxes per key (one map) / value row
   int kbu;              // key boxes of the head's own part; the others hold the part shared by all heads
   int k_stages, v_stages;       // depth of the K and V rings
   int tab_stride;       // floats between the bias rows of two heads
@@ -71,7 +74,32 @@ __device__ __forceinline__ uint32_t bit_range(int a, int b) {
   return hi & ~lo;
 }
 
-template <bool CAP, bool BIAS, bool BOUNDED>
+// sigmoid of a gate logit
+__device__ __forceinline__ float wp_open(float z) { return 1.0f / (1.0f + __expf(-z)); }
+
+// 16 channels of a row, times f, channel by channel times their gate's opening where `gate` is given
+__device__ __forceinline__ void wp_store16(__nv_bfloat16* dst, const float (&v)[16], float f, const __nv_bfloat16* gate) {
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    float o[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) o[e] = v[x * 8 + e] * f;
+    if (gate) {
+      const uint4 z = *reinterpret_cast<const uint4*>(gate + x * 8);
+      const uint32_t zw[4] = {z.x, z.y, z.z, z.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 g = unpack_bf16(zw[e]);
+        o[2 * e] *= wp_open(g.x);
+        o[2 * e + 1] *= wp_open(g.y);
+      }
+    }
+    *reinterpret_cast<uint4*>(dst + x * 8) = make_uint4(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]), pack_bf16(o[4], o[5]),
+                                                        pack_bf16(o[6], o[7]));
+  }
+}
+
+template <bool CAP, bool BIAS, bool BOUNDED, bool PAIR>
 __global__ void __launch_bounds__(WP_THREADS, 1)
 attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                            const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmS,
@@ -90,8 +118,9 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   const int row0 = p.q_start[seq] + off;                     // first batch row of the block
   const int n_seq = p.q_start[seq + 1] - p.q_start[seq];
   const int ctx = p.context[seq];
-  const int nt = min(w.nq * w.TT, n_seq - off);               // tokens of the block
-  const int n_qt = nt > w.TT ? 2 : 1;
+  const int nt = min((PAIR ? 1 : w.nq) * w.TT, n_seq - off);  // tokens of the block
+  const int n_qt = PAIR || nt > w.TT ? 2 : 1;
+  const int tile_tokens = PAIR ? 0 : w.TT;                   // tokens from one query tile to the next
   const int p_first = ctx + off, p_last = p_first + nt - 1;
   const int lo_chunk = p.window > 0 ? max(0, p_first - p.window + 1) / 32 : 0;
   const int kept = min(lo_chunk, (p.keep_first + 31) / 32);       // chunks of the kept first tokens
@@ -99,7 +128,8 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   auto chunk_of = [&](int u) { return u < kept ? u : lo_chunk + u - kept; };
 
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  const uint32_t q_tile = w.kb * WP_BOX, k_tile = q_tile, v_tile = w.vb * WP_BOX;
+  const int k_boxes = PAIR ? 2 * w.kb : w.kb;
+  const uint32_t q_tile = w.kb * WP_BOX, k_tile = k_boxes * WP_BOX, v_tile = w.vb * WP_BOX;
   const uint32_t sQ = base, sK = base + w.nq * q_tile, sV = sK + w.k_stages * k_tile;
   float* tab = reinterpret_cast<float*>(smem_raw + (sV + w.v_stages * v_tile - smem_u32(smem_raw)));
   const int tab_floats = w.R * w.tab_stride;
@@ -148,7 +178,7 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       for (int t = 0; t < n_qt; ++t)
         for (int x = 0; x < w.kb; ++x)
           tma_load_4d(sQ + t * q_tile + x * WP_BOX, &tmQ, qb, x < w.kbu ? 64 * x : p.dp_u + 64 * (x - w.kbu), 0,
-                      row0 + t * w.TT, g);
+                      row0 + t * tile_tokens, PAIR ? 2 * g + t : g);
     }
     const int* bt = p.block_tables + (long)seq * p.bt_stride;
     const int bs = p.key_start ? 32 : p.block_size, last_page = (ctx + n_seq - 1) / bs;
@@ -177,9 +207,10 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       mbar_wait(smem_u32(&k_empty[ks]), ((j / w.k_stages) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
       if (lane == 0) mbar_expect_tx(kbar, k_tile);
       __syncwarp();
-      for (int x = x_first; x < w.kb; x += x_step) {
+      for (int x = x_first; x < k_boxes; x += x_step) {
         const uint32_t dst = sK + ks * k_tile + x * WP_BOX + my_box * box_bytes;
-        if (x < w.kbu) tma_load_3d(dst, &tmK, kbar, 64 * x, r, g);
+        if (PAIR) tma_load_3d(dst, &tmK, kbar, 64 * (x < w.kb ? x : x - w.kb), r, 2 * g + (x < w.kb ? 0 : 1));
+        else if (x < w.kbu) tma_load_3d(dst, &tmK, kbar, 64 * x, r, g);
         else tma_load_3d(dst, &tmS, kbar, 64 * (x - w.kbu), r, 0);
       }
       mbar_wait(smem_u32(&v_empty[vs]), ((j / w.v_stages) & 1) ^ 1, &s_abort, status, ERR_WAIT_EMPTY);
@@ -198,7 +229,7 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       const uint64_t dV = umma_desc_sw128(sV, WP_BOX, 1024);
       const int ks = p.dp >> 4, ksu = p.dp_u >> 4;
       auto issue_s = [&](int t, int st) {
-        const uint64_t a0 = dQ + (uint64_t)t * q16, b0 = dK + (uint64_t)st * k16;
+        const uint64_t a0 = dQ + (uint64_t)t * q16, b0 = dK + (uint64_t)st * k16 + (PAIR ? (uint64_t)t * q16 : 0ull);
         auto step = [&](int k0) {
           const int k = k0 < ksu ? k0 : 4 * w.kbu + k0 - ksu;       // the shared part starts a box of its own
           const uint64_t o = (uint64_t)(k >> 2) * box16 + (uint64_t)((k & 3) * 2);   // 16 channels = 32 bytes of a row
@@ -207,6 +238,9 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         if (ks == 8 && ksu == 8) {
 #pragma unroll
           for (int k = 0; k < 8; ++k) step(k);
+        } else if (ks == 4 && ksu == 4) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k) step(k);
         } else {
           for (int k = 0; k < ks; ++k) step(k);
         }
@@ -281,9 +315,9 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     const int row = q * 32 + lane;
     const int tok = row / w.R, r = row - tok * w.R;
     const bool tile_used = t < n_qt;
-    const bool row_ok = tile_used && tok < w.TT && t * w.TT + tok < nt;
+    const bool row_ok = tile_used && tok < w.TT && t * tile_tokens + tok < nt;
     const bool rows_used = __any_sync(0xffffffffu, row_ok);
-    const int pos = p_first + t * w.TT + tok;
+    const int pos = p_first + t * tile_tokens + tok;
     const uint32_t lane_addr = (uint32_t)(q * 32) << 16;
     const uint32_t tS = tmem_base + lane_addr + t * 128, tO = tmem_base + lane_addr + 256 + t * 128;
     const int h = g * w.R + min(r, w.R - 1);
@@ -304,7 +338,7 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       m = ref;
       b_const = C - ref;
     }
-    const float* my_tab = tab + min(r, w.R - 1) * w.tab_stride + min(t * w.TT + tok, 2 * w.TT - 1) + 127;
+    const float* my_tab = tab + min(r, w.R - 1) * w.tab_stride + min(t * tile_tokens + tok, 2 * w.TT - 1) + 127;
     for (int j = 0; tile_used && j < n_kv; ++j) {
       mbar_wait(smem_u32(&s_full[t]), j & 1, &s_abort, status, ERR_WAIT_FULL);
       if (!rows_used) {
@@ -458,31 +492,62 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     if (rows_used) {
       mbar_wait(smem_u32(&o_done[t]), 0, &s_abort, status, ERR_WAIT_PV);
       tc_fence_after_sync();
-      const long orow = row0 + t * w.TT + tok;
+      const long orow = row0 + t * tile_tokens + tok;
       float s0, s1, s2, s3;
       unpack2(l2a, s0, s1);
       unpack2(l2b, s2, s3);
       float f = 1.0f / ((s0 + s1) + (s2 + s3));
-      if (p.gate && row_ok) {
-        const float z = (float)static_cast<const __nv_bfloat16*>(p.gate)[orow * p.g_rs + h];
-        f *= 1.0f / (1.0f + __expf(-z));
-      }
+      const __nv_bfloat16* gate = p.gate && row_ok ? static_cast<const __nv_bfloat16*>(p.gate) + orow * p.g_rs + (long)h * p.g_hs : nullptr;
+      const float head_gate = gate && p.g_cs == 0 ? wp_open((float)gate[0]) : 1.f;
+      if (p.g_cs == 0) gate = nullptr;
       __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + orow * p.o_rs + (long)h * p.vp;
-#pragma unroll 1
-      for (int c = 0; c < p.vp; c += 16) {
-        uint32_t v[16];
-        tmem_ld_32x16(tO + c, v);
-        tmem_wait_ld();
-        if (row_ok) {
+      if constexpr (PAIR) {
+        mbar_wait(smem_u32(&o_done[t ^ 1]), 0, &s_abort, status, ERR_WAIT_PV);
+        tc_fence_after_sync();
+        // every product is done: the query tiles' memory takes the exchanged numbers
+        float* ex = reinterpret_cast<float*>(smem_raw + (sQ - smem_u32(smem_raw)));
+        auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(1 + q) : "memory"); };
+        ex[t * 128 + row] = f;
+        pair_sync();
+        const float f0 = ex[row], f1 = -p.lam * ex[128 + row];
+        const uint32_t o0 = tmem_base + lane_addr + 256, o1 = o0 + 128;
+        float ss = 0.f;
+        auto combined = [&](int c, float (&u)[16]) {
+          uint32_t a[16], b[16];
+          tmem_ld_32x16(o0 + c, a);
+          tmem_ld_32x16(o1 + c, b);
+          tmem_wait_ld();
 #pragma unroll
-          for (int x = 0; x < 2; ++x) {
-            uint4 o;
-            o.x = pack_bf16(__uint_as_float(v[x * 8 + 0]) * f, __uint_as_float(v[x * 8 + 1]) * f);
-            o.y = pack_bf16(__uint_as_float(v[x * 8 + 2]) * f, __uint_as_float(v[x * 8 + 3]) * f);
-            o.z = pack_bf16(__uint_as_float(v[x * 8 + 4]) * f, __uint_as_float(v[x * 8 + 5]) * f);
-            o.w = pack_bf16(__uint_as_float(v[x * 8 + 6]) * f, __uint_as_float(v[x * 8 + 7]) * f);
-            *reinterpret_cast<uint4*>(dst + c + x * 8) = o;
-          }
+          for (int e = 0; e < 16; ++e) u[e] = fmaf(__uint_as_float(a[e]), f0, __uint_as_float(b[e]) * f1);
+        };
+#pragma unroll 1
+        for (int c = 16 * t; c < p.vp; c += 32) {
+          float u[16];
+          combined(c, u);
+#pragma unroll
+          for (int e = 0; e < 16; ++e) ss = fmaf(u[e], u[e], ss);
+        }
+        ex[256 + t * 128 + row] = ss;
+        pair_sync();
+        ss = ex[256 + row] + ex[384 + row];
+        f = p.out_mul * head_gate / sqrtf(ss / (float)p.vdim + p.out_eps);
+#pragma unroll 1
+        for (int c = 16 * t; c < p.vp; c += 32) {
+          float u[16];
+          combined(c, u);
+          if (row_ok) wp_store16(dst + c, u, f, gate ? gate + c : nullptr);
+        }
+      } else {
+        f *= head_gate;
+#pragma unroll 1
+        for (int c = 0; c < p.vp; c += 16) {
+          uint32_t v[16];
+          tmem_ld_32x16(tO + c, v);
+          tmem_wait_ld();
+          float u[16];
+#pragma unroll
+          for (int e = 0; e < 16; ++e) u[e] = __uint_as_float(v[e]);
+          if (row_ok) wp_store16(dst + c, u, f, gate ? gate + c : nullptr);
         }
       }
     }
@@ -499,12 +564,12 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
-// Q as (channel, head of the group, token, KV head)
+// Q as (channel, head of the group, token, KV head and map)
 static int make_q_tmap(CUtensorMap* tm, const WinAttn& p, int R, int TT) {
   EncodeTiledFn enc = get_encode_tiled();
   if (!enc) return RC_NO_DRIVER;
   if ((reinterpret_cast<uintptr_t>(p.q) & 15) || (p.q_rs & 7)) return RC_BAD_ARG;
-  cuuint64_t gdim[4] = {(cuuint64_t)p.dp, (cuuint64_t)R, (cuuint64_t)p.T, (cuuint64_t)p.G};
+  cuuint64_t gdim[4] = {(cuuint64_t)p.dp, (cuuint64_t)R, (cuuint64_t)p.T, (cuuint64_t)p.G * (p.maps == 2 ? 2 : 1)};
   cuuint64_t gstr[3] = {(cuuint64_t)p.dp * 2, (cuuint64_t)p.q_rs * 2, (cuuint64_t)R * p.dp * 2};
   cuuint32_t box[4] = {64, (cuuint32_t)R, (cuuint32_t)TT, 1};
   cuuint32_t estr[4] = {1, 1, 1, 1};
@@ -514,12 +579,12 @@ static int make_q_tmap(CUtensorMap* tm, const WinAttn& p, int R, int TT) {
   return r == CUDA_SUCCESS ? RC_OK : RC_TMAP;
 }
 
-template <bool CAP, bool BIAS, bool BOUNDED>
+template <bool CAP, bool BIAS, bool BOUNDED, bool PAIR = false>
 static int launch_prefill(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& ts, const WinPrefill& w,
                           int smem, cudaStream_t st) {
   static unsigned long long prep = 0;
-  if (int e = ensure_dynamic_smem((const void*)attn_window_prefill_kernel<CAP, BIAS, BOUNDED>, 227 * 1024 - 512, prep)) return e;
-  attn_window_prefill_kernel<CAP, BIAS, BOUNDED><<<dim3(w.a.G, w.a.n_items), WP_THREADS, smem, st>>>(tq, tk, tv, ts, w);
+  if (int e = ensure_dynamic_smem((const void*)attn_window_prefill_kernel<CAP, BIAS, BOUNDED, PAIR>, 227 * 1024 - 512, prep)) return e;
+  attn_window_prefill_kernel<CAP, BIAS, BOUNDED, PAIR><<<dim3(w.a.G, w.a.n_items), WP_THREADS, smem, st>>>(tq, tk, tv, ts, w);
   return (int)cudaGetLastError();
 }
 
@@ -545,7 +610,11 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   if (w.R > 128) return RC_BAD_ARG;
   w.TT = 128 / w.R;
   if (p.block_tokens != w.TT && p.block_tokens != 2 * w.TT) return RC_BAD_ARG;
-  w.nq = p.block_tokens / w.TT;
+  const bool pair = p.maps == 2;
+  if (pair && (p.block_tokens != w.TT || p.dp_u != p.dp || p.key_start || p.r1 || p.sink || p.cap > 0.f || p.vdim <= 0 || p.vdim > p.vp))
+    return RC_BAD_ARG;
+  if (p.g_cs && ((reinterpret_cast<uintptr_t>(p.gate) & 15) || (p.g_rs & 7) || (p.g_hs & 7) || p.g_cs != 1)) return RC_BAD_ARG;
+  w.nq = pair ? 2 : p.block_tokens / w.TT;
   w.kbu = (p.dp_u + 63) / 64;
   w.kb = w.kbu + (p.dp - p.dp_u + 63) / 64;
   w.vb = (p.vp + 63) / 64;
@@ -557,7 +626,7 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   while (w.tab_stride % 32 != want) ++w.tab_stride;
   const int tab_bytes = p.r1 ? 3 * w.R * w.tab_stride * 4 : 0;
   const int limit = 227 * 1024 - 1024 - 512;                 // less the alignment slack and the static barriers
-  const int q_bytes = w.nq * w.kb * WP_BOX, k_bytes = w.kb * WP_BOX, v_bytes = w.vb * WP_BOX;
+  const int q_bytes = w.nq * w.kb * WP_BOX, k_bytes = (pair ? 2 : 1) * w.kb * WP_BOX, v_bytes = w.vb * WP_BOX;
   w.k_stages = w.v_stages = 1;
   int used = q_bytes + tab_bytes + k_bytes + v_bytes;
   if (used > limit) return RC_TOO_LARGE;
@@ -572,7 +641,7 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
   const uint64_t slots = p.key_start ? (uint64_t)p.key_rows : (uint64_t)p.num_blocks * p.block_size;
   const uint32_t box_rows = p.key_start ? 32 : (p.block_size < 32 ? p.block_size : 32);
   int rc = make_q_tmap(&tq, p, w.R, w.TT);
-  if (!rc) rc = make_tmap_3d(&tk, p.k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dp_u, slots, p.G, (uint64_t)p.k_ts * 2,
+  if (!rc) rc = make_tmap_3d(&tk, p.k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dp_u, slots, p.G * (pair ? 2 : 1), (uint64_t)p.k_ts * 2,
                              (uint64_t)p.dp_u * 2, 64, box_rows);
   if (!rc) rc = make_tmap_3d(&tv, p.v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.vp, slots, p.G, (uint64_t)p.v_ts * 2,
                              (uint64_t)p.vp * 2, 64, box_rows);
@@ -582,6 +651,7 @@ extern "C" int omni_attn_window_prefill(const WinAttn* args, void* stream) {
                       (uint64_t)p.ks_ts * 2, 64, box_rows);
   if (rc) return rc;
   cudaStream_t st = (cudaStream_t)stream;
+  if (pair) return launch_prefill<false, false, false, true>(tq, tk, tv, ts, w, smem, st);
   if (p.cap > 0.f && p.bounded)
     return p.r1 ? launch_prefill<true, true, true>(tq, tk, tv, ts, w, smem, st) : launch_prefill<true, false, true>(tq, tk, tv, ts, w, smem, st);
   if (p.cap > 0.f)

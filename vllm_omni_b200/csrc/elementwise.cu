@@ -13,7 +13,7 @@
 //  omni_cfg_euler_step  guidance mix neg + s (pos - neg), optional norm rescale, flow-match
 //                       Euler update x += dt * v, bf16 copy of the new latents
 //                       (reference: vllm_omni/diffusion/distributed/cfg_parallel.py:99-137)
-//  omni_silu_mul        SwiGLU gate: silu(x[:, :N]) * x[:, N:]
+//  omni_silu_mul        SwiGLU gate: silu(x[:, :N]) * x[:, N:] (_f32: the same in fp32)
 //  omni_rel_l1_partial / omni_rel_l1_finish
 //                       TeaCache residual metric sum|a-b| / sum|b| with the polynomial
 //                       rescale, accumulation and skip decision kept on the device
@@ -411,6 +411,18 @@ silu_mul_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__
   }
 }
 
+// the same in fp32 (exact mode)
+__global__ void __launch_bounds__(256)
+silu_mul_f32_kernel(const float* __restrict__ x, float* __restrict__ y, long rows, int N, long ldx, long ldy) {
+  const long total = rows * N;
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
+    const long r = i / N;
+    const int c = (int)(i - r * N);
+    const float g = x[r * ldx + c];
+    y[r * ldy + c] = g / (1.0f + expf(-g)) * x[r * ldx + N + c];
+  }
+}
+
 // --------------------------------------------------------- TeaCache rel-L1 metric
 // Stage 1: every CTA writes its partial (sum|a-b|, sum|b|) into scratch[2*blockIdx.x].
 // Stage 2 (one CTA): reduces the partials, applies the polynomial rescale, accumulates
@@ -565,6 +577,14 @@ extern "C" int omni_silu_mul(const void* x, void* y, long rows, int N, int ldx, 
   long blocks = (nchunk + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   silu_mul_kernel<<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, N, ldx, ldy);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_silu_mul_f32(const float* x, float* y, long rows, int N, long ldx, long ldy, void* stream) {
+  if (rows <= 0 || N <= 0) return RC_OK;
+  long blocks = (rows * N + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  silu_mul_f32_kernel<<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>(x, y, rows, N, ldx, ldy);
   return (int)cudaGetLastError();
 }
 

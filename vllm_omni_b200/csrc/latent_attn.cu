@@ -3,11 +3,13 @@
 // W_uv[h] c; queries are [dim_p unrotated | rot_p rotated] channels per head.  All sizes are multiples of 16 with
 // zero padding.
 //
-//   omni_latent_rows     rotates the queries in place, norms and rotates a token's row, writes it to its page
+//   omni_latent_rows     rotates the queries in place, norms and rotates a token's row, writes it to its page, norms a
+//                        latent of the queries in place (each part optional)
 //   omni_latent_gather   rows of several sequences from their pages to one buffer (prompts expand them to keys and
 //                        values with one GEMM and run on attn_window_sm100.cu)
 //   omni_head_gemm       one small product per head: queries into the latent space (W_uk^T q) and attention results
 //                        out of it (W_uv o, times the output gate); weights are read once per 16 rows
+//   omni_gate_channels   out *= sigmoid(gate), channel by channel (where no other kernel's epilogue does it)
 //   omni_latent_decode   decoded tokens (and rows of short portions): scores and weighted sums directly on the
 //                        latent rows, so a row is read once per 16 or 32 heads.  A block owns one token's heads and a
 //                        share of its keys; a producer warp copies 32-key tiles into a ring (bulk copies), two groups of
@@ -26,15 +28,19 @@ typedef __nv_bfloat16 bf16;
 
 // ------------------------------------------------------------------------------- rows and pages
 struct LatentRows {
-  void* proj; long ldp;            // [T, ldp]: q (H heads of dim_p + rot_p) | latent rank_p | rot_p
+  void* q; long ldq;               // [T, H, dim_p + rot_p] or nullptr: rotated parts are turned in place
   int T, H, dim_p, rot, rot_p;
+  const void* z; long ldz;         // [T, rank_p | rot_p] or nullptr: the layer writes no row
   int rank, rank_p;
   const float* turns;              // [T, rot / 2, 2] cos, sin
   const int* slots;                // [T], < 0: not written
   void* pages; long num_slots;     // [num_slots, rank_p + rot_p]
-  const float* norm;               // [rank_p]; nullptr: the layer writes no row
+  const float* norm;               // [rank_p]
   float eps;
   int* status;
+  void* qc; long ldqc;             // [T, q_rank_p] or nullptr: latent of the queries, normed in place
+  int q_rank, q_rank_p;
+  const float* q_norm;             // [q_rank_p]
 };
 
 // four rotated pairs: channels 8 i .. 8 i + 7 of a part of 2 `half` rotated channels (padding passes unchanged)
@@ -53,29 +59,46 @@ __device__ __forceinline__ void turn8(float (&v)[8], const float2* turn, int i, 
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_rows_kernel(const LatentRows p) {
-  __shared__ float sh[32];
+  __shared__ float sh[64];
   const long t = blockIdx.x;
-  T* row = static_cast<T*>(p.proj) + t * p.ldp;
   const float2* turn = reinterpret_cast<const float2*>(p.turns) + t * (p.rot / 2);
   const int half = p.rot / 2, hc = p.dim_p + p.rot_p, rv = (p.rot + 7) / 8;
-  for (int i = threadIdx.x; i < p.H * rv; i += 128) {
-    const int h = i / rv, c = i - h * rv;
-    T* q = row + h * hc + p.dim_p + 8 * c;
-    float v[8];
-    load8<T>(q, v);
-    turn8(v, turn, c, half);
-    store8<T>(q, v);
+  if (p.q) {
+    T* row = static_cast<T*>(p.q) + t * p.ldq;
+    for (int i = threadIdx.x; i < p.H * rv; i += 128) {
+      const int h = i / rv, c = i - h * rv;
+      T* q = row + h * hc + p.dim_p + 8 * c;
+      float v[8];
+      load8<T>(q, v);
+      turn8(v, turn, c, half);
+      store8<T>(q, v);
+    }
   }
-  if (p.norm == nullptr) return;
-  const T* z = row + p.H * hc;
-  float ss[1] = {0.f};
-  for (int i = threadIdx.x; i < p.rank_p / 8; i += 128) {
-    float v[8];
-    load8<T>(z + 8 * i, v);
+  if (p.z == nullptr && p.qc == nullptr) return;
+  const T* z = static_cast<const T*>(p.z) + t * p.ldz;
+  T* qc = static_cast<T*>(p.qc) + t * p.ldqc;
+  float ss[2] = {0.f, 0.f};
+  auto add = [&](const T* src, int n, float& sum) {
+    for (int i = threadIdx.x; i < n / 8; i += 128) {
+      float v[8];
+      load8<T>(src + 8 * i, v);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) ss[0] = fmaf(v[e], v[e], ss[0]);
+      for (int e = 0; e < 8; ++e) sum = fmaf(v[e], v[e], sum);
+    }
+  };
+  if (p.z) add(z, p.rank_p, ss[0]);
+  if (p.qc) add(qc, p.q_rank_p, ss[1]);
+  block_sum<2>(ss, sh);
+  if (p.qc) {
+    const float s = rms_scale(ss[1], p.q_rank, p.eps);
+    for (int i = threadIdx.x; i < p.q_rank_p / 8; i += 128) {
+      float v[8];
+      load8<T>(qc + 8 * i, v);
+      scale_gain8(v, s, p.q_norm, 1, 8 * i);
+      store8<T>(qc + 8 * i, v);
+    }
   }
-  block_sum<1>(ss, sh);
+  if (p.z == nullptr) return;
   const float s = rms_scale(ss[0], p.rank, p.eps);
   const long slot = p.slots[t];
   if (slot >= p.num_slots && p.status && threadIdx.x == 0) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
@@ -90,10 +113,30 @@ latent_rows_kernel(const LatentRows p) {
   }
 }
 
-// members: (sequence, first row of the output) pairs closed by (-1, rows); 16-byte pieces.
+// out[t, c] *= sigmoid(gate[t, c])
+template <typename T>
+__global__ void __launch_bounds__(256)
+gate_channels_kernel(T* __restrict__ out, long ldo, const T* __restrict__ gate, long ldg, long rows, int n) {
+  const int chunks = n / 8;
+  const long total = rows * chunks;
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
+    const long r = i / chunks;
+    const int c = (int)(i - r * chunks) * 8;
+    float v[8], g[8];
+    load8<T>(out + r * ldo + c, v);
+    load8<T>(gate + r * ldg + c, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= 1.0f / (1.0f + expf(-g[e]));
+    store8<T>(out + r * ldo + c, v);
+  }
+}
+
+// members: (sequence, first row of the output) pairs closed by (-1, rows); key_start[s]: row of the output that position 0 of
+// sequence s has or would have (negative where a window leaves its first positions out); 16-byte pieces.
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const uint4* __restrict__ pages, int row16, const int* __restrict__ tables, int bt_stride, int block_size,
-                     int num_blocks, const int* __restrict__ members, int n_members, uint4* __restrict__ out, long rows) {
+                     int num_blocks, const int* __restrict__ members, int n_members, const int* __restrict__ key_start,
+                     uint4* __restrict__ out, long rows) {
   const long total = rows * row16;
   for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
     const int r = (int)(i / row16), c = (int)(i - (long)r * row16);
@@ -102,8 +145,8 @@ latent_gather_kernel(const uint4* __restrict__ pages, int row16, const int* __re
       const int mid = (lo + hi + 1) >> 1;
       if (members[2 * mid + 1] <= r) lo = mid; else hi = mid - 1;
     }
-    const int pos = r - members[2 * lo + 1];
-    int pg = tables[(long)members[2 * lo] * bt_stride + pos / block_size];
+    const int seq = members[2 * lo], pos = r - key_start[seq];
+    int pg = tables[(long)seq * bt_stride + pos / block_size];
     pg = min(max(pg, 0), num_blocks - 1);
     out[i] = pages[((long)pg * block_size + pos % block_size) * row16 + c];
   }
@@ -116,6 +159,7 @@ struct HeadGemm {
   bf16* C; long c_row, c_head; const int* c_rows;
   const bf16* gate; long g_row;                             // logits at the row of C and head, or nullptr
   int M, N, K, H, rows_a, rows_c;
+  long g_head; int g_col;                                   // pitch of heads; 1: one logit per channel, 0: one per head
 };
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
@@ -175,9 +219,16 @@ head_gemm_kernel(const HeadGemm p) {
   }
   int row = p.c_rows ? p.c_rows[m0 + r] : m0 + r;
   row = min(max(row, 0), p.rows_c - 1);
-  float f = 1.f;
-  if (p.gate) f = 1.0f / (1.0f + __expf(-(float)p.gate[row * p.g_row + h]));
-  *reinterpret_cast<uint2*>(p.C + row * p.c_row + h * p.c_head + n0 + c) = make_uint2(pack_bf16(o.x * f, o.y * f), pack_bf16(o.z * f, o.w * f));
+  if (p.gate) {
+    const bf16* z = p.gate + row * p.g_row + h * p.g_head + (n0 + c) * p.g_col;
+    auto open = [](bf16 v) { return 1.0f / (1.0f + __expf(-(float)v)); };
+    const float f = open(z[0]);
+    o.x *= f;
+    o.y *= p.g_col ? open(z[1]) : f;
+    o.z *= p.g_col ? open(z[2]) : f;
+    o.w *= p.g_col ? open(z[3]) : f;
+  }
+  *reinterpret_cast<uint2*>(p.C + row * p.c_row + h * p.c_head + n0 + c) = make_uint2(pack_bf16(o.x, o.y), pack_bf16(o.z, o.w));
 }
 
 // ---------------------------------------------------------------------------------- decode
@@ -193,6 +244,7 @@ struct LatentDecode {
   int H, splits;
   float* part_o; float* part_ml;       // [n, H, splits, rank_p], [n, H, splits, 2]
   int* status;
+  int window;                          // a row sees its last `window` positions; <= 0: all
 };
 
 constexpr int LD_KEYS = 32, LD_ROWS = 16, LD_MAX_STAGES = 8;
@@ -243,7 +295,9 @@ latent_decode_kernel(const LatentDecode p, const int stages) {
   const int h0 = blockIdx.y * QROWS, split = blockIdx.z;
   const int row = min(max(p.rows[blockIdx.x], 0), p.T - 1);
   const int seq = min(max(p.row_seq[row], 0), p.num_seqs - 1);
-  const int n_vis = p.context[seq] + row - p.q_start[seq] + 1;
+  const int pos = p.context[seq] + row - p.q_start[seq];
+  const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;         // keys are counted from the first visible one
+  const int n_vis = pos - first + 1;
   const int tiles_all = (n_vis + LD_KEYS - 1) / LD_KEYS;
   const int per = (tiles_all + p.splits - 1) / p.splits;
   const int t0 = min(tiles_all, split * per), n_tiles = min(tiles_all, t0 + per) - t0;
@@ -284,9 +338,9 @@ latent_decode_kernel(const LatentDecode p, const int stages) {
     // ------------------------------------------- producer: a lane copies one key row, pages are looked up a tile ahead
     const int* bt = p.block_tables + (long)seq * p.bt_stride;
     auto src_row = [&](int t) {
-      const int pos = min((t0 + t) * LD_KEYS + lane, n_vis - 1);           // past the end: a valid key, masked below
-      const int pg = min(max(bt[pos / p.block_size], 0), p.num_blocks - 1);
-      return p.pages + ((long)pg * p.block_size + pos % p.block_size) * ch;
+      const int j = first + min((t0 + t) * LD_KEYS + lane, n_vis - 1);     // past the end: a valid key, masked below
+      const int pg = min(max(bt[j / p.block_size], 0), p.num_blocks - 1);
+      return p.pages + ((long)pg * p.block_size + j % p.block_size) * ch;
     };
     const bf16* next = n_tiles > 0 ? src_row(0) : nullptr;
     int st = 0;
@@ -515,22 +569,37 @@ using namespace omni;
 extern "C" int omni_latent_rows(const LatentRows* args, int is_bf16, void* stream) {
   const LatentRows& p = *args;
   if (p.T <= 0) return RC_OK;
-  if (p.H < 0 || p.rot < 0 || (p.rot & 1) || p.rot > p.rot_p || (p.dim_p & 15) || (p.rot_p & 15) || (p.rank_p & 15) || (p.ldp & 7))
+  if (p.H < 0 || p.rot < 0 || (p.rot & 1) || p.rot > p.rot_p || (p.dim_p & 15) || (p.rot_p & 15) || (p.q && (p.ldq & 7))) return RC_BAD_ARG;
+  if ((p.q || p.z) && p.turns == nullptr) return RC_BAD_ARG;
+  if (p.z && (p.pages == nullptr || p.norm == nullptr || p.slots == nullptr || (p.rank_p & 15) || (p.ldz & 7) || p.rank <= 0 ||
+              p.rank > p.rank_p || p.num_slots <= 0))
     return RC_BAD_ARG;
-  if (p.norm && (p.pages == nullptr || p.rank <= 0 || p.rank > p.rank_p || p.num_slots <= 0)) return RC_BAD_ARG;
+  if (p.qc && (p.q_norm == nullptr || (p.q_rank_p & 7) || (p.ldqc & 7) || p.q_rank <= 0 || p.q_rank > p.q_rank_p)) return RC_BAD_ARG;
   if (is_bf16) latent_rows_kernel<bf16><<<p.T, 128, 0, (cudaStream_t)stream>>>(p);
   else latent_rows_kernel<float><<<p.T, 128, 0, (cudaStream_t)stream>>>(p);
   return (int)cudaGetLastError();
 }
 
 extern "C" int omni_latent_gather(const void* pages, int row_bytes, const int* tables, int bt_stride, int block_size, int num_blocks,
-                                  const int* members, int n_members, void* out, long rows, void* stream) {
+                                  const int* members, int n_members, const int* key_start, void* out, long rows, void* stream) {
   if (rows <= 0) return RC_OK;
-  if ((row_bytes & 15) || row_bytes <= 0 || n_members <= 0 || block_size <= 0 || num_blocks <= 0) return RC_BAD_ARG;
+  if (key_start == nullptr || (row_bytes & 15) || row_bytes <= 0 || n_members <= 0 || block_size <= 0 || num_blocks <= 0) return RC_BAD_ARG;
   long blocks = (rows * (row_bytes / 16) + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   latent_gather_kernel<<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>((const uint4*)pages, row_bytes / 16, tables, bt_stride,
-                                                                          block_size, num_blocks, members, n_members, (uint4*)out, rows);
+                                                                          block_size, num_blocks, members, n_members, key_start, (uint4*)out,
+                                                                          rows);
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_gate_channels(void* out, long ldo, const void* gate, long ldg, long rows, int n, int is_bf16, void* stream) {
+  if (rows <= 0 || n <= 0) return RC_OK;
+  if ((n & 7) || (ldo & 7) || (ldg & 7)) return RC_BAD_ARG;
+  long blocks = (rows * (n / 8) + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (is_bf16) gate_channels_kernel<bf16><<<(unsigned)blocks, 256, 0, st>>>((bf16*)out, ldo, (const bf16*)gate, ldg, rows, n);
+  else gate_channels_kernel<float><<<(unsigned)blocks, 256, 0, st>>>((float*)out, ldo, (const float*)gate, ldg, rows, n);
   return (int)cudaGetLastError();
 }
 

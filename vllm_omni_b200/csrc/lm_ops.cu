@@ -5,9 +5,10 @@
 //   omni_add_norm       x += rms(y) * g_y, xn = rms(x) * g_n                          (one launch)
 //   omni_poly_norm      a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's rms
 //   omni_conv_heads     short causal convolution over time of the packed q/k/v projection, per-head
-//                       RMS norm of q and k, mixing of v with an earlier layer's values, K/V rows
-//                       written to their pages, convolution history written to the state pool
-//   omni_logit_softcap  cap * tanh(logit / cap) -> fp32
+//                       RMS norm of q and k, growth of q with the position, mixing of v with an earlier
+//                       layer's values, K/V rows written to their pages, convolution history written to
+//                       the state pool
+//   omni_logit_softcap  mult * logit, bounded to cap * tanh(. / cap) -> fp32
 //
 // Norm gains are fp32, either one number for the whole row (stride 0) or one per channel (stride 1).
 // Rows are padded to a multiple of 8 channels; padding channels hold zeros and do not count in means.
@@ -166,7 +167,7 @@ poly_norm_kernel(const T* __restrict__ z, int ldz, T* __restrict__ out, int ldo,
 }
 
 // ------------------------------------------ short convolution, head norms, value mixing, pages
-// The packed projection has columns [q: H * dp | k: G * dp | v: G * vp | ...], heads padded to dp / vp
+// The packed projection has columns [q: H * dp | k: G * dp | v: GV * vp | ...], heads padded to dp / vp
 // channels (multiples of 8).  A group of `lph` lanes owns one (row, head); a lane holds 8 channels.
 // The history of a sequence (its last K-1 projected rows) comes from the state pool when it lies before
 // the rows of this launch; pool rows are double-buffered (read index != write index), so the groups that
@@ -174,7 +175,7 @@ poly_norm_kernel(const T* __restrict__ z, int ldz, T* __restrict__ out, int ldo,
 struct ConvHeads {
   const void* proj; long ldp;
   int T, H, G, dp, vp, d, taps;
-  const float* conv;        // [taps, H * dp + G * dp + G * vp] or nullptr
+  const float* conv;        // [taps, H * dp + G * dp + GV * vp] or nullptr
   const float* q_norm;      // [dp] or nullptr (no norm)
   const float* k_norm;
   float eps;
@@ -186,15 +187,22 @@ struct ConvHeads {
   const int* state_in;      // [S]
   const int* state_out;     // [S], < 0: not written
   void* q_out;              // [T, H * dp]
-  void* k_cache; void* v_cache;     // [slots, G, dp], [slots, G, vp]
-  void* v_first;            // [T, G * vp]
+  void* k_cache; void* v_cache;     // [slots, G, dp], [slots, GV, vp]
+  void* v_first;            // [T, GV * vp]
   int v_mode;               // 0: as they are, 1: also saved to v_first, 2: mixed with v_first
   const float* lambda;
   long num_slots;           // page slots of the caches / rows of the pool (bounds of the index operands)
   int num_state, num_seqs;
   int* status;
   int lph;                  // lanes per head: a power of two, 32 at most
+  int GV;                   // value heads
+  float q_coef;             // q grows by 1 + q_coef ln(floor((position + 1) / q_every) + 1); 0: not at all
+  double q_every;
 };
+
+__device__ __forceinline__ float query_growth(const ConvHeads& p, int pos) {
+  return fmaf(p.q_coef, logf((float)floor((double)(pos + 1) / p.q_every) + 1.0f), 1.0f);
+}
 
 template <typename T, int IT>
 __global__ void __launch_bounds__(256)
@@ -207,7 +215,7 @@ conv_heads_kernel(ConvHeads p) {
   const int kind = head < p.H ? 0 : (head < p.H + p.G ? 1 : 2);
   const int width = kind == 2 ? p.vp : p.dp;
   const int hk = kind == 0 ? head : (kind == 1 ? head - p.H : head - p.H - p.G);
-  const int C = (p.H + p.G) * p.dp + p.G * p.vp;
+  const int C = (p.H + p.G) * p.dp + p.GV * p.vp;
   const int col0 = kind == 0 ? hk * p.dp : (kind == 1 ? (p.H + hk) * p.dp : (p.H + p.G) * p.dp + hk * p.vp);
   const T* proj = static_cast<const T*>(p.proj);
   T* state = static_cast<T*>(p.state);
@@ -281,6 +289,13 @@ conv_heads_kernel(ConvHeads p) {
     }
   }
   if (!live) return;
+  if (kind == 0 && p.q_coef != 0.f) {
+    const float grow = query_growth(p, ctx + off);
+#pragma unroll
+    for (int i = 0; i < IT; ++i)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] *= grow;
+  }
   int slot = kind == 0 ? 0 : p.slots[row];
   if (slot >= p.num_slots && kind != 0) {
     if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
@@ -296,7 +311,7 @@ conv_heads_kernel(ConvHeads p) {
     } else if (kind == 1) {
       if (slot >= 0) store8<T>(static_cast<T*>(p.k_cache) + ((long)slot * p.G + hk) * p.dp + c, v[i]);
     } else {
-      T* vf = static_cast<T*>(p.v_first) + (long)row * p.G * p.vp + hk * p.vp + c;
+      T* vf = static_cast<T*>(p.v_first) + (long)row * p.GV * p.vp + hk * p.vp + c;
       if (p.v_mode == 1) store8<T>(vf, v[i]);
       if (p.v_mode == 2) {
         float f[8];
@@ -304,7 +319,7 @@ conv_heads_kernel(ConvHeads p) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[i][e] = (1.f - lam) * v[i][e] + lam * f[e];
       }
-      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + ((long)slot * p.G + hk) * p.vp + c, v[i]);
+      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + ((long)slot * p.GV + hk) * p.vp + c, v[i]);
     }
   }
 }
@@ -323,7 +338,7 @@ conv_heads_run_kernel(ConvHeads p) {
   const int kind = head < p.H ? 0 : (head < p.H + p.G ? 1 : 2);
   const int width = kind == 2 ? p.vp : p.dp;
   const int hk = kind == 0 ? head : (kind == 1 ? head - p.H : head - p.H - p.G);
-  const int C = (p.H + p.G) * p.dp + p.G * p.vp;
+  const int C = (p.H + p.G) * p.dp + p.GV * p.vp;
   const int c = lane * 8;
   const int col = (kind == 0 ? hk * p.dp : (kind == 1 ? (p.H + hk) * p.dp : (p.H + p.G) * p.dp + hk * p.vp)) + c;
   const bool in = c < width;
@@ -400,6 +415,11 @@ conv_heads_run_kernel(ConvHeads p) {
     }
     if (!live || !in) continue;
     if (kind == 0) {
+      if (p.q_coef != 0.f) {
+        const float grow = query_growth(p, ctx + row - q0);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= grow;
+      }
       store8<T>(static_cast<T*>(p.q_out) + (long)row * p.H * p.dp + col, v);
       continue;
     }
@@ -411,7 +431,7 @@ conv_heads_run_kernel(ConvHeads p) {
     if (kind == 1) {
       if (slot >= 0) store8<T>(static_cast<T*>(p.k_cache) + ((long)slot * p.G + hk) * p.dp + c, v);
     } else {
-      T* vf = static_cast<T*>(p.v_first) + (long)row * p.G * p.vp + hk * p.vp + c;
+      T* vf = static_cast<T*>(p.v_first) + (long)row * p.GV * p.vp + hk * p.vp + c;
       if (p.v_mode == 1) store8<T>(vf, v);
       if (p.v_mode == 2) {
         float f[8];
@@ -419,7 +439,7 @@ conv_heads_run_kernel(ConvHeads p) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) v[e] = (1.f - lam) * v[e] + lam * f[e];
       }
-      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + ((long)slot * p.G + hk) * p.vp + c, v);
+      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + ((long)slot * p.GV + hk) * p.vp + c, v);
     }
   }
 }
@@ -427,12 +447,12 @@ conv_heads_run_kernel(ConvHeads p) {
 // ------------------------------------------------------------------------------ logit cap
 template <typename T>
 __global__ void __launch_bounds__(256)
-logit_softcap_kernel(const T* __restrict__ in, long ldi, float* __restrict__ out, long ldo, long rows, int V, float cap) {
+logit_softcap_kernel(const T* __restrict__ in, long ldi, float* __restrict__ out, long ldo, long rows, int V, float cap, float mult) {
   const long total = rows * V;
   for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
     const long r = i / V;
     const int c = (int)(i - r * V);
-    const float z = (float)in[r * ldi + c];
+    const float z = mult * (float)in[r * ldi + c];
     out[r * ldo + c] = cap > 0.f ? cap * tanhf(z / cap) : z;
   }
 }
@@ -505,7 +525,7 @@ extern "C" int omni_poly_norm(const void* z, int ldz, void* out, int ldo, const 
 extern "C" int omni_conv_heads(const ConvHeads* args, int is_bf16, void* stream) {
   ConvHeads p = *args;
   if (p.T <= 0) return RC_OK;
-  if (p.num_seqs <= 0 || p.H <= 0 || p.G <= 0 || (p.dp & 7) || (p.vp & 7) || (p.ldp & 7) || p.d > p.dp || p.taps < 1)
+  if (p.num_seqs <= 0 || p.H <= 0 || p.G <= 0 || p.GV <= 0 || (p.q_coef != 0.f && !(p.q_every > 0)) || (p.dp & 7) || (p.vp & 7) || (p.ldp & 7) || p.d > p.dp || p.taps < 1)
     return RC_BAD_ARG;
   if ((p.conv == nullptr && p.taps != 1) || (p.taps > 1 && (p.state == nullptr || p.num_state <= 0))) return RC_BAD_ARG;
   if (p.v_mode != 0 && p.v_first == nullptr) return RC_BAD_ARG;
@@ -514,12 +534,12 @@ extern "C" int omni_conv_heads(const ConvHeads* args, int is_bf16, void* stream)
   p.lph = 1;
   while (p.lph < lanes && p.lph < 32) p.lph *= 2;
   const int rows_per_cta = 256 / p.lph;
-  dim3 grid((p.T + rows_per_cta - 1) / rows_per_cta, p.H + 2 * p.G);
+  dim3 grid((p.T + rows_per_cta - 1) / rows_per_cta, p.H + p.G + p.GV);
   cudaStream_t st = (cudaStream_t)stream;
   constexpr int RUN = 8;
   if (is_bf16 && lanes <= 32 && p.T >= 256 && p.taps <= 4 && p.conv != nullptr) {
     const int rows = rows_per_cta * RUN;
-    dim3 rgrid((p.T + rows - 1) / rows, p.H + 2 * p.G);
+    dim3 rgrid((p.T + rows - 1) / rows, p.H + p.G + p.GV);
     switch (p.taps) {
       case 1: conv_heads_run_kernel<1, RUN><<<rgrid, 256, 0, st>>>(p); break;
       case 2: conv_heads_run_kernel<2, RUN><<<rgrid, 256, 0, st>>>(p); break;
@@ -538,13 +558,13 @@ extern "C" int omni_conv_heads(const ConvHeads* args, int is_bf16, void* stream)
   return (int)cudaGetLastError();
 }
 
-extern "C" int omni_logit_softcap(const void* in, long ldi, float* out, long ldo, long rows, int V, float cap, int is_bf16,
-                                  void* stream) {
+extern "C" int omni_logit_softcap(const void* in, long ldi, float* out, long ldo, long rows, int V, float cap, float mult,
+                                  int is_bf16, void* stream) {
   if (rows <= 0) return RC_OK;
   long blocks = (rows * V + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   cudaStream_t st = (cudaStream_t)stream;
-  if (is_bf16) logit_softcap_kernel<bf16><<<(unsigned)blocks, 256, 0, st>>>((const bf16*)in, ldi, out, ldo, rows, V, cap);
-  else logit_softcap_kernel<float><<<(unsigned)blocks, 256, 0, st>>>((const float*)in, ldi, out, ldo, rows, V, cap);
+  if (is_bf16) logit_softcap_kernel<bf16><<<(unsigned)blocks, 256, 0, st>>>((const bf16*)in, ldi, out, ldo, rows, V, cap, mult);
+  else logit_softcap_kernel<float><<<(unsigned)blocks, 256, 0, st>>>((const float*)in, ldi, out, ldo, rows, V, cap, mult);
   return (int)cudaGetLastError();
 }

@@ -2,7 +2,7 @@
 //
 //   omni_moe_route     softmax over expert logits, top-k, optional renormalisation
 //   omni_moe_router    router product and choice in one launch: fp32 logits with a bias, the top-k largest, softmax
-//                      among them (bf16 rows)
+//                      among them, or sigmoid scores divided by their sum, of the best groups of experts (bf16 rows)
 //   omni_moe_topk      the same choice from fp32 logits
 //   omni_moe_pairs_f32 y[p] = act(W[expert of pair p] x[p / per]) in true fp32 (exact mode)
 //   omni_moe_plan      per-expert counts -> segment offsets padded to 128 rows (the GEMM's M
@@ -78,28 +78,89 @@ moe_route_kernel(const __nv_bfloat16* __restrict__ logits, int ld, int T, int E,
   }
 }
 
-// Choice of one token by one warp: the k largest of v (lane + 32 i holds expert lane + 32 i), ties to the lower index;
-// weights are the softmax of the chosen logits.  E <= 256, k <= 16.
-__device__ __forceinline__ void topk_softmax(float (&v)[8], int E, int k, int lane, int* ids, float* weights) {
+// What turns logits into a choice.  sigmoid = 0: softmax among the k largest.  sigmoid = 1: scores 1 / (1 + e^-z); with
+// groups > 0 only the `keep` groups of neighbours with the largest sums of their two best scores take part; weights are
+// scale * score / (sum of the chosen scores + 1e-20).
+struct RouterRule {
+  int sigmoid, groups, keep;
+  float scale;
+};
+
+// the largest of 256 values, value lane + 32 i in v[i]; ties go to the lower index
+__device__ __forceinline__ void warp_best(const float (&v)[8], int lane, float& best, int& bi) {
+  best = -INFINITY;
+  bi = 0x7fffffff;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int e = lane + i * 32;
+    if (v[i] > best || (v[i] == best && v[i] != -INFINITY && e < bi)) { best = v[i]; bi = e; }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+  }
+}
+
+// Leaves the experts of the kept groups in v (scores), -inf elsewhere.  `sh`: 256 floats of this warp.
+__device__ __forceinline__ void keep_groups(float (&v)[8], int E, const RouterRule& rule, int lane, float* sh) {
+  const int size = E / rule.groups;
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (lane + i * 32 < E) sh[lane + i * 32] = v[i];
+  __syncwarp();
+  float sum[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int g = lane + i * 32;
+    sum[i] = -INFINITY;
+    if (g < rule.groups) {
+      float a = sh[g * size], b = size > 1 ? -INFINITY : 0.f;
+      for (int j = 1; j < size; ++j) {
+        const float x = sh[g * size + j];
+        b = fmaxf(b, fminf(a, x));
+        a = fmaxf(a, x);
+      }
+      sum[i] = a + b;
+    }
+  }
+  __syncwarp();
+  unsigned live = 0u;
+  for (int j = 0; j < rule.keep; ++j) {
+    float best;
+    int g;
+    warp_best(sum, lane, best, g);
+    if (g >= rule.groups) break;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (lane + i * 32 == g) sum[i] = -INFINITY;
+      if ((lane + i * 32) / size == g) live |= 1u << i;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (!(live & (1u << i))) v[i] = -INFINITY;
+}
+
+// Choice of one token by one warp from logits v (lane + 32 i holds expert lane + 32 i, -inf past the last), ties to the
+// lower index.  E <= 256, k <= 16.  `sh`: 256 floats of this warp (groups only).
+__device__ __forceinline__ void choose_experts(float (&v)[8], int E, int k, const RouterRule& rule, int lane, float* sh, int* ids,
+                                               float* weights) {
+  if (rule.sigmoid) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = lane + i * 32 < E ? 1.0f / (1.0f + expf(-v[i])) : -INFINITY;
+    if (rule.groups > 0) keep_groups(v, E, rule, lane, sh);
+  }
   float top = 0.f, sum = 0.f, mine = 0.f;
   int mine_id = 0;
   for (int j = 0; j < k; ++j) {
-    float best = -INFINITY;
-    int bi = 0x7fffffff;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int e = lane + i * 32;
-      if (e < E && (v[i] > best || (v[i] == best && e < bi))) { best = v[i]; bi = e; }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
-    }
-    if (bi >= E) bi = j;                       // no finite logit left: any index inside the range
+    float best;
+    int bi;
+    warp_best(v, lane, best, bi);
+    if (bi >= E) bi = j;                       // no finite value left: any index inside the range
     if (j == 0) top = best;
-    const float w = expf(best - top);
+    const float w = rule.sigmoid ? best : expf(best - top);
     sum += w;
     if (lane == j) { mine = w; mine_id = bi; }
 #pragma unroll
@@ -108,13 +169,14 @@ __device__ __forceinline__ void topk_softmax(float (&v)[8], int E, int k, int la
   }
   if (lane < k) {
     ids[lane] = mine_id;
-    weights[lane] = mine / sum;
+    weights[lane] = rule.sigmoid ? mine / (sum + 1e-20f) * rule.scale : mine / sum;
   }
 }
 
 __global__ void __launch_bounds__(256)
-moe_topk_kernel(const float* __restrict__ logits, long ld, int T, int E, int k, int* __restrict__ ids,
+moe_topk_kernel(const float* __restrict__ logits, long ld, int T, int E, int k, RouterRule rule, int* __restrict__ ids,
                 float* __restrict__ weights) {
+  __shared__ float sh[8][256];
   const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= T) return;
   float v[8];
@@ -123,7 +185,7 @@ moe_topk_kernel(const float* __restrict__ logits, long ld, int T, int E, int k, 
     const int e = lane + i * 32;
     v[i] = e < E ? logits[t * ld + e] : -INFINITY;
   }
-  topk_softmax(v, E, k, lane, ids + (long)t * k, weights + (long)t * k);
+  choose_experts(v, E, k, rule, lane, sh[threadIdx.x >> 5], ids + (long)t * k, weights + (long)t * k);
 }
 
 // Router of MT * 16 tokens per block: NW warps share the contraction (each takes every NW-th 32-channel chunk), 64 experts
@@ -133,8 +195,8 @@ moe_topk_kernel(const float* __restrict__ logits, long ld, int T, int E, int k, 
 template <int MT, int NW>
 __global__ void __launch_bounds__(32 * NW)
 moe_router_kernel(const __nv_bfloat16* __restrict__ x, long ldx, const __nv_bfloat16* __restrict__ w, long ldw,
-                  const float* __restrict__ bias, int T, int D, int E, int Ep, int k, int* __restrict__ ids,
-                  float* __restrict__ weights) {
+                  const float* __restrict__ bias, int T, int D, int E, int Ep, int k, RouterRule rule,
+                  int* __restrict__ ids, float* __restrict__ weights) {
   extern __shared__ float sm[];
   float* part = sm;                            // [NW][MT * 16][64]
   float* logit = sm + NW * MT * 16 * 64;        // [MT * 16][256]
@@ -205,7 +267,8 @@ moe_router_kernel(const __nv_bfloat16* __restrict__ x, long ldx, const __nv_bflo
     float v[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) v[i] = lane + i * 32 < E ? logit[r * 256 + lane + i * 32] : -INFINITY;
-    topk_softmax(v, E, k, lane, ids + (long)t * k, weights + (long)t * k);
+    __syncwarp();                              // the row's logits become scratch
+    choose_experts(v, E, k, rule, lane, logit + r * 256, ids + (long)t * k, weights + (long)t * k);
   }
 }
 
@@ -468,18 +531,24 @@ extern "C" int omni_moe_route(const void* logits, int ld, int T, int E, int k, i
   return (int)cudaGetLastError();
 }
 
-extern "C" int omni_moe_topk(const float* logits, long ld, int T, int E, int k, int* ids, float* weights, void* stream) {
+static bool router_rule_ok(const RouterRule& r, int E, int k) {
+  if (E > 256 || E < 1 || k > 16 || k > E || k < 1) return false;
+  return r.groups == 0 || (r.sigmoid && r.groups > 0 && E % r.groups == 0 && r.keep >= 1 && r.keep <= r.groups && r.keep * (E / r.groups) >= k);
+}
+
+extern "C" int omni_moe_topk(const float* logits, long ld, int T, int E, int k, const RouterRule* rule, int* ids, float* weights,
+                             void* stream) {
   if (T <= 0) return RC_OK;
-  if (E > 256 || k > 16 || k > E || k < 1) return RC_BAD_ARG;
-  moe_topk_kernel<<<(T + 7) / 8, 256, 0, (cudaStream_t)stream>>>(logits, ld, T, E, k, ids, weights);
+  if (!router_rule_ok(*rule, E, k)) return RC_BAD_ARG;
+  moe_topk_kernel<<<(T + 7) / 8, 256, 0, (cudaStream_t)stream>>>(logits, ld, T, E, k, *rule, ids, weights);
   return (int)cudaGetLastError();
 }
 
 // x [T, D] and w [Ep >= E, D] bf16 (D, pitches multiples of 8), bias [E] fp32 or null.
 extern "C" int omni_moe_router(const void* x, long ldx, const void* w, long ldw, const float* bias, int T, int D, int E, int Ep,
-                               int k, int* ids, float* weights, void* stream) {
+                               int k, const RouterRule* rule, int* ids, float* weights, void* stream) {
   if (T <= 0) return RC_OK;
-  if (E > 256 || k > 16 || k > E || k < 1 || D <= 0 || (D & 7) || (ldx & 7) || (ldw & 7)) return RC_BAD_ARG;
+  if (!router_rule_ok(*rule, E, k) || D <= 0 || (D & 7) || (ldx & 7) || (ldw & 7)) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
   const bf16* xb = (const bf16*)x;
   const bf16* wb = (const bf16*)w;
@@ -487,11 +556,11 @@ extern "C" int omni_moe_router(const void* x, long ldx, const void* w, long ldw,
   if (T > 148 * 16) {
     const int smem = (8 * 32 * 64 + 32 * 256) * 4;
     if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<2, 8>, smem, prep[0])) return e;
-    moe_router_kernel<2, 8><<<(T + 31) / 32, 256, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
+    moe_router_kernel<2, 8><<<(T + 31) / 32, 256, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, *rule, ids, weights);
   } else {
     const int smem = (16 * 16 * 64 + 16 * 256) * 4;
     if (int e = ensure_dynamic_smem((const void*)moe_router_kernel<1, 16>, smem, prep[1])) return e;
-    moe_router_kernel<1, 16><<<(T + 15) / 16, 512, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, ids, weights);
+    moe_router_kernel<1, 16><<<(T + 15) / 16, 512, smem, st>>>(xb, ldx, wb, ldw, bias, T, D, E, Ep, k, *rule, ids, weights);
   }
   return (int)cudaGetLastError();
 }

@@ -1,11 +1,12 @@
-// Steps of decoders whose fp32 residual stream takes scaled branches and whose norms have no statistics, for bf16
-// activations (serving) and fp32 activations (exact mode):
+// Steps of decoders whose fp32 residual stream takes scaled branches, for bf16 activations (serving) and fp32
+// activations (exact mode):
 //
-//   omni_stream_step    x += mult * branch, then the rows the next GEMM reads (one launch).  The branch is a row, a
-//                       row divided by its rms with a gain per channel, or the weighted sum of a token's expert
-//                       rows plus a shared expert's row; or x starts as an embedding row.  Output: nothing, x in the
-//                       activations' type, or w tanh(alpha x) + b.
-//   omni_rotary_rows    cos / sin of position * frequency, angles reduced in fp64
+//   omni_stream_step    x += mult * branch, then the rows the next GEMM reads (one launch).  The branch is a row or the
+//                       weighted sum of a token's expert rows plus a shared expert's row (times the sigmoid of one
+//                       logit per token, where given); with a gain per channel either is divided by its rms first.
+//                       Or x starts as mult * an embedding row, or as a row that replaces it.  Output: nothing, x in the activations' type,
+//                       w tanh(alpha x) + b, or x divided by its rms times w.
+//   omni_rotary_rows    magnitude * cos / sin of position * frequency, angles reduced in fp64
 //   omni_gelu_lookup    z = gelu(z) * a token's row of a table
 //
 // Rows are padded to a multiple of 8 channels with zeros; padding does not count in means.
@@ -14,8 +15,8 @@
 
 namespace omni {
 
-enum StreamSource : int { SRC_EMBED = 0, SRC_ROW = 1, SRC_NORMED = 2, SRC_EXPERTS = 3 };
-enum StreamOut : int { OUT_NONE = 0, OUT_CAST = 1, OUT_TANH = 2 };
+enum StreamSource : int { SRC_EMBED = 0, SRC_ROW = 1, SRC_NORMED = 2, SRC_EXPERTS = 3, SRC_EXPERTS_NORMED = 4 };
+enum StreamOut : int { OUT_NONE = 0, OUT_CAST = 1, OUT_TANH = 2, OUT_RMS = 3 };
 
 struct StreamStep {
   float* x;
@@ -32,6 +33,8 @@ struct StreamStep {
   void* out;                           // [rows, Dp]
   const float* alpha; const float* w; const float* b;
   int* status;
+  const void* shared_gate; long ldsg;  // [rows] logits at this pitch, or nullptr
+  float out_eps;                       // OUT_RMS
 };
 
 // tanh for values that are rounded to bf16 next: absolute error about 1e-7
@@ -43,26 +46,34 @@ template <> __device__ __forceinline__ float tanh_for<__nv_bfloat16>(float z) { 
 template <typename T, int SRC, int NV>
 __global__ void __launch_bounds__(1024)
 stream_step_kernel(const StreamStep p) {
+  constexpr bool EXPERTS = SRC == SRC_EXPERTS || SRC == SRC_EXPERTS_NORMED;
+  constexpr bool NORMED = SRC == SRC_NORMED || SRC == SRC_EXPERTS_NORMED;
   __shared__ float sh[32];
   const long r = blockIdx.x;
   float xv[NV][8], yv[NV][8];
   float ss[1] = {0.f};
   const T* src = nullptr;
+  float scale = p.mult;
   if (SRC == SRC_EMBED) {
     long id = p.ids[r];
     id = id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id);
     const bool over = p.overlay != nullptr && (p.overlay_mask == nullptr || p.overlay_mask[r]);
+    if (over) scale = 1.f;
     src = over ? static_cast<const T*>(p.overlay) + r * p.Dp : static_cast<const T*>(p.embed) + id * p.Dp;
-  } else if (SRC != SRC_EXPERTS) {
+  } else if (!EXPERTS) {
     src = static_cast<const T*>(p.y) + r * p.ldy;
   }
+  float sg = 1.f;
+  if (EXPERTS && p.shared_gate) sg = 1.0f / (1.0f + expf(-(float)static_cast<const T*>(p.shared_gate)[r * p.ldsg]));
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * 8;
     if (c >= p.Dp) continue;
-    if (SRC == SRC_EXPERTS) {
+    if (EXPERTS) {
       if (p.shared) {
         load8<T>(static_cast<const T*>(p.shared) + r * p.lds + c, yv[i]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) yv[i][e] *= sg;
       } else {
 #pragma unroll
         for (int e = 0; e < 8; ++e) yv[i][e] = 0.f;
@@ -84,25 +95,25 @@ stream_step_kernel(const StreamStep p) {
       load8<T>(src + c, yv[i]);
     }
     if (SRC != SRC_EMBED) load8<float>(p.x + r * p.Dp + c, xv[i]);
-    if (SRC == SRC_NORMED) {
+    if (NORMED) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss[0] = fmaf(yv[i][e], yv[i][e], ss[0]);
     }
   }
-  float scale = p.mult;
-  if (SRC == SRC_NORMED) {
+  if (NORMED) {
     block_sum<1>(ss, sh);
     scale = p.mult * rms_scale(ss[0], p.D, p.eps);
   }
   const float alpha = p.out_mode == OUT_TANH ? p.alpha[0] : 0.f;
+  float so[1] = {0.f};
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * 8;
     if (c >= p.Dp) continue;
     if (SRC == SRC_EMBED) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) xv[i][e] = yv[i][e];
-    } else if (SRC == SRC_NORMED) {
+      for (int e = 0; e < 8; ++e) xv[i][e] = scale * yv[i][e];
+    } else if (NORMED) {
       float g[8];
       load8<float>(p.gain + c, g);
 #pragma unroll
@@ -121,20 +132,34 @@ stream_step_kernel(const StreamStep p) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) w[e] = fmaf(w[e], tanh_for<T>(alpha * xv[i][e]), b[e]);
       store8<T>(static_cast<T*>(p.out) + r * p.Dp + c, w);
+    } else if (p.out_mode == OUT_RMS) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) so[0] = fmaf(xv[i][e], xv[i][e], so[0]);
     }
+  }
+  if (p.out_mode != OUT_RMS) return;
+  block_sum<1>(so, sh);
+  const float scale_out = rms_scale(so[0], p.D, p.out_eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c >= p.Dp) continue;
+    scale_gain8(xv[i], scale_out, p.w, 1, c);
+    store8<T>(static_cast<T*>(p.out) + r * p.Dp + c, xv[i]);
   }
 }
 
-// out[t, i] = (cos, sin) of pos[t] * freq[i]
+// out[t, i] = mag (cos, sin) of pos[t] * freq[i]
 __global__ void __launch_bounds__(256)
-rotary_rows_kernel(const long* __restrict__ pos, const double* __restrict__ freq, float2* __restrict__ out, int T, int half) {
+rotary_rows_kernel(const long* __restrict__ pos, const double* __restrict__ freq, float mag, float2* __restrict__ out, int T,
+                   int half) {
   const long n = (long)T * half;
   for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long)gridDim.x * blockDim.x) {
     const double two_pi = 6.283185307179586476925;
     const double a = (double)pos[i / half] * freq[i % half];
     float s, c;
     sincosf((float)(a - two_pi * rint(a / two_pi)), &s, &c);
-    out[i] = make_float2(c, s);
+    out[i] = make_float2(mag * c, mag * s);
   }
 }
 
@@ -169,6 +194,7 @@ static int launch_source(const StreamStep& p, int threads, int nv, cudaStream_t 
     case SRC_ROW: return launch_step<T, SRC_ROW>(p, threads, nv, st);
     case SRC_NORMED: return launch_step<T, SRC_NORMED>(p, threads, nv, st);
     case SRC_EXPERTS: return launch_step<T, SRC_EXPERTS>(p, threads, nv, st);
+    case SRC_EXPERTS_NORMED: return launch_step<T, SRC_EXPERTS_NORMED>(p, threads, nv, st);
     default: return RC_BAD_ARG;
   }
 }
@@ -183,17 +209,19 @@ extern "C" int omni_stream_step(const StreamStep* args, int is_bf16, void* strea
   int threads, nv;
   if ((p.Dp & 7) || (p.ldy & 7) || (p.lds & 7) || p.D > p.Dp || !row_shape(p.Dp, threads, nv)) return RC_BAD_ARG;
   if (p.source == SRC_EMBED ? (!p.ids || !p.embed || p.vocab <= 0) : !p.y) return RC_BAD_ARG;
-  if ((p.source == SRC_NORMED && !p.gain) || (p.source == SRC_EXPERTS && (!p.weights || p.k <= 0))) return RC_BAD_ARG;
-  if ((p.out_mode != OUT_NONE && !p.out) || (p.out_mode == OUT_TANH && (!p.alpha || !p.w || !p.b))) return RC_BAD_ARG;
+  const bool experts = p.source == SRC_EXPERTS || p.source == SRC_EXPERTS_NORMED;
+  if (((p.source == SRC_NORMED || p.source == SRC_EXPERTS_NORMED) && !p.gain) || (experts && (!p.weights || p.k <= 0))) return RC_BAD_ARG;
+  if ((p.out_mode != OUT_NONE && !p.out) || (p.out_mode == OUT_TANH && (!p.alpha || !p.w || !p.b)) || (p.out_mode == OUT_RMS && !p.w))
+    return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
   return is_bf16 ? launch_source<__nv_bfloat16>(p, threads, nv, st) : launch_source<float>(p, threads, nv, st);
 }
 
-extern "C" int omni_rotary_rows(const long* pos, const double* freq, float* out, int T, int half, void* stream) {
+extern "C" int omni_rotary_rows(const long* pos, const double* freq, float mag, float* out, int T, int half, void* stream) {
   if (T <= 0 || half <= 0) return RC_OK;
   long blocks = ((long)T * half + 255) / 256;
   if (blocks > 148 * 8) blocks = 148 * 8;
-  rotary_rows_kernel<<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>(pos, freq, reinterpret_cast<float2*>(out), T, half);
+  rotary_rows_kernel<<<(unsigned)blocks, 256, 0, (cudaStream_t)stream>>>(pos, freq, mag, reinterpret_cast<float2*>(out), T, half);
   return (int)cudaGetLastError();
 }
 

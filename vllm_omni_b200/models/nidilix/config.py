@@ -6,6 +6,7 @@ from dataclasses import dataclass, field
 import torch
 
 from ...ops.latent_attention import LatentShape
+from ...ops.moe import Router
 from ...ops.recurrent import GatedScanShape
 from ..packed_decoder import round_up
 from ..seq_table import StateTensor
@@ -56,9 +57,12 @@ class ExpertsConfig:
             raise ValueError(f"unknown feed-forward kind {d['kind']!r}")
         m = cls(int(d["router"]["experts"]), int(d["router"]["top"]), int(d["expert"]["ff"]),
                 int(d["shared"]["ff"]) if d.get("shared") else None)
-        if not 1 <= m.top <= m.experts:
-            raise ValueError(f"router.top ({m.top}) must be between 1 and experts ({m.experts})")
+        m.router                        # refuses a choice that cannot be made
         return m
+
+    @property
+    def router(self) -> Router:
+        return Router(self.experts, self.top)
 
 
 @dataclass

@@ -159,8 +159,7 @@ class _Experts(nn.Module):
     def forward(self, xn):
         """(rows of the chosen experts with their weights, shared expert's rows or None)."""
         shared = self.shared_down(self.shared_up(xn, act="relu2")) if self.m.shared_ff else None
-        return moe.expert_rows(xn, self.router, self.router_b, self.m.experts, self.m.top, self.up, self.down, act="relu2",
-                               ws=self.ws), shared
+        return moe.expert_rows(xn, self.router, self.router_b, self.m.router, self.up, self.down, act="relu2", ws=self.ws), shared
 
 
 class NidilixLayer(nn.Module):

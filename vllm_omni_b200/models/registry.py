@@ -13,6 +13,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "Qwen3MoeForCausalLM": ("vllm_omni_b200.models.text", "build_text_model"),
     "Tavulix": ("vllm_omni_b200.models.tavulix.model", "build_tavulix"),
     "Nidilix": ("vllm_omni_b200.models.nidilix.model", "build_nidilix"),
+    "Milivik": ("vllm_omni_b200.models.milivik.model", "build_milivik"),
     "BagelForConditionalGeneration": ("vllm_omni_b200.models.text", "build_text_model"),
 }
 

@@ -33,7 +33,8 @@ def round_up4(n: int) -> int:
 @dataclass
 class KeyGroup:
     """Sequences whose keys lie back to back in one buffer (``SeqTable.long_groups``)."""
-    key_start: torch.Tensor                    # int32 [S of the batch]: first key of a member
+    key_start: torch.Tensor                    # int32 [S of the batch]: where position 0 of a member is, or (< first key)
+                                               # would be if a window did not leave its first positions out
     members: torch.Tensor                      # int32 [2 (members + 1)]: (sequence, first key), closed by (-1, keys)
     n_members: int
     keys: int
@@ -108,34 +109,42 @@ class SeqTable:
             self._items[("short", limit)] = got
         return got
 
-    def long_groups(self, limit: int, max_keys: int, rows_per_block: int):
-        """The sequences with more than ``limit`` rows in groups whose keys (context and new tokens) fit ``max_keys``
-        together, at least one sequence each: ``KeyGroup`` list, for kernels that want a group's keys back to back."""
-        got = self._items.get(("long", limit, max_keys, rows_per_block))
+    def _first_key(self, s: int, window: int | None) -> int:
+        """First position that a row of sequence s sees, rounded down to the 32 keys a kernel reads at a time."""
+        return 0 if window is None else max(0, self.contexts[s] - window + 1) // 32 * 32
+
+    def long_groups(self, limit: int, max_keys: int, rows_per_block: int, window: int | None = None):
+        """The sequences with more than ``limit`` rows in groups whose keys (context and new tokens, with a ``window`` only
+        those some row sees) fit ``max_keys`` together, at least one sequence each: ``KeyGroup`` list, for kernels that want
+        a group's keys back to back."""
+        key = ("long", limit, max_keys, rows_per_block, window)
+        got = self._items.get(key)
         if got is None:
             got, cur, keys = [], [], 0
             for s, n in enumerate(self.lens):
                 if n <= limit:
                     continue
-                k = n + self.contexts[s]
+                k = n + self.contexts[s] - self._first_key(s, window)
                 if cur and keys + k > max_keys:
-                    got.append(self._key_group(cur, rows_per_block))
+                    got.append(self._key_group(cur, rows_per_block, window))
                     cur, keys = [], 0
                 cur.append(s)
                 keys += k
             if cur:
-                got.append(self._key_group(cur, rows_per_block))
-            self._items[("long", limit, max_keys, rows_per_block)] = got
+                got.append(self._key_group(cur, rows_per_block, window))
+            self._items[key] = got
         return got
 
-    def _key_group(self, seqs, rows_per_block):
-        start, at = [0] * self.n_seqs, 0
+    def _key_group(self, seqs, rows_per_block, window):
+        start, firsts, at = [0] * self.n_seqs, [], 0
         for s in seqs:
-            start[s] = at
-            at += self.lens[s] + self.contexts[s]
+            lo = self._first_key(s, window)
+            start[s] = at - lo
+            firsts += [s, at]
+            at += self.lens[s] + self.contexts[s] - lo
         items = sorted(((s, o) for s in seqs for o in range(0, self.lens[s], rows_per_block)),
                        key=lambda it: -(self.contexts[it[0]] + it[1]))     # most keys first
-        members = [v for s in seqs for v in (s, start[s])] + [-1, at]      # (sequence, first key) pairs, then the end
+        members = firsts + [-1, at]                                        # (sequence, first key) pairs, then the end
         flat = start + [0] * (-len(start) % 4) + members + [0] * (-len(members) % 4) + [v for it in items for v in it]
         buf = torch.tensor(flat, dtype=torch.int32).to(self.q_start.device)
         o1 = round_up4(len(start))

@@ -191,10 +191,15 @@ def silu_mul(x, out=None):
             return out
         return y
     x2 = x.reshape(-1, 2 * N)
-    assert x2.stride(1) == 1 and x.dtype == torch.bfloat16
+    assert x2.stride(1) == 1 and x.dtype in (torch.bfloat16, torch.float32)
     if out is None:
         out = torch.empty(*x.shape[:-1], N, dtype=x.dtype, device=x.device)
     o2 = out.view(-1, N)
+    if x.dtype == torch.float32:
+        rc = nv.lib("elementwise").omni_silu_mul_f32(nv.ptr(x2), nv.ptr(o2), c_long(x2.shape[0]), c_int(N), c_long(x2.stride(0)),
+                                                     c_long(o2.stride(0)), nv.stream_ptr())
+        nv.check_rc(rc, "omni_silu_mul_f32")
+        return out
     rc = nv.lib("elementwise").omni_silu_mul(nv.ptr(x2), nv.ptr(o2), c_long(x2.shape[0]), c_int(N),
                                              c_int(x2.stride(0)), c_int(o2.stride(0)), nv.stream_ptr())
     nv.check_rc(rc, "omni_silu_mul")

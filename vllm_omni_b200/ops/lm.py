@@ -88,14 +88,14 @@ def poly_norm(z, coef, n: int, eps: float, out=None):
     return out
 
 
-def logit_softcap(logits, cap: float | None, n: int):
-    """First ``n`` columns of ``logits`` as fp32, bounded to cap * tanh(logit / cap) when ``cap`` is set."""
+def logit_softcap(logits, cap: float | None, n: int, mult: float = 1.0):
+    """``mult`` times the first ``n`` columns of ``logits`` as fp32, bounded to cap * tanh(. / cap) when ``cap`` is set."""
     if not logits.is_cuda:
-        f = logits[:, :n].float()
+        f = mult * logits[:, :n].float()
         return f if not cap else cap * torch.tanh(f / cap)
     out = torch.empty(logits.shape[0], n, dtype=torch.float32, device=logits.device)
     rc = nv.lib("lm_ops").omni_logit_softcap(nv.ptr(logits), c_long(logits.stride(0)), nv.ptr(out), c_long(n),
-                                             c_long(logits.shape[0]), c_int(n), c_float(cap or 0.0), _bf(logits),
+                                             c_long(logits.shape[0]), c_int(n), c_float(cap or 0.0), c_float(mult), _bf(logits),
                                              nv.stream_ptr())
     nv.check_rc(rc, "omni_logit_softcap")
     return out
@@ -109,7 +109,8 @@ class _ConvHeads(ctypes.Structure):
                 ("context", c_void_p), ("slots", c_void_p), ("state", c_void_p), ("state_in", c_void_p),
                 ("state_out", c_void_p), ("q_out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p),
                 ("v_first", c_void_p), ("v_mode", c_int), ("lam", c_void_p), ("num_slots", c_long),
-                ("num_state", c_int), ("num_seqs", c_int), ("status", c_void_p), ("lph", c_int)]
+                ("num_state", c_int), ("num_seqs", c_int), ("status", c_void_p), ("lph", c_int), ("GV", c_int),
+                ("q_coef", c_float), ("q_every", ctypes.c_double)]
 
 
 @dataclass
@@ -122,17 +123,29 @@ class HeadShape:
     dp: int
     vp: int
     taps: int = 0                     # convolution taps, 0 = no convolution
+    v_heads: int = 0                  # value heads where they are fewer than key heads, 0 = kv_heads
+
+    @property
+    def values(self) -> int:
+        return self.v_heads or self.kv_heads
 
     @property
     def channels(self) -> int:        # convolved channels: q, k and v
-        return (self.heads + self.kv_heads) * self.dp + self.kv_heads * self.vp
+        return (self.heads + self.kv_heads) * self.dp + self.values * self.vp
+
+
+@dataclass(frozen=True)
+class QueryGrowth:
+    """Queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    coef: float
+    every: float
 
 
 def conv_heads(proj, hs: HeadShape, seqs, slots, k_cache, v_cache, *, conv=None, state=None, q_norm=None, k_norm=None,
-               eps: float = 1e-6, v_first=None, v_mode: str = "plain", lam=None):
+               eps: float = 1e-6, v_first=None, v_mode: str = "plain", lam=None, growth: QueryGrowth | None = None):
     """One pass over the packed projection ``proj`` [T, >= channels] (columns q | k | v): causal convolution
-    over time per channel, RMS norm of every q and k head, value mixing, K/V to their pages, convolution
-    history to the state pool.  Returns q [T, H, dp].
+    over time per channel, RMS norm of every q and k head, ``growth`` of q, value mixing, K/V to their pages,
+    convolution history to the state pool.  Returns q [T, H, dp].
 
     ``conv``: fp32 [taps, channels]; ``state``: [rows, taps - 1, channels], read at ``seqs.state_in`` and
     written at ``seqs.state_out`` (distinct rows; < 0 = not written).  ``v_mode``: "plain", "save" (the
@@ -143,9 +156,9 @@ def conv_heads(proj, hs: HeadShape, seqs, slots, k_cache, v_cache, *, conv=None,
     q_out = torch.empty(T, H, dp, dtype=proj.dtype, device=proj.device)
     if not proj.is_cuda:
         return _conv_heads_cpu(proj, hs, seqs, slots, k_cache, v_cache, conv, state, q_norm, k_norm, eps, v_first, v_mode,
-                               lam, q_out, taps)
+                               lam, q_out, taps, growth)
     assert proj.stride(1) == 1 and slots.dtype == torch.int32 and k_cache.is_contiguous() and v_cache.is_contiguous()
-    assert k_cache.shape[2:] == (G, dp) and v_cache.shape[2:] == (G, vp) and k_cache.dtype == proj.dtype
+    assert k_cache.shape[2:].numel() == G * dp and v_cache.shape[2:] == (hs.values, vp) and k_cache.dtype == proj.dtype
     a = _ConvHeads()
     P = lambda t: 0 if t is None else t.data_ptr()
     a.proj, a.ldp, a.T, a.H, a.G, a.dp, a.vp, a.d, a.taps = P(proj), proj.stride(0), T, H, G, dp, vp, hs.dim, taps
@@ -156,14 +169,16 @@ def conv_heads(proj, hs: HeadShape, seqs, slots, k_cache, v_cache, *, conv=None,
         a.state, a.state_in, a.state_out, a.num_state = P(state), P(seqs.state_in), P(seqs.state_out), state.shape[0]
     a.q_out, a.k_cache, a.v_cache = P(q_out), P(k_cache), P(v_cache)
     a.v_first, a.v_mode, a.lam = P(v_first), {"plain": 0, "save": 1, "mix": 2}[v_mode], P(lam)
-    a.num_slots, a.num_seqs = k_cache.shape[0] * k_cache.shape[1], seqs.n_seqs
+    a.num_slots, a.num_seqs, a.GV = k_cache.shape[0] * k_cache.shape[1], seqs.n_seqs, hs.values
+    if growth is not None:
+        a.q_coef, a.q_every = growth.coef, growth.every
     a.status = P(nv.status_word(proj.device))
     nv.check_rc(nv.lib("lm_ops").omni_conv_heads(ctypes.byref(a), _bf(proj), nv.stream_ptr()), "omni_conv_heads")
     return q_out
 
 
 def _conv_heads_cpu(proj, hs, seqs, slots, k_cache, v_cache, conv, state, q_norm, k_norm, eps, v_first, v_mode, lam,
-                    q_out, taps):
+                    q_out, taps, growth):
     H, G, dp, vp, C = hs.heads, hs.kv_heads, hs.dp, hs.vp, hs.channels
     T, hist = proj.shape[0], taps - 1
     u = proj[:, :C].float()
@@ -187,6 +202,9 @@ def _conv_heads_cpu(proj, hs, seqs, slots, k_cache, v_cache, conv, state, q_norm
         q = _rms(q, hs.dim, eps) * q_norm
     if k_norm is not None:
         k = _rms(k, hs.dim, eps) * k_norm
+    if growth is not None:
+        pos = torch.cat([torch.arange(int(c), int(c) + int(b - a)) for a, b, c in zip(seqs.q_start, seqs.q_start[1:], seqs.context)])
+        q = q * (1 + growth.coef * torch.log(torch.floor((pos + 1).double() / growth.every) + 1)).float()[:, None, None]
     if v_mode == "save":
         v_first.copy_(v)
     elif v_mode == "mix":
@@ -195,5 +213,5 @@ def _conv_heads_cpu(proj, hs, seqs, slots, k_cache, v_cache, conv, state, q_norm
     ok = slots >= 0
     where = slots[ok].long()
     k_cache.view(-1, G * dp)[where] = k.reshape(T, -1)[ok].to(k_cache.dtype)
-    v_cache.view(-1, G * vp)[where] = v[ok].to(v_cache.dtype)
+    v_cache.view(-1, hs.values * vp)[where] = v[ok].to(v_cache.dtype)
     return q_out

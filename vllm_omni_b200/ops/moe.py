@@ -155,45 +155,102 @@ def _plan_and_dispatch(ws, x, E, e_lo, e_hi, k):
                                       c_int(D), nv.ptr(ws.xp), st), "omni_moe_dispatch")
 
 
-def expert_rows(x, router_w, router_b, experts: int, k: int, up, down, act: str, ws: MoEWorkspace | None = None) -> ExpertRows:
-    """Two-matrix experts behind a router with fp32 logits: the k largest of ``router_w x + router_b`` (rows past
-    ``experts`` are padding), weighted by the softmax among themselves; y = down[e] act(up[e] x) per choice.
+class _RouterRule(ctypes.Structure):
+    _fields_ = [("sigmoid", c_int), ("groups", c_int), ("keep", c_int), ("scale", ctypes.c_float)]
 
-    x [T, D]; router_w [>= E, D]; router_b fp32; up [E, F, D]; down [E, D, F].  The weighted sum is the caller's
-    (ops/stream.py add_expert_rows_ fuses it with the residual add)."""
-    assert act == "relu2"
+
+@dataclass(frozen=True)
+class Router:
+    """How logits become a choice.  Without ``sigmoid``: the ``top`` largest, weighted by the softmax among themselves.  With
+    it: scores 1 / (1 + e^-z), weights ``scale`` * score / (sum of the chosen scores + 1e-20); with ``groups`` only experts
+    of the ``keep`` groups of neighbours with the largest sums of their two best scores take part."""
+    experts: int
+    top: int
+    sigmoid: bool = False
+    groups: int = 0
+    keep: int = 0
+    scale: float = 1.0
+
+    def __post_init__(self):
+        if not 1 <= self.top <= self.experts:
+            raise ValueError(f"router: top ({self.top}) must be between 1 and experts ({self.experts})")
+        if self.experts > 256 or self.top > 16:
+            raise ValueError(f"router: at most 256 experts and 16 per token, got {self.experts} and {self.top}")
+        if self.groups:
+            if self.experts % self.groups:
+                raise ValueError(f"router: experts ({self.experts}) must be a multiple of groups ({self.groups})")
+            if not 1 <= self.keep <= self.groups or self.keep * (self.experts // self.groups) < self.top:
+                raise ValueError(f"router: {self.keep} of {self.groups} groups do not hold {self.top} of {self.experts} experts")
+
+    @property
+    def rule(self) -> _RouterRule:
+        return _RouterRule(int(self.sigmoid), self.groups, self.keep, self.scale)
+
+    def choose(self, logits):
+        """(ids, weights) [T, top] of logits [T, >= experts]: PyTorch restatement."""
+        z = logits[:, :self.experts].float()
+        if not self.sigmoid:
+            val, ids = torch.topk(z, self.top, dim=-1)
+            return ids, torch.softmax(val, -1)
+        s = pick = torch.sigmoid(z)
+        if self.groups:
+            per = s.view(-1, self.groups, self.experts // self.groups)
+            best = per.topk(min(2, per.shape[2]), -1).values.sum(-1).topk(self.keep, -1).indices
+            live = torch.zeros(per.shape[:2], dtype=torch.bool, device=z.device).scatter_(1, best, True)
+            pick = per.masked_fill(~live[:, :, None], float("-inf")).flatten(1)
+        ids = pick.topk(self.top, -1).indices
+        w = s.gather(1, ids)
+        return ids, w / (w.sum(-1, keepdim=True) + 1e-20) * self.scale
+
+
+def expert_rows(x, router_w, router_b, router: Router, up, down, act: str, ws: MoEWorkspace | None = None) -> ExpertRows:
+    """Experts behind a router with fp32 logits ``router_w x + router_b`` (rows past ``router.experts`` are padding); per choice
+    y = down[e] relu(up[e] x)^2 (``act="relu2"``) or down[e] (silu(gate) * lift) with [gate | lift] = up[e] x (``"swiglu"``).
+
+    x [T, D]; router_w [>= E, D]; router_b fp32 or None; up [E, F or 2 F, D]; down [E, D, F].  The weighted sum is the
+    caller's (ops/stream.py add_expert_rows_ fuses it with the residual add)."""
+    assert act in ("relu2", "swiglu")
     T, D = x.shape
-    Fd = down.shape[2]
+    Fd, experts, k = down.shape[2], router.experts, router.top
+    assert up.shape[1] == (2 * Fd if act == "swiglu" else Fd)
     if not x.is_cuda:
-        logits = F.linear(x.float(), router_w.float(), router_b)[:, :experts]
-        val, ids = torch.topk(logits, k, dim=-1)
+        ids, w = router.choose(F.linear(x.float(), router_w.float(), router_b))
         y = torch.empty(T * k, D)
         for e in range(experts):
             hit = (ids.reshape(-1) == e).nonzero()[:, 0]
             if hit.numel():
-                h = F.relu(F.linear(x[hit // k].float(), up[e].float())).square().to(x.dtype).float()
-                y[hit] = F.linear(h, down[e].float())
-        return ExpertRows(y.to(x.dtype), None, torch.softmax(val, -1))
-    assert x.stride(1) == 1 and router_b.dtype == torch.float32 and up.is_contiguous() and down.is_contiguous()
-    lib, st = nv.lib("moe"), nv.stream_ptr()
+                h = F.linear(x[hit // k].float(), up[e].float())
+                h = F.silu(h[:, :Fd]) * h[:, Fd:] if act == "swiglu" else F.relu(h).square()
+                y[hit] = F.linear(h.to(x.dtype).float(), down[e].float())
+        return ExpertRows(y.to(x.dtype), None, w)
+    assert x.stride(1) == 1 and up.is_contiguous() and down.is_contiguous()
+    assert router_b is None or router_b.dtype == torch.float32
+    lib, st, rule = nv.lib("moe"), nv.stream_ptr(), router.rule
     if x.dtype == torch.float32:
         logits = gemm.linear(x, router_w, router_b)
         ids = torch.empty(T, k, dtype=torch.int32, device=x.device)
         w = torch.empty(T, k, dtype=torch.float32, device=x.device)
-        nv.check_rc(lib.omni_moe_topk(nv.ptr(logits), c_long(logits.stride(0)), c_int(T), c_int(experts), c_int(k), nv.ptr(ids),
-                                      nv.ptr(w), st), "omni_moe_topk")
-        h, y = (torch.empty(T * k, n, dtype=x.dtype, device=x.device) for n in (Fd, D))
-        for a, per, m, out, relu in ((x, k, up, h, 1), (h, 1, down, y, 0)):
+        nv.check_rc(lib.omni_moe_topk(nv.ptr(logits), c_long(logits.stride(0)), c_int(T), c_int(experts), c_int(k), ctypes.byref(rule),
+                                      nv.ptr(ids), nv.ptr(w), st), "omni_moe_topk")
+
+        def pairs(a, per, m, relu2=0):
+            out = torch.empty(T * k, m.shape[1], dtype=x.dtype, device=x.device)
             nv.check_rc(lib.omni_moe_pairs_f32(nv.ptr(a), c_long(a.stride(0)), c_int(per), nv.ptr(ids), nv.ptr(m), c_int(experts),
                                                nv.ptr(out), c_long(out.stride(0)), c_long(T * k), c_int(m.shape[1]),
-                                               c_int(m.shape[2]), c_int(relu), st), "omni_moe_pairs_f32")
-        return ExpertRows(y, None, w)
+                                               c_int(m.shape[2]), c_int(relu2), st), "omni_moe_pairs_f32")
+            return out
+        h = fused.silu_mul(pairs(x, k, up)) if act == "swiglu" else pairs(x, k, up, 1)
+        return ExpertRows(pairs(h, 1, down), None, w)
     ws = (ws or MoEWorkspace()).get(T, k, experts, D, Fd, x.device, x.dtype)
     nv.check_rc(lib.omni_moe_router(nv.ptr(x), c_long(x.stride(0)), nv.ptr(router_w), c_long(router_w.stride(0)), nv.ptr(router_b),
-                                    c_int(T), c_int(D), c_int(experts), c_int(router_w.shape[0]), c_int(k), nv.ptr(ws.ids),
-                                    nv.ptr(ws.weights), st), "omni_moe_router")
+                                    c_int(T), c_int(D), c_int(experts), c_int(router_w.shape[0]), c_int(k), ctypes.byref(rule),
+                                    nv.ptr(ws.ids), nv.ptr(ws.weights), st), "omni_moe_router")
     _plan_and_dispatch(ws, x, experts, 0, experts, k)
-    _grouped(ws, ws.xp, D, up, ws.h, Fd, Fd, D, ws.tile_expert, gemm.ACT[act])
+    if act == "swiglu":
+        _grouped(ws, ws.xp, D, up, ws.h13, 2 * Fd, 2 * Fd, D, ws.tile_expert)
+        fused.silu_mul(ws.h13, out=ws.h)
+    else:
+        _grouped(ws, ws.xp, D, up, ws.h, Fd, Fd, D, ws.tile_expert, gemm.ACT[act])
     _grouped(ws, ws.h, Fd, down, ws.y, D, D, Fd, ws.tile_expert)
     return ExpertRows(ws.y, ws.row_of_pair, ws.weights)
 

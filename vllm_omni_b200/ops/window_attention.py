@@ -1,6 +1,6 @@
 """Attention of a mixed batch (prompt portions and single decoded tokens) over the paged cache, with a
-sliding window that keeps the first tokens, bounded scores, a logarithmic distance bias, a softmax sink
-and a per-head output gate — each optional.  Kernels: csrc/attn_window_sm100.cu (tcgen05, portions of two
+sliding window that keeps the first tokens, bounded scores, a logarithmic distance bias, a softmax sink,
+two maps per head whose results are subtracted, and an output gate — each optional.  Kernels: csrc/attn_window_sm100.cu (tcgen05, portions of two
 tokens and more), csrc/attn_window.cu (single tokens; and one block per row for fp32 and head sizes the
 tensor-core kernels do not take)."""
 from __future__ import annotations
@@ -26,7 +26,27 @@ class _WinAttn(ctypes.Structure):
                 ("keep_first", c_int), ("T", c_int), ("H", c_int), ("G", c_int), ("dp", c_int), ("vp", c_int),
                 ("num_seqs", c_int), ("num_blocks", c_int), ("block_size", c_int), ("splits", c_int),
                 ("part_o", c_void_p), ("part_ml", c_void_p), ("status", c_void_p), ("k_ts", c_long), ("v_ts", c_long),
-                ("k_shared", c_void_p), ("ks_ts", c_long), ("dp_u", c_int), ("key_start", c_void_p), ("key_rows", c_long)]
+                ("k_shared", c_void_p), ("ks_ts", c_long), ("dp_u", c_int), ("key_start", c_void_p), ("key_rows", c_long),
+                ("g_hs", c_long), ("g_cs", c_int), ("maps", c_int), ("lam", c_float), ("out_mul", c_float), ("out_eps", c_float),
+                ("vdim", c_int)]
+
+    def set_gate(self, gate, heads: int):
+        """``gate``: logits [T, heads] or [T, heads * channels of a head], a view with unit column stride."""
+        if gate is None:
+            return
+        assert gate.stride(1) == 1 and gate.shape[1] % heads == 0
+        self.gate, self.g_rs, self.g_hs = gate.data_ptr(), gate.stride(0), gate.shape[1] // heads
+        self.g_cs = 0 if gate.shape[1] == heads else 1
+
+
+@dataclass(frozen=True)
+class DiffRule:
+    """Differential attention: head h's result is u / sqrt(<u^2> + eps) * mult for u = a1 - lam a2, a1 and a2 the results of
+    its two maps over the same values; ``vdim``: real channels of a value head."""
+    lam: float
+    mult: float
+    eps: float
+    vdim: int
 
 
 @dataclass
@@ -40,6 +60,7 @@ class ScoreRule:
     window: int | None = None
     keep_first: int = 0
     bounded: bool = False                 # see ``bounded_scores``
+    diff: DiffRule | None = None          # two maps per head; not together with a bias or a sink
 
 
 def bounded_scores(softcap, r1=None, r2=None) -> bool:
@@ -54,10 +75,10 @@ def bounded_scores(softcap, r1=None, r2=None) -> bool:
     return 2.0 * softcap * math.log2(math.e) <= 90.0
 
 
-def prefill_rows_per_block(heads: int, kv_heads: int, dp: int) -> int:
+def prefill_rows_per_block(heads: int, kv_heads: int, dp: int, maps: int = 1) -> int:
     """Tokens one block of the tcgen05 kernel serves: two 128-row tiles of (token, head of the KV group) rows,
-    one when two tiles of the widest heads do not fit in shared memory."""
-    return (1 if dp > 192 else 2) * (128 // (heads // kv_heads))
+    one when two tiles of the widest heads do not fit in shared memory or the second one is the second map."""
+    return (1 if dp > 192 or maps == 2 else 2) * (128 // (heads // kv_heads))
 
 
 def prefill_kernel_ok(heads: int, kv_heads: int, dp: int, vp: int, block_size: int) -> bool:
@@ -65,9 +86,9 @@ def prefill_kernel_ok(heads: int, kv_heads: int, dp: int, vp: int, block_size: i
         and 128 % block_size == 0
 
 
-def decode_splits(n: int, kv_heads: int, group: int, max_keys: int) -> int:
+def decode_splits(n: int, kv_heads: int, group: int, max_keys: int, heads_per_block: int = 16) -> int:
     """Blocks that share one sequence's visible keys: enough for about two blocks per SM, at least 64 keys each."""
-    blocks = n * kv_heads * ((group + 15) // 16)
+    blocks = n * kv_heads * -(-group // heads_per_block)
     want = max(1, (2 * 148) // max(1, blocks))
     return max(1, min(want, 32, (max_keys + 63) // 64))
 
@@ -87,12 +108,16 @@ def _parts(device, n: int, vp: int):
 
 def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None, impl: str | None = None):
     """q [T, H, dp]; caches [num_blocks, block_size, G, dp | vp] that already hold this step's tokens;
-    ``seqs``: the batch's ``SeqTable``; ``out`` [T, H * vp]; ``gate`` [T, H] logits (a view is fine).
+    ``seqs``: the batch's ``SeqTable``; ``out`` [T, H * vp]; ``gate`` [T, H] or [T, H * vp] logits (a view is fine).
+    With ``rule.diff`` q is [T, 2 H, dp], heads ordered (KV head, map, head of the group), and a cached key has
+    2 dp channels, its two maps side by side.
 
     ``impl="rows"`` forces the row-per-block kernel for every row."""
-    T, H, dp = q.shape
+    maps = 1 if rule.diff is None else 2
+    T, H, dp = q.shape[0], q.shape[1] // maps, q.shape[2]
     nb, bs, G, _ = k_cache.shape
     vp = v_cache.shape[3]
+    assert k_cache.shape[3] == maps * dp and out.shape[1] == H * vp
     if not q.is_cuda:
         return _cpu(q, k_cache, v_cache, seqs, rule, out, gate)
     assert q.is_contiguous() and out.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
@@ -103,23 +128,25 @@ def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None,
     a.block_tables, a.bt_stride = P(seqs.block_tables), seqs.block_tables.stride(0)
     a.q_start, a.context, a.row_seq = P(seqs.q_start), P(seqs.context), P(seqs.row_seq)
     a.out, a.o_rs = P(out), out.stride(0)
-    a.gate, a.g_rs = P(gate), 0 if gate is None else gate.stride(0)
+    a.set_gate(gate, H)
     a.r1, a.r2, a.sink = P(rule.r1), P(rule.r2), P(rule.sink)
     a.scale, a.cap = rule.scale, rule.softcap or 0.0
     a.bounded, a.window, a.keep_first = int(rule.bounded), rule.window or 0, rule.keep_first
     a.T, a.H, a.G, a.dp, a.vp, a.num_seqs, a.num_blocks, a.block_size = T, H, G, dp, vp, seqs.n_seqs, nb, bs
-    a.k_ts, a.v_ts, a.dp_u = G * dp, G * vp, dp
+    a.k_ts, a.v_ts, a.dp_u, a.maps = G * maps * dp, G * vp, dp, maps
+    if rule.diff is not None:
+        a.lam, a.out_mul, a.out_eps, a.vdim = rule.diff.lam, rule.diff.mult, rule.diff.eps, rule.diff.vdim
     a.splits = 1
     a.status = P(nv.status_word(q.device))
     bf = q.dtype == torch.bfloat16
-    rows_only = impl == "rows" or not bf or dp > 256 or vp > 256 or not (
+    rows_only = impl == "rows" or not bf or dp > (256 if maps == 1 else 128) or vp > 256 or (maps == 2 and rule.softcap) or not (
         seqs.n_decode == seqs.n_seqs or prefill_kernel_ok(H, G, dp, vp, bs))
     if rows_only:
         rc = nv.lib("attn_window").omni_attn_window_rows(ctypes.byref(a), c_int(1 if bf else 0), nv.stream_ptr())
         nv.check_rc(rc, "omni_attn_window_rows")
         return out
     if seqs.n_decode < seqs.n_seqs:
-        a.block_tokens = prefill_rows_per_block(H, G, dp)
+        a.block_tokens = prefill_rows_per_block(H, G, dp, maps)
         items, a.n_items = seqs.prefill_items(a.block_tokens)
         a.items = P(items)
         rc = nv.lib("attn_window_sm100").omni_attn_window_prefill(ctypes.byref(a), nv.stream_ptr())
@@ -129,9 +156,9 @@ def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None,
         keys = seqs.max_context + 1
         if rule.window:
             keys = min(keys, rule.window + rule.keep_first)
-        a.splits = decode_splits(seqs.n_decode, G, H // G, keys)
+        a.splits = decode_splits(seqs.n_decode, G, H // G, keys, 16 // maps)
         if a.splits > 1:
-            po, pml = _parts(q.device, seqs.n_decode * H * a.splits, vp)
+            po, pml = _parts(q.device, seqs.n_decode * H * maps * a.splits, vp)
             a.part_o, a.part_ml = P(po), P(pml)
         nv.check_rc(nv.lib("attn_window").omni_attn_window_decode(ctypes.byref(a), nv.stream_ptr()),
                     "omni_attn_window_decode")
@@ -139,19 +166,21 @@ def window_attention(q, k_cache, v_cache, seqs, rule: ScoreRule, out, gate=None,
 
 
 def _cpu(q, k_cache, v_cache, seqs, rule, out, gate):
-    T, H, dp = q.shape
+    maps = 1 if rule.diff is None else 2
+    T, H, dp = q.shape[0], q.shape[1] // maps, q.shape[2]
     nb, bs, G, _ = k_cache.shape
-    vp = v_cache.shape[3]
-    kf, vf = k_cache.view(nb * bs, G, dp), v_cache.view(nb * bs, G, vp)
-    o = torch.empty(T, H, vp)
+    vp, R = v_cache.shape[3], H // G
+    qm = q.float().view(T, G, maps, R, dp).permute(2, 0, 1, 3, 4).reshape(maps, T, H, dp)
+    kf, vf = k_cache.view(nb * bs, G, maps, dp), v_cache.view(nb * bs, G, vp)
+    o = torch.empty(maps, T, H, vp)
     for s in range(seqs.n_seqs):
         a, b, ctx = int(seqs.q_start[s]), int(seqs.q_start[s + 1]), int(seqs.context[s])
         j = torch.arange(ctx + b - a)
         i = torch.arange(ctx, ctx + b - a)[:, None]
         slot = seqs.block_tables[s].long()[j // bs] * bs + j % bs
-        k = kf[slot].float().repeat_interleave(H // G, 1)
-        v = vf[slot].float().repeat_interleave(H // G, 1)
-        sc = torch.einsum("thd,jhd->htj", q[a:b].float(), k) * rule.scale
+        k = kf[slot].float().repeat_interleave(R, 1)
+        v = vf[slot].float().repeat_interleave(R, 1)
+        sc = torch.einsum("mthd,jhmd->mhtj", qm[:, a:b], k) * rule.scale
         if rule.softcap:
             sc = rule.softcap * torch.tanh(sc / rule.softcap)
         dist = (i - j).float()
@@ -162,10 +191,15 @@ def _cpu(q, k_cache, v_cache, seqs, rule, out, gate):
             see &= (dist < rule.window) | (j < rule.keep_first)
         sc = sc.masked_fill(~see, float("-inf"))
         if rule.sink is not None:
-            sc = torch.cat([sc, rule.sink.float()[:, None, None].expand(H, b - a, 1)], -1)
+            sc = torch.cat([sc, rule.sink.float()[:, None, None].expand(maps, H, b - a, 1)], -1)
         w = sc.softmax(-1)[..., : j.numel()]
-        o[a:b] = torch.einsum("htj,jhd->thd", w, v)
+        o[:, a:b] = torch.einsum("mhtj,jhd->mthd", w, v)
+    if rule.diff is None:
+        o = o[0]
+    else:
+        u = o[0] - rule.diff.lam * o[1]
+        o = u * torch.rsqrt(u.pow(2).sum(-1, keepdim=True) / rule.diff.vdim + rule.diff.eps) * rule.diff.mult
     if gate is not None:
-        o = o * torch.sigmoid(gate.float())[:, :, None]
+        o = o * torch.sigmoid(gate.float()).view(T, H, -1)
     out.copy_(o.reshape(T, H * vp))
     return out
