@@ -152,14 +152,24 @@ def route(z, top, count=None, keep=None, scale=1.0):
     return ids, [s[e] / total * scale for e in ids]
 
 
-def mixture(h, W, p, m):
+def steady(z, spread, *rule):
+    """Does the choice of one token stay the same when its logits move by about ``spread``?"""
+    g = torch.Generator().manual_seed(0)
+    ids = set(route(z, *rule)[0])
+    return all(set(route(z + spread * torch.randn(z.shape, generator=g, dtype=z.dtype), *rule)[0]) == ids for _ in range(8))
+
+
+def mixture(h, W, p, m, clear=None):
     r = m["router"]
     g = r.get("groups") or {}
     z = h @ W[p + "router"].T
     weight = torch.zeros_like(z)
     for t in range(h.shape[0]):
-        for e, w in zip(*route(z[t], r["top"], g.get("count"), g.get("keep"), r["scale"])):
+        rule = r["top"], g.get("count"), g.get("keep"), r["scale"]
+        for e, w in zip(*route(z[t], *rule)):
             weight[t, e] = w
+        if clear is not None:
+            clear[t] &= steady(z[t], 0.03, *rule)
     out = sum(weight[:, e:e + 1] * gated_ff(h, W, f"{p}e{e}.") for e in range(r["experts"]))
     if m.get("shared"):
         out = out + sigmoid(h @ W[p + "shared.sg"].T) * gated_ff(h, W, p + "shared.")
@@ -167,8 +177,9 @@ def mixture(h, W, p, m):
 
 
 # ---------------------------------------------------------------------------------------------- model
-def forward(cfg, weights, tokens, dtype=torch.float64, trace=None):
-    """Logits [T, vocab] of one sequence.  ``trace``: a list that receives the stream after every layer."""
+def forward(cfg, weights, tokens, dtype=torch.float64, trace=None, clear=None):
+    """Logits [T, vocab] of one sequence.  ``trace``: a list that receives the stream after every layer; ``clear`` (bool
+    [T]): cleared where a router's choice is so close that rounding to bf16 may turn it."""
     W = {n: t.to(dtype) for n, t in weights.items()}
     ids = torch.as_tensor(tokens, dtype=torch.long)
     eps = cfg["norm"]["eps"]
@@ -178,7 +189,7 @@ def forward(cfg, weights, tokens, dtype=torch.float64, trace=None):
         x = x + branch_norm(mix(x, W, p + "mix.", layer["mixer"], eps), W[p + "norm1"], eps)
         m = layer.get("mlp")
         if m is not None:
-            y = gated_ff(x, W, p + "mlp.") if m["kind"] == "dense" else mixture(x, W, p + "mlp.", m)
+            y = gated_ff(x, W, p + "mlp.") if m["kind"] == "dense" else mixture(x, W, p + "mlp.", m, clear)
             x = x + branch_norm(y, W[p + "norm2"], eps)
         if trace is not None:
             trace.append(x.clone())

@@ -3,6 +3,7 @@ logits) against the plain restatements, one mechanism at a time."""
 import pytest
 import torch
 
+import milivik_oracle as M
 import tavulix_oracle as O
 from vllm_omni_b200.models.seq_table import SeqTable
 from vllm_omni_b200.ops import lm
@@ -256,3 +257,54 @@ def test_fp32_linear_is_exact(m, n, k):
     want = x.double() @ w.double().T + b.double()
     assert (got.cpu().double() - want).abs().max() < 1e-5 * k ** 0.5
     assert torch.equal(linear(x[:1].cuda(), w.cuda(), b.cuda()), got[:1])       # a row alone: the same bits
+
+
+@pytest.mark.parametrize("device,dtype", DEVICES)
+@pytest.mark.parametrize("taps", [0, 3])
+@pytest.mark.parametrize("coef,every", [(0.3, 64), (0.5, 1), (0.2, 7.0), (-0.1, 300)])
+def test_queries_grow_with_the_position(device, dtype, taps, coef, every):
+    """Fewer value heads than key heads; positions at both sides of a whole period, in portions and one by one."""
+    c = ConvCase((4, 2, 20, 36), taps, dtype, device)
+    c.hs = lm.HeadShape(8, 4, 20, 36, 32, 48, taps, v_heads=2)
+    h = c.hs
+    cols, o = [], 0
+    for heads, d, p in ((8, 20, 32), (4, 20, 32), (2, 36, 48)):
+        for _ in range(heads):
+            cols += range(o, o + d)
+            o += p
+    assert o == h.channels
+    T = 330
+    u = torch.randn(T, len(cols), generator=torch.Generator().manual_seed(4)).bfloat16()
+    w = torch.randn(max(taps, 1), len(cols), generator=torch.Generator().manual_seed(5))
+    conv = state = None
+    if taps:
+        conv = torch.zeros(taps, h.channels)
+        conv[:, cols] = w
+        conv, state = conv.to(device), torch.zeros(2, taps - 1, h.channels, dtype=dtype, device=device)
+    qn, kn = torch.rand(20) + 0.5, torch.rand(20) + 0.5
+    kc, vc = (torch.full((T // 8 + 2, 8, 2, n), 5.0, dtype=dtype, device=device) for n in (64, 48))
+    pages = torch.randperm(T // 8 + 2, generator=torch.Generator().manual_seed(6)).tolist()
+    at, qs, phase = 0, [], 0
+    for n in [1, 1, 2, 5, 290] + [1] * 31:
+        proj = torch.zeros(n, h.channels + 8, dtype=dtype)
+        proj[:, cols] = u[at:at + n].to(dtype)
+        t = torch.arange(at, at + n)
+        slots = (torch.tensor(pages)[t // 8] * 8 + t % 8).int().to(device)
+        seqs = SeqTable.build([n], [at], [pages], [(phase, 1 - phase)], device)
+        qs.append(lm.conv_heads(proj.to(device), h, seqs, slots, kc, vc, conv=conv, state=state, q_norm=_pad(qn, 32).to(device),
+                                k_norm=_pad(kn, 32).to(device), eps=1e-5, growth=lm.QueryGrowth(coef, every)).float().cpu())
+        at, phase = at + n, phase ^ 1
+    y = O.causal_conv(u.double(), w.double().T) if taps else u.double()
+    q, k, v = y.split([160, 80, 72], 1)
+    q = O.rms_unit(q.reshape(T, 8, 20), 1e-5) * qn.double() * M.query_temperature(range(T), coef, every)[:, None, None]
+    _close(torch.cat(qs)[..., :20], q, dtype, scale=3)
+    flat = (torch.tensor(pages)[torch.arange(T) // 8] * 8 + torch.arange(T) % 8).to(device)
+    _close(kc.view(-1, 4, 32)[flat][..., :20], O.rms_unit(k.reshape(T, 4, 20), 1e-5) * kn.double(), dtype)
+    _close(vc.view(-1, 2, 48)[flat][..., :36], v.reshape(T, 2, 36), dtype)
+
+
+@pytest.mark.parametrize("device,dtype", DEVICES)
+def test_scaled_logits(device, dtype):
+    z = (torch.randn(3, 304) * 8).to(dtype)
+    _close(lm.logit_softcap(z.to(device), None, 300, 0.25), 0.25 * z[:, :300].double(), torch.float32)
+    _close(lm.logit_softcap(z.to(device), 5.0, 300, 0.25), O.soft_cap(0.25 * z[:, :300].double(), 5.0), torch.float32)

@@ -46,12 +46,10 @@ def kv_gather(k_cache, v_cache, block_table, T, out_k=None, out_v=None):
     live in another GPU's peer-mapped memory)."""
     nb, bs, Hkv, D = k_cache.shape
     if out_k is None:
-        out_k = torch.empty(T, Hkv, D, dtype=k_cache.dtype, device=k_cache.device)
-        out_v = torch.empty_like(out_k)
-    if not k_cache.is_cuda:
-        idx = (block_table[: (T + bs - 1) // bs].long()[:, None] * bs + torch.arange(bs)[None, :]).reshape(-1)[:T]
-        out_k.copy_(k_cache.view(-1, Hkv, D)[idx])
-        out_v.copy_(v_cache.view(-1, Hkv, D)[idx])
+        out_k, out_v = (torch.empty(T, *c.shape[2:], dtype=c.dtype, device=c.device) for c in (k_cache, v_cache))
+    if not k_cache.is_cuda or k_cache.shape != v_cache.shape or k_cache.dtype != torch.bfloat16:
+        out_k.copy_(rows_gather(k_cache, block_table, T))
+        out_v.copy_(rows_gather(v_cache, block_table, T))
         return out_k, out_v
     _set_bounds(k_cache)
     rc = nv.lib("kv_cache").omni_kv_gather(nv.ptr(k_cache), nv.ptr(v_cache), nv.ptr(block_table), c_int(bs), c_int(T),
