@@ -77,16 +77,15 @@ __device__ __forceinline__ uint32_t bit_range(int a, int b) {
 // sigmoid of a gate logit
 __device__ __forceinline__ float wp_open(float z) { return 1.0f / (1.0f + __expf(-z)); }
 
-// 16 channels of a row, times f, channel by channel times their gate's opening where `gate` is given
-__device__ __forceinline__ void wp_store16(__nv_bfloat16* dst, const float (&v)[16], float f, const __nv_bfloat16* gate) {
+// 16 channels of a row, times f, channel by channel times the opening of their logits z where `gated`
+__device__ __forceinline__ void wp_store16(__nv_bfloat16* dst, const float (&v)[16], float f, bool gated, const uint4 (&z)[2]) {
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     float o[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) o[e] = v[x * 8 + e] * f;
-    if (gate) {
-      const uint4 z = *reinterpret_cast<const uint4*>(gate + x * 8);
-      const uint32_t zw[4] = {z.x, z.y, z.z, z.w};
+    if (gated) {
+      const uint32_t zw[4] = {z[x].x, z[x].y, z[x].z, z[x].w};
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float2 g = unpack_bf16(zw[e]);
@@ -338,6 +337,11 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       m = ref;
       b_const = C - ref;
     }
+    const long orow = row0 + t * tile_tokens + tok;
+    const __nv_bfloat16* gate = p.gate && row_ok ? static_cast<const __nv_bfloat16*>(p.gate) + orow * p.g_rs + (long)h * p.g_hs : nullptr;
+    if (gate && p.g_cs) {                        // fetched after the last tile
+      for (int c = 0; c < p.vp; c += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(gate + c));
+    }
     const float* my_tab = tab + min(r, w.R - 1) * w.tab_stride + min(t * tile_tokens + tok, 2 * w.TT - 1) + 127;
     for (int j = 0; tile_used && j < n_kv; ++j) {
       mbar_wait(smem_u32(&s_full[t]), j & 1, &s_abort, status, ERR_WAIT_FULL);
@@ -490,16 +494,24 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       weights(v3, 3, negm2);
     }
     if (rows_used) {
+      // the gate's logits, on their way while the last products finish
+      const bool channels = gate && p.g_cs;
+      const float head_gate = gate && p.g_cs == 0 ? wp_open((float)gate[0]) : 1.f;
+      uint4 gz[8][2];
+      if (channels) {
+#pragma unroll
+        for (int c = 0; c < 8; ++c)
+          if (c * 16 < p.vp) {
+            gz[c][0] = *reinterpret_cast<const uint4*>(gate + c * 16);
+            gz[c][1] = *reinterpret_cast<const uint4*>(gate + c * 16 + 8);
+          }
+      }
       mbar_wait(smem_u32(&o_done[t]), 0, &s_abort, status, ERR_WAIT_PV);
       tc_fence_after_sync();
-      const long orow = row0 + t * tile_tokens + tok;
       float s0, s1, s2, s3;
       unpack2(l2a, s0, s1);
       unpack2(l2b, s2, s3);
       float f = 1.0f / ((s0 + s1) + (s2 + s3));
-      const __nv_bfloat16* gate = p.gate && row_ok ? static_cast<const __nv_bfloat16*>(p.gate) + orow * p.g_rs + (long)h * p.g_hs : nullptr;
-      const float head_gate = gate && p.g_cs == 0 ? wp_open((float)gate[0]) : 1.f;
-      if (p.g_cs == 0) gate = nullptr;
       __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + orow * p.o_rs + (long)h * p.vp;
       if constexpr (PAIR) {
         mbar_wait(smem_u32(&o_done[t ^ 1]), 0, &s_abort, status, ERR_WAIT_PV);
@@ -531,23 +543,29 @@ attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         pair_sync();
         ss = ex[256 + row] + ex[384 + row];
         f = p.out_mul * head_gate / sqrtf(ss / (float)p.vdim + p.out_eps);
-#pragma unroll 1
-        for (int c = 16 * t; c < p.vp; c += 32) {
-          float u[16];
-          combined(c, u);
-          if (row_ok) wp_store16(dst + c, u, f, gate ? gate + c : nullptr);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int c = 16 * t + 32 * i;
+          if (c < p.vp) {
+            float u[16];
+            combined(c, u);
+            if (row_ok) wp_store16(dst + c, u, f, channels, t ? gz[2 * i + 1] : gz[2 * i]);
+          }
         }
       } else {
         f *= head_gate;
-#pragma unroll 1
-        for (int c = 0; c < p.vp; c += 16) {
-          uint32_t v[16];
-          tmem_ld_32x16(tO + c, v);
-          tmem_wait_ld();
-          float u[16];
 #pragma unroll
-          for (int e = 0; e < 16; ++e) u[e] = __uint_as_float(v[e]);
-          if (row_ok) wp_store16(dst + c, u, f, gate ? gate + c : nullptr);
+        for (int i = 0; i < 8; ++i) {
+          const int c = 16 * i;
+          if (c < p.vp) {
+            uint32_t v[16];
+            tmem_ld_32x16(tO + c, v);
+            tmem_wait_ld();
+            float u[16];
+#pragma unroll
+            for (int e = 0; e < 16; ++e) u[e] = __uint_as_float(v[e]);
+            if (row_ok) wp_store16(dst + c, u, f, channels, gz[i]);
+          }
         }
       }
     }

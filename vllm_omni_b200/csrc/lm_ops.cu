@@ -197,11 +197,15 @@ struct ConvHeads {
   int lph;                  // lanes per head: a power of two, 32 at most
   int GV;                   // value heads
   float q_coef;             // q grows by 1 + q_coef ln(floor((position + 1) / q_every) + 1); 0: not at all
-  double q_every;
+  float q_every;
 };
 
 __device__ __forceinline__ float query_growth(const ConvHeads& p, int pos) {
-  return fmaf(p.q_coef, logf((float)floor((double)(pos + 1) / p.q_every) + 1.0f), 1.0f);
+  const float x = (float)(pos + 1);
+  float n = floorf(__fdividef(x, p.q_every));             // off by one at most: put right by the products
+  if (n * p.q_every > x) n -= 1.0f;
+  else if ((n + 1.0f) * p.q_every <= x) n += 1.0f;
+  return fmaf(p.q_coef, logf(n + 1.0f), 1.0f);
 }
 
 template <typename T, int IT>
@@ -444,6 +448,76 @@ conv_heads_run_kernel(ConvHeads p) {
   }
 }
 
+// Without a convolution: a group owns RUN rows of one head, all loads of the run (rows, page slots, positions) in flight at
+// once.
+template <int RUN>
+__global__ void __launch_bounds__(256)
+heads_run_kernel(ConvHeads p) {
+  typedef __nv_bfloat16 T;
+  const int lane = threadIdx.x & (p.lph - 1);
+  const int groups = blockDim.x / p.lph, t0 = blockIdx.x * groups * RUN + threadIdx.x / p.lph;   // rows t0 + i * groups
+  const int head = blockIdx.y;
+  const int kind = head < p.H ? 0 : (head < p.H + p.G ? 1 : 2);
+  const int width = kind == 2 ? p.vp : p.dp;
+  const int hk = kind == 0 ? head : (kind == 1 ? head - p.H : head - p.H - p.G);
+  const int c = lane * 8;
+  const int col = (kind == 0 ? hk * p.dp : (kind == 1 ? (p.H + hk) * p.dp : (p.H + p.G) * p.dp + hk * p.vp)) + c;
+  const bool in = c < width;
+  const T* proj = static_cast<const T*>(p.proj) + col;
+  uint4 raw[RUN];
+  int at[RUN];                                              // page slot (k, v), position (q)
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    const int row = t0 + i * groups;
+    raw[i] = make_uint4(0u, 0u, 0u, 0u);
+    at[i] = -1;
+    if (row >= p.T) continue;
+    if (in) raw[i] = *reinterpret_cast<const uint4*>(proj + (long)row * p.ldp);
+    if (kind != 0) at[i] = p.slots[row];
+    else if (p.q_coef != 0.f) at[i] = min(max(p.row_seq[row], 0), p.num_seqs - 1);
+  }
+  if (kind == 0 && p.q_coef != 0.f) {
+#pragma unroll
+    for (int i = 0; i < RUN; ++i)
+      if (at[i] >= 0) at[i] = p.context[at[i]] + t0 + i * groups - p.q_start[at[i]];
+  }
+  const float* nw = kind == 0 ? p.q_norm : (kind == 1 ? p.k_norm : nullptr);
+  float w[8];
+  if (nw != nullptr && in) load8<float>(nw + c, w);
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    const int row = t0 + i * groups;
+    float v[8];
+    load8<T>(reinterpret_cast<const T*>(&raw[i]), v);
+    if (nw != nullptr) {                                    // uniform over the block
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+      for (int o = p.lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      float s = rms_scale(ss, p.d, p.eps);
+      if (kind == 0 && p.q_coef != 0.f) s *= query_growth(p, max(at[i], 0));
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= s * w[e];
+    } else if (kind == 0 && p.q_coef != 0.f) {
+      const float s = query_growth(p, max(at[i], 0));
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= s;
+    }
+    if (row >= p.T || !in) continue;
+    if (kind == 0) {
+      store8<T>(static_cast<T*>(p.q_out) + (long)row * p.H * p.dp + col, v);
+      continue;
+    }
+    if (at[i] >= p.num_slots) {
+      if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+      continue;
+    }
+    if (at[i] < 0) continue;
+    T* dst = kind == 1 ? static_cast<T*>(p.k_cache) + ((long)at[i] * p.G + hk) * p.dp : static_cast<T*>(p.v_cache) + ((long)at[i] * p.GV + hk) * p.vp;
+    store8<T>(dst + c, v);
+  }
+}
+
 // ------------------------------------------------------------------------------ logit cap
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -546,6 +620,11 @@ extern "C" int omni_conv_heads(const ConvHeads* args, int is_bf16, void* stream)
       case 3: conv_heads_run_kernel<3, RUN><<<rgrid, 256, 0, st>>>(p); break;
       default: conv_heads_run_kernel<4, RUN><<<rgrid, 256, 0, st>>>(p); break;
     }
+    return (int)cudaGetLastError();
+  }
+  if (is_bf16 && lanes <= 32 && p.T >= 256 && p.conv == nullptr && p.v_mode == 0) {
+    const int rows = rows_per_cta * 4;
+    heads_run_kernel<4><<<dim3((p.T + rows - 1) / rows, p.H + p.G + p.GV), 256, 0, st>>>(p);
     return (int)cudaGetLastError();
   }
   if (is_bf16) {

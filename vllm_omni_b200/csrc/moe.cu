@@ -86,15 +86,16 @@ struct RouterRule {
   float scale;
 };
 
-// the largest of 256 values, value lane + 32 i in v[i]; ties go to the lower index
-__device__ __forceinline__ void warp_best(const float (&v)[8], int lane, float& best, int& bi) {
+// the largest of n <= 256 values, value lane + 32 i in v[i]; ties go to the lower index
+__device__ __forceinline__ void warp_best(const float (&v)[8], int n, int lane, float& best, int& bi) {
   best = -INFINITY;
   bi = 0x7fffffff;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const int e = lane + i * 32;
-    if (v[i] > best || (v[i] == best && v[i] != -INFINITY && e < bi)) { best = v[i]; bi = e; }
-  }
+  for (int i = 0; i < 8; ++i)
+    if (i * 32 < n) {
+      const int e = lane + i * 32;
+      if (v[i] > best || (v[i] == best && v[i] != -INFINITY && e < bi)) { best = v[i]; bi = e; }
+    }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
     const float ob = __shfl_xor_sync(0xffffffffu, best, o);
@@ -115,7 +116,7 @@ __device__ __forceinline__ void keep_groups(float (&v)[8], int E, const RouterRu
   for (int i = 0; i < 8; ++i) {
     const int g = lane + i * 32;
     sum[i] = -INFINITY;
-    if (g < rule.groups) {
+    if (i * 32 < rule.groups && g < rule.groups) {
       float a = sh[g * size], b = size > 1 ? -INFINITY : 0.f;
       for (int j = 1; j < size; ++j) {
         const float x = sh[g * size + j];
@@ -130,12 +131,13 @@ __device__ __forceinline__ void keep_groups(float (&v)[8], int E, const RouterRu
   for (int j = 0; j < rule.keep; ++j) {
     float best;
     int g;
-    warp_best(sum, lane, best, g);
+    warp_best(sum, rule.groups, lane, best, g);
     if (g >= rule.groups) break;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      if (lane + i * 32 == g) sum[i] = -INFINITY;
-      if ((lane + i * 32) / size == g) live |= 1u << i;
+      const int e = lane + i * 32;
+      if (e == g) sum[i] = -INFINITY;
+      if (i * 32 < E && e >= g * size && e < (g + 1) * size) live |= 1u << i;
     }
   }
 #pragma unroll
@@ -149,7 +151,8 @@ __device__ __forceinline__ void choose_experts(float (&v)[8], int E, int k, cons
                                                float* weights) {
   if (rule.sigmoid) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = lane + i * 32 < E ? 1.0f / (1.0f + expf(-v[i])) : -INFINITY;
+    for (int i = 0; i < 8; ++i)
+      if (i * 32 < E) v[i] = lane + i * 32 < E ? 1.0f / (1.0f + expf(-v[i])) : -INFINITY;
     if (rule.groups > 0) keep_groups(v, E, rule, lane, sh);
   }
   float top = 0.f, sum = 0.f, mine = 0.f;
@@ -157,7 +160,7 @@ __device__ __forceinline__ void choose_experts(float (&v)[8], int E, int k, cons
   for (int j = 0; j < k; ++j) {
     float best;
     int bi;
-    warp_best(v, lane, best, bi);
+    warp_best(v, E, lane, best, bi);
     if (bi >= E) bi = j;                       // no finite value left: any index inside the range
     if (j == 0) top = best;
     const float w = rule.sigmoid ? best : expf(best - top);

@@ -110,7 +110,7 @@ class _ConvHeads(ctypes.Structure):
                 ("state_out", c_void_p), ("q_out", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p),
                 ("v_first", c_void_p), ("v_mode", c_int), ("lam", c_void_p), ("num_slots", c_long),
                 ("num_state", c_int), ("num_seqs", c_int), ("status", c_void_p), ("lph", c_int), ("GV", c_int),
-                ("q_coef", c_float), ("q_every", ctypes.c_double)]
+                ("q_coef", c_float), ("q_every", c_float)]
 
 
 @dataclass
