@@ -75,7 +75,7 @@ __device__ __forceinline__ uint32_t bit_range(int a, int b) {
 }
 
 // sigmoid of a gate logit
-__device__ __forceinline__ float wp_open(float z) { return 1.0f / (1.0f + __expf(-z)); }
+__device__ __forceinline__ float wp_open(float z) { return wp_rcp(1.0f + wp_ex2(-WP_LOG2E * z)); }
 
 // 16 channels of a row, times f, channel by channel times the opening of their logits z where `gated`
 __device__ __forceinline__ void wp_store16(__nv_bfloat16* dst, const float (&v)[16], float f, bool gated, const uint4 (&z)[2]) {
