@@ -454,18 +454,20 @@ template <int RUN>
 __global__ void __launch_bounds__(256)
 heads_run_kernel(ConvHeads p) {
   typedef __nv_bfloat16 T;
-  const int lane = threadIdx.x & (p.lph - 1);
-  const int groups = blockDim.x / p.lph, t0 = blockIdx.x * groups * RUN + threadIdx.x / p.lph;   // rows t0 + i * groups
   const int head = blockIdx.y;
   const int kind = head < p.H ? 0 : (head < p.H + p.G ? 1 : 2);
   const int width = kind == 2 ? p.vp : p.dp;
+  const int lph = width <= 16 ? 2 : (width <= 32 ? 4 : (width <= 64 ? 8 : (width <= 128 ? 16 : 32)));
+  const int lane = threadIdx.x & (lph - 1);
+  const int groups = 256 / lph, t0 = blockIdx.x * groups * RUN + threadIdx.x / lph;   // rows t0 + i * groups
+  if (blockIdx.x * groups * RUN >= p.T) return;             // the grid is made for the widest heads
   const int hk = kind == 0 ? head : (kind == 1 ? head - p.H : head - p.H - p.G);
   const int c = lane * 8;
   const int col = (kind == 0 ? hk * p.dp : (kind == 1 ? (p.H + hk) * p.dp : (p.H + p.G) * p.dp + hk * p.vp)) + c;
   const bool in = c < width;
   const T* proj = static_cast<const T*>(p.proj) + col;
   uint4 raw[RUN];
-  int at[RUN];                                              // page slot (k, v), position (q)
+  int at[RUN];                                              // page slot of a row (k, v)
 #pragma unroll
   for (int i = 0; i < RUN; ++i) {
     const int row = t0 + i * groups;
@@ -474,12 +476,31 @@ heads_run_kernel(ConvHeads p) {
     if (row >= p.T) continue;
     if (in) raw[i] = *reinterpret_cast<const uint4*>(proj + (long)row * p.ldp);
     if (kind != 0) at[i] = p.slots[row];
-    else if (p.q_coef != 0.f) at[i] = min(max(p.row_seq[row], 0), p.num_seqs - 1);
   }
-  if (kind == 0 && p.q_coef != 0.f) {
+  float grow[RUN];
 #pragma unroll
-    for (int i = 0; i < RUN; ++i)
-      if (at[i] >= 0) at[i] = p.context[at[i]] + t0 + i * groups - p.q_start[at[i]];
+  for (int i = 0; i < RUN; ++i) grow[i] = 1.f;
+  if (kind == 0 && p.q_coef != 0.f) {                       // a lane computes one row's growth for all lanes of its group
+    float mine[RUN];
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) {
+      const int row = t0 + (i * lph + lane) * groups;
+      mine[i] = 1.f;
+      if (i * lph >= RUN) break;
+      if (i * lph + lane < RUN && row < p.T) {
+        const int seq = min(max(p.row_seq[row], 0), p.num_seqs - 1);
+        mine[i] = query_growth(p, max(p.context[seq] + row - p.q_start[seq], 0));
+      }
+    }
+    const int first = threadIdx.x & 31 & ~(lph - 1);
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) {
+      float m = mine[0];
+#pragma unroll
+      for (int k = 1; k < RUN; ++k)
+        if (i >= k * lph) m = mine[k];
+      grow[i] = __shfl_sync(0xffffffffu, m, first + (i & (lph - 1)));
+    }
   }
   const float* nw = kind == 0 ? p.q_norm : (kind == 1 ? p.k_norm : nullptr);
   float w[8];
@@ -493,15 +514,13 @@ heads_run_kernel(ConvHeads p) {
       float ss = 0.f;
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
-      for (int o = p.lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      float s = rms_scale(ss, p.d, p.eps);
-      if (kind == 0 && p.q_coef != 0.f) s *= query_growth(p, max(at[i], 0));
+      for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      const float s = rsqrtf(fmaf(ss, 1.0f / (float)p.d, p.eps)) * grow[i];
 #pragma unroll
       for (int e = 0; e < 8; ++e) v[e] *= s * w[e];
-    } else if (kind == 0 && p.q_coef != 0.f) {
-      const float s = query_growth(p, max(at[i], 0));
+    } else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[e] *= s;
+      for (int e = 0; e < 8; ++e) v[e] *= grow[i];
     }
     if (row >= p.T || !in) continue;
     if (kind == 0) {
