@@ -261,7 +261,7 @@ def test_fp32_linear_is_exact(m, n, k):
 
 @pytest.mark.parametrize("device,dtype", DEVICES)
 @pytest.mark.parametrize("taps", [0, 3])
-@pytest.mark.parametrize("coef,every", [(0.3, 64), (0.5, 1), (0.2, 7.0), (-0.1, 300)])
+@pytest.mark.parametrize("coef,every", [(0.35, 50), (0.5, 1), (0.2, 7.0), (-0.1, 300)])
 def test_queries_grow_with_the_position(device, dtype, taps, coef, every):
     """Fewer value heads than key heads; positions at both sides of a whole period, in portions and one by one."""
     c = ConvCase((4, 2, 20, 36), taps, dtype, device)
@@ -306,5 +306,5 @@ def test_queries_grow_with_the_position(device, dtype, taps, coef, every):
 @pytest.mark.parametrize("device,dtype", DEVICES)
 def test_scaled_logits(device, dtype):
     z = (torch.randn(3, 304) * 8).to(dtype)
-    _close(lm.logit_softcap(z.to(device), None, 300, 0.25), 0.25 * z[:, :300].double(), torch.float32)
-    _close(lm.logit_softcap(z.to(device), 5.0, 300, 0.25), O.soft_cap(0.25 * z[:, :300].double(), 5.0), torch.float32)
+    _close(lm.logit_softcap(z.to(device), None, 300, 0.4), 0.4 * z[:, :300].double(), torch.float32)
+    _close(lm.logit_softcap(z.to(device), 5.0, 300, 0.4), O.soft_cap(0.4 * z[:, :300].double(), 5.0), torch.float32)

@@ -191,7 +191,7 @@ def test_scaled_embedding(mode):
     near(out, M.branch_norm(want, w, 1e-5), tol)
 
 
-YARN = [(None, 10000.0, 32), ((2.0, 512, 32.0, 1.0), 20000.0, 64), ((8.0, 64, 4.0, 3.9), 300.0, 10), ((1.0, 4096, 32.0, 1.0), 10000.0, 64),
+YARN = [(None, 10000.0, 32), ((2.5, 700, 24.0, 1.5), 30000.0, 64), ((8.0, 64, 4.0, 3.9), 300.0, 10), ((1.0, 4096, 32.0, 1.0), 10000.0, 64),
         ((16.0, 8, 32.0, 1.0), 10000.0, 16), ((3.0, 100000, 1.0, 1.0), 50.0, 6), ((4.0, 256, 16.0, 2.0), 10000.0, 2)]
 
 
