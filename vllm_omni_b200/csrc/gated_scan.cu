@@ -4,8 +4,6 @@
 //                     channels of one part; convolution to shared memory, both gates on 16 x 8 x 16 tensor-core
 //                     products (weights straight from global memory, each byte read once per 16 tokens), state
 //                     update and output in the epilogue
-//   omni_scan_conv_bf16   convolution of prompt portions to bf16 rows and their new history; a thread slides over eight
-//                     rows of eight channels (gated_scan_sm100.cu does the rest)
 //   omni_scan_conv    convolution to fp32 and the new history \ plain kernels, bf16 or fp32: the exact mode, and
 //   omni_scan_plain   scan, one thread per channel            / sizes the other kernels do not take
 #include "gated_scan.cuh"
@@ -65,86 +63,6 @@ scan_plain_kernel(const GatedScan p) {
     static_cast<T*>(p.out)[t * p.C + c] = (T)(S * (0.5f * y * (1.0f + th)));
   }
   if (sout >= 0) p.state[(long)sout * p.C + c] = S;
-}
-
-// --------------------------------------------------------------- convolution of long batches
-// TAPS > 0: the taps of the thread's channels and the rows before the current one stay in registers.
-template <int TAPS>
-__global__ void __launch_bounds__(256)
-scan_conv_bf16_kernel(const GatedScan p) {
-  constexpr int RUN = 8, H = TAPS > 1 ? TAPS - 1 : 1;
-  const int vecs = p.C / 8;
-  const long idx = (long)blockIdx.x * 256 + threadIdx.x;
-  const int c = (int)(idx % vecs) * 8;
-  const long r0 = idx / vecs * RUN;
-  if (r0 >= p.T) return;
-  const int taps = TAPS > 0 ? TAPS : p.taps, h = taps - 1;
-  const bf16* x = static_cast<const bf16*>(p.proj) + p.C + c;
-  bf16* hist = static_cast<bf16*>(p.hist) + c;
-  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-  int seq = -1, q0 = 0, q1 = 0, ctx = 0, sin = 0, sout = -1;
-  auto raw_x = [&](int b) {                                  // row b of the portion; negative: history
-    if (b >= 0) return *reinterpret_cast<const uint4*>(x + (long)(q0 + b) * p.ldp);
-    if (ctx + b >= 0) return *reinterpret_cast<const uint4*>(hist + ((long)sin * h + h + b) * p.C);
-    return zero;
-  };
-  uint4 raw[RUN], win[H];
-  float w[TAPS > 0 ? TAPS : 1][8], bias[8];
-  load8<float>(p.conv_b + c, bias);
-  if (TAPS > 0) {
-#pragma unroll
-    for (int i = 0; i < RUN; ++i) raw[i] = r0 + i < p.T ? *reinterpret_cast<const uint4*>(x + (r0 + i) * p.ldp) : zero;
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) load8<float>(p.conv + (long)j * p.C + c, w[j]);
-  }
-#pragma unroll
-  for (int i = 0; i < RUN; ++i) {
-    const long row = r0 + i;
-    if (row >= p.T) break;
-    const int s = min(max(p.row_seq[row], 0), p.num_seqs - 1);
-    if (s != seq) {                                          // first row of the run or of a sequence
-      seq = s;
-      q0 = p.q_start[seq];
-      q1 = p.q_start[seq + 1];
-      ctx = p.context[seq];
-      scan_rows(p, seq, sin, sout);
-      if (TAPS > 1) {
-#pragma unroll
-        for (int m = 0; m < H; ++m) win[m] = raw_x((int)(row - q0) - H + m);
-      }
-    }
-    float o[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) o[e] = bias[e];
-    if (TAPS > 0) {
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) {
-        float f[8];
-        load8<bf16>(reinterpret_cast<const bf16*>(j < TAPS - 1 ? &win[j < H ? j : 0] : &raw[i]), f);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = fmaf(w[j][e], f[e], o[e]);
-      }
-      if (TAPS > 1) {
-#pragma unroll
-        for (int m = 0; m + 1 < H; ++m) win[m] = win[m + 1];
-        win[H - 1] = raw[i];
-      }
-    } else {
-      for (int j = 0; j < taps; ++j) {
-        float f[8], wj[8];
-        const uint4 q = raw_x((int)(row - q0) - h + j);
-        load8<bf16>(reinterpret_cast<const bf16*>(&q), f);
-        load8<float>(p.conv + (long)j * p.C + c, wj);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = fmaf(wj[e], f[e], o[e]);
-      }
-    }
-    store8<bf16>(static_cast<bf16*>(p.u) + row * p.C + c, o);
-    // single rows leave their history to omni_scan_step
-    if (row == q1 - 1 && q1 - q0 > 1 && sout >= 0)
-      for (int m = 0; m < h; ++m)
-        *reinterpret_cast<uint4*>(hist + ((long)sout * h + m) * p.C) = raw_x((int)(row - q0) + 1 - h + m);
-  }
 }
 
 // ---------------------------------------------------------------------------- one token each
@@ -270,23 +188,6 @@ extern "C" int omni_scan_plain(const GatedScan* args, int is_bf16, void* stream)
   dim3 grid((p.C + 127) / 128, p.num_seqs);
   if (is_bf16) scan_plain_kernel<bf16><<<grid, 128, 0, (cudaStream_t)stream>>>(p);
   else scan_plain_kernel<float><<<grid, 128, 0, (cudaStream_t)stream>>>(p);
-  return (int)cudaGetLastError();
-}
-
-extern "C" int omni_scan_conv_bf16(const GatedScan* args, void* stream) {
-  const GatedScan& p = *args;
-  if (p.T <= 0) return RC_OK;
-  if (!scan_args_ok(p) || !p.u || !p.row_seq) return RC_BAD_ARG;
-  const long blocks = ((long)((p.T + 7) / 8) * (p.C / 8) + 255) / 256;
-  if (blocks > 0x7fffffffl) return RC_BAD_ARG;
-  cudaStream_t st = (cudaStream_t)stream;
-  switch (p.taps) {
-    case 1: scan_conv_bf16_kernel<1><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    case 2: scan_conv_bf16_kernel<2><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    case 3: scan_conv_bf16_kernel<3><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    case 4: scan_conv_bf16_kernel<4><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    default: scan_conv_bf16_kernel<0><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-  }
   return (int)cudaGetLastError();
 }
 

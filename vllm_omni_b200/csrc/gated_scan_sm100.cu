@@ -1,5 +1,5 @@
 // Gated linear recurrence of prompt portions on tcgen05 tensor cores (gated_scan.cuh says what is computed; the
-// convolution's rows come from gated_scan.cu).
+// convolution's rows come from short_conv.cu).
 //
 // A portion is cut into runs of consecutive tokens.  One block owns 128 channels of one part and four runs (streams),
 // and keeps the gate weights of its channels in shared memory; a run is walked in tiles of 32 tokens.  The gates are

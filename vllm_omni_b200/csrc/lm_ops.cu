@@ -8,6 +8,8 @@
 //                       RMS norm of q and k, growth of q with the position, mixing of v with an earlier
 //                       layer's values, K/V rows written to their pages, convolution history written to
 //                       the state pool
+//   omni_rotary_heads   norm of whole query and key rows, rotation of the first channels of every head, norm of value heads,
+//                       K/V rows written to their pages
 //   omni_logit_softcap  mult * logit, bounded to cap * tanh(. / cap) -> fp32
 //
 // Norm gains are fp32, either one number for the whole row (stride 0) or one per channel (stride 1).
@@ -537,6 +539,98 @@ heads_run_kernel(ConvHeads p) {
   }
 }
 
+// ------------------------------------------- row norms, rotation, value head norms, pages
+// One block per row of the packed projection [q: H * dp | k: G * dp | v: G * vp | ...]; a thread holds NV vectors of eight
+// channels.  Rotated pairs are neighbours, so a rotation stays within a vector.
+struct RotaryHeads {
+  const void* proj; long ldp;
+  int T, H, G, dp, vp;
+  int rot;                  // rotated channels of a q / k head, even
+  const float* turns;       // [T, rot / 2, 2]: cos, sin
+  const float* q_gain;      // [H * dp] or nullptr (no norm): norm over the whole row
+  const float* k_gain;      // [G * dp] or nullptr
+  int nq, nk, vdim;         // real channels of a query row, a key row, a value head
+  int v_norm;               // every value head over its root mean square
+  float v_mult, eps;
+  const int* slots;         // [T] page slot of each row, < 0: not written
+  void* q_out;              // [T, H * dp]
+  void* k_cache; void* v_cache;     // [slots, G, dp], [slots, G, vp]
+  long num_slots;
+  int* status;
+};
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(1024)
+rotary_heads_kernel(const RotaryHeads p) {
+  extern __shared__ float s_v[];                            // sums of squares of the value vectors
+  __shared__ float sh[64];
+  const long row = blockIdx.x;
+  const int nq = p.H * p.dp, nk = p.G * p.dp, C = nq + nk + p.G * p.vp;
+  const T* proj = static_cast<const T*>(p.proj) + row * p.ldp;
+  float v[NV][8];
+  float ss[2] = {0.f, 0.f};                                 // of the query row, of the key row
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c >= C) continue;
+    load8<T>(proj + c, v[i]);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s = fmaf(v[i][e], v[i][e], s);
+    if (c < nq) ss[0] += s;
+    else if (c < nq + nk) ss[1] += s;
+    else if (p.v_norm) s_v[(c - nq - nk) / 8] = s;
+  }
+  float sq = 1.f, sk = 1.f;
+  if (p.q_gain || p.k_gain || p.v_norm) {                   // uniform
+    block_sum<2>(ss, sh);                                   // also: the value sums are in place
+    sq = rms_scale(ss[0], p.nq, p.eps);
+    sk = rms_scale(ss[1], p.nk, p.eps);
+  }
+  int slot = p.slots[row];
+  if (slot >= p.num_slots) {
+    if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+    slot = -1;
+  }
+  const float* turns = p.turns + row * p.rot;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 8;
+    if (c >= C) continue;
+    if (c >= nq + nk) {
+      const int cv = c - nq - nk;
+      float s = p.v_mult;
+      if (p.v_norm) {
+        const int per = p.vp / 8, first = cv / p.vp * per;
+        float t = 0.f;
+        for (int x = 0; x < per; ++x) t += s_v[first + x];
+        s *= rms_scale(t, p.vdim, p.eps);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] *= s;
+      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + (long)slot * p.G * p.vp + cv, v[i]);
+      continue;
+    }
+    const bool is_q = c < nq;
+    const int ck = is_q ? c : c - nq;
+    const float* gain = is_q ? p.q_gain : p.k_gain;
+    if (gain) scale_gain8(v[i], is_q ? sq : sk, gain, 1, ck);
+    const int in = ck % p.dp;
+    if (in < p.rot) {
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        if (in + e >= p.rot) break;
+        const float2 t = *reinterpret_cast<const float2*>(turns + in + e);
+        const float a = v[i][e], b = v[i][e + 1];
+        v[i][e] = a * t.x - b * t.y;
+        v[i][e + 1] = b * t.x + a * t.y;
+      }
+    }
+    if (is_q) store8<T>(static_cast<T*>(p.q_out) + row * nq + ck, v[i]);
+    else if (slot >= 0) store8<T>(static_cast<T*>(p.k_cache) + (long)slot * nk + ck, v[i]);
+  }
+}
+
 // ------------------------------------------------------------------------------ logit cap
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -653,6 +747,29 @@ extern "C" int omni_conv_heads(const ConvHeads* args, int is_bf16, void* stream)
     if (lanes <= 32) conv_heads_kernel<float, 1><<<grid, 256, 0, st>>>(p);
     else conv_heads_kernel<float, 4><<<grid, 256, 0, st>>>(p);
   }
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_rotary_heads(const RotaryHeads* args, int is_bf16, void* stream) {
+  const RotaryHeads& p = *args;
+  if (p.T <= 0) return RC_OK;
+  if (p.H <= 0 || p.G <= 0 || (p.dp & 7) || (p.vp & 7) || p.dp <= 0 || p.vp <= 0 || (p.ldp & 7) || (p.rot & 1) || p.rot < 0 ||
+      p.rot > p.dp || (p.rot && !p.turns) || !p.slots || !p.q_out || !p.k_cache || !p.v_cache || p.nq <= 0 || p.nk <= 0 || p.vdim <= 0)
+    return RC_BAD_ARG;
+  const int C = (p.H + p.G) * p.dp + p.G * p.vp;
+  int threads, nv;
+  if (C > p.ldp || !row_shape(C, threads, nv)) return RC_BAD_ARG;
+  const int smem = p.v_norm ? p.G * p.vp / 8 * 4 : 0;
+  if (smem > 47 * 1024) return RC_TOO_LARGE;
+  cudaStream_t st = (cudaStream_t)stream;
+#define OMNI_ROTARY(ELT)                                                                \
+  do {                                                                                \
+    if (nv == 1) rotary_heads_kernel<ELT, 1><<<p.T, threads, smem, st>>>(p);            \
+    else if (nv == 2) rotary_heads_kernel<ELT, 2><<<p.T, threads, smem, st>>>(p);       \
+    else rotary_heads_kernel<ELT, 4><<<p.T, threads, smem, st>>>(p);                    \
+  } while (0)
+  if (is_bf16) OMNI_ROTARY(bf16); else OMNI_ROTARY(float);
+#undef OMNI_ROTARY
   return (int)cudaGetLastError();
 }
 

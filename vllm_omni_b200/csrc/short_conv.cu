@@ -1,0 +1,138 @@
+// Short causal convolution over time of a mixed batch's bf16 rows, per channel, with an optional bias and silu:
+// out_t = act(bias + sum_j conv[j] x_(t - taps + 1 + j)).  Rows before a portion come from the history pool where the
+// position says that there are any, zeros otherwise; the portion's last rows become the sequence's new history.  Pool rows
+// are double-buffered (read row != write row), so readers of the old history never race with the writer of the new one.
+// A thread slides over eight rows of eight channels; with up to four taps weights and earlier rows stay in registers.
+#include "host_util.h"
+#include "row_ops.cuh"
+
+namespace omni {
+
+typedef __nv_bfloat16 bf16;
+
+struct ConvRows {
+  const void* x; long ldx;
+  int T, C, taps;
+  const float* conv;                            // [taps, C]
+  const float* bias;                            // [C] or nullptr
+  int act;                                      // 0 none, 1 silu
+  int skip_single;                              // sequences with one row: their history is another kernel's
+  const int* row_seq; const int* q_start; const int* context;
+  const int* state_in; const int* state_out;    // [S] rows of the pool; out < 0: not written
+  void* hist;                                   // [num_state, taps - 1, C]
+  int num_state, num_seqs;
+  void* out;                                    // [T, C]
+  int* status;
+};
+
+template <int TAPS>
+__global__ void __launch_bounds__(256)
+conv_rows_kernel(const ConvRows p) {
+  constexpr int RUN = 8, H = TAPS > 1 ? TAPS - 1 : 1;
+  const int vecs = p.C / 8;
+  const long idx = (long)blockIdx.x * 256 + threadIdx.x;
+  const int c = (int)(idx % vecs) * 8;
+  const long r0 = idx / vecs * RUN;
+  if (r0 >= p.T) return;
+  const int taps = TAPS > 0 ? TAPS : p.taps, h = taps - 1;
+  const bf16* x = static_cast<const bf16*>(p.x) + c;
+  bf16* hist = static_cast<bf16*>(p.hist) + c;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  int seq = -1, q0 = 0, q1 = 0, ctx = 0, sin = 0, sout = -1;
+  auto raw_x = [&](int b) {                                  // row b of the portion; negative: history
+    if (b >= 0) return *reinterpret_cast<const uint4*>(x + (long)(q0 + b) * p.ldx);
+    if (ctx + b >= 0) return *reinterpret_cast<const uint4*>(hist + ((long)sin * h + h + b) * p.C);
+    return zero;
+  };
+  uint4 raw[RUN], win[H];
+  float w[TAPS > 0 ? TAPS : 1][8], bias[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (p.bias) load8<float>(p.bias + c, bias);
+  if (TAPS > 0) {
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) raw[i] = r0 + i < p.T ? *reinterpret_cast<const uint4*>(x + (r0 + i) * p.ldx) : zero;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load8<float>(p.conv + (long)j * p.C + c, w[j]);
+  }
+#pragma unroll
+  for (int i = 0; i < RUN; ++i) {
+    const long row = r0 + i;
+    if (row >= p.T) break;
+    const int s = min(max(p.row_seq[row], 0), p.num_seqs - 1);
+    if (s != seq) {                                          // first row of the run or of a sequence
+      seq = s;
+      q0 = p.q_start[seq];
+      q1 = p.q_start[seq + 1];
+      ctx = p.context[seq];
+      if (h > 0) {
+        sin = p.state_in[seq];
+        sout = p.state_out[seq];
+        if (sin < 0 || sin >= p.num_state || sout >= p.num_state) {
+          if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+          sin = 0;
+          sout = -1;
+        }
+      }
+      if (TAPS > 1) {
+#pragma unroll
+        for (int m = 0; m < H; ++m) win[m] = raw_x((int)(row - q0) - H + m);
+      }
+    }
+    float o[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) o[e] = bias[e];
+    if (TAPS > 0) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        float f[8];
+        load8<bf16>(reinterpret_cast<const bf16*>(j < TAPS - 1 ? &win[j < H ? j : 0] : &raw[i]), f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = fmaf(w[j][e], f[e], o[e]);
+      }
+      if (TAPS > 1) {
+#pragma unroll
+        for (int m = 0; m + 1 < H; ++m) win[m] = win[m + 1];
+        win[H - 1] = raw[i];
+      }
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        float f[8], wj[8];
+        const uint4 q = raw_x((int)(row - q0) - h + j);
+        load8<bf16>(reinterpret_cast<const bf16*>(&q), f);
+        load8<float>(p.conv + (long)j * p.C + c, wj);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = fmaf(wj[e], f[e], o[e]);
+      }
+    }
+    if (p.act == 1) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) o[e] = __fdividef(o[e], 1.0f + __expf(-o[e]));
+    }
+    store8<bf16>(static_cast<bf16*>(p.out) + row * p.C + c, o);
+    if (row == q1 - 1 && sout >= 0 && !(p.skip_single && q1 - q0 == 1))
+      for (int m = 0; m < h; ++m)
+        *reinterpret_cast<uint4*>(hist + ((long)sout * h + m) * p.C) = raw_x((int)(row - q0) + 1 - h + m);
+  }
+}
+
+}  // namespace omni
+
+using namespace omni;
+
+extern "C" int omni_conv_rows(const ConvRows* args, void* stream) {
+  const ConvRows& p = *args;
+  if (p.T <= 0) return RC_OK;
+  if (p.C <= 0 || (p.C & 7) || (p.ldx & 7) || p.ldx < p.C || p.taps < 1 || !p.conv || !p.x || !p.out || !p.row_seq || p.num_seqs <= 0 ||
+      (reinterpret_cast<uintptr_t>(p.x) & 15) || (p.taps > 1 && (!p.hist || !p.state_in || !p.state_out || p.num_state <= 0)))
+    return RC_BAD_ARG;
+  const long blocks = ((long)((p.T + 7) / 8) * (p.C / 8) + 255) / 256;
+  if (blocks > 0x7fffffffl) return RC_BAD_ARG;
+  cudaStream_t st = (cudaStream_t)stream;
+  switch (p.taps) {
+    case 1: conv_rows_kernel<1><<<(unsigned)blocks, 256, 0, st>>>(p); break;
+    case 2: conv_rows_kernel<2><<<(unsigned)blocks, 256, 0, st>>>(p); break;
+    case 3: conv_rows_kernel<3><<<(unsigned)blocks, 256, 0, st>>>(p); break;
+    case 4: conv_rows_kernel<4><<<(unsigned)blocks, 256, 0, st>>>(p); break;
+    default: conv_rows_kernel<0><<<(unsigned)blocks, 256, 0, st>>>(p); break;
+  }
+  return (int)cudaGetLastError();
+}

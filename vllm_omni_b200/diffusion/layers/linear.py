@@ -44,7 +44,7 @@ class FusedLinear(nn.Module):
             y = gemm.linear(x, self.weight, self.bias)
             for (A, B, scale) in self.lora:
                 y = y + scale * gemm.linear(gemm.linear(x, A), B)
-            y = _epilogue(y, act, residual, gate, out)
+            y = _epilogue(y, act, residual, gate, out, kw.get("coef"))
         else:
             y = gemm.linear(x, self.weight, self.bias, act=act, residual=residual, gate=gate, out=out, **kw)
         return y
@@ -53,7 +53,7 @@ class FusedLinear(nn.Module):
         return f"in={self.in_features}, out={self.out_features}, bias={self.bias is not None}"
 
 
-def _epilogue(y, act, residual, gate, out):
+def _epilogue(y, act, residual, gate, out, coef=None):
     import torch.nn.functional as F
     if act == "gelu_tanh":
         y = F.gelu(y.float(), approximate="tanh").to(y.dtype)
@@ -61,6 +61,10 @@ def _epilogue(y, act, residual, gate, out):
         y = F.silu(y)
     elif act == "relu2":
         y = F.relu(y).square()
+    elif act == "tanh":
+        y = torch.tanh(y)
+    elif act == "xielu":
+        y = gemm.xielu(y.float(), coef).to(y.dtype)
     if gate is not None:
         B = gate.shape[0]
         y = (y.reshape(B, -1, y.shape[-1]) * gate.unsqueeze(1)).reshape(y.shape)

@@ -9,7 +9,7 @@ from .decoder import NidilixDecoder
 
 # libraries under csrc/ that serving this model loads on a GPU
 NATIVE_LIBS = ("gemm_sm100", "gemm_f32", "lm_ops", "stream_ops", "moe", "latent_attn", "attn_window", "attn_window_sm100",
-               "gated_scan", "gated_scan_sm100", "sampler", "rt_host", "io_host")
+               "short_conv", "gated_scan", "gated_scan_sm100", "sampler", "rt_host", "io_host")
 
 
 class NidilixForCausalLM(StageModel):

@@ -32,6 +32,10 @@ class PackedDecoder(nn.Module):
         """Checkpoint name -> list of (destination view, selection of the checkpoint tensor that goes there)."""
         raise NotImplementedError
 
+    def resize(self, name: str, shape: tuple[int, ...]) -> None:
+        """Makes room for a checkpoint tensor whose size only the checkpoint tells (None in ``cfg.tensor_shapes()``)."""
+        raise NotImplementedError
+
     def weights_loaded(self) -> None:
         """Called when every tensor is in place: values derived from the weights are computed here."""
 
@@ -42,7 +46,12 @@ class PackedDecoder(nn.Module):
         for name, w in weights:
             if name not in targets:
                 continue
-            if tuple(w.shape) != shapes[name]:
+            if None in shapes[name]:
+                if len(w.shape) != len(shapes[name]) or any(b not in (None, a) for a, b in zip(w.shape, shapes[name])):
+                    raise ValueError(f"{name}: shape {tuple(w.shape)}, expected {shapes[name]}")
+                self.resize(name, tuple(w.shape))
+                targets = self.targets()
+            elif tuple(w.shape) != shapes[name]:
                 raise ValueError(f"{name}: shape {tuple(w.shape)}, expected {shapes[name]}")
             w = w.reshape(1) if w.dim() == 0 else w
             if any(sel != slice(None) for _, sel in targets[name]):

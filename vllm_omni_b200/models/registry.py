@@ -14,6 +14,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "Tavulix": ("vllm_omni_b200.models.tavulix.model", "build_tavulix"),
     "Nidilix": ("vllm_omni_b200.models.nidilix.model", "build_nidilix"),
     "Milivik": ("vllm_omni_b200.models.milivik.model", "build_milivik"),
+    "Fikizen": ("vllm_omni_b200.models.fikizen.model", "build_fikizen"),
     "BagelForConditionalGeneration": ("vllm_omni_b200.models.text", "build_text_model"),
 }
 

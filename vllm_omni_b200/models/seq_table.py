@@ -44,6 +44,15 @@ class KeyGroup:
 
 
 @dataclass
+class Chunks:
+    """Short runs of rows for recurrences that take several tokens at a time (``SeqTable.chunks``)."""
+    table: torch.Tensor                        # int32 [n, 4]: (sequence, first row in the portion, rows, 0), a portion's in order
+    n: int
+    seqs: torch.Tensor                         # int32 [n_seqs, 2]: (sequence, its first chunk), longest portions first
+    n_seqs: int
+
+
+@dataclass
 class SeqTable:
     """Sequence s owns rows [q_start[s], q_start[s + 1]) of the batch; context[s] of its tokens came before."""
     q_start: torch.Tensor                      # int32 [S + 1]
@@ -167,6 +176,22 @@ class SeqTable:
                     several |= len(runs) - first > 1
             got = (torch.tensor(runs, dtype=torch.int32).to(self.q_start.device), len(runs), several)
             self._items[("time", key)] = got
+        return got
+
+    def chunks(self, size: int) -> Chunks:
+        """The portions of more than one row, cut into chunks of ``size`` rows."""
+        got = self._items.get(("chunks", size))
+        if got is None:
+            rows, long = [], []
+            for s, n in enumerate(self.lens):
+                if n > 1:
+                    long.append((s, len(rows) // 4))
+                    for o in range(0, n, size):
+                        rows += (s, o, min(size, n - o), 0)
+            long.sort(key=lambda it: -self.lens[it[0]])
+            buf = torch.tensor(rows + [v for it in long for v in it], dtype=torch.int32).to(self.q_start.device)
+            got = Chunks(buf[:len(rows)].view(-1, 4), len(rows) // 4, buf[len(rows):].view(-1, 2), len(long))
+            self._items[("chunks", size)] = got
         return got
 
     def prefill_items(self, rows_per_block: int):

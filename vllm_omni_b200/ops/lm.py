@@ -177,6 +177,61 @@ def conv_heads(proj, hs: HeadShape, seqs, slots, k_cache, v_cache, *, conv=None,
     return q_out
 
 
+class _RotaryHeads(ctypes.Structure):
+    _fields_ = [("proj", c_void_p), ("ldp", c_long), ("T", c_int), ("H", c_int), ("G", c_int), ("dp", c_int), ("vp", c_int),
+                ("rot", c_int), ("turns", c_void_p), ("q_gain", c_void_p), ("k_gain", c_void_p), ("nq", c_int), ("nk", c_int),
+                ("vdim", c_int), ("v_norm", c_int), ("v_mult", c_float), ("eps", c_float), ("slots", c_void_p), ("q_out", c_void_p),
+                ("k_cache", c_void_p), ("v_cache", c_void_p), ("num_slots", c_long), ("status", c_void_p)]
+
+
+def rotary_heads(proj, hs: HeadShape, slots, k_cache, v_cache, turns, rot: int, *, q_gain=None, k_gain=None, v_norm: bool = False,
+                 v_mult: float = 1.0, eps: float = 1e-6):
+    """One pass over the packed projection ``proj`` [T, >= channels] (columns q | k | v): where gains are given, RMS norm of
+    the whole query row and of the whole key row (all heads' channels at once); rotation of the first ``rot`` channels of
+    every q and k head in interleaved pairs; with ``v_norm`` every value head over its root mean square, times
+    ``v_mult``; K/V to their pages.  Returns q [T, H, dp].
+
+    ``turns``: fp32 [T, rot / 2, 2] (ops/stream.py rotary_rows); ``q_gain`` fp32 [H * dp], ``k_gain`` [G * dp]."""
+    T, H, G, dp, vp = proj.shape[0], hs.heads, hs.kv_heads, hs.dp, hs.vp
+    q_out = torch.empty(T, H, dp, dtype=proj.dtype, device=proj.device)
+    if not proj.is_cuda:
+        f = proj.float()
+        q, k, v = f[:, :H * dp], f[:, H * dp:(H + G) * dp], f[:, (H + G) * dp:hs.channels].reshape(T, G, vp)
+        if q_gain is not None:
+            q = _rms(q, H * hs.dim, eps) * q_gain
+        if k_gain is not None:
+            k = _rms(k, G * hs.dim, eps) * k_gain
+        if v_norm:
+            v = _rms(v, hs.vdim, eps)
+        if rot:
+            c, s = turns[:, None, :, 0], turns[:, None, :, 1]
+
+            def turn(x):
+                x = x.clone()
+                a, b = x[..., 0:rot:2].clone(), x[..., 1:rot:2].clone()
+                x[..., 0:rot:2], x[..., 1:rot:2] = a * c - b * s, b * c + a * s
+                return x
+            q, k = turn(q.reshape(T, H, dp)), turn(k.reshape(T, G, dp))
+        q_out.copy_(q.reshape(T, H, dp))
+        ok = slots >= 0
+        where = slots[ok].long()
+        k_cache.view(-1, G * dp)[where] = k.reshape(T, -1)[ok].to(k_cache.dtype)
+        v_cache.view(-1, G * vp)[where] = (v_mult * v).reshape(T, -1)[ok].to(v_cache.dtype)
+        return q_out
+    assert proj.stride(1) == 1 and slots.dtype == torch.int32 and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.shape[2:] == (G, dp) and v_cache.shape[2:] == (G, vp) and k_cache.dtype == proj.dtype and rot % 2 == 0
+    assert not rot or (turns.is_contiguous() and turns.shape == (T, rot // 2, 2))
+    a = _RotaryHeads()
+    P = lambda t: 0 if t is None else t.data_ptr()
+    a.proj, a.ldp, a.T, a.H, a.G, a.dp, a.vp, a.rot, a.turns = P(proj), proj.stride(0), T, H, G, dp, vp, rot, P(turns) if rot else 0
+    a.q_gain, a.k_gain, a.nq, a.nk, a.vdim = P(q_gain), P(k_gain), H * hs.dim, G * hs.dim, hs.vdim
+    a.v_norm, a.v_mult, a.eps, a.slots, a.q_out = int(v_norm), v_mult, eps, P(slots), P(q_out)
+    a.k_cache, a.v_cache, a.num_slots = P(k_cache), P(v_cache), k_cache.shape[0] * k_cache.shape[1]
+    a.status = P(nv.status_word(proj.device))
+    nv.check_rc(nv.lib("lm_ops").omni_rotary_heads(ctypes.byref(a), _bf(proj), nv.stream_ptr()), "omni_rotary_heads")
+    return q_out
+
+
 def _conv_heads_cpu(proj, hs, seqs, slots, k_cache, v_cache, conv, state, q_norm, k_norm, eps, v_first, v_mode, lam,
                     q_out, taps, growth):
     H, G, dp, vp, C = hs.heads, hs.kv_heads, hs.dp, hs.vp, hs.channels

@@ -2,7 +2,7 @@
 channel, block-diagonal gates on its result, the scan S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with
 ln a_t = decay r_t, and the product with a gelu branch.  Convolution history and state live in the runner's pools.
 
-Kernels: csrc/gated_scan_sm100.cu (tcgen05, portions of two tokens and more), csrc/gated_scan.cu (single tokens on
+Kernels: csrc/short_conv.cu and csrc/gated_scan_sm100.cu (tcgen05, portions of two tokens and more), csrc/gated_scan.cu (single tokens on
 tensor cores; and plain kernels for fp32 and block sizes the tensor-core kernels do not take)."""
 from __future__ import annotations
 
@@ -14,6 +14,7 @@ import torch.nn.functional as F
 
 from . import _native as nv
 from . import gemm
+from .short_conv import conv_rows
 
 c_int, c_long, c_float, c_void_p = ctypes.c_int, ctypes.c_long, ctypes.c_float, ctypes.c_void_p
 
@@ -103,9 +104,8 @@ def gated_scan(proj, s: GatedScanShape, seqs, conv, conv_b, gates, gates_b, deca
         a.seq_list, a.n_list = P(seqs.decode_list), seqs.n_decode
         nv.check_rc(lib.omni_scan_step(ctypes.byref(a), nv.stream_ptr()), "omni_scan_step")
     if seqs.n_decode < seqs.n_seqs:
-        u = torch.empty(T, C, dtype=proj.dtype, device=proj.device)
+        u = conv_rows(proj[:, C:], seqs, s.taps, C, conv, hist, bias=conv_b, skip_single=True)
         a.u = P(u)
-        nv.check_rc(lib.omni_scan_conv_bf16(ctypes.byref(a), nv.stream_ptr()), "omni_scan_conv_bf16")
         tiles = s.blocks * ((s.part_p + 127) // 128)
         runs, a.n_runs, several = seqs.time_runs(tiles, lambda lens: run_length(lens, tiles))
         a.runs = P(runs)
