@@ -44,7 +44,7 @@ def parse_args():
     ap.add_argument("--workload", default="image", choices=["image", "lm"],
                     help="image: the headline (default); lm: decoder layers of the causal-LM models")
     ap.add_argument("--lm-sizes", default="2048,4096", help="lm workload: widths to run")
-    ap.add_argument("--lm-design", default="tavulix", choices=["tavulix", "nidilix", "milivik"], help="lm workload: decoder to measure")
+    ap.add_argument("--lm-design", default="tavulix", choices=["tavulix", "nidilix", "milivik", "fikizen"], help="lm workload: decoder to measure")
     ap.add_argument("--lm-parts", default="steps,kernels", help="lm workload: which tables to fill")
     ap.add_argument("--ref-eager", action="store_true", help="reference arm: skip its regional torch.compile")
     return ap.parse_args()

@@ -222,7 +222,7 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
 def run(steps: int, warmup: int, widths, parts=("steps", "kernels"), design: str = "tavulix") -> dict:
     import importlib
     from ..ops import _native as nv
-    tables = importlib.import_module({"nidilix": ".lm_nidilix", "milivik": ".lm_milivik"}.get(design, ".lm_layers"), __package__)
+    tables = importlib.import_module({"nidilix": ".lm_nidilix", "milivik": ".lm_milivik", "fikizen": ".lm_fikizen"}.get(design, ".lm_layers"), __package__)
     timer = Timer(steps, warmup)
     n0 = nv.launch_count
     rec = {"metric": "lm_layers", "design": design, "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16", "data": "synthetic (random weights)",
