@@ -1,4 +1,4 @@
-// Delta-rule recurrences of prompt portions in chunks of 16 tokens on tensor cores (delta_rule.cuh says what is computed).
+// Delta-rule recurrences of prompt portions in chunks of 16 or 32 tokens on tensor cores (delta_rule.cuh says what is computed).
 //
 // Within a chunk the recurrence is a triangular system.  With G_t the chunk's decays through token t (scalars, or one per
 // key channel), S the state before the chunk, and rows over tokens:
@@ -9,8 +9,8 @@
 //             O = R0 S + N V - L Y,  R0_t = r_t e^G_t,  N_ts, L_ts = R0_t . (k_s, a_s u_s) e^-G_s up to the diagonal
 //             S <- e^G_last S + (e^(G_last - G) k)^T V - (e^(G_last - G) a u)^T Y
 //
-//   prepare   one warp per (chunk, head), all chunks at once: the 16 x 16 matrices and the inverse T of I + A, left in memory
-//             as tensor-core operands; gated: the tokens' factors; channel: the decayed rows
+//   prepare   a warp per 16 tokens of a (chunk, head), all chunks at once: the lower tiles (16 x 16) of the matrices and of
+//             T = (I + A)^-1, left in memory as tensor-core operands; gated: the tokens' factors; channel: the decayed rows
 //   sequence  one block per (portion, head, 32 value columns); a warp owns eight columns of the state, in registers from the
 //             first chunk to the last, and walks the chunks without talking to the others; operands come through a
 //             cp.async ring that the block shares
@@ -25,7 +25,7 @@ namespace omni {
 
 typedef __nv_bfloat16 bf16;
 
-constexpr int DC_TOK = 16;
+constexpr int DC_TOK = 16;             // tokens of a tile; a chunk is one or two tiles
 constexpr int DC_COLS = 32;            // value columns per block of the sequence kernel
 constexpr int DC_WARPS = 4;
 
@@ -117,52 +117,106 @@ __device__ __forceinline__ void dc_read_tiles(const float (*a)[20], int lane, fl
   }
 }
 
+// Lower left tile of the inverse, -T1 A10 T0, from the tile A10 (result layout) and the inverses of the two diagonal tiles
+__device__ __forceinline__ void dc_corner(const float (&a0)[4], const float (&a1)[4], const float (*t0)[20], const float (*t1)[20],
+                                          int lane, float (&c0)[4], float (&c1)[4]) {
+  auto product = [&](const float (&x0)[4], const float (&x1)[4], const float (&y0)[4], const float (&y1)[4], float (&r0)[4],
+                     float (&r1)[4]) {
+    uint32_t h[4], l[4];
+    dc_split(x0[0], x0[1], h[0], l[0]);
+    dc_split(x0[2], x0[3], h[1], l[1]);
+    dc_split(x1[0], x1[1], h[2], l[2]);
+    dc_split(x1[2], x1[3], h[3], l[3]);
+    SplitB b;
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      float (&r)[4] = n ? r1 : r0;
+      b.from(n ? y1 : y0);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) r[e] = 0.f;
+      dc_mma(r, h, b.h0, b.h1);
+      dc_mma(r, h, b.l0, b.l1);
+      dc_mma(r, l, b.h0, b.h1);
+    }
+  };
+  float x0[4], x1[4], w0[4], w1[4];
+  dc_read_tiles(t0, lane, x0, x1);
+  product(a0, a1, x0, x1, w0, w1);
+  dc_read_tiles(t1, lane, x0, x1);
+  product(x0, x1, w0, w1, c0, c1);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    c0[e] = -c0[e];
+    c1[e] = -c1[e];
+  }
+}
+
 // rows of a chunk
 struct ChunkRows {
   int seq, n;
   long row0;
 };
+template <int M>
 __device__ __forceinline__ ChunkRows dc_chunk(const DeltaRule& p, int i) {
   const int4 c = *reinterpret_cast<const int4*>(p.chunks + 4 * i);
   ChunkRows r;
   r.seq = min(max(c.x, 0), p.num_seqs - 1);
-  r.n = min(max(c.z, 1), DC_TOK);
+  r.n = min(max(c.z, 1), DC_TOK * M);
   r.row0 = p.q_start[r.seq] + c.y;
   return r;
 }
 
+// Matrices of a (chunk, head): `kinds` kinds of the lower tiles, in the order (0, 0), (1, 0), (1, 1); 64 uint4 each
+template <int M> __host__ __device__ constexpr int dc_tiles() { return M * (M + 1) / 2; }
+__device__ __forceinline__ int dc_tile(int m, int n) { return m * (m + 1) / 2 + n; }
+
 // ------------------------------------------------------------------------------ prepare: gated
+template <int M>
 __global__ void __launch_bounds__(128)
 delta_prepare_gated_kernel(const DeltaRule p) {
-  __shared__ float s_a[4][DC_TOK][20], s_tok[4][4][DC_TOK];
+  constexpr int HEADS = 4 / M, C = DC_TOK * M, NT = dc_tiles<M>();
+  __shared__ float s_a[4][DC_TOK][20], s_tok[HEADS][3][C];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
-  const int h = blockIdx.y * 4 + warp;
-  if (h >= p.H) return;
-  const ChunkRows ch = dc_chunk(p, blockIdx.x);
-  float* s_G = s_tok[warp][0];         // cumulative log decay
-  float* s_b = s_tok[warp][1];
-  float* s_ik = s_tok[warp][2];
-  const bf16* proj = static_cast<const bf16*>(p.proj);
+  const int m = warp % M, slot = warp / M;                   // token tile, head of the block
+  const bool live = blockIdx.y * HEADS + slot < p.H;
+  const int h = min((int)blockIdx.y * HEADS + slot, p.H - 1);
+  const ChunkRows ch = dc_chunk<M>(p, blockIdx.x);
+  float* s_G = s_tok[slot][0];         // cumulative log decay
+  float* s_b = s_tok[slot][1];
+  float* s_ik = s_tok[slot][2];
   const int hk = h / (p.H / p.G);
-  // q and k of rows g and g + 8: 8 channels per lane and turn, the same order in both operands
-  const bf16* u = static_cast<const bf16*>(p.u);
-  const long ra = (ch.row0 + min(g, ch.n - 1)) * p.ldu + hk * p.dp, rb = (ch.row0 + min(g + 8, ch.n - 1)) * p.ldu + hk * p.dp;
+  // rows g and g + 8 of a tile: 8 channels per lane and turn, the same order in both operands
+  const bf16* u = static_cast<const bf16*>(p.u) + hk * p.dp;
   const int ko = p.G * p.dp;
-  float kk0[4] = {}, kk1[4] = {}, qk0[4] = {}, qk1[4] = {};
+  auto row = [&](int tile, int r) { return (ch.row0 + min(tile * DC_TOK + r, ch.n - 1)) * p.ldu; };
+  const long ra = row(m, g), rb = row(m, g + 8);
+  float kk[M][2][4] = {}, qk[M][2][4] = {};
   float ss[4] = {};                    // sums of squares: k rows g, g + 8, q rows g, g + 8
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  auto load = [&](long at) { return *reinterpret_cast<const uint4*>(u + at); };
   for (int c = j * 8; c < p.dp + j * 8; c += 32) {
     const bool in = c < p.dp;
-    const uint4 ka = in ? *reinterpret_cast<const uint4*>(u + ra + ko + c) : zero, kb = in ? *reinterpret_cast<const uint4*>(u + rb + ko + c) : zero;
-    const uint4 qa = in ? *reinterpret_cast<const uint4*>(u + ra + c) : zero, qb = in ? *reinterpret_cast<const uint4*>(u + rb + c) : zero;
+    const uint4 ka = in ? load(ra + ko + c) : zero, kb = in ? load(rb + ko + c) : zero;
+    const uint4 qa = in ? load(ra + c) : zero, qb = in ? load(rb + c) : zero;
     const uint32_t kf[2][4] = {{ka.x, kb.x, ka.y, kb.y}, {ka.z, kb.z, ka.w, kb.w}};
     const uint32_t qf[2][4] = {{qa.x, qb.x, qa.y, qb.y}, {qa.z, qb.z, qa.w, qb.w}};
+    uint32_t cf[2][4];                 // keys of the first tile
+    if (M == 2 && m == 1) {
+      const uint4 a = in ? load(row(0, g) + ko + c) : zero, b = in ? load(row(0, g + 8) + ko + c) : zero;
+      cf[0][0] = a.x; cf[0][1] = b.x; cf[0][2] = a.y; cf[0][3] = b.y;
+      cf[1][0] = a.z; cf[1][1] = b.z; cf[1][2] = a.w; cf[1][3] = b.w;
+    }
 #pragma unroll
     for (int s = 0; s < 2; ++s) {
-      dc_mma(kk0, kf[s], kf[s][0], kf[s][2]);
-      dc_mma(kk1, kf[s], kf[s][1], kf[s][3]);
-      dc_mma(qk0, qf[s], kf[s][0], kf[s][2]);
-      dc_mma(qk1, qf[s], kf[s][1], kf[s][3]);
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        dc_mma(kk[0][n], kf[s], kf[s][n], kf[s][n + 2]);
+        dc_mma(qk[0][n], qf[s], kf[s][n], kf[s][n + 2]);
+        if (M == 2 && m == 1) {
+          dc_mma(kk[M - 1][n], kf[s], cf[s][n], cf[s][n + 2]);
+          dc_mma(qk[M - 1][n], qf[s], cf[s][n], cf[s][n + 2]);
+        }
+      }
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const float2 fk = unpack_bf16(kf[s][e]), fq = unpack_bf16(qf[s][e]);
@@ -179,90 +233,110 @@ delta_prepare_gated_kernel(const DeltaRule p) {
   const float ik[2] = {1.0f / sqrtf(ss[0] + p.unit_eps), 1.0f / sqrtf(ss[1] + p.unit_eps)};
   const float iq[2] = {p.q_mul / sqrtf(ss[2] + p.unit_eps), p.q_mul / sqrtf(ss[3] + p.unit_eps)};
   if (j == 0) {
-    s_ik[g] = ik[0];
-    s_ik[g + 8] = ik[1];
+    s_ik[m * DC_TOK + g] = ik[0];
+    s_ik[m * DC_TOK + g + 8] = ik[1];
   }
   // a lane per token: step size, cumulative log decay
-  const int t = lane & 15;
-  const bool live = t < ch.n;
-  const bf16* pr = proj + (ch.row0 + min(t, ch.n - 1)) * p.ldp;
-  const float beta = live ? dr_sigmoid((float)pr[p.b_col + h]) : 0.f;
-  float G = live ? p.rate[h] * dr_softplus((float)pr[p.a_col + h] + p.dt_bias[h]) : 0.f;
+  const int t = lane & (C - 1);
+  const bf16* pr = static_cast<const bf16*>(p.proj) + (ch.row0 + min(t, ch.n - 1)) * p.ldp;
+  const float beta = t < ch.n ? dr_sigmoid((float)pr[p.b_col + h]) : 0.f;
+  float G = t < ch.n ? p.rate[h] * dr_softplus((float)pr[p.a_col + h] + p.dt_bias[h]) : 0.f;
 #pragma unroll
-  for (int o = 1; o < 16; o <<= 1) {
-    const float v = __shfl_up_sync(0xffffffffu, G, o, 16);
+  for (int o = 1; o < C; o <<= 1) {
+    const float v = __shfl_up_sync(0xffffffffu, G, o, C);
     if (t >= o) G += v;
   }
-  const float G_last = __shfl_sync(0xffffffffu, G, 15, 16);
-  if (lane < 16) {
+  const float G_last = __shfl_sync(0xffffffffu, G, C - 1, C);
+  if (m == 0 && lane < C) {
     s_G[t] = G;
     s_b[t] = beta;
   }
-  __syncwarp();
+  __syncthreads();
   const long at = (long)blockIdx.x * p.H + h;
-  uint4* mats = static_cast<uint4*>(p.mats) + at * 128;
-  float* coef = p.coef + at * (4 * DC_TOK + 4);
-  float p0[4], p1[4];
+  uint4* mats = static_cast<uint4*>(p.mats) + at * (2 * NT * 64);
+  float* coef = p.coef + at * (4 * C + 4);
+  // tile (m, n) of the system and of the output matrix
+  auto finish = [&](int n, float (&a)[2][4], float (&q)[2][4]) {
 #pragma unroll
-  for (int e = 0; e < 4; ++e) {
-    const int r = g + (e >> 1) * 8;
+    for (int e = 0; e < 4; ++e) {
+      const int r = m * DC_TOK + g + (e >> 1) * 8;
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int s = half * 8 + j * 2 + (e & 1);
-      const float d = r >= s ? expf(s_G[r] - s_G[s]) * s_ik[s] : 0.f;
-      s_a[warp][r][s] = r > s ? s_b[r] * ik[e >> 1] * (half ? kk1[e] : kk0[e]) * d : 0.f;
-      (half ? p1[e] : p0[e]) = iq[e >> 1] * (half ? qk1[e] : qk0[e]) * d;
+      for (int half = 0; half < 2; ++half) {
+        const int s = n * DC_TOK + half * 8 + j * 2 + (e & 1);
+        const float d = r >= s ? expf(s_G[r] - s_G[s]) * s_ik[s] : 0.f;
+        a[half][e] *= r > s ? s_b[r] * ik[e >> 1] * d : 0.f;
+        q[half][e] *= iq[e >> 1] * d;
+      }
     }
-  }
-  dc_store_mat(mats + 64, lane, p0, p1);
-  if (j == 0) {
+    if (live) dc_store_mat(mats + (NT + dc_tile(m, n)) * 64, lane, q[0], q[1]);
+  };
+  finish(m, kk[0], qk[0]);
+  if (M == 2 && m == 1) finish(0, kk[M - 1], qk[M - 1]);
+#pragma unroll
+  for (int e = 0; e < 4; ++e)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) s_a[warp][g + (e >> 1) * 8][half * 8 + j * 2 + (e & 1)] = kk[0][half][e];
+  if (live && j == 0) {
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int r = g + 8 * half;
+      const int r = m * DC_TOK + g + 8 * half;
       const float e = expf(s_G[r]);
       const float4 c = make_float4(s_b[r], -s_b[r] * e * ik[half], e * iq[half], r < ch.n ? expf(G_last - s_G[r]) * ik[half] : 0.f);
       *reinterpret_cast<float4*>(coef + 4 * r) = c;
     }
   }
-  if (lane == 0) *reinterpret_cast<float4*>(coef + 4 * DC_TOK) = make_float4(expf(G_last), 0.f, 0.f, 0.f);
+  if (live && m == 0 && lane == 0) *reinterpret_cast<float4*>(coef + 4 * C) = make_float4(expf(G_last), 0.f, 0.f, 0.f);
   __syncwarp();
   dc_invert(s_a[warp], lane);
   float c0[4], c1[4];
   dc_read_tiles(s_a[warp], lane, c0, c1);
-  dc_store_mat(mats, lane, c0, c1);
+  if (live) dc_store_mat(mats + dc_tile(m, m) * 64, lane, c0, c1);
+  if (M == 2) {
+    __syncthreads();                                         // the first tile's inverse is there
+    if (m == 1) {
+      dc_corner(kk[M - 1][0], kk[M - 1][1], s_a[warp - 1], s_a[warp], lane, c0, c1);
+      if (live) dc_store_mat(mats + dc_tile(1, 0) * 64, lane, c0, c1);
+    }
+  }
 }
 
 // ---------------------------------------------------------------------------- prepare: channel
-constexpr int PC_WARPS = 2, PC_PITCH = 64 * 2 + 16;          // bytes of a row of 64 channels
-constexpr int PC_WARP_BYTES = 8 * DC_TOK * PC_PITCH;
+constexpr int PC_PITCH = 64 * 2 + 16;  // bytes of a row of 64 channels
 
-__global__ void __launch_bounds__(32 * PC_WARPS)
+template <int M>
+__global__ void __launch_bounds__(32 * M)
 delta_prepare_channel_kernel(const DeltaRule p) {
-  __shared__ __align__(16) uint8_t s_rows[PC_WARPS][PC_WARP_BYTES];      // decayed rows: b0, r0, k / G, a u / G (high, low)
-  __shared__ float s_a[PC_WARPS][DC_TOK][20];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
-  const int h = blockIdx.y * PC_WARPS + warp;
-  if (h >= p.H) return;
-  const ChunkRows ch = dc_chunk(p, blockIdx.x);
+  constexpr int C = DC_TOK * M, NT = dc_tiles<M>();
+  constexpr int ROW32 = PC_PITCH / 4, ARR32 = C * ROW32;
+  __shared__ __align__(16) uint32_t s_rows[8 * ARR32];       // decayed rows: b0, r0, k / G, a u / G (high, low)
+  __shared__ float s_a[M][DC_TOK][20];
+  __shared__ float2 s_tot[M][32];                            // log decay of a tile's tokens
+  const int m = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+  const int h = blockIdx.y;
+  const ChunkRows ch = dc_chunk<M>(p, blockIdx.x);
   const bf16* proj = static_cast<const bf16*>(p.proj) + (long)h * p.dp;
   const bf16* z = static_cast<const bf16*>(p.z) + (long)h * p.dp;
   const long at = (long)blockIdx.x * p.H + h;
-  uint32_t* tiles = static_cast<uint32_t*>(p.tiles) + at * (8 * DC_TOK * (p.dp / 2));
-  uint4* mats = static_cast<uint4*>(p.mats) + at * 256;
-  const int tile = DC_TOK * (p.dp / 2);                      // channel pairs of an operand
-  auto pair = [&](const bf16* base, long ld, int t, int c) {  // two channels of token t
-    return unpack_bf16(*reinterpret_cast<const uint32_t*>(base + (ch.row0 + t) * ld + c));
+  const int tile = C * (p.dp / 2);                           // channel pairs of an operand
+  uint32_t* tiles = static_cast<uint32_t*>(p.tiles) + at * (8 * tile);
+  uint4* mats = static_cast<uint4*>(p.mats) + at * (4 * NT * 64);
+  // two channels of the tile's token t (past the end: another token's, not used)
+  auto raw = [&](const bf16* base, long ld, int t, int c) {
+    return *reinterpret_cast<const uint32_t*>(base + (ch.row0 + min(m * DC_TOK + t, ch.n - 1)) * ld + c);
   };
   // lengths of the keys
   float ik[DC_TOK];
 #pragma unroll
-  for (int t = 0; t < DC_TOK; ++t) {
-    ik[t] = 0.f;
-    if (t < ch.n)
-      for (int c = lane * 2; c < p.dp; c += 64) {
-        const float2 k = pair(proj + p.k_col, p.ldp, t, c);
-        ik[t] = fmaf(k.x, k.x, fmaf(k.y, k.y, ik[t]));
-      }
+  for (int t = 0; t < DC_TOK; ++t) ik[t] = 0.f;
+  for (int c = lane * 2; c < p.dp; c += 64) {
+    uint32_t k[DC_TOK];
+#pragma unroll
+    for (int t = 0; t < DC_TOK; ++t) k[t] = raw(proj + p.k_col, p.ldp, t, c);
+#pragma unroll
+    for (int t = 0; t < DC_TOK; ++t) {
+      const float2 f = unpack_bf16(k[t]);
+      ik[t] = fmaf(f.x, f.x, fmaf(f.y, f.y, ik[t]));
+    }
   }
 #pragma unroll
   for (int t = 0; t < DC_TOK; ++t) {
@@ -270,92 +344,108 @@ delta_prepare_channel_kernel(const DeltaRule p) {
     for (int o = 16; o > 0; o >>= 1) ik[t] += __shfl_xor_sync(0xffffffffu, ik[t], o);
     ik[t] = 1.0f / sqrtf(ik[t] + p.unit_eps);
   }
-  float am[2][4] = {}, mm[2][4] = {}, nm[2][4] = {}, lm[2][4] = {};
-  const uint32_t base = smem_u32(s_rows[warp]);
-  uint32_t* rows = reinterpret_cast<uint32_t*>(s_rows[warp]);
-  constexpr int ROW32 = PC_PITCH / 4, ARR32 = DC_TOK * ROW32;
+  float am[M][2][4] = {}, mm[M][2][4] = {}, nm[M][2][4] = {}, lm[M][2][4] = {};      // [0]: diagonal tile, [1]: left of it
+  const uint32_t base = smem_u32(s_rows);
   for (int cb = 0; cb < p.dp; cb += 64) {
     const int c = cb + lane * 2;
     const bool in = c < p.dp;
     const int cc = in ? c : 0;
     const float2 db = *reinterpret_cast<const float2*>(p.decay_bias + h * p.dp + cc);
     const float2 rb = *reinterpret_cast<const float2*>(p.removal_bias + h * p.dp + cc);
-    float e0 = 1.f, e1 = 1.f, G0 = 0.f, G1 = 0.f;            // decays so far
-    float kx[DC_TOK], ky[DC_TOK], ax[DC_TOK], ay[DC_TOK];    // k / G, a u / G
-    __syncwarp();                                            // the products of the last 64 channels are done
+    uint32_t r_[DC_TOK], k_[DC_TOK], a_[DC_TOK];
+    float2 G[DC_TOK];                                        // cumulative log decay
 #pragma unroll
     for (int t = 0; t < DC_TOK; ++t) {
-      float2 b0 = make_float2(0.f, 0.f), r0 = b0;
-      kx[t] = ky[t] = ax[t] = ay[t] = 0.f;
-      if (t < ch.n && in) {
-        const float2 r = pair(proj + p.q_col, p.ldp, t, c), k = pair(proj + p.k_col, p.ldp, t, c);
-        const float2 a = pair(proj + p.a_col, p.ldp, t, c), zz = pair(z, p.ldz, t, c);
-        b0 = make_float2(k.x * ik[t] * e0, k.y * ik[t] * e1);
-        G0 = fmaf(p.decay_scale, __fdividef(1.0f, 1.0f + __expf(-(zz.x + db.x))), G0);
-        G1 = fmaf(p.decay_scale, __fdividef(1.0f, 1.0f + __expf(-(zz.y + db.y))), G1);
-        e0 = __expf(G0);
-        e1 = __expf(G1);
-        r0 = make_float2(r.x * e0, r.y * e1);
-        const float i0 = __expf(-G0), i1 = __expf(-G1);
-        kx[t] = k.x * i0;
-        ky[t] = k.y * i1;
-        ax[t] = __fdividef(ik[t], 1.0f + __expf(-(a.x + rb.x))) * kx[t];
-        ay[t] = __fdividef(ik[t], 1.0f + __expf(-(a.y + rb.y))) * ky[t];
-      }
-      uint32_t hi, lo;
-      uint32_t* dst = rows + t * ROW32 + lane;
-      uint32_t* out = tiles + t * (p.dp / 2) + c / 2;
-      dc_split(b0.x, b0.y, hi, lo);
-      dst[0] = hi;
-      dst[ARR32] = lo;
-      if (in) { out[0] = hi; out[tile] = lo; }
-      dc_split(r0.x, r0.y, hi, lo);
-      dst[2 * ARR32] = hi;
-      dst[3 * ARR32] = lo;
-      if (in) { out[2 * tile] = hi; out[3 * tile] = lo; }
-      dc_split(kx[t], ky[t], hi, lo);
-      dst[4 * ARR32] = hi;
-      dst[5 * ARR32] = lo;
-      dc_split(ax[t], ay[t], hi, lo);
-      dst[6 * ARR32] = hi;
-      dst[7 * ARR32] = lo;
+      const float2 f = unpack_bf16(raw(z, p.ldz, t, cc));
+      G[t] = make_float2(f.x + db.x, f.y + db.y);
+      r_[t] = raw(proj + p.q_col, p.ldp, t, cc);
+      k_[t] = raw(proj + p.k_col, p.ldp, t, cc);
+      a_[t] = raw(proj + p.a_col, p.ldp, t, cc);
     }
-    if (in) {
-      *reinterpret_cast<float2*>(p.coef + at * p.dp + c) = make_float2(e0, e1);
+    float2 sum = make_float2(0.f, 0.f);
 #pragma unroll
-      for (int t = 0; t < DC_TOK; ++t) {
-        uint32_t hi, lo;
-        uint32_t* out = tiles + 4 * tile + t * (p.dp / 2) + c / 2;
-        dc_split(kx[t] * e0, ky[t] * e1, hi, lo);
-        out[0] = hi;
-        out[tile] = lo;
-        dc_split(-ax[t] * e0, -ay[t] * e1, hi, lo);
-        out[2 * tile] = hi;
-        out[3 * tile] = lo;
+    for (int t = 0; t < DC_TOK; ++t) {
+      if (m * DC_TOK + t < ch.n) {
+        sum.x = fmaf(p.decay_scale, __fdividef(1.0f, 1.0f + __expf(-G[t].x)), sum.x);
+        sum.y = fmaf(p.decay_scale, __fdividef(1.0f, 1.0f + __expf(-G[t].y)), sum.y);
       }
+      G[t] = sum;
     }
-    __syncwarp();
-    const uint32_t a0 = base + ((lane & 7) + ((lane >> 3) & 1) * 8) * PC_PITCH + (lane >> 4) * 16;
-    constexpr uint32_t ARR = DC_TOK * PC_PITCH;
+    s_tot[m][lane] = sum;
+    __syncthreads();                                         // totals; and the products of the last 64 channels are done
+    float2 before = make_float2(0.f, 0.f), total = s_tot[0][lane];
+    if (M == 2) {
+      if (m == 1) before = total;
+      total.x += s_tot[M - 1][lane].x;
+      total.y += s_tot[M - 1][lane].y;
+    }
+    const float tx = __expf(total.x), ty = __expf(total.y);
+    float e0 = __expf(before.x), e1 = __expf(before.y);      // decays so far
+#pragma unroll
+    for (int t = 0; t < DC_TOK; ++t) {
+      float2 b0 = make_float2(0.f, 0.f), r0 = b0, ki = b0, ai = b0;
+      if (m * DC_TOK + t < ch.n && in) {
+        const float2 r = unpack_bf16(r_[t]), k = unpack_bf16(k_[t]), a = unpack_bf16(a_[t]);
+        b0 = make_float2(k.x * ik[t] * e0, k.y * ik[t] * e1);
+        const float gx = G[t].x + before.x, gy = G[t].y + before.y;
+        e0 = __expf(gx);
+        e1 = __expf(gy);
+        r0 = make_float2(r.x * e0, r.y * e1);
+        ki = make_float2(k.x * __expf(-gx), k.y * __expf(-gy));
+        ai = make_float2(__fdividef(ik[t], 1.0f + __expf(-(a.x + rb.x))) * ki.x, __fdividef(ik[t], 1.0f + __expf(-(a.y + rb.y))) * ki.y);
+      }
+      const int tok = m * DC_TOK + t;
+      uint32_t hi, lo;
+      uint32_t* dst = s_rows + tok * ROW32 + lane;
+      uint32_t* out = tiles + tok * (p.dp / 2) + c / 2;
+      auto put = [&](int x, float2 v, bool shared, int global) {           // a pair of channels of operand x, high and low parts
+        dc_split(v.x, v.y, hi, lo);
+        if (shared) {
+          dst[x * ARR32] = hi;
+          dst[(x + 1) * ARR32] = lo;
+        }
+        if (in && global >= 0) {
+          out[global * tile] = hi;
+          out[(global + 1) * tile] = lo;
+        }
+      };
+      put(0, b0, true, 0);
+      put(2, r0, true, 2);
+      put(4, ki, true, -1);
+      put(6, ai, true, -1);
+      put(0, make_float2(ki.x * tx, ki.y * ty), false, 4);
+      put(0, make_float2(-ai.x * tx, -ai.y * ty), false, 6);
+    }
+    if (in && m == 0) *reinterpret_cast<float2*>(p.coef + at * p.dp + c) = make_float2(tx, ty);
+    __syncthreads();
+    constexpr uint32_t ARR = C * PC_PITCH;
+    const uint32_t a0 = base + ((lane & 7) + ((lane >> 3) & 1) * 8) * PC_PITCH + (lane >> 4) * 16, mine = a0 + m * DC_TOK * PC_PITCH;
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       if (cb + k * 16 >= p.dp) break;
-      uint32_t f[8][4];
+      uint32_t x[4][4];                                      // b0, r0 of this tile
 #pragma unroll
-      for (int x = 0; x < 8; ++x) dc_ldsm4(a0 + x * ARR + k * 32, f[x]);
-      // rows x (0: b0, 2: r0) times columns y (4: k / G, 6: a u / G): high high, high low, low high
-      auto product = [&](float (&c)[2][4], int x, int y) {
+      for (int i = 0; i < 4; ++i) dc_ldsm4(mine + i * ARR + k * 32, x[i]);
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          dc_mma(c[n], f[x], f[y][n], f[y][n + 2]);
-          dc_mma(c[n], f[x], f[y + 1][n], f[y + 1][n + 2]);
-          dc_mma(c[n], f[x + 1], f[y][n], f[y][n + 2]);
-        }
-      };
-      product(am, 0, 6);
-      product(mm, 0, 4);
-      product(nm, 2, 4);
-      product(lm, 2, 6);
+      for (int n = 0; n < M; ++n) {                          // columns: this tile, then the one before
+        if (n > m) continue;
+        uint32_t y[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) dc_ldsm4((n ? a0 : mine) + (4 + i) * ARR + k * 32, y[i]);
+        // high high, high low, low high
+        auto product = [&](float (&r)[2][4], int i, int q) {
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            dc_mma(r[half], x[i], y[q][half], y[q][half + 2]);
+            dc_mma(r[half], x[i], y[q + 1][half], y[q + 1][half + 2]);
+            dc_mma(r[half], x[i + 1], y[q][half], y[q][half + 2]);
+          }
+        };
+        product(am[n], 0, 2);
+        product(mm[n], 0, 0);
+        product(nm[n], 2, 0);
+        product(lm[n], 2, 2);
+      }
     }
   }
 #pragma unroll
@@ -363,76 +453,96 @@ delta_prepare_channel_kernel(const DeltaRule p) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int r = g + (e >> 1) * 8, s = n * 8 + j * 2 + (e & 1);
-      s_a[warp][r][s] = r > s ? am[n][e] : 0.f;
-      if (r <= s) mm[n][e] = 0.f;
-      if (r < s) nm[n][e] = 0.f;
-      lm[n][e] = r < s ? 0.f : -lm[n][e];
+      s_a[m][r][s] = r > s ? am[0][n][e] : 0.f;
+      if (r <= s) mm[0][n][e] = 0.f;
+      if (r < s) nm[0][n][e] = 0.f;
+      lm[0][n][e] = r < s ? 0.f : -lm[0][n][e];
+      if (M == 2) lm[M - 1][n][e] = m == 1 ? -lm[M - 1][n][e] : lm[M - 1][n][e];
     }
-  dc_store_mat(mats + 64, lane, mm[0], mm[1]);
-  dc_store_mat(mats + 128, lane, nm[0], nm[1]);
-  dc_store_mat(mats + 192, lane, lm[0], lm[1]);
+#pragma unroll
+  for (int n = 0; n < M; ++n) {
+    if (n > m) continue;
+    const int i = dc_tile(m, m - n);
+    dc_store_mat(mats + (NT + i) * 64, lane, mm[n][0], mm[n][1]);
+    dc_store_mat(mats + (2 * NT + i) * 64, lane, nm[n][0], nm[n][1]);
+    dc_store_mat(mats + (3 * NT + i) * 64, lane, lm[n][0], lm[n][1]);
+  }
   __syncwarp();
-  dc_invert(s_a[warp], lane);
+  dc_invert(s_a[m], lane);
   float c0[4], c1[4];
-  dc_read_tiles(s_a[warp], lane, c0, c1);
-  dc_store_mat(mats, lane, c0, c1);
+  dc_read_tiles(s_a[m], lane, c0, c1);
+  dc_store_mat(mats + dc_tile(m, m) * 64, lane, c0, c1);
+  if (M == 2) {
+    __syncthreads();                                         // the first tile's inverse is there
+    if (m == 1) {
+      dc_corner(am[M - 1][0], am[M - 1][1], s_a[0], s_a[M - 1], lane, c0, c1);
+      dc_store_mat(mats + dc_tile(1, 0) * 64, lane, c0, c1);
+    }
+  }
 }
 
 // ----------------------------------------------------------------------------------- sequence
+constexpr int DC_VPITCH = DC_COLS * 2 + 16;
+
 // Bytes of a stage: rows of the operands (gated: k, q; channel: eight), values, matrices, factors
 struct DeltaStage {
   int pitch, arr, values, mats, coef, bytes;
 };
-__host__ __device__ __forceinline__ DeltaStage delta_stage(int dp, bool channel) {
+template <bool CHANNEL, int M>
+__host__ __device__ __forceinline__ DeltaStage delta_stage(int dp) {
   DeltaStage s;
   s.pitch = dp * 2 + 16;               // an odd multiple of 16 bytes: conflict-free ldmatrix
-  s.arr = DC_TOK * s.pitch;
-  s.values = (channel ? 8 : 2) * s.arr;
-  s.mats = s.values + DC_TOK * (DC_COLS * 2 + 16);
-  s.coef = s.mats + (channel ? 4096 : 2048);
-  s.bytes = s.coef + (channel ? dp * 4 : (4 * DC_TOK + 4) * 4);
+  s.arr = M * DC_TOK * s.pitch;
+  s.values = (CHANNEL ? 8 : 2) * s.arr;
+  s.mats = s.values + M * DC_TOK * DC_VPITCH;
+  s.coef = s.mats + (CHANNEL ? 4 : 2) * dc_tiles<M>() * 1024;
+  s.bytes = s.coef + (CHANNEL ? dp * 4 : (4 * M * DC_TOK + 4) * 4);
   return s;
 }
-constexpr int DC_VPITCH = DC_COLS * 2 + 16;
 
-// KS: 16-channel steps of the key channels that the state's registers hold (dp <= 16 KS)
-template <bool CHANNEL, int KS>
+// KS: 16-channel steps of the key channels that the state's registers hold.  EXACT: dp = 16 KS, so that a chunk's products
+// are straight-line code; otherwise dp <= 16 KS.  M: tiles of 16 tokens in a chunk.
+template <bool CHANNEL, int KS, bool EXACT, int M>
 __global__ void __launch_bounds__(32 * DC_WARPS)
 delta_sequence_kernel(const DeltaRule p, const int stages) {
+  constexpr int C = M * DC_TOK, NT = dc_tiles<M>();
   extern __shared__ __align__(16) uint8_t smem[];
+  const int dp = EXACT ? 16 * KS : p.dp;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, j2 = (lane & 3) * 2;
   const int seq = min(max(p.long_list[2 * blockIdx.z], 0), p.num_seqs - 1), first = p.long_list[2 * blockIdx.z + 1];
   const int h = blockIdx.y, col0 = blockIdx.x * DC_COLS, hk = h / (p.H / p.G);
   const long row0 = p.q_start[seq];
   const int n = (int)(p.q_start[seq + 1] - row0);
-  const int n_chunks = min((n + DC_TOK - 1) / DC_TOK, p.n_chunks - first);
-  const DeltaStage lay = delta_stage(p.dp, CHANNEL);
+  const int n_chunks = min((n + C - 1) / C, p.n_chunks - first);
+  const DeltaStage lay = delta_stage<CHANNEL, M>(dp);
   const uint32_t base = smem_u32(smem);
-  const int vecs = p.dp / 8, v_vecs = min(DC_COLS, p.vp - col0) / 8;
+  const int vecs = dp / 8, v_vecs = min(DC_COLS, p.vp - col0) / 8;
 
   auto fetch = [&](int i) {
     const uint32_t st = base + (i % stages) * lay.bytes;
     const long at = (long)(first + i) * p.H + h;
-    auto row = [&](int t) { return row0 + min(i * DC_TOK + t, n - 1); };       // past the end: finite, its factors are zero
+    auto row = [&](int t) { return row0 + min(i * C + t, n - 1); };        // past the end: finite, its factors are zero
     if (CHANNEL) {
-      const uint4* src = static_cast<const uint4*>(p.tiles) + at * (8 * DC_TOK * vecs);
-      for (int x = tid; x < 8 * DC_TOK * vecs; x += 32 * DC_WARPS) dc_copy16(st + (x / vecs) * lay.pitch + (x % vecs) * 16, src + x);
+      const uint4* src = static_cast<const uint4*>(p.tiles) + at * (8 * C * vecs);
+      for (int x = tid; x < 8 * C * vecs; x += 32 * DC_WARPS) dc_copy16(st + (x / vecs) * lay.pitch + (x % vecs) * 16, src + x);
     } else {
-      const bf16* u = static_cast<const bf16*>(p.u) + hk * p.dp;
-      for (int x = tid; x < 2 * DC_TOK * vecs; x += 32 * DC_WARPS) {
+      const bf16* u = static_cast<const bf16*>(p.u) + hk * dp;
+      for (int x = tid; x < 2 * C * vecs; x += 32 * DC_WARPS) {
         const int r = x / vecs, c = x - r * vecs;            // rows of k, then of q
-        dc_copy16(st + r * lay.pitch + c * 16, u + row(r & 15) * p.ldu + (r < DC_TOK ? p.G * p.dp : 0) + c * 8);
+        dc_copy16(st + r * lay.pitch + c * 16, u + row(r & (C - 1)) * p.ldu + (r < C ? p.G * dp : 0) + c * 8);
       }
     }
-    const bf16* v = CHANNEL ? static_cast<const bf16*>(p.proj) + p.v_col : static_cast<const bf16*>(p.u) + 2 * p.G * p.dp;
+    const bf16* v = CHANNEL ? static_cast<const bf16*>(p.proj) + p.v_col : static_cast<const bf16*>(p.u) + 2 * p.G * dp;
     const long ldv = CHANNEL ? p.ldp : p.ldu;
-    for (int x = tid; x < DC_TOK * v_vecs; x += 32 * DC_WARPS) {
-      const int r = x / v_vecs, c = x - r * v_vecs;
-      dc_copy16(st + lay.values + r * DC_VPITCH + c * 16, v + row(r) * ldv + (long)h * p.vp + col0 + c * 8);
+    for (int x = tid; x < C * (DC_COLS / 8); x += 32 * DC_WARPS) {
+      const int r = x / (DC_COLS / 8), c = x % (DC_COLS / 8);
+      if (c < v_vecs) dc_copy16(st + lay.values + r * DC_VPITCH + c * 16, v + row(r) * ldv + (long)h * p.vp + col0 + c * 8);
     }
-    const int nm = CHANNEL ? 256 : 128;
-    for (int x = tid; x < nm; x += 32 * DC_WARPS) dc_copy16(st + lay.mats + x * 16, static_cast<const uint4*>(p.mats) + at * nm + x);
-    const int nf = CHANNEL ? p.dp / 4 : DC_TOK + 1;
+    constexpr int nm = (CHANNEL ? 4 : 2) * NT * 64;
+    const uint4* mats = static_cast<const uint4*>(p.mats) + at * nm;
+#pragma unroll
+    for (int x = 0; x < nm; x += 32 * DC_WARPS) dc_copy16(st + lay.mats + (x + tid) * 16, mats + x + tid);
+    const int nf = CHANNEL ? dp / 4 : C + 1;
     for (int x = tid; x < nf; x += 32 * DC_WARPS) dc_copy16(st + lay.coef + x * 16, reinterpret_cast<const float4*>(p.coef) + at * nf + x);
   };
 
@@ -442,14 +552,14 @@ delta_sequence_kernel(const DeltaRule p, const int stages) {
   const bool used = col < p.vp;
   float S[KS][4];                                            // rows g, g + 8 of 16 key channels, columns j2, j2 + 1
   {
-    const float* src = p.state + ((long)sin * p.H + h) * p.dp * p.vp + col + j2;
+    const float* src = p.state + ((long)sin * p.H + h) * dp * p.vp + col + j2;
     const bool have = used && p.context[seq] > 0;
 #pragma unroll
     for (int k = 0; k < KS; ++k)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int r = k * 16 + g + 8 * e;
-        const float2 v = have && k * 16 < p.dp ? *reinterpret_cast<const float2*>(src + (long)r * p.vp) : make_float2(0.f, 0.f);
+        const float2 v = have && (EXACT || k * 16 < dp) ? *reinterpret_cast<const float2*>(src + (long)r * p.vp) : make_float2(0.f, 0.f);
         S[k][2 * e] = v.x;
         S[k][2 * e + 1] = v.y;
       }
@@ -458,186 +568,253 @@ delta_sequence_kernel(const DeltaRule p, const int stages) {
     if (i < n_chunks) fetch(i);
     asm volatile("cp.async.commit_group;" ::: "memory");
   }
-  bf16* raw = static_cast<bf16*>(p.raw) + (long)h * p.vp + col + j2;
-  const uint32_t a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * lay.pitch + (lane >> 4) * 16;      // tokens x channels
-  const uint32_t t_off = ((lane & 7) + (lane >> 4) * 8) * lay.pitch + ((lane >> 3) & 1) * 16;      // channels x tokens
-  for (int i = 0; i < n_chunks; ++i) {
-    if (stages == 4) asm volatile("cp.async.wait_group 2;" ::: "memory");
-    else if (stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
-    else asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                         // chunk i is here, chunk i - 1 is done with
+  auto next = [&](int i) {                                   // into the place of chunk i - 1
     if (i + stages - 1 < n_chunks) fetch(i + stages - 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
-    if (!used) continue;
+  };
+  bf16* out = static_cast<bf16*>(p.raw) + (long)h * p.vp + col + j2;
+  const uint32_t a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * lay.pitch + (lane >> 4) * 16;      // tokens x channels
+  const uint32_t t_off = ((lane & 7) + (lane >> 4) * 8) * lay.pitch + ((lane >> 3) & 1) * 16;      // channels x tokens
+  const uint32_t tile = DC_TOK * lay.pitch;
+  for (int i = 0; i < n_chunks; ++i) {
+    if (stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+    else asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                         // chunk i is here, chunk i - 1 is done with
+    if (!used) {
+      next(i);
+      continue;
+    }
     const int so = (i % stages) * lay.bytes;
     const uint32_t st = base + so;
     const uint4* mats = reinterpret_cast<const uint4*>(smem + so + lay.mats) + lane;
-    auto mat = [&](int m, uint32_t (&a)[4]) {
-      const uint4 v = mats[32 * m];
-      a[0] = v.x; a[1] = v.y; a[2] = v.z; a[3] = v.w;
-    };
     // what the state gives for the chunk's keys (x) and queries (o)
-    float x0[4] = {}, x1[4] = {}, o0[4] = {}, o1[4] = {};
-    SplitB s[KS];
+    float x[M][2][4] = {}, o[M][2][4] = {};
 #pragma unroll
     for (int k = 0; k < KS; ++k) {
-      if (k * 16 >= p.dp) break;
-      s[k].from(S[k]);
-      uint32_t a[4];
-      dc_ldsm4(st + a_off + k * 32, a);
-      dc_mma(x0, a, s[k].h0, s[k].h1);
-      dc_mma(x1, a, s[k].l0, s[k].l1);
-      if (CHANNEL) {
-        dc_ldsm4(st + lay.arr + a_off + k * 32, a);
-        dc_mma(x1, a, s[k].h0, s[k].h1);
-      }
-    }
+      if (!EXACT && k * 16 >= dp) break;
+      SplitB s;
+      s.from(S[k]);
 #pragma unroll
-    for (int k = 0; k < KS; ++k) {
-      if (k * 16 >= p.dp) break;
-      uint32_t a[4];
-      dc_ldsm4(st + (CHANNEL ? 2 : 1) * lay.arr + a_off + k * 32, a);
-      dc_mma(o0, a, s[k].h0, s[k].h1);
-      dc_mma(o1, a, s[k].l0, s[k].l1);
-      if (CHANNEL) {
-        dc_ldsm4(st + 3 * lay.arr + a_off + k * 32, a);
-        dc_mma(o1, a, s[k].h0, s[k].h1);
+      for (int m = 0; m < M; ++m) {
+        uint32_t a[4];
+        dc_ldsm4(st + a_off + m * tile + k * 32, a);
+        dc_mma(x[m][0], a, s.h0, s.h1);
+        dc_mma(x[m][1], a, s.l0, s.l1);
+        if (CHANNEL) {
+          dc_ldsm4(st + lay.arr + a_off + m * tile + k * 32, a);
+          dc_mma(x[m][1], a, s.h0, s.h1);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        uint32_t a[4];
+        dc_ldsm4(st + (CHANNEL ? 2 : 1) * lay.arr + a_off + m * tile + k * 32, a);
+        dc_mma(o[m][0], a, s.h0, s.h1);
+        dc_mma(o[m][1], a, s.l0, s.l1);
+        if (CHANNEL) {
+          dc_ldsm4(st + 3 * lay.arr + a_off + m * tile + k * 32, a);
+          dc_mma(o[m][1], a, s.h0, s.h1);
+        }
       }
     }
-    float y[4] = {}, o[4];
-    uint32_t mh[4], ml[4];
-    // product of a 16 x 16 matrix with split rows
-    auto times = [&](float (&c)[4], int m, const SplitB& b) {
-      mat(m, mh);
-      mat(m + 1, ml);
-      dc_mma(c, mh, b.h0, b.h1);
-      dc_mma(c, mh, b.l0, b.l1);
-      dc_mma(c, ml, b.h0, b.h1);
+    next(i);
+    // r += tile (m, n) of matrix `kind` times split rows, or times bf16 rows
+    auto times = [&](float (&r)[4], int kind, int m, int n, const SplitB& b) {
+      const uint4 h4 = mats[(kind * NT + dc_tile(m, n)) * 64], l4 = mats[(kind * NT + dc_tile(m, n)) * 64 + 32];
+      const uint32_t hi[4] = {h4.x, h4.y, h4.z, h4.w}, lo[4] = {l4.x, l4.y, l4.z, l4.w};
+      dc_mma(r, hi, b.h0, b.h1);
+      dc_mma(r, hi, b.l0, b.l1);
+      dc_mma(r, lo, b.h0, b.h1);
     };
-    SplitB b;
-    if (CHANNEL) {
-      uint32_t v0, v1;
-      dc_ldsm2_t(st + lay.values + (lane & 15) * DC_VPITCH + warp * 16, v0, v1);
+    auto times_raw = [&](float (&r)[4], int kind, int m, int n, const uint32_t (&b)[2]) {
+      const uint4 h4 = mats[(kind * NT + dc_tile(m, n)) * 64], l4 = mats[(kind * NT + dc_tile(m, n)) * 64 + 32];
+      const uint32_t hi[4] = {h4.x, h4.y, h4.z, h4.w}, lo[4] = {l4.x, l4.y, l4.z, l4.w};
+      dc_mma(r, hi, b[0], b[1]);
+      dc_mma(r, lo, b[0], b[1]);
+    };
+    float y[M][4], y2[4] = {};                               // y2: the lower left tile's share, a chain of its own
+    SplitB b[M];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        x0[e] += x1[e];
-        o[e] = o0[e] + o1[e];
+    for (int m = 0; m < M; ++m)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[m][e] = 0.f;
+    if (CHANNEL) {
+      uint32_t v[M][2];
+#pragma unroll
+      for (int m = 0; m < M; ++m) dc_ldsm2_t(st + lay.values + (m * DC_TOK + (lane & 15)) * DC_VPITCH + warp * 16, v[m][0], v[m][1]);
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+#pragma unroll
+        for (int q = 0; q <= m; ++q) times_raw(x[m][1], 1, m, q, v[q]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[m][0][e] += x[m][1][e];
+        b[m].from(x[m][0]);
       }
-      mat(2, mh);
-      mat(3, ml);
-      dc_mma(x0, mh, v0, v1);
-      dc_mma(x0, ml, v0, v1);
-      b.from(x0);
-      times(y, 0, b);
-      b.from(y);
-      mat(4, mh);
-      mat(5, ml);
-      dc_mma(o, mh, v0, v1);
-      dc_mma(o, ml, v0, v1);
-      times(o, 6, b);
+#pragma unroll
+      for (int m = 0; m < M; ++m) times(y[m], 0, m, m, b[m]);
+      if (M == 2) times(y2, 0, 1, 0, b[0]);
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        if (m == 1)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[m][e] += y2[e];
+        b[m].from(y[m]);
+      }
+#pragma unroll
+      for (int m = 0; m < M; ++m)
+#pragma unroll
+        for (int q = 0; q <= m; ++q) {
+          times_raw(o[m][0], 2, m, q, v[q]);
+          times(o[m][1], 3, m, q, b[q]);
+        }
+#pragma unroll
+      for (int m = 0; m < M; ++m)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[m][0][e] += o[m][1][e];
       const float* decay = reinterpret_cast<const float*>(smem + so + lay.coef);
 #pragma unroll
       for (int k = 0; k < KS; ++k) {
-        if (k * 16 >= p.dp) break;
+        if (!EXACT && k * 16 >= dp) break;
         const float d0 = decay[k * 16 + g], d1 = decay[k * 16 + g + 8];
         S[k][0] *= d0;
         S[k][1] *= d0;
         S[k][2] *= d1;
         S[k][3] *= d1;
-        uint32_t a[4];
-        dc_ldsm4_t(st + 4 * lay.arr + t_off + k * 32, a);
-        dc_mma(S[k], a, v0, v1);
-        dc_ldsm4_t(st + 5 * lay.arr + t_off + k * 32, a);
-        dc_mma(S[k], a, v0, v1);
-        dc_ldsm4_t(st + 6 * lay.arr + t_off + k * 32, a);
-        dc_mma(S[k], a, b.h0, b.h1);
-        dc_mma(S[k], a, b.l0, b.l1);
-        dc_ldsm4_t(st + 7 * lay.arr + t_off + k * 32, a);
-        dc_mma(S[k], a, b.h0, b.h1);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          const uint32_t at = st + t_off + m * tile + k * 32;
+          uint32_t a[4];
+          dc_ldsm4_t(at + 4 * lay.arr, a);
+          dc_mma(S[k], a, v[m][0], v[m][1]);
+          dc_ldsm4_t(at + 5 * lay.arr, a);
+          dc_mma(S[k], a, v[m][0], v[m][1]);
+          dc_ldsm4_t(at + 6 * lay.arr, a);
+          dc_mma(S[k], a, b[m].h0, b[m].h1);
+          dc_mma(S[k], a, b[m].l0, b[m].l1);
+          dc_ldsm4_t(at + 7 * lay.arr, a);
+          dc_mma(S[k], a, b[m].h0, b[m].h1);
+        }
       }
     } else {
       const float* coef = reinterpret_cast<const float*>(smem + so + lay.coef);
-      const float4 ca = *reinterpret_cast<const float4*>(coef + 4 * g), cb = *reinterpret_cast<const float4*>(coef + 4 * (g + 8));
-      const uint8_t* vp = smem + so + lay.values + g * DC_VPITCH + (warp * 8 + j2) * 2;
-      const float2 va = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp)), vb = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp + 8 * DC_VPITCH));
-      x0[0] = fmaf(ca.y, x0[0] + x1[0], ca.x * va.x);
-      x0[1] = fmaf(ca.y, x0[1] + x1[1], ca.x * va.y);
-      x0[2] = fmaf(cb.y, x0[2] + x1[2], cb.x * vb.x);
-      x0[3] = fmaf(cb.y, x0[3] + x1[3], cb.x * vb.y);
-      b.from(x0);
-      times(y, 0, b);
-      b.from(y);
-      o[0] = ca.z * (o0[0] + o1[0]);
-      o[1] = ca.z * (o0[1] + o1[1]);
-      o[2] = cb.z * (o0[2] + o1[2]);
-      o[3] = cb.z * (o0[3] + o1[3]);
-      times(o, 2, b);
-      y[0] *= ca.w;
-      y[1] *= ca.w;
-      y[2] *= cb.w;
-      y[3] *= cb.w;
-      b.from(y);
-      const float decay = coef[4 * DC_TOK];
+      float4 ca[M], cb[M];                                   // factors of rows g, g + 8
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        ca[m] = *reinterpret_cast<const float4*>(coef + 4 * (m * DC_TOK + g));
+        cb[m] = *reinterpret_cast<const float4*>(coef + 4 * (m * DC_TOK + g + 8));
+        const uint8_t* vp = smem + so + lay.values + (m * DC_TOK + g) * DC_VPITCH + (warp * 8 + j2) * 2;
+        const float2 va = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp)), vb = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp + 8 * DC_VPITCH));
+        float (&x0)[4] = x[m][0];
+        x0[0] = fmaf(ca[m].y, x0[0] + x[m][1][0], ca[m].x * va.x);
+        x0[1] = fmaf(ca[m].y, x0[1] + x[m][1][1], ca[m].x * va.y);
+        x0[2] = fmaf(cb[m].y, x0[2] + x[m][1][2], cb[m].x * vb.x);
+        x0[3] = fmaf(cb[m].y, x0[3] + x[m][1][3], cb[m].x * vb.y);
+        b[m].from(x0);
+      }
+#pragma unroll
+      for (int m = 0; m < M; ++m) times(y[m], 0, m, m, b[m]);
+      if (M == 2) times(y2, 0, 1, 0, b[0]);
+      SplitB w[M];                                           // what is written, with the decays to the chunk's end
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        if (m == 1)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[m][e] += y2[e];
+        const float u[4] = {y[m][0] * ca[m].w, y[m][1] * ca[m].w, y[m][2] * cb[m].w, y[m][3] * cb[m].w};
+        w[m].from(u);
+      }
+      const float decay = coef[4 * C];
 #pragma unroll
       for (int k = 0; k < KS; ++k) {
-        if (k * 16 >= p.dp) break;
+        if (!EXACT && k * 16 >= dp) break;
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[k][e] *= decay;
-        uint32_t a[4];
-        dc_ldsm4_t(st + t_off + k * 32, a);
-        dc_mma(S[k], a, b.h0, b.h1);
-        dc_mma(S[k], a, b.l0, b.l1);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          uint32_t a[4];
+          dc_ldsm4_t(st + t_off + m * tile + k * 32, a);
+          dc_mma(S[k], a, w[m].h0, w[m].h1);
+          dc_mma(S[k], a, w[m].l0, w[m].l1);
+        }
       }
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        b[m].from(y[m]);
+        o[m][0][0] = ca[m].z * (o[m][0][0] + o[m][1][0]);
+        o[m][0][1] = ca[m].z * (o[m][0][1] + o[m][1][1]);
+        o[m][0][2] = cb[m].z * (o[m][0][2] + o[m][1][2]);
+        o[m][0][3] = cb[m].z * (o[m][0][3] + o[m][1][3]);
+      }
+#pragma unroll
+      for (int m = 0; m < M; ++m)
+#pragma unroll
+        for (int q = 0; q <= m; ++q) times(o[m][0], 1, m, q, b[q]);
     }
-    const int t = i * DC_TOK + g;
-    if (t < n) *reinterpret_cast<uint32_t*>(raw + (row0 + t) * p.H * p.vp) = pack_bf16(o[0], o[1]);
-    if (t + 8 < n) *reinterpret_cast<uint32_t*>(raw + (row0 + t + 8) * p.H * p.vp) = pack_bf16(o[2], o[3]);
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+      const int t = i * C + m * DC_TOK + g;
+      if (t < n) *reinterpret_cast<uint32_t*>(out + (row0 + t) * p.H * p.vp) = pack_bf16(o[m][0][0], o[m][0][1]);
+      if (t + 8 < n) *reinterpret_cast<uint32_t*>(out + (row0 + t + 8) * p.H * p.vp) = pack_bf16(o[m][0][2], o[m][0][3]);
+    }
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   if (!used || sout < 0) return;
-  float* dst = p.state + ((long)sout * p.H + h) * p.dp * p.vp + col + j2;
+  float* dst = p.state + ((long)sout * p.H + h) * dp * p.vp + col + j2;
 #pragma unroll
   for (int k = 0; k < KS; ++k)
 #pragma unroll
     for (int e = 0; e < 2; ++e)
-      if (k * 16 < p.dp) *reinterpret_cast<float2*>(dst + (long)(k * 16 + g + 8 * e) * p.vp) = make_float2(S[k][2 * e], S[k][2 * e + 1]);
+      if (EXACT || k * 16 < dp) *reinterpret_cast<float2*>(dst + (long)(k * 16 + g + 8 * e) * p.vp) = make_float2(S[k][2 * e], S[k][2 * e + 1]);
 }
 
-template <bool CHANNEL, int KS>
+template <bool CHANNEL, int KS, bool EXACT, int M>
 static int launch_sequence(const DeltaRule& p, cudaStream_t st) {
-  const DeltaStage lay = delta_stage(p.dp, CHANNEL);
+  const DeltaStage lay = delta_stage<CHANNEL, M>(p.dp);
   const int limit = 226 * 1024;
-  int stages = 4;
-  while (stages > 2 && stages * lay.bytes > (stages == 4 ? 64 : 226) * 1024) --stages;
+  const dim3 grid((p.vp + DC_COLS - 1) / DC_COLS, p.H, p.n_long);
+  // two stages leave room for more blocks on an SM, three hide more of a fetch
+  const int stages = (long)grid.x * grid.y * grid.z <= 2l * sm_count() && 3 * lay.bytes <= limit / (CHANNEL ? 1 : 2) ? 3 : 2;
   const int smem = stages * lay.bytes;
   if (smem > limit) return RC_TOO_LARGE;
   static unsigned long long prep = 0;
-  if (int e = ensure_dynamic_smem((const void*)delta_sequence_kernel<CHANNEL, KS>, limit, prep)) return e;
-  delta_sequence_kernel<CHANNEL, KS><<<dim3((p.vp + DC_COLS - 1) / DC_COLS, p.H, p.n_long), 32 * DC_WARPS, smem, st>>>(p, stages);
+  if (int e = ensure_dynamic_smem((const void*)delta_sequence_kernel<CHANNEL, KS, EXACT, M>, limit, prep)) return e;
+  delta_sequence_kernel<CHANNEL, KS, EXACT, M><<<grid, 32 * DC_WARPS, smem, st>>>(p, stages);
   return (int)cudaGetLastError();
 }
 
-template <bool CHANNEL>
+template <bool CHANNEL, int M>
 static int launch_chunks(const DeltaRule& p, cudaStream_t st) {
-  if (CHANNEL) delta_prepare_channel_kernel<<<dim3(p.n_chunks, (p.H + PC_WARPS - 1) / PC_WARPS), 32 * PC_WARPS, 0, st>>>(p);
-  else delta_prepare_gated_kernel<<<dim3(p.n_chunks, (p.H + 3) / 4), 128, 0, st>>>(p);
+  if (CHANNEL) delta_prepare_channel_kernel<M><<<dim3(p.n_chunks, p.H), 32 * M, 0, st>>>(p);
+  else delta_prepare_gated_kernel<M><<<dim3(p.n_chunks, (p.H * M + 3) / 4), 128, 0, st>>>(p);
   if (int e = (int)cudaGetLastError()) return e;
-  if (p.dp <= 64) return launch_sequence<CHANNEL, 4>(p, st);
-  if (p.dp <= 128) return launch_sequence<CHANNEL, 8>(p, st);
-  return launch_sequence<CHANNEL, 16>(p, st);
+  if constexpr (M == 1) {
+    return launch_sequence<CHANNEL, 16, false, 1>(p, st);
+  } else {
+    switch (p.dp) {
+      case 64: return launch_sequence<CHANNEL, 4, true, 2>(p, st);
+      case 96: return launch_sequence<CHANNEL, 6, true, 2>(p, st);
+      case 128: return launch_sequence<CHANNEL, 8, true, 2>(p, st);
+      default: break;
+    }
+    if (p.dp <= 128) return launch_sequence<CHANNEL, 8, false, 2>(p, st);
+    if constexpr (CHANNEL) return RC_TOO_LARGE;
+    else return launch_sequence<CHANNEL, 16, false, 2>(p, st);
+  }
 }
 
 }  // namespace omni
 
 using namespace omni;
 
-// Portions of more than one row (`chunks`, `long_list`); results before their norm go to `raw`.
-extern "C" int omni_delta_chunks(const DeltaRule* args, int channel, void* stream) {
+// Portions of more than one row (`chunks` of 32 tokens, channel also 16; `long_list`); results before their norm go to `raw`.
+extern "C" int omni_delta_chunks(const DeltaRule* args, int channel, int chunk, void* stream) {
   const DeltaRule& p = *args;
   if (p.n_chunks <= 0 || p.n_long <= 0) return RC_OK;
-  if (!delta_args_ok(p, channel) || !p.chunks || !p.long_list || !p.raw || !p.mats || !p.coef || p.dp > 256 || p.n_long > 65535)
+  if (!delta_args_ok(p, channel) || !p.chunks || !p.long_list || !p.raw || !p.mats || !p.coef || p.dp > 256 || p.n_long > 65535 ||
+      chunk != 32 && !(channel && chunk == 16))
     return RC_BAD_ARG;
   if (channel ? !p.tiles : (!p.u || (p.ldu & 7) || p.ldu < 2l * p.G * p.dp + (long)p.H * p.vp)) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
-  return channel ? launch_chunks<true>(p, st) : launch_chunks<false>(p, st);
+  if (!channel) return launch_chunks<false, 2>(p, st);
+  return chunk == 16 ? launch_chunks<true, 1>(p, st) : launch_chunks<true, 2>(p, st);
 }

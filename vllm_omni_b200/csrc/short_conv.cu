@@ -25,6 +25,17 @@ struct ConvRows {
   int* status;
 };
 
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 template <int TAPS>
 __global__ void __launch_bounds__(256)
 conv_rows_kernel(const ConvRows p) {
@@ -44,6 +55,8 @@ conv_rows_kernel(const ConvRows p) {
     if (ctx + b >= 0) return *reinterpret_cast<const uint4*>(hist + ((long)sin * h + h + b) * p.C);
     return zero;
   };
+  // portions are contiguous: rows that begin and end in the same one need no look at those between
+  const int s_first = min(max(p.row_seq[r0], 0), p.num_seqs - 1), s_last = min(max(p.row_seq[min(r0 + RUN, (long)p.T) - 1], 0), p.num_seqs - 1);
   uint4 raw[RUN], win[H];
   float w[TAPS > 0 ? TAPS : 1][8], bias[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
   if (p.bias) load8<float>(p.bias + c, bias);
@@ -57,7 +70,7 @@ conv_rows_kernel(const ConvRows p) {
   for (int i = 0; i < RUN; ++i) {
     const long row = r0 + i;
     if (row >= p.T) break;
-    const int s = min(max(p.row_seq[row], 0), p.num_seqs - 1);
+    const int s = i == 0 || s_first == s_last ? s_first : min(max(p.row_seq[row], 0), p.num_seqs - 1);
     if (s != seq) {                                          // first row of the run or of a sequence
       seq = s;
       q0 = p.q_start[seq];
@@ -105,7 +118,7 @@ conv_rows_kernel(const ConvRows p) {
     }
     if (p.act == 1) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) o[e] = __fdividef(o[e], 1.0f + __expf(-o[e]));
+      for (int e = 0; e < 8; ++e) o[e] *= rcp_approx(1.0f + ex2_approx(-1.4426950408889634f * o[e]));
     }
     store8<bf16>(static_cast<bf16*>(p.out) + row * p.C + c, o);
     if (row == q1 - 1 && sout >= 0 && !(p.skip_single && q1 - q0 == 1))

@@ -7,7 +7,7 @@
                channel; o / rms(o) * gain * sigmoid(gate)
 
 Kernels: csrc/delta_rule.cu (token by token: decoded tokens in one launch; every row in the exact mode and for sizes the
-others do not take), csrc/delta_chunks.cu (prompt portions in chunks of 16 tokens on tensor cores).  Convolution history
+others do not take), csrc/delta_chunks.cu (prompt portions in chunks of 32 tokens on tensor cores).  Convolution history
 and state live in the runner's pools.  CPU tensors take a PyTorch restatement."""
 from __future__ import annotations
 
@@ -22,8 +22,7 @@ from .short_conv import conv_rows
 
 c_int, c_long, c_float, c_void_p = ctypes.c_int, ctypes.c_long, ctypes.c_float, ctypes.c_void_p
 
-CHUNK = 16               # tokens the chunked kernels take at a time
-MAX_DIM = 256            # key channels they take
+MAX_DIM = 256            # key channels the chunked kernels take
 
 
 @dataclass(frozen=True)
@@ -95,9 +94,15 @@ class _Delta(ctypes.Structure):
                 ("tiles", c_void_p), ("status", c_void_p)]
 
 
-def _chunked(s: DeltaShape, rule, proj) -> bool:
-    """Do the chunked kernels take this?  A chunk's decays are undone within it, so their product must stay in range."""
-    return proj.dtype == torch.bfloat16 and s.dp <= MAX_DIM and (not rule.channel or -rule.decay_scale * CHUNK <= 40.0)
+def _chunk(s: DeltaShape, rule, proj) -> int:
+    """Tokens the chunked kernels take at a time, 0 where they do not take this.  Decays per channel are undone within a
+    chunk, so their product must stay in range; their operands fill shared memory."""
+    if proj.dtype != torch.bfloat16 or s.dp > MAX_DIM:
+        return 0
+    if not rule.channel:
+        return 32
+    n = 32 if s.dp <= 128 else 16
+    return n if -rule.decay_scale * n <= 40.0 else 0
 
 
 def delta_rule(proj, s: DeltaShape, seqs, rule, state, out, *, hist=None, decay=None, impl: str | None = None):
@@ -132,7 +137,8 @@ def delta_rule(proj, s: DeltaShape, seqs, rule, state, out, *, hist=None, decay=
     a.status = P(nv.status_word(proj.device))
     bf, kind, st = c_int(proj.dtype == torch.bfloat16), c_int(rule.channel), nv.stream_ptr()
     lib = nv.lib("delta_rule")
-    chunked = seqs.n_decode < seqs.n_seqs and impl != "steps" and _chunked(s, rule, proj)
+    size = _chunk(s, rule, proj) if seqs.n_decode < seqs.n_seqs and impl != "steps" else 0
+    chunked = size > 0
     wide = s.dp * s.vp > 16384                              # a head's state does not fit the registers of one block
     raw = torch.empty(T, s.v_cols, dtype=proj.dtype, device=proj.device) if chunked or wide else None
     a.raw = P(raw)
@@ -141,19 +147,20 @@ def delta_rule(proj, s: DeltaShape, seqs, rule, state, out, *, hist=None, decay=
         a.seq_list = P(seqs.decode_list) if chunked else 0  # none: every sequence
         nv.check_rc(lib.omni_delta_steps(ctypes.byref(a), kind, bf, c_int(wide), st), "omni_delta_steps")
     if chunked:
-        chunks = seqs.chunks(CHUNK)
+        chunks = seqs.chunks(size)
         a.chunks, a.n_chunks, a.long_list, a.n_long = P(chunks.table), chunks.n, P(chunks.seqs), chunks.n_seqs
         dev, n = proj.device, chunks.n * s.heads
+        lower = 512 * (3 if size == 32 else 1)              # lower tiles of a chunk's matrix, high and low parts
         if rule.channel:
-            mats, coef = torch.empty(n, 8 * 256, dtype=torch.bfloat16, device=dev), torch.empty(n, s.dp, device=dev)
-            tiles = torch.empty(n, 8, CHUNK, s.dp, dtype=torch.bfloat16, device=dev)
+            mats, coef = torch.empty(n, 4 * lower, dtype=torch.bfloat16, device=dev), torch.empty(n, s.dp, device=dev)
+            tiles = torch.empty(n, 8, size, s.dp, dtype=torch.bfloat16, device=dev)
             a.tiles = P(tiles)
         else:
-            mats, coef = torch.empty(n, 4 * 256, dtype=torch.bfloat16, device=dev), torch.empty(n, 4 * CHUNK + 4, device=dev)
+            mats, coef = torch.empty(n, 2 * lower, dtype=torch.bfloat16, device=dev), torch.empty(n, 4 * size + 4, device=dev)
             u = conv_rows(proj, seqs, s.taps, s.channels, rule.conv, hist, act="silu", skip_single=True)
             a.u, a.ldu = P(u), u.stride(0)
         a.mats, a.coef = P(mats), P(coef)
-        nv.check_rc(nv.lib("delta_chunks").omni_delta_chunks(ctypes.byref(a), kind, st), "omni_delta_chunks")
+        nv.check_rc(nv.lib("delta_chunks").omni_delta_chunks(ctypes.byref(a), kind, c_int(size), st), "omni_delta_chunks")
     if raw is not None:
         # rows of single tokens are finished already unless their state was too wide
         nv.check_rc(lib.omni_delta_finish(ctypes.byref(a), kind, bf, c_int(not wide), st), "omni_delta_finish")
