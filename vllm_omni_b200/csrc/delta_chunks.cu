@@ -11,9 +11,9 @@
 //
 //   prepare   a warp per 16 tokens of a (chunk, head), all chunks at once: the lower tiles (16 x 16) of the matrices and of
 //             T = (I + A)^-1, left in memory as tensor-core operands; gated: the tokens' factors; channel: the decayed rows
-//   sequence  one block per (portion, head, 32 value columns); a warp owns eight columns of the state, in registers from the
-//             first chunk to the last, and walks the chunks without talking to the others; operands come through a
-//             cp.async ring that the block shares
+//   sequence  one block per (portion, head, 32 or 16 value columns); a warp (or two, see there) owns eight columns of the
+//             state, in registers from the first chunk to the last, and walks the chunks; operands come through a ring of
+//             TMA copies that the block shares.  Every wait is bounded
 //
 // Everything that is not a GEMM's or convolution's bf16 result keeps fp32 precision on the way through the tensor cores: such
 // an operand is two bf16 numbers, high and low part, and a product of two of them three products (16 bits and more of
@@ -26,8 +26,7 @@ namespace omni {
 typedef __nv_bfloat16 bf16;
 
 constexpr int DC_TOK = 16;             // tokens of a tile; a chunk is one or two tiles
-constexpr int DC_COLS = 32;            // value columns per block of the sequence kernel
-constexpr int DC_WARPS = 4;
+constexpr int DC_WARPS = 4;            // of the sequence kernel (and one that copies, where two share columns)
 
 __device__ __forceinline__ void dc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
@@ -52,8 +51,10 @@ __device__ __forceinline__ uint32_t dc_trans(uint32_t x) {
   asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
   return y;
 }
-__device__ __forceinline__ void dc_copy16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+__device__ __forceinline__ void dc_bulk(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes),
+               "r"(bar)
+               : "memory");
 }
 // two numbers as pairs of bf16: high parts, and what the high parts leave
 __device__ __forceinline__ void dc_split(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -317,7 +318,7 @@ delta_prepare_channel_kernel(const DeltaRule p) {
   const bf16* proj = static_cast<const bf16*>(p.proj) + (long)h * p.dp;
   const bf16* z = static_cast<const bf16*>(p.z) + (long)h * p.dp;
   const long at = (long)blockIdx.x * p.H + h;
-  const int tile = C * (p.dp / 2);                           // channel pairs of an operand
+  const int pitch = p.dp / 2 + 4, tile = C * pitch;          // channel pairs of a row (padded as in shared memory), of an operand
   uint32_t* tiles = static_cast<uint32_t*>(p.tiles) + at * (8 * tile);
   uint4* mats = static_cast<uint4*>(p.mats) + at * (4 * NT * 64);
   // two channels of the tile's token t (past the end: another token's, not used)
@@ -397,7 +398,7 @@ delta_prepare_channel_kernel(const DeltaRule p) {
       const int tok = m * DC_TOK + t;
       uint32_t hi, lo;
       uint32_t* dst = s_rows + tok * ROW32 + lane;
-      uint32_t* out = tiles + tok * (p.dp / 2) + c / 2;
+      uint32_t* out = tiles + tok * pitch + c / 2;
       auto put = [&](int x, float2 v, bool shared, int global) {           // a pair of channels of operand x, high and low parts
         dc_split(v.x, v.y, hi, lo);
         if (shared) {
@@ -482,304 +483,389 @@ delta_prepare_channel_kernel(const DeltaRule p) {
 }
 
 // ----------------------------------------------------------------------------------- sequence
-constexpr int DC_VPITCH = DC_COLS * 2 + 16;
-
-// Bytes of a stage: rows of the operands (gated: k, q; channel: eight), values, matrices, factors
+// Bytes of a stage: rows of the operands, values, matrices, factors.  Gated: k, then q, in boxes of 64 channels of all
+// tokens, 128-byte swizzle.  Channel: eight operands as prepared, rows of `pitch` bytes (an odd multiple of 16:
+// conflict-free ldmatrix).
 struct DeltaStage {
   int pitch, arr, values, mats, coef, bytes;
 };
-template <bool CHANNEL, int M>
+template <bool CHANNEL, int M, int COLS>
 __host__ __device__ __forceinline__ DeltaStage delta_stage(int dp) {
   DeltaStage s;
-  s.pitch = dp * 2 + 16;               // an odd multiple of 16 bytes: conflict-free ldmatrix
-  s.arr = M * DC_TOK * s.pitch;
-  s.values = (CHANNEL ? 8 : 2) * s.arr;
-  s.mats = s.values + M * DC_TOK * DC_VPITCH;
+  s.pitch = CHANNEL ? dp * 2 + 16 : 128;
+  s.arr = M * DC_TOK * (CHANNEL ? s.pitch : (dp + 63) / 64 * 128);
+  s.values = ((CHANNEL ? 8 : 2) * s.arr + 127) / 128 * 128;
+  s.mats = s.values + M * DC_TOK * COLS * 2;
   s.coef = s.mats + (CHANNEL ? 4 : 2) * dc_tiles<M>() * 1024;
-  s.bytes = s.coef + (CHANNEL ? dp * 4 : (4 * M * DC_TOK + 4) * 4);
+  s.bytes = (s.coef + (CHANNEL ? dp * 4 : (4 * M * DC_TOK + 4) * 4) + 1023) / 1024 * 1024;
   return s;
 }
 
 // KS: 16-channel steps of the key channels that the state's registers hold.  EXACT: dp = 16 KS, so that a chunk's products
-// are straight-line code; otherwise dp <= 16 KS.  M: tiles of 16 tokens in a chunk.
-template <bool CHANNEL, int KS, bool EXACT, int M>
-__global__ void __launch_bounds__(32 * DC_WARPS)
-delta_sequence_kernel(const DeltaRule p, const int stages) {
-  constexpr int C = M * DC_TOK, NT = dc_tiles<M>();
-  extern __shared__ __align__(16) uint8_t smem[];
+// are straight-line code; otherwise dp <= 16 KS.  M: tiles of 16 tokens in a chunk.  SPLIT = 2: two warps share eight
+// columns, each has half of the key channels; they add up what the state answers in shared memory, and each finishes the
+// output of one token tile.  For few portions and heads, where the chain of a chunk's products is what takes the time.
+template <bool CHANNEL, int KS, bool EXACT, int M, int SPLIT>
+__global__ void __launch_bounds__(32 * (DC_WARPS + SPLIT - 1), SPLIT == 1 && KS <= 8 ? 4 : 1)
+delta_sequence_kernel(const __grid_constant__ CUtensorMap tmU, const __grid_constant__ CUtensorMap tmV,
+                      const __grid_constant__ DeltaRule p, const int stages) {
+  constexpr int C = M * DC_TOK, NT = dc_tiles<M>(), GROUPS = DC_WARPS / SPLIT, COLS = 8 * GROUPS, VPITCH = COLS * 2;
+  constexpr int KW = KS / SPLIT, NM = (CHANNEL ? 4 : 2) * NT * 64;
+  static_assert(SPLIT == 1 || (SPLIT == 2 && M == 2), "a warp of a pair finishes one tile");
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ __align__(8) uint64_t full[3], empty[3];
+  __shared__ __align__(16) float4 s_ex[SPLIT == 2 ? 2 : 1][DC_WARPS][3][SPLIT == 2 ? 32 : 1];
+  __shared__ int s_abort;
   const int dp = EXACT ? 16 * KS : p.dp;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, j2 = (lane & 3) * 2;
   const int seq = min(max(p.long_list[2 * blockIdx.z], 0), p.num_seqs - 1), first = p.long_list[2 * blockIdx.z + 1];
-  const int h = blockIdx.y, col0 = blockIdx.x * DC_COLS, hk = h / (p.H / p.G);
+  const int h = blockIdx.y, col0 = blockIdx.x * COLS, hk = h / (p.H / p.G);
   const long row0 = p.q_start[seq];
   const int n = (int)(p.q_start[seq + 1] - row0);
   const int n_chunks = min((n + C - 1) / C, p.n_chunks - first);
-  const DeltaStage lay = delta_stage<CHANNEL, M>(dp);
-  const uint32_t base = smem_u32(smem);
-  const int vecs = dp / 8, v_vecs = min(DC_COLS, p.vp - col0) / 8;
+  const DeltaStage lay = delta_stage<CHANNEL, M, COLS>(dp);
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  const uint8_t* smem = smem_raw + (base - smem_u32(smem_raw));
+  if (tid == 0) {
+    s_abort = 0;
+    tma_prefetch_desc(&tmU);
+    tma_prefetch_desc(&tmV);
+    for (int i = 0; i < 3; ++i) {
+      mbar_init(smem_u32(&full[i]), 1);
+      mbar_init(smem_u32(&empty[i]), DC_WARPS);
+    }
+    fence_mbar_init();
+  }
+  __syncthreads();
 
-  auto fetch = [&](int i) {
-    const uint32_t st = base + (i % stages) * lay.bytes;
+  // the copies of chunk i (one thread); rows past the portion's end are another's or zero: finite, and their factors are zero
+  auto copy = [&](int i) {
+    const int slot = i % stages, boxes = (dp + 63) / 64, row = (int)row0 + i * C;
+    const uint32_t bar = smem_u32(&full[slot]), dst = base + slot * lay.bytes;
+    const uint32_t f_bytes = CHANNEL ? dp * 4 : (4 * C + 4) * 4;
     const long at = (long)(first + i) * p.H + h;
-    auto row = [&](int t) { return row0 + min(i * C + t, n - 1); };        // past the end: finite, its factors are zero
+    mbar_wait(smem_u32(&empty[slot]), ((i / stages) & 1) ^ 1, &s_abort, p.status, ERR_WAIT_EMPTY);
+    mbar_expect_tx(bar, (CHANNEL ? 8 : 2) * lay.arr + C * VPITCH + NM * 16 + f_bytes);
     if (CHANNEL) {
-      const uint4* src = static_cast<const uint4*>(p.tiles) + at * (8 * C * vecs);
-      for (int x = tid; x < 8 * C * vecs; x += 32 * DC_WARPS) dc_copy16(st + (x / vecs) * lay.pitch + (x % vecs) * 16, src + x);
+      dc_bulk(dst, static_cast<const uint8_t*>(p.tiles) + at * (8 * lay.arr), 8 * lay.arr, bar);
     } else {
-      const bf16* u = static_cast<const bf16*>(p.u) + hk * dp;
-      for (int x = tid; x < 2 * C * vecs; x += 32 * DC_WARPS) {
-        const int r = x / vecs, c = x - r * vecs;            // rows of k, then of q
-        dc_copy16(st + r * lay.pitch + c * 16, u + row(r & (C - 1)) * p.ldu + (r < C ? p.G * dp : 0) + c * 8);
-      }
+      for (int x = 0; x < boxes; ++x) tma_load_2d(dst + x * C * 128, &tmU, bar, (p.G + hk) * dp + 64 * x, row);
+      for (int x = 0; x < boxes; ++x) tma_load_2d(dst + lay.arr + x * C * 128, &tmU, bar, hk * dp + 64 * x, row);
     }
-    const bf16* v = CHANNEL ? static_cast<const bf16*>(p.proj) + p.v_col : static_cast<const bf16*>(p.u) + 2 * p.G * dp;
-    const long ldv = CHANNEL ? p.ldp : p.ldu;
-    for (int x = tid; x < C * (DC_COLS / 8); x += 32 * DC_WARPS) {
-      const int r = x / (DC_COLS / 8), c = x % (DC_COLS / 8);
-      if (c < v_vecs) dc_copy16(st + lay.values + r * DC_VPITCH + c * 16, v + row(r) * ldv + (long)h * p.vp + col0 + c * 8);
-    }
-    constexpr int nm = (CHANNEL ? 4 : 2) * NT * 64;
-    const uint4* mats = static_cast<const uint4*>(p.mats) + at * nm;
-#pragma unroll
-    for (int x = 0; x < nm; x += 32 * DC_WARPS) dc_copy16(st + lay.mats + (x + tid) * 16, mats + x + tid);
-    const int nf = CHANNEL ? dp / 4 : C + 1;
-    for (int x = tid; x < nf; x += 32 * DC_WARPS) dc_copy16(st + lay.coef + x * 16, reinterpret_cast<const float4*>(p.coef) + at * nf + x);
+    tma_load_2d(dst + lay.values, &tmV, bar, h * p.vp + col0, row);
+    dc_bulk(dst + lay.mats, static_cast<const uint4*>(p.mats) + at * NM, NM * 16, bar);
+    dc_bulk(dst + lay.coef, reinterpret_cast<const uint8_t*>(p.coef) + at * f_bytes, f_bytes, bar);
   };
 
-  int sin, sout;
-  delta_rows(p, seq, sin, sout);
-  const int col = col0 + warp * 8;                           // this warp's columns
-  const bool used = col < p.vp;
-  float S[KS][4];                                            // rows g, g + 8 of 16 key channels, columns j2, j2 + 1
-  {
-    const float* src = p.state + ((long)sin * p.H + h) * dp * p.vp + col + j2;
-    const bool have = used && p.context[seq] > 0;
+  if (SPLIT == 2 && warp == DC_WARPS) {                      // a warp of its own where the chain of products counts
+    if (elect_one())
+      for (int i = 0; i < n_chunks; ++i) copy(i);
+  } else {
+    if (SPLIT == 1 && warp == 0 && elect_one())
+      for (int i = 0; i < min(stages - 1, n_chunks); ++i) copy(i);
+    __syncwarp();
+    int sin, sout;
+    delta_rows(p, seq, sin, sout);
+    const int grp = warp % GROUPS, kh = warp / GROUPS, k0 = kh * KW;
+    const int col = col0 + grp * 8;                          // this warp's columns
+    const bool used = col < p.vp;
+    float S[KW][4];                                          // rows g, g + 8 of 16 key channels, columns j2, j2 + 1
+    {
+      const float* src = p.state + ((long)sin * p.H + h) * dp * p.vp + col + j2;
+      const bool have = used && p.context[seq] > 0;
 #pragma unroll
-    for (int k = 0; k < KS; ++k)
+      for (int k = 0; k < KW; ++k)
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int r = k * 16 + g + 8 * e;
-        const float2 v = have && (EXACT || k * 16 < dp) ? *reinterpret_cast<const float2*>(src + (long)r * p.vp) : make_float2(0.f, 0.f);
-        S[k][2 * e] = v.x;
-        S[k][2 * e + 1] = v.y;
-      }
-  }
-  for (int i = 0; i < stages - 1; ++i) {
-    if (i < n_chunks) fetch(i);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  }
-  auto next = [&](int i) {                                   // into the place of chunk i - 1
-    if (i + stages - 1 < n_chunks) fetch(i + stages - 1);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  bf16* out = static_cast<bf16*>(p.raw) + (long)h * p.vp + col + j2;
-  const uint32_t a_off = ((lane & 7) + ((lane >> 3) & 1) * 8) * lay.pitch + (lane >> 4) * 16;      // tokens x channels
-  const uint32_t t_off = ((lane & 7) + (lane >> 4) * 8) * lay.pitch + ((lane >> 3) & 1) * 16;      // channels x tokens
-  const uint32_t tile = DC_TOK * lay.pitch;
-  for (int i = 0; i < n_chunks; ++i) {
-    if (stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
-    else asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                         // chunk i is here, chunk i - 1 is done with
-    if (!used) {
-      next(i);
-      continue;
+        for (int e = 0; e < 2; ++e) {
+          const int r = (k0 + k) * 16 + g + 8 * e;
+          const float2 v = have && (EXACT || (k0 + k) * 16 < dp) ? *reinterpret_cast<const float2*>(src + (long)r * p.vp) : make_float2(0.f, 0.f);
+          S[k][2 * e] = v.x;
+          S[k][2 * e + 1] = v.y;
+        }
     }
-    const int so = (i % stages) * lay.bytes;
-    const uint32_t st = base + so;
-    const uint4* mats = reinterpret_cast<const uint4*>(smem + so + lay.mats) + lane;
-    // what the state gives for the chunk's keys (x) and queries (o)
-    float x[M][2][4] = {}, o[M][2][4] = {};
-#pragma unroll
-    for (int k = 0; k < KS; ++k) {
-      if (!EXACT && k * 16 >= dp) break;
-      SplitB s;
-      s.from(S[k]);
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-        uint32_t a[4];
-        dc_ldsm4(st + a_off + m * tile + k * 32, a);
-        dc_mma(x[m][0], a, s.h0, s.h1);
-        dc_mma(x[m][1], a, s.l0, s.l1);
-        if (CHANNEL) {
-          dc_ldsm4(st + lay.arr + a_off + m * tile + k * 32, a);
-          dc_mma(x[m][1], a, s.h0, s.h1);
-        }
-      }
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-        uint32_t a[4];
-        dc_ldsm4(st + (CHANNEL ? 2 : 1) * lay.arr + a_off + m * tile + k * 32, a);
-        dc_mma(o[m][0], a, s.h0, s.h1);
-        dc_mma(o[m][1], a, s.l0, s.l1);
-        if (CHANNEL) {
-          dc_ldsm4(st + 3 * lay.arr + a_off + m * tile + k * 32, a);
-          dc_mma(o[m][1], a, s.h0, s.h1);
-        }
-      }
-    }
-    next(i);
-    // r += tile (m, n) of matrix `kind` times split rows, or times bf16 rows
-    auto times = [&](float (&r)[4], int kind, int m, int n, const SplitB& b) {
-      const uint4 h4 = mats[(kind * NT + dc_tile(m, n)) * 64], l4 = mats[(kind * NT + dc_tile(m, n)) * 64 + 32];
-      const uint32_t hi[4] = {h4.x, h4.y, h4.z, h4.w}, lo[4] = {l4.x, l4.y, l4.z, l4.w};
-      dc_mma(r, hi, b.h0, b.h1);
-      dc_mma(r, hi, b.l0, b.l1);
-      dc_mma(r, lo, b.h0, b.h1);
+    bf16* out = static_cast<bf16*>(p.raw) + row0 * p.H * p.vp + (long)h * p.vp + col + j2;
+    // where a lane's 16 bytes of a 16 x 16 operand are: tokens x channels, and channels x tokens (transposed on the way)
+    const uint32_t a_row = ((lane & 7) + ((lane >> 3) & 1) * 8) * lay.pitch, t_row = ((lane & 7) + (lane >> 4) * 8) * lay.pitch;
+    const uint32_t a_vec = (CHANNEL ? lane >> 4 : (lane >> 4) ^ (lane & 7)) * 16;
+    const uint32_t t_vec = (CHANNEL ? (lane >> 3) & 1 : ((lane >> 3) & 1) ^ (lane & 7)) * 16;
+    auto place = [&](uint32_t row, uint32_t vec, int arr, int m, int k) {
+      const uint32_t at = row + arr * lay.arr + m * DC_TOK * lay.pitch;
+      k += k0;
+      return CHANNEL ? at + vec + k * 32 : at + (k >> 2) * (C * 128) + (vec ^ ((k & 3) * 32));
     };
-    auto times_raw = [&](float (&r)[4], int kind, int m, int n, const uint32_t (&b)[2]) {
-      const uint4 h4 = mats[(kind * NT + dc_tile(m, n)) * 64], l4 = mats[(kind * NT + dc_tile(m, n)) * 64 + 32];
-      const uint32_t hi[4] = {h4.x, h4.y, h4.z, h4.w}, lo[4] = {l4.x, l4.y, l4.z, l4.w};
-      dc_mma(r, hi, b[0], b[1]);
-      dc_mma(r, lo, b[0], b[1]);
-    };
-    float y[M][4], y2[4] = {};                               // y2: the lower left tile's share, a chain of its own
-    SplitB b[M];
-#pragma unroll
-    for (int m = 0; m < M; ++m)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) y[m][e] = 0.f;
-    if (CHANNEL) {
-      uint32_t v[M][2];
-#pragma unroll
-      for (int m = 0; m < M; ++m) dc_ldsm2_t(st + lay.values + (m * DC_TOK + (lane & 15)) * DC_VPITCH + warp * 16, v[m][0], v[m][1]);
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-#pragma unroll
-        for (int q = 0; q <= m; ++q) times_raw(x[m][1], 1, m, q, v[q]);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) x[m][0][e] += x[m][1][e];
-        b[m].from(x[m][0]);
+    auto at_a = [&](int arr, int m, int k) { return place(a_row, a_vec, arr, m, k); };
+    auto at_t = [&](int arr, int m, int k) { return place(t_row, t_vec, arr, m, k); };
+    int stage = 0;
+    uint32_t ph = 0;
+    for (int i = 0; i < n_chunks; ++i) {
+      mbar_wait(smem_u32(&full[stage]), ph, &s_abort, p.status, ERR_WAIT_FULL);
+      const int so = stage * lay.bytes;
+      const uint32_t bar = smem_u32(&empty[stage]);
+      if (++stage == stages) {
+        stage = 0;
+        ph ^= 1;
       }
-#pragma unroll
-      for (int m = 0; m < M; ++m) times(y[m], 0, m, m, b[m]);
-      if (M == 2) times(y2, 0, 1, 0, b[0]);
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-        if (m == 1)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) y[m][e] += y2[e];
-        b[m].from(y[m]);
+      if (!used) {
+        if (lane == 0) mbar_arrive(bar);
+        continue;
       }
+      const uint32_t st = base + so;
+      const uint4* mats = reinterpret_cast<const uint4*>(smem + so + lay.mats) + lane;
+      // what the state gives for the chunk's keys (x) and queries (o)
+      float x[M][2][4] = {}, o[M][2][4] = {};
 #pragma unroll
-      for (int m = 0; m < M; ++m)
-#pragma unroll
-        for (int q = 0; q <= m; ++q) {
-          times_raw(o[m][0], 2, m, q, v[q]);
-          times(o[m][1], 3, m, q, b[q]);
-        }
-#pragma unroll
-      for (int m = 0; m < M; ++m)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) o[m][0][e] += o[m][1][e];
-      const float* decay = reinterpret_cast<const float*>(smem + so + lay.coef);
-#pragma unroll
-      for (int k = 0; k < KS; ++k) {
-        if (!EXACT && k * 16 >= dp) break;
-        const float d0 = decay[k * 16 + g], d1 = decay[k * 16 + g + 8];
-        S[k][0] *= d0;
-        S[k][1] *= d0;
-        S[k][2] *= d1;
-        S[k][3] *= d1;
-#pragma unroll
-        for (int m = 0; m < M; ++m) {
-          const uint32_t at = st + t_off + m * tile + k * 32;
-          uint32_t a[4];
-          dc_ldsm4_t(at + 4 * lay.arr, a);
-          dc_mma(S[k], a, v[m][0], v[m][1]);
-          dc_ldsm4_t(at + 5 * lay.arr, a);
-          dc_mma(S[k], a, v[m][0], v[m][1]);
-          dc_ldsm4_t(at + 6 * lay.arr, a);
-          dc_mma(S[k], a, b[m].h0, b[m].h1);
-          dc_mma(S[k], a, b[m].l0, b[m].l1);
-          dc_ldsm4_t(at + 7 * lay.arr, a);
-          dc_mma(S[k], a, b[m].h0, b[m].h1);
-        }
-      }
-    } else {
-      const float* coef = reinterpret_cast<const float*>(smem + so + lay.coef);
-      float4 ca[M], cb[M];                                   // factors of rows g, g + 8
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-        ca[m] = *reinterpret_cast<const float4*>(coef + 4 * (m * DC_TOK + g));
-        cb[m] = *reinterpret_cast<const float4*>(coef + 4 * (m * DC_TOK + g + 8));
-        const uint8_t* vp = smem + so + lay.values + (m * DC_TOK + g) * DC_VPITCH + (warp * 8 + j2) * 2;
-        const float2 va = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp)), vb = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp + 8 * DC_VPITCH));
-        float (&x0)[4] = x[m][0];
-        x0[0] = fmaf(ca[m].y, x0[0] + x[m][1][0], ca[m].x * va.x);
-        x0[1] = fmaf(ca[m].y, x0[1] + x[m][1][1], ca[m].x * va.y);
-        x0[2] = fmaf(cb[m].y, x0[2] + x[m][1][2], cb[m].x * vb.x);
-        x0[3] = fmaf(cb[m].y, x0[3] + x[m][1][3], cb[m].x * vb.y);
-        b[m].from(x0);
-      }
-#pragma unroll
-      for (int m = 0; m < M; ++m) times(y[m], 0, m, m, b[m]);
-      if (M == 2) times(y2, 0, 1, 0, b[0]);
-      SplitB w[M];                                           // what is written, with the decays to the chunk's end
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-        if (m == 1)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) y[m][e] += y2[e];
-        const float u[4] = {y[m][0] * ca[m].w, y[m][1] * ca[m].w, y[m][2] * cb[m].w, y[m][3] * cb[m].w};
-        w[m].from(u);
-      }
-      const float decay = coef[4 * C];
-#pragma unroll
-      for (int k = 0; k < KS; ++k) {
-        if (!EXACT && k * 16 >= dp) break;
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[k][e] *= decay;
+      for (int k = 0; k < KW; ++k) {
+        if (!EXACT && (k0 + k) * 16 >= dp) break;
+        SplitB s;
+        s.from(S[k]);
 #pragma unroll
         for (int m = 0; m < M; ++m) {
           uint32_t a[4];
-          dc_ldsm4_t(st + t_off + m * tile + k * 32, a);
-          dc_mma(S[k], a, w[m].h0, w[m].h1);
-          dc_mma(S[k], a, w[m].l0, w[m].l1);
+          dc_ldsm4(st + at_a(0, m, k), a);
+          dc_mma(x[m][0], a, s.h0, s.h1);
+          dc_mma(x[m][1], a, s.l0, s.l1);
+          if (CHANNEL) {
+            dc_ldsm4(st + at_a(1, m, k), a);
+            dc_mma(x[m][1], a, s.h0, s.h1);
+          }
         }
-      }
 #pragma unroll
-      for (int m = 0; m < M; ++m) {
-        b[m].from(y[m]);
-        o[m][0][0] = ca[m].z * (o[m][0][0] + o[m][1][0]);
-        o[m][0][1] = ca[m].z * (o[m][0][1] + o[m][1][1]);
-        o[m][0][2] = cb[m].z * (o[m][0][2] + o[m][1][2]);
-        o[m][0][3] = cb[m].z * (o[m][0][3] + o[m][1][3]);
+        for (int m = 0; m < M; ++m) {
+          uint32_t a[4];
+          dc_ldsm4(st + at_a(CHANNEL ? 2 : 1, m, k), a);
+          dc_mma(o[m][0], a, s.h0, s.h1);
+          dc_mma(o[m][1], a, s.l0, s.l1);
+          if (CHANNEL) {
+            dc_ldsm4(st + at_a(3, m, k), a);
+            dc_mma(o[m][1], a, s.h0, s.h1);
+          }
+        }
       }
 #pragma unroll
       for (int m = 0; m < M; ++m)
 #pragma unroll
-        for (int q = 0; q <= m; ++q) times(o[m][0], 1, m, q, b[q]);
-    }
+        for (int e = 0; e < 4; ++e) {
+          x[m][0][e] += x[m][1][e];
+          o[m][0][e] += o[m][1][e];
+          x[m][1][e] = o[m][1][e] = 0.f;
+        }
+      if constexpr (SPLIT == 2) {
+        auto as4 = [](const float (&v)[4]) { return make_float4(v[0], v[1], v[2], v[3]); };
+        float4(*mine)[32] = s_ex[i & 1][warp], (*other)[32] = s_ex[i & 1][warp ^ GROUPS];
+        mine[0][lane] = as4(x[0][0]);
+        mine[1][lane] = as4(x[1][0]);
+        mine[2][lane] = kh ? as4(o[0][0]) : as4(o[1][0]);
+        asm volatile("bar.sync %0, 64;" ::"r"(1 + grp) : "memory");
+        const float4 a = other[0][lane], b = other[1][lane], c = other[2][lane];
+        x[0][0][0] += a.x; x[0][0][1] += a.y; x[0][0][2] += a.z; x[0][0][3] += a.w;
+        x[1][0][0] += b.x; x[1][0][1] += b.y; x[1][0][2] += b.z; x[1][0][3] += b.w;
+        float (&mo)[4] = o[0][0], (&so_)[4] = o[1][0];         // only one of the two is used
+        mo[0] += c.x; mo[1] += c.y; mo[2] += c.z; mo[3] += c.w;
+        so_[0] += c.x; so_[1] += c.y; so_[2] += c.z; so_[3] += c.w;
+      }
+      if (SPLIT == 1 && warp == 0) {                         // into the place of chunk i - 1
+        if (elect_one() && i + stages - 1 < n_chunks) copy(i + stages - 1);
+        __syncwarp();
+      }
+      const bool has[2] = {SPLIT == 1 || kh == 0, SPLIT == 1 || kh == 1};     // token tiles whose output this warp finishes
+      // r += tile (m, n) of matrix `kind` times split rows, or times bf16 rows
+      auto times = [&](float (&r)[4], int kind, int m, int n, const SplitB& b) {
+        const uint4 h4 = mats[(kind * NT + dc_tile(m, n)) * 64], l4 = mats[(kind * NT + dc_tile(m, n)) * 64 + 32];
+        const uint32_t hi[4] = {h4.x, h4.y, h4.z, h4.w}, lo[4] = {l4.x, l4.y, l4.z, l4.w};
+        dc_mma(r, hi, b.h0, b.h1);
+        dc_mma(r, hi, b.l0, b.l1);
+        dc_mma(r, lo, b.h0, b.h1);
+      };
+      auto times_raw = [&](float (&r)[4], int kind, int m, int n, const uint32_t (&b)[2]) {
+        const uint4 h4 = mats[(kind * NT + dc_tile(m, n)) * 64], l4 = mats[(kind * NT + dc_tile(m, n)) * 64 + 32];
+        const uint32_t hi[4] = {h4.x, h4.y, h4.z, h4.w}, lo[4] = {l4.x, l4.y, l4.z, l4.w};
+        dc_mma(r, hi, b[0], b[1]);
+        dc_mma(r, lo, b[0], b[1]);
+      };
+      float y[M][4] = {}, y2[4] = {};                        // y2: the lower left tile's share, a chain of its own
+      SplitB b[M];
+      if (CHANNEL) {
+        uint32_t v[M][2];
 #pragma unroll
-    for (int m = 0; m < M; ++m) {
-      const int t = i * C + m * DC_TOK + g;
-      if (t < n) *reinterpret_cast<uint32_t*>(out + (row0 + t) * p.H * p.vp) = pack_bf16(o[m][0][0], o[m][0][1]);
-      if (t + 8 < n) *reinterpret_cast<uint32_t*>(out + (row0 + t + 8) * p.H * p.vp) = pack_bf16(o[m][0][2], o[m][0][3]);
+        for (int m = 0; m < M; ++m) dc_ldsm2_t(st + lay.values + (m * DC_TOK + (lane & 15)) * VPITCH + grp * 16, v[m][0], v[m][1]);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+#pragma unroll
+          for (int q = 0; q <= m; ++q) times_raw(x[m][1], 1, m, q, v[q]);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) x[m][0][e] += x[m][1][e];
+          b[m].from(x[m][0]);
+        }
+#pragma unroll
+        for (int m = 0; m < M; ++m) times(y[m], 0, m, m, b[m]);
+        if (M == 2) times(y2, 0, 1, 0, b[0]);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          if (m == 1)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[m][e] += y2[e];
+          b[m].from(y[m]);
+        }
+        const float* decay = reinterpret_cast<const float*>(smem + so + lay.coef) + k0 * 16 + g;
+#pragma unroll
+        for (int k = 0; k < KW; ++k) {
+          if (!EXACT && (k0 + k) * 16 >= dp) break;
+          const float d0 = decay[k * 16], d1 = decay[k * 16 + 8];
+          S[k][0] *= d0;
+          S[k][1] *= d0;
+          S[k][2] *= d1;
+          S[k][3] *= d1;
+#pragma unroll
+          for (int m = 0; m < M; ++m) {
+            uint32_t a[4];
+            dc_ldsm4_t(st + at_t(4, m, k), a);
+            dc_mma(S[k], a, v[m][0], v[m][1]);
+            dc_ldsm4_t(st + at_t(5, m, k), a);
+            dc_mma(S[k], a, v[m][0], v[m][1]);
+            dc_ldsm4_t(st + at_t(6, m, k), a);
+            dc_mma(S[k], a, b[m].h0, b[m].h1);
+            dc_mma(S[k], a, b[m].l0, b[m].l1);
+            dc_ldsm4_t(st + at_t(7, m, k), a);
+            dc_mma(S[k], a, b[m].h0, b[m].h1);
+          }
+        }
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          if (!has[m]) continue;
+#pragma unroll
+          for (int q = 0; q <= m; ++q) {
+            times_raw(o[m][0], 2, m, q, v[q]);
+            times(o[m][1], 3, m, q, b[q]);
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) o[m][0][e] += o[m][1][e];
+        }
+      } else {
+        const float* coef = reinterpret_cast<const float*>(smem + so + lay.coef);
+        float4 ca[M], cb[M];                                 // factors of rows g, g + 8
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          ca[m] = *reinterpret_cast<const float4*>(coef + 4 * (m * DC_TOK + g));
+          cb[m] = *reinterpret_cast<const float4*>(coef + 4 * (m * DC_TOK + g + 8));
+          const uint8_t* vp = smem + so + lay.values + (m * DC_TOK + g) * VPITCH + (grp * 8 + j2) * 2;
+          const float2 va = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp)), vb = unpack_bf16(*reinterpret_cast<const uint32_t*>(vp + 8 * VPITCH));
+          float (&x0)[4] = x[m][0];
+          x0[0] = fmaf(ca[m].y, x0[0], ca[m].x * va.x);
+          x0[1] = fmaf(ca[m].y, x0[1], ca[m].x * va.y);
+          x0[2] = fmaf(cb[m].y, x0[2], cb[m].x * vb.x);
+          x0[3] = fmaf(cb[m].y, x0[3], cb[m].x * vb.y);
+          b[m].from(x0);
+        }
+#pragma unroll
+        for (int m = 0; m < M; ++m) times(y[m], 0, m, m, b[m]);
+        if (M == 2) times(y2, 0, 1, 0, b[0]);
+        SplitB w[M];                                         // what is written, with the decays to the chunk's end
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          if (m == 1)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[m][e] += y2[e];
+          const float u[4] = {y[m][0] * ca[m].w, y[m][1] * ca[m].w, y[m][2] * cb[m].w, y[m][3] * cb[m].w};
+          w[m].from(u);
+        }
+        const float decay = coef[4 * C];
+#pragma unroll
+        for (int k = 0; k < KW; ++k) {
+          if (!EXACT && (k0 + k) * 16 >= dp) break;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) S[k][e] *= decay;
+#pragma unroll
+          for (int m = 0; m < M; ++m) {
+            uint32_t a[4];
+            dc_ldsm4_t(st + at_t(0, m, k), a);
+            dc_mma(S[k], a, w[m].h0, w[m].h1);
+            dc_mma(S[k], a, w[m].l0, w[m].l1);
+          }
+        }
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          b[m].from(y[m]);
+          o[m][0][0] *= ca[m].z;
+          o[m][0][1] *= ca[m].z;
+          o[m][0][2] *= cb[m].z;
+          o[m][0][3] *= cb[m].z;
+        }
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          if (!has[m]) continue;
+#pragma unroll
+          for (int q = 0; q <= m; ++q) times(o[m][0], 1, m, q, b[q]);
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar);
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        if (!has[m]) continue;
+        const int t = i * C + m * DC_TOK + g;
+        if (t < n) *reinterpret_cast<uint32_t*>(out + (long)t * p.H * p.vp) = pack_bf16(o[m][0][0], o[m][0][1]);
+        if (t + 8 < n) *reinterpret_cast<uint32_t*>(out + (long)(t + 8) * p.H * p.vp) = pack_bf16(o[m][0][2], o[m][0][3]);
+      }
+    }
+    if (used && sout >= 0) {
+      float* dst = p.state + ((long)sout * p.H + h) * dp * p.vp + col + j2;
+#pragma unroll
+      for (int k = 0; k < KW; ++k)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          if (EXACT || (k0 + k) * 16 < dp)
+            *reinterpret_cast<float2*>(dst + (long)((k0 + k) * 16 + g + 8 * e) * p.vp) = make_float2(S[k][2 * e], S[k][2 * e + 1]);
     }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-  if (!used || sout < 0) return;
-  float* dst = p.state + ((long)sout * p.H + h) * dp * p.vp + col + j2;
-#pragma unroll
-  for (int k = 0; k < KS; ++k)
-#pragma unroll
-    for (int e = 0; e < 2; ++e)
-      if (EXACT || k * 16 < dp) *reinterpret_cast<float2*>(dst + (long)(k * 16 + g + 8 * e) * p.vp) = make_float2(S[k][2 * e], S[k][2 * e + 1]);
+  __syncthreads();
+  if (s_abort) {
+    // a wait ran out: give copies in flight time to finish before their memory goes
+    const unsigned long long t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) {
+    }
+  }
 }
 
-template <bool CHANNEL, int KS, bool EXACT, int M>
+// [rows, cols] bf16 as boxes of box_rows x box_cols without swizzle
+static int rows_tmap(CUtensorMap* out, const void* ptr, uint64_t rows, uint64_t cols, uint64_t pitch, uint32_t box_rows, uint32_t box_cols) {
+  EncodeTiledFn enc = get_encode_tiled();
+  if (!enc) return RC_NO_DRIVER;
+  if ((reinterpret_cast<uintptr_t>(ptr) & 15) || (pitch & 15)) return RC_BAD_ARG;
+  cuuint64_t gdim[2] = {cols, rows}, gstr[1] = {pitch};
+  cuuint32_t box[2] = {box_cols, box_rows}, estr[2] = {1, 1};
+  const CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), gdim, gstr, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                         CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? RC_OK : RC_TMAP;
+}
+
+template <bool CHANNEL, int KS, bool EXACT, int M, int SPLIT>
 static int launch_sequence(const DeltaRule& p, cudaStream_t st) {
-  const DeltaStage lay = delta_stage<CHANNEL, M>(p.dp);
-  const int limit = 226 * 1024;
-  const dim3 grid((p.vp + DC_COLS - 1) / DC_COLS, p.H, p.n_long);
+  constexpr int COLS = 8 * DC_WARPS / SPLIT;
+  const DeltaStage lay = delta_stage<CHANNEL, M, COLS>(p.dp);
+  const int limit = 212 * 1024;                              // less the exchange and the barriers
+  const dim3 grid((p.vp + COLS - 1) / COLS, p.H, p.n_long);
   // two stages leave room for more blocks on an SM, three hide more of a fetch
-  const int stages = (long)grid.x * grid.y * grid.z <= 2l * sm_count() && 3 * lay.bytes <= limit / (CHANNEL ? 1 : 2) ? 3 : 2;
-  const int smem = stages * lay.bytes;
+  const int stages = (long)grid.x * grid.y * grid.z <= sm_count() && 3 * lay.bytes <= limit ? 3 : 2;
+  const int smem = stages * lay.bytes + 1024;
   if (smem > limit) return RC_TOO_LARGE;
+  CUtensorMap tu, tv;
+  const bf16* v = CHANNEL ? static_cast<const bf16*>(p.proj) + p.v_col : static_cast<const bf16*>(p.u) + 2 * p.G * p.dp;
+  const uint64_t ldv = (uint64_t)(CHANNEL ? p.ldp : p.ldu) * 2;
+  if (int rc = rows_tmap(&tv, v, p.T, p.H * p.vp, ldv, M * DC_TOK, COLS)) return rc;
+  tu = tv;
+  if (!CHANNEL)
+    if (int rc = make_tmap_2d(&tu, p.u, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.T, 2 * p.G * p.dp, (uint64_t)p.ldu * 2, M * DC_TOK, 64)) return rc;
   static unsigned long long prep = 0;
-  if (int e = ensure_dynamic_smem((const void*)delta_sequence_kernel<CHANNEL, KS, EXACT, M>, limit, prep)) return e;
-  delta_sequence_kernel<CHANNEL, KS, EXACT, M><<<grid, 32 * DC_WARPS, smem, st>>>(p, stages);
+  if (int e = ensure_dynamic_smem((const void*)delta_sequence_kernel<CHANNEL, KS, EXACT, M, SPLIT>, limit, prep)) return e;
+  delta_sequence_kernel<CHANNEL, KS, EXACT, M, SPLIT><<<grid, 32 * (DC_WARPS + SPLIT - 1), smem, st>>>(tu, tv, p, stages);
   return (int)cudaGetLastError();
+}
+
+template <bool CHANNEL, int KS>
+static int launch_exact(const DeltaRule& p, cudaStream_t st) {
+  // SMs to spare: two warps to eight columns
+  const long blocks = (long)((p.vp + 4 * DC_WARPS - 1) / (4 * DC_WARPS)) * p.H * p.n_long;
+  return blocks <= sm_count() ? launch_sequence<CHANNEL, KS, true, 2, 2>(p, st) : launch_sequence<CHANNEL, KS, true, 2, 1>(p, st);
 }
 
 template <bool CHANNEL, int M>
@@ -788,17 +874,17 @@ static int launch_chunks(const DeltaRule& p, cudaStream_t st) {
   else delta_prepare_gated_kernel<M><<<dim3(p.n_chunks, (p.H * M + 3) / 4), 128, 0, st>>>(p);
   if (int e = (int)cudaGetLastError()) return e;
   if constexpr (M == 1) {
-    return launch_sequence<CHANNEL, 16, false, 1>(p, st);
+    return launch_sequence<CHANNEL, 16, false, 1, 1>(p, st);
   } else {
     switch (p.dp) {
-      case 64: return launch_sequence<CHANNEL, 4, true, 2>(p, st);
-      case 96: return launch_sequence<CHANNEL, 6, true, 2>(p, st);
-      case 128: return launch_sequence<CHANNEL, 8, true, 2>(p, st);
+      case 64: return launch_exact<CHANNEL, 4>(p, st);
+      case 96: return launch_exact<CHANNEL, 6>(p, st);
+      case 128: return launch_exact<CHANNEL, 8>(p, st);
       default: break;
     }
-    if (p.dp <= 128) return launch_sequence<CHANNEL, 8, false, 2>(p, st);
+    if (p.dp <= 128) return launch_sequence<CHANNEL, 8, false, 2, 1>(p, st);
     if constexpr (CHANNEL) return RC_TOO_LARGE;
-    else return launch_sequence<CHANNEL, 16, false, 2>(p, st);
+    else return launch_sequence<CHANNEL, 16, false, 2, 1>(p, st);
   }
 }
 
@@ -811,7 +897,7 @@ extern "C" int omni_delta_chunks(const DeltaRule* args, int channel, int chunk, 
   const DeltaRule& p = *args;
   if (p.n_chunks <= 0 || p.n_long <= 0) return RC_OK;
   if (!delta_args_ok(p, channel) || !p.chunks || !p.long_list || !p.raw || !p.mats || !p.coef || p.dp > 256 || p.n_long > 65535 ||
-      chunk != 32 && !(channel && chunk == 16))
+      (chunk != 32 && !(channel && chunk == 16 && p.dp > 128)) || (channel && chunk == 32 && p.dp > 128))
     return RC_BAD_ARG;
   if (channel ? !p.tiles : (!p.u || (p.ldu & 7) || p.ldu < 2l * p.G * p.dp + (long)p.H * p.vp)) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;

@@ -205,36 +205,40 @@ delta_steps_kernel(const DeltaRule p, const int cw) {
   }
 }
 
-// One group of lanes per (row, head), eight channels per lane and turn.
-template <typename T, bool CHANNEL>
+// One group of lanes per (row, head), eight channels per lane and turn; ONE turn is enough where a group covers the head.
+template <typename T, bool CHANNEL, bool ONE>
 __global__ void __launch_bounds__(256)
 delta_finish_kernel(const DeltaRule p, const int lph, const int skip_single) {
   const int lane = threadIdx.x & (lph - 1);
   const int t = blockIdx.x * (256 / lph) + threadIdx.x / lph, h = blockIdx.y;
   bool live = t < p.T;
   const long row = live ? t : p.T - 1;                       // idle groups keep the shuffles company
+  const T* raw = static_cast<const T*>(p.raw) + row * p.H * p.vp + (long)h * p.vp;
+  const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.g_col + (long)h * p.vp;
+  const float* gain = p.gain + (long)h * p.gain_hs;
+  T* out = static_cast<T*>(p.out) + row * p.ldo + (long)h * p.vp;
+  float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, z[8];
+  float ss = 0.f;
+  for (int c = lane * 8; c < p.vp; c += lph * 8) {
+    load8<T>(raw + c, v);
+    if (ONE) load8<T>(gate + c, z);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+  }
   if (skip_single) {
     const int seq = min(max(p.row_seq[row], 0), p.num_seqs - 1);
     live = live && p.q_start[seq + 1] - p.q_start[seq] > 1;
   }
-  const T* raw = static_cast<const T*>(p.raw) + row * p.H * p.vp + (long)h * p.vp;
-  const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.g_col + (long)h * p.vp;
-  float ss = 0.f;
-  for (int c = lane * 8; c < p.vp; c += lph * 8) {
-    float v[8];
-    load8<T>(raw + c, v);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
-  }
   for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
   if (!live) return;
   const float s = rms_scale(ss, p.dv, p.eps);
-  T* out = static_cast<T*>(p.out) + row * p.ldo + (long)h * p.vp;
   for (int c = lane * 8; c < p.vp; c += lph * 8) {
-    float v[8], z[8], gn[8];
-    load8<T>(raw + c, v);
-    load8<T>(gate + c, z);
-    load8<float>(p.gain + (long)h * p.gain_hs + c, gn);
+    float gn[8];
+    if (!ONE) {
+      load8<T>(raw + c, v);
+      load8<T>(gate + c, z);
+    }
+    load8<float>(gain + c, gn);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       const float open = sizeof(T) == 4 ? dr_sigmoid(z[e]) : __fdividef(1.0f, 1.0f + __expf(-z[e]));
@@ -263,7 +267,9 @@ static int launch_finish(const DeltaRule& p, int skip_single, cudaStream_t st) {
   int lph = 1;
   while (lph < 32 && lph * 8 < p.vp) lph *= 2;
   const int rows = 256 / lph;
-  delta_finish_kernel<T, CHANNEL><<<dim3((p.T + rows - 1) / rows, p.H), 256, 0, st>>>(p, lph, skip_single);
+  const dim3 grid((p.T + rows - 1) / rows, p.H);
+  if (lph * 8 >= p.vp) delta_finish_kernel<T, CHANNEL, true><<<grid, 256, 0, st>>>(p, lph, skip_single);
+  else delta_finish_kernel<T, CHANNEL, false><<<grid, 256, 0, st>>>(p, lph, skip_single);
   return (int)cudaGetLastError();
 }
 

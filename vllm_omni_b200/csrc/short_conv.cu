@@ -3,6 +3,7 @@
 // position says that there are any, zeros otherwise; the portion's last rows become the sequence's new history.  Pool rows
 // are double-buffered (read row != write row), so readers of the old history never race with the writer of the new one.
 // A thread slides over eight rows of eight channels; with up to four taps weights and earlier rows stay in registers.
+#include "f32x2.cuh"
 #include "host_util.h"
 #include "row_ops.cuh"
 
@@ -37,17 +38,18 @@ __device__ __forceinline__ float rcp_approx(float x) {
 }
 
 template <int TAPS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(128, 4)
 conv_rows_kernel(const ConvRows p) {
-  constexpr int RUN = 8, H = TAPS > 1 ? TAPS - 1 : 1;
+  constexpr int RUN = 8, H = TAPS > 1 ? TAPS - 1 : 1, HALF = RUN / 2;
   const int vecs = p.C / 8;
-  const long idx = (long)blockIdx.x * 256 + threadIdx.x;
+  const long idx = (long)blockIdx.x * 128 + threadIdx.x;
   const int c = (int)(idx % vecs) * 8;
   const long r0 = idx / vecs * RUN;
   if (r0 >= p.T) return;
   const int taps = TAPS > 0 ? TAPS : p.taps, h = taps - 1;
   const bf16* x = static_cast<const bf16*>(p.x) + c;
   bf16* hist = static_cast<bf16*>(p.hist) + c;
+  bf16* out = static_cast<bf16*>(p.out) + c;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   int seq = -1, q0 = 0, q1 = 0, ctx = 0, sin = 0, sout = -1;
   auto raw_x = [&](int b) {                                  // row b of the portion; negative: history
@@ -55,58 +57,43 @@ conv_rows_kernel(const ConvRows p) {
     if (ctx + b >= 0) return *reinterpret_cast<const uint4*>(hist + ((long)sin * h + h + b) * p.C);
     return zero;
   };
-  // portions are contiguous: rows that begin and end in the same one need no look at those between
-  const int s_first = min(max(p.row_seq[r0], 0), p.num_seqs - 1), s_last = min(max(p.row_seq[min(r0 + RUN, (long)p.T) - 1], 0), p.num_seqs - 1);
-  uint4 raw[RUN], win[H];
-  float w[TAPS > 0 ? TAPS : 1][8], bias[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-  if (p.bias) load8<float>(p.bias + c, bias);
-  if (TAPS > 0) {
-#pragma unroll
-    for (int i = 0; i < RUN; ++i) raw[i] = r0 + i < p.T ? *reinterpret_cast<const uint4*>(x + (r0 + i) * p.ldx) : zero;
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) load8<float>(p.conv + (long)j * p.C + c, w[j]);
-  }
-#pragma unroll
-  for (int i = 0; i < RUN; ++i) {
-    const long row = r0 + i;
-    if (row >= p.T) break;
-    const int s = i == 0 || s_first == s_last ? s_first : min(max(p.row_seq[row], 0), p.num_seqs - 1);
-    if (s != seq) {                                          // first row of the run or of a sequence
-      seq = s;
-      q0 = p.q_start[seq];
-      q1 = p.q_start[seq + 1];
-      ctx = p.context[seq];
-      if (h > 0) {
-        sin = p.state_in[seq];
-        sout = p.state_out[seq];
-        if (sin < 0 || sin >= p.num_state || sout >= p.num_state) {
-          if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
-          sin = 0;
-          sout = -1;
-        }
-      }
-      if (TAPS > 1) {
-#pragma unroll
-        for (int m = 0; m < H; ++m) win[m] = raw_x((int)(row - q0) - H + m);
+  auto enter = [&](int s) {                                  // a sequence's numbers
+    seq = s;
+    q0 = p.q_start[seq];
+    q1 = p.q_start[seq + 1];
+    ctx = p.context[seq];
+    if (h > 0) {
+      sin = p.state_in[seq];
+      sout = p.state_out[seq];
+      if (sin < 0 || sin >= p.num_state || sout >= p.num_state) {
+        if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
+        sin = 0;
+        sout = -1;
       }
     }
-    float o[8];
+  };
+  auto seq_of = [&](long row) { return min(max(p.row_seq[row], 0), p.num_seqs - 1); };
+  auto finish = [&](float (&o)[8], long row) {
+    if (p.act == 1) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) o[e] = bias[e];
-    if (TAPS > 0) {
+      for (int e = 0; e < 8; ++e) o[e] *= rcp_approx(1.0f + ex2_approx(-1.4426950408889634f * o[e]));
+    }
+    store8<bf16>(out + row * p.C, o);
+  };
+  auto new_history = [&](long row) {                         // after the portion's last row
+    if (row == q1 - 1 && sout >= 0 && !(p.skip_single && q1 - q0 == 1))
+      for (int m = 0; m < h; ++m)
+        *reinterpret_cast<uint4*>(hist + ((long)sout * h + m) * p.C) = raw_x((int)(row - q0) + 1 - h + m);
+  };
+  float bias[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (p.bias) load8<float>(p.bias + c, bias);
+  if constexpr (TAPS == 0) {
+    for (long row = r0; row < min(r0 + RUN, (long)p.T); ++row) {
+      const int s = seq_of(row);
+      if (s != seq) enter(s);
+      float o[8];
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) {
-        float f[8];
-        load8<bf16>(reinterpret_cast<const bf16*>(j < TAPS - 1 ? &win[j < H ? j : 0] : &raw[i]), f);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = fmaf(w[j][e], f[e], o[e]);
-      }
-      if (TAPS > 1) {
-#pragma unroll
-        for (int m = 0; m + 1 < H; ++m) win[m] = win[m + 1];
-        win[H - 1] = raw[i];
-      }
-    } else {
+      for (int e = 0; e < 8; ++e) o[e] = bias[e];
       for (int j = 0; j < taps; ++j) {
         float f[8], wj[8];
         const uint4 q = raw_x((int)(row - q0) - h + j);
@@ -115,15 +102,53 @@ conv_rows_kernel(const ConvRows p) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) o[e] = fmaf(wj[e], f[e], o[e]);
       }
+      finish(o, row);
+      new_history(row);
     }
-    if (p.act == 1) {
+  } else {
+    // portions are contiguous: rows that begin and end in the same one need no look at those between
+    const int s_first = seq_of(r0);
+    const bool same = s_first == seq_of(min(r0 + RUN, (long)p.T) - 1);
+    uint4 raw[HALF];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) o[e] *= rcp_approx(1.0f + ex2_approx(-1.4426950408889634f * o[e]));
+    for (int i = 0; i < HALF; ++i) raw[i] = r0 + i < p.T ? *reinterpret_cast<const uint4*>(x + (r0 + i) * p.ldx) : zero;
+    float w[TAPS][8], win[TAPS][8];                          // win: rows t - taps + 1 .. t, row t at t % TAPS
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load8<float>(p.conv + (long)j * p.C + c, w[j]);
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) {
+      const long row = r0 + i;
+      if (row >= p.T) break;
+      if (i == HALF) {
+#pragma unroll
+        for (int k = 0; k < HALF; ++k) raw[k] = row + k < p.T ? *reinterpret_cast<const uint4*>(x + (row + k) * p.ldx) : zero;
+      }
+      const int s = i == 0 || same ? s_first : seq_of(row);
+      if (s != seq) {                                        // first row of the run or of a sequence
+        enter(s);
+        if (TAPS > 1) {
+#pragma unroll
+          for (int m = 0; m < H; ++m) {
+            const uint4 q = raw_x((int)(row - q0) - H + m);
+            load8<bf16>(reinterpret_cast<const bf16*>(&q), win[(i + m + 1) % TAPS]);
+          }
+        }
+      }
+      load8<bf16>(reinterpret_cast<const bf16*>(&raw[i % HALF]), win[i % TAPS]);
+      uint64_t o2[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o2[e] = pack2(bias[2 * e], bias[2 * e + 1]);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          o2[e] = fma2(pack2(w[j][2 * e], w[j][2 * e + 1]), pack2(win[(i + j + 1) % TAPS][2 * e], win[(i + j + 1) % TAPS][2 * e + 1]), o2[e]);
+      float o[8];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) unpack2(o2[e], o[2 * e], o[2 * e + 1]);
+      finish(o, row);
+      new_history(row);
     }
-    store8<bf16>(static_cast<bf16*>(p.out) + row * p.C + c, o);
-    if (row == q1 - 1 && sout >= 0 && !(p.skip_single && q1 - q0 == 1))
-      for (int m = 0; m < h; ++m)
-        *reinterpret_cast<uint4*>(hist + ((long)sout * h + m) * p.C) = raw_x((int)(row - q0) + 1 - h + m);
   }
 }
 
@@ -137,15 +162,15 @@ extern "C" int omni_conv_rows(const ConvRows* args, void* stream) {
   if (p.C <= 0 || (p.C & 7) || (p.ldx & 7) || p.ldx < p.C || p.taps < 1 || !p.conv || !p.x || !p.out || !p.row_seq || p.num_seqs <= 0 ||
       (reinterpret_cast<uintptr_t>(p.x) & 15) || (p.taps > 1 && (!p.hist || !p.state_in || !p.state_out || p.num_state <= 0)))
     return RC_BAD_ARG;
-  const long blocks = ((long)((p.T + 7) / 8) * (p.C / 8) + 255) / 256;
+  const long blocks = ((long)((p.T + 7) / 8) * (p.C / 8) + 127) / 128;
   if (blocks > 0x7fffffffl) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
   switch (p.taps) {
-    case 1: conv_rows_kernel<1><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    case 2: conv_rows_kernel<2><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    case 3: conv_rows_kernel<3><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    case 4: conv_rows_kernel<4><<<(unsigned)blocks, 256, 0, st>>>(p); break;
-    default: conv_rows_kernel<0><<<(unsigned)blocks, 256, 0, st>>>(p); break;
+    case 1: conv_rows_kernel<1><<<(unsigned)blocks, 128, 0, st>>>(p); break;
+    case 2: conv_rows_kernel<2><<<(unsigned)blocks, 128, 0, st>>>(p); break;
+    case 3: conv_rows_kernel<3><<<(unsigned)blocks, 128, 0, st>>>(p); break;
+    case 4: conv_rows_kernel<4><<<(unsigned)blocks, 128, 0, st>>>(p); break;
+    default: conv_rows_kernel<0><<<(unsigned)blocks, 128, 0, st>>>(p); break;
   }
   return (int)cudaGetLastError();
 }

@@ -153,7 +153,7 @@ def delta_rule(proj, s: DeltaShape, seqs, rule, state, out, *, hist=None, decay=
         lower = 512 * (3 if size == 32 else 1)              # lower tiles of a chunk's matrix, high and low parts
         if rule.channel:
             mats, coef = torch.empty(n, 4 * lower, dtype=torch.bfloat16, device=dev), torch.empty(n, s.dp, device=dev)
-            tiles = torch.empty(n, 8, size, s.dp, dtype=torch.bfloat16, device=dev)
+            tiles = torch.empty(n, 8, size, s.dp + 8, dtype=torch.bfloat16, device=dev)
             a.tiles = P(tiles)
         else:
             mats, coef = torch.empty(n, 2 * lower, dtype=torch.bfloat16, device=dev), torch.empty(n, 4 * size + 4, device=dev)
