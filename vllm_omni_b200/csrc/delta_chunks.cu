@@ -51,6 +51,9 @@ __device__ __forceinline__ uint32_t dc_trans(uint32_t x) {
   asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
   return y;
 }
+__device__ __forceinline__ void dc_copy16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
 __device__ __forceinline__ void dc_bulk(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes),
                "r"(bar)
@@ -312,6 +315,7 @@ delta_prepare_channel_kernel(const DeltaRule p) {
   __shared__ __align__(16) uint32_t s_rows[8 * ARR32];       // decayed rows: b0, r0, k / G, a u / G (high, low)
   __shared__ float s_a[M][DC_TOK][20];
   __shared__ float2 s_tot[M][32];                            // log decay of a tile's tokens
+  __shared__ float s_ik[M][DC_TOK];                          // one over the length of a key
   const int m = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
   const int h = blockIdx.y;
   const ChunkRows ch = dc_chunk<M>(p, blockIdx.x);
@@ -321,79 +325,88 @@ delta_prepare_channel_kernel(const DeltaRule p) {
   const int pitch = p.dp / 2 + 4, tile = C * pitch;          // channel pairs of a row (padded as in shared memory), of an operand
   uint32_t* tiles = static_cast<uint32_t*>(p.tiles) + at * (8 * tile);
   uint4* mats = static_cast<uint4*>(p.mats) + at * (4 * NT * 64);
-  // two channels of the tile's token t (past the end: another token's, not used)
-  auto raw = [&](const bf16* base, long ld, int t, int c) {
-    return *reinterpret_cast<const uint32_t*>(base + (ch.row0 + min(m * DC_TOK + t, ch.n - 1)) * ld + c);
-  };
-  // lengths of the keys
-  float ik[DC_TOK];
-#pragma unroll
-  for (int t = 0; t < DC_TOK; ++t) ik[t] = 0.f;
-  for (int c = lane * 2; c < p.dp; c += 64) {
-    uint32_t k[DC_TOK];
-#pragma unroll
-    for (int t = 0; t < DC_TOK; ++t) k[t] = raw(proj + p.k_col, p.ldp, t, c);
-#pragma unroll
-    for (int t = 0; t < DC_TOK; ++t) {
-      const float2 f = unpack_bf16(k[t]);
-      ik[t] = fmaf(f.x, f.x, fmaf(f.y, f.y, ik[t]));
+  const uint32_t base = smem_u32(s_rows);
+  constexpr uint32_t ARR = C * PC_PITCH;
+  // the raw rows of 64 channels, where the operands k / G and a u / G take their places channel by channel: r, k, a, z
+  auto fetch = [&](int cb) {
+    for (int x = threadIdx.x; x < 4 * C * 8; x += 32 * M) {
+      const int arr = x / (C * 8), t = x / 8 % C, c = cb + x % 8 * 8;
+      const bf16* src = arr == 3 ? z : proj + (arr == 0 ? p.q_col : (arr == 1 ? p.k_col : p.a_col));
+      const long ld = arr == 3 ? p.ldz : p.ldp;
+      if (c < p.dp) dc_copy16(base + (4 + arr) * ARR + t * PC_PITCH + x % 8 * 16, src + (ch.row0 + min(t, ch.n - 1)) * ld + c);
     }
-  }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(0);
+  // lengths of the keys: two lanes per token
+  {
+    const int t = lane & 15;
+    const bf16* k = proj + p.k_col + (ch.row0 + min(m * DC_TOK + t, ch.n - 1)) * p.ldp;
+    float ss = 0.f;
+    for (int c = (lane >> 4) * 8; c < p.dp; c += 16) {
+      float v[8];
+      load8<bf16>(k + c, v);
 #pragma unroll
-  for (int t = 0; t < DC_TOK; ++t) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) ik[t] += __shfl_xor_sync(0xffffffffu, ik[t], o);
-    ik[t] = 1.0f / sqrtf(ik[t] + p.unit_eps);
+      for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+    }
+    ss += __shfl_xor_sync(0xffffffffu, ss, 16);
+    if (lane < 16) s_ik[m][t] = 1.0f / sqrtf(ss + p.unit_eps);
+    __syncwarp();
   }
   float am[M][2][4] = {}, mm[M][2][4] = {}, nm[M][2][4] = {}, lm[M][2][4] = {};      // [0]: diagonal tile, [1]: left of it
-  const uint32_t base = smem_u32(s_rows);
   for (int cb = 0; cb < p.dp; cb += 64) {
+    if (cb > 0) {
+      __syncthreads();                                       // the products of the last 64 channels are done
+      fetch(cb);
+    }
     const int c = cb + lane * 2;
     const bool in = c < p.dp;
     const int cc = in ? c : 0;
     const float2 db = *reinterpret_cast<const float2*>(p.decay_bias + h * p.dp + cc);
     const float2 rb = *reinterpret_cast<const float2*>(p.removal_bias + h * p.dp + cc);
-    uint32_t r_[DC_TOK], k_[DC_TOK], a_[DC_TOK];
-    float2 G[DC_TOK];                                        // cumulative log decay
-#pragma unroll
-    for (int t = 0; t < DC_TOK; ++t) {
-      const float2 f = unpack_bf16(raw(z, p.ldz, t, cc));
-      G[t] = make_float2(f.x + db.x, f.y + db.y);
-      r_[t] = raw(proj + p.q_col, p.ldp, t, cc);
-      k_[t] = raw(proj + p.k_col, p.ldp, t, cc);
-      a_[t] = raw(proj + p.a_col, p.ldp, t, cc);
-    }
+    const int nt = min(max(ch.n - m * DC_TOK, 0), DC_TOK);   // tokens of the tile
+    auto log_decay = [&](uint32_t w) {
+      const float2 f = unpack_bf16(w);
+      return make_float2(p.decay_scale * __fdividef(1.0f, 1.0f + __expf(-(f.x + db.x))),
+                         p.decay_scale * __fdividef(1.0f, 1.0f + __expf(-(f.y + db.y))));
+    };
+    auto raw = [&](int arr, int t) { return s_rows[(4 + arr) * ARR32 + (m * DC_TOK + t) * ROW32 + lane]; };
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
     float2 sum = make_float2(0.f, 0.f);
-#pragma unroll
+#pragma unroll 8
     for (int t = 0; t < DC_TOK; ++t) {
-      if (m * DC_TOK + t < ch.n) {
-        sum.x = fmaf(p.decay_scale, __fdividef(1.0f, 1.0f + __expf(-G[t].x)), sum.x);
-        sum.y = fmaf(p.decay_scale, __fdividef(1.0f, 1.0f + __expf(-G[t].y)), sum.y);
+      const float2 l = log_decay(raw(3, t));
+      if (t < nt) {
+        sum.x += l.x;
+        sum.y += l.y;
       }
-      G[t] = sum;
     }
     s_tot[m][lane] = sum;
-    __syncthreads();                                         // totals; and the products of the last 64 channels are done
-    float2 before = make_float2(0.f, 0.f), total = s_tot[0][lane];
+    __syncthreads();
+    float2 G = make_float2(0.f, 0.f), total = s_tot[0][lane];               // cumulative log decay
     if (M == 2) {
-      if (m == 1) before = total;
+      if (m == 1) G = total;
       total.x += s_tot[M - 1][lane].x;
       total.y += s_tot[M - 1][lane].y;
     }
     const float tx = __expf(total.x), ty = __expf(total.y);
-    float e0 = __expf(before.x), e1 = __expf(before.y);      // decays so far
-#pragma unroll
+    float e0 = __expf(G.x), e1 = __expf(G.y);                // decays so far
+#pragma unroll 4
     for (int t = 0; t < DC_TOK; ++t) {
+      const uint32_t rw = raw(0, t), kw = raw(1, t), aw = raw(2, t), zw = raw(3, t);
       float2 b0 = make_float2(0.f, 0.f), r0 = b0, ki = b0, ai = b0;
-      if (m * DC_TOK + t < ch.n && in) {
-        const float2 r = unpack_bf16(r_[t]), k = unpack_bf16(k_[t]), a = unpack_bf16(a_[t]);
-        b0 = make_float2(k.x * ik[t] * e0, k.y * ik[t] * e1);
-        const float gx = G[t].x + before.x, gy = G[t].y + before.y;
-        e0 = __expf(gx);
-        e1 = __expf(gy);
+      if (t < nt && in) {
+        const float2 r = unpack_bf16(rw), k = unpack_bf16(kw), a = unpack_bf16(aw), l = log_decay(zw);
+        const float ik = s_ik[m][t];
+        b0 = make_float2(k.x * ik * e0, k.y * ik * e1);
+        G.x += l.x;
+        G.y += l.y;
+        e0 = __expf(G.x);
+        e1 = __expf(G.y);
         r0 = make_float2(r.x * e0, r.y * e1);
-        ki = make_float2(k.x * __expf(-gx), k.y * __expf(-gy));
-        ai = make_float2(__fdividef(ik[t], 1.0f + __expf(-(a.x + rb.x))) * ki.x, __fdividef(ik[t], 1.0f + __expf(-(a.y + rb.y))) * ki.y);
+        ki = make_float2(k.x * __expf(-G.x), k.y * __expf(-G.y));
+        ai = make_float2(__fdividef(ik, 1.0f + __expf(-(a.x + rb.x))) * ki.x, __fdividef(ik, 1.0f + __expf(-(a.y + rb.y))) * ki.y);
       }
       const int tok = m * DC_TOK + t;
       uint32_t hi, lo;
@@ -419,7 +432,6 @@ delta_prepare_channel_kernel(const DeltaRule p) {
     }
     if (in && m == 0) *reinterpret_cast<float2*>(p.coef + at * p.dp + c) = make_float2(tx, ty);
     __syncthreads();
-    constexpr uint32_t ARR = C * PC_PITCH;
     const uint32_t a0 = base + ((lane & 7) + ((lane >> 3) & 1) * 8) * PC_PITCH + (lane >> 4) * 16, mine = a0 + m * DC_TOK * PC_PITCH;
 #pragma unroll
     for (int k = 0; k < 4; ++k) {

@@ -205,46 +205,63 @@ delta_steps_kernel(const DeltaRule p, const int cw) {
   }
 }
 
-// One group of lanes per (row, head), eight channels per lane and turn; ONE turn is enough where a group covers the head.
+// One group of lanes per (row, head), eight channels per lane and turn.  ONE: a turn covers the head, and a group takes two
+// rows with all loads in flight.
 template <typename T, bool CHANNEL, bool ONE>
 __global__ void __launch_bounds__(256)
-delta_finish_kernel(const DeltaRule p, const int lph, const int skip_single) {
-  const int lane = threadIdx.x & (lph - 1);
-  const int t = blockIdx.x * (256 / lph) + threadIdx.x / lph, h = blockIdx.y;
-  bool live = t < p.T;
-  const long row = live ? t : p.T - 1;                       // idle groups keep the shuffles company
-  const T* raw = static_cast<const T*>(p.raw) + row * p.H * p.vp + (long)h * p.vp;
-  const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.g_col + (long)h * p.vp;
+delta_finish_kernel(const DeltaRule p, const int lph) {
+  constexpr int ROWS = ONE ? 2 : 1;
+  const int lane = threadIdx.x & (lph - 1), h = blockIdx.y;
+  const int t0 = (blockIdx.x * (256 / lph) + threadIdx.x / lph) * ROWS;
   const float* gain = p.gain + (long)h * p.gain_hs;
-  T* out = static_cast<T*>(p.out) + row * p.ldo + (long)h * p.vp;
-  float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, z[8];
-  float ss = 0.f;
-  for (int c = lane * 8; c < p.vp; c += lph * 8) {
-    load8<T>(raw + c, v);
-    if (ONE) load8<T>(gate + c, z);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
-  }
-  if (skip_single) {
-    const int seq = min(max(p.row_seq[row], 0), p.num_seqs - 1);
-    live = live && p.q_start[seq + 1] - p.q_start[seq] > 1;
-  }
-  for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if (!live) return;
-  const float s = rms_scale(ss, p.dv, p.eps);
-  for (int c = lane * 8; c < p.vp; c += lph * 8) {
+  auto opened = [&](float (&v)[8], const float (&z)[8], float s, int c) {
     float gn[8];
-    if (!ONE) {
-      load8<T>(raw + c, v);
-      load8<T>(gate + c, z);
-    }
     load8<float>(gain + c, gn);
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       const float open = sizeof(T) == 4 ? dr_sigmoid(z[e]) : __fdividef(1.0f, 1.0f + __expf(-z[e]));
       v[e] *= s * gn[e] * (CHANNEL ? open : z[e] * open);
     }
-    store8<T>(out + c, v);
+  };
+  float v[ROWS][8], z[ROWS][8], ss[ROWS];
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    const long row = min(t0 + i, p.T - 1);                   // idle groups keep the shuffles company
+    const T* raw = static_cast<const T*>(p.raw) + row * p.H * p.vp + (long)h * p.vp;
+    const T* gate = static_cast<const T*>(p.proj) + row * p.ldp + p.g_col + (long)h * p.vp;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[i][e] = z[i][e] = 0.f;
+    ss[i] = 0.f;
+    for (int c = lane * 8; c < p.vp; c += lph * 8) {
+      load8<T>(raw + c, v[i]);
+      if (ONE) load8<T>(gate + c, z[i]);
+      else
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss[i] = fmaf(v[i][e], v[i][e], ss[i]);
+      if (ONE) break;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    if (ONE)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss[i] = fmaf(v[i][e], v[i][e], ss[i]);
+    for (int o = lph >> 1; o > 0; o >>= 1) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+  }
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    const long row = t0 + i;
+    if (row >= p.T) return;
+    const float s = rms_scale(ss[i], p.dv, p.eps);
+    T* out = static_cast<T*>(p.out) + row * p.ldo + (long)h * p.vp;
+    for (int c = lane * 8; c < p.vp; c += lph * 8) {
+      if (!ONE) {
+        load8<T>(static_cast<const T*>(p.raw) + row * p.H * p.vp + (long)h * p.vp + c, v[i]);
+        load8<T>(static_cast<const T*>(p.proj) + row * p.ldp + p.g_col + (long)h * p.vp + c, z[i]);
+      }
+      opened(v[i], z[i], s, c);
+      store8<T>(out + c, v[i]);
+    }
   }
 }
 
@@ -263,13 +280,14 @@ static int launch_steps(const DeltaRule& p, int cw, cudaStream_t st) {
 }
 
 template <typename T, bool CHANNEL>
-static int launch_finish(const DeltaRule& p, int skip_single, cudaStream_t st) {
+static int launch_finish(const DeltaRule& p, cudaStream_t st) {
   int lph = 1;
   while (lph < 32 && lph * 8 < p.vp) lph *= 2;
-  const int rows = 256 / lph;
+  const bool one = lph * 8 >= p.vp;
+  const int rows = 256 / lph * (one ? 2 : 1);
   const dim3 grid((p.T + rows - 1) / rows, p.H);
-  if (lph * 8 >= p.vp) delta_finish_kernel<T, CHANNEL, true><<<grid, 256, 0, st>>>(p, lph, skip_single);
-  else delta_finish_kernel<T, CHANNEL, false><<<grid, 256, 0, st>>>(p, lph, skip_single);
+  if (one) delta_finish_kernel<T, CHANNEL, true><<<grid, 256, 0, st>>>(p, lph);
+  else delta_finish_kernel<T, CHANNEL, false><<<grid, 256, 0, st>>>(p, lph);
   return (int)cudaGetLastError();
 }
 
@@ -297,12 +315,11 @@ extern "C" int omni_delta_steps(const DeltaRule* args, int channel, int is_bf16,
   return channel ? launch_steps<float, true>(p, cw, st) : launch_steps<float, false>(p, cw, st);
 }
 
-// skip_single: rows of sequences with one row are finished already.
-extern "C" int omni_delta_finish(const DeltaRule* args, int channel, int is_bf16, int skip_single, void* stream) {
+extern "C" int omni_delta_finish(const DeltaRule* args, int channel, int is_bf16, void* stream) {
   const DeltaRule& p = *args;
   if (p.T <= 0) return RC_OK;
-  if (!delta_args_ok(p, channel) || !p.raw || (skip_single && !p.row_seq)) return RC_BAD_ARG;
+  if (!delta_args_ok(p, channel) || !p.raw) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
-  if (is_bf16) return channel ? launch_finish<bf16, true>(p, skip_single, st) : launch_finish<bf16, false>(p, skip_single, st);
-  return channel ? launch_finish<float, true>(p, skip_single, st) : launch_finish<float, false>(p, skip_single, st);
+  if (is_bf16) return channel ? launch_finish<bf16, true>(p, st) : launch_finish<bf16, false>(p, st);
+  return channel ? launch_finish<float, true>(p, st) : launch_finish<float, false>(p, st);
 }

@@ -2,7 +2,7 @@
 // out_t = act(bias + sum_j conv[j] x_(t - taps + 1 + j)).  Rows before a portion come from the history pool where the
 // position says that there are any, zeros otherwise; the portion's last rows become the sequence's new history.  Pool rows
 // are double-buffered (read row != write row), so readers of the old history never race with the writer of the new one.
-// A thread slides over eight rows of eight channels; with up to four taps weights and earlier rows stay in registers.
+// A thread slides over eight rows of four channels; with up to four taps weights and earlier rows stay in registers.
 #include "f32x2.cuh"
 #include "host_util.h"
 #include "row_ops.cuh"
@@ -37,26 +37,32 @@ __device__ __forceinline__ float rcp_approx(float x) {
   return y;
 }
 
+// four channels of a row
+__device__ __forceinline__ void unpack4(const uint2& q, uint64_t (&v)[2]) {
+  const float2 a = unpack_bf16(q.x), b = unpack_bf16(q.y);
+  v[0] = pack2(a.x, a.y);
+  v[1] = pack2(b.x, b.y);
+}
+
 template <int TAPS>
-__global__ void __launch_bounds__(128, 4)
+__global__ void __launch_bounds__(128)
 conv_rows_kernel(const ConvRows p) {
-  constexpr int RUN = 8, H = TAPS > 1 ? TAPS - 1 : 1, HALF = RUN / 2;
-  const int vecs = p.C / 8;
+  constexpr int RUN = 8, H = TAPS > 1 ? TAPS - 1 : 1;
+  const int vecs = p.C / 4;
   const long idx = (long)blockIdx.x * 128 + threadIdx.x;
-  const int c = (int)(idx % vecs) * 8;
+  const int c = (int)(idx % vecs) * 4;
   const long r0 = idx / vecs * RUN;
   if (r0 >= p.T) return;
   const int taps = TAPS > 0 ? TAPS : p.taps, h = taps - 1;
   const bf16* x = static_cast<const bf16*>(p.x) + c;
   bf16* hist = static_cast<bf16*>(p.hist) + c;
   bf16* out = static_cast<bf16*>(p.out) + c;
-  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   int seq = -1, q0 = 0, q1 = 0, ctx = 0, sin = 0, sout = -1;
-  auto raw_x = [&](int b) {                                  // row b of the portion; negative: history
-    if (b >= 0) return *reinterpret_cast<const uint4*>(x + (long)(q0 + b) * p.ldx);
-    if (ctx + b >= 0) return *reinterpret_cast<const uint4*>(hist + ((long)sin * h + h + b) * p.C);
-    return zero;
+  auto row_x = [&](long row) { return __ldg(reinterpret_cast<const uint2*>(x + row * p.ldx)); };
+  auto past = [&](int b) {                                   // row b < 0 of the portion
+    return ctx + b >= 0 ? *reinterpret_cast<const uint2*>(hist + ((long)sin * h + h + b) * p.C) : make_uint2(0u, 0u);
   };
+  auto raw_x = [&](int b) { return b >= 0 ? row_x(q0 + b) : past(b); };
   auto enter = [&](int s) {                                  // a sequence's numbers
     seq = s;
     q0 = p.q_start[seq];
@@ -73,79 +79,78 @@ conv_rows_kernel(const ConvRows p) {
     }
   };
   auto seq_of = [&](long row) { return min(max(p.row_seq[row], 0), p.num_seqs - 1); };
-  auto finish = [&](float (&o)[8], long row) {
+  auto finish = [&](const uint64_t (&v)[2], long row) {
+    float o[4];
+    unpack2(v[0], o[0], o[1]);
+    unpack2(v[1], o[2], o[3]);
     if (p.act == 1) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) o[e] *= rcp_approx(1.0f + ex2_approx(-1.4426950408889634f * o[e]));
+      for (int e = 0; e < 4; ++e) o[e] *= rcp_approx(1.0f + ex2_approx(-1.4426950408889634f * o[e]));
     }
-    store8<bf16>(out + row * p.C, o);
+    *reinterpret_cast<uint2*>(out + row * p.C) = make_uint2(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]));
   };
   auto new_history = [&](long row) {                         // after the portion's last row
     if (row == q1 - 1 && sout >= 0 && !(p.skip_single && q1 - q0 == 1))
       for (int m = 0; m < h; ++m)
-        *reinterpret_cast<uint4*>(hist + ((long)sout * h + m) * p.C) = raw_x((int)(row - q0) + 1 - h + m);
+        *reinterpret_cast<uint2*>(hist + ((long)sout * h + m) * p.C) = raw_x((int)(row - q0) + 1 - h + m);
   };
-  float bias[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-  if (p.bias) load8<float>(p.bias + c, bias);
+  uint64_t bias[2] = {0ull, 0ull};
+  auto load_pairs = [&](const float* src, uint64_t (&v)[2]) {
+    const float4 f = *reinterpret_cast<const float4*>(src);
+    v[0] = pack2(f.x, f.y);
+    v[1] = pack2(f.z, f.w);
+  };
+  if (p.bias) load_pairs(p.bias + c, bias);
   if constexpr (TAPS == 0) {
     for (long row = r0; row < min(r0 + RUN, (long)p.T); ++row) {
       const int s = seq_of(row);
       if (s != seq) enter(s);
-      float o[8];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) o[e] = bias[e];
+      uint64_t o[2] = {bias[0], bias[1]};
       for (int j = 0; j < taps; ++j) {
-        float f[8], wj[8];
-        const uint4 q = raw_x((int)(row - q0) - h + j);
-        load8<bf16>(reinterpret_cast<const bf16*>(&q), f);
-        load8<float>(p.conv + (long)j * p.C + c, wj);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = fmaf(wj[e], f[e], o[e]);
+        uint64_t f[2], w[2];
+        unpack4(raw_x((int)(row - q0) - h + j), f);
+        load_pairs(p.conv + (long)j * p.C + c, w);
+        o[0] = fma2(w[0], f[0], o[0]);
+        o[1] = fma2(w[1], f[1], o[1]);
       }
       finish(o, row);
       new_history(row);
     }
   } else {
+    // all loads of the run in flight at once, the rows before it as if the portion began earlier
+    uint2 raw[RUN], before[H];
+#pragma unroll
+    for (int i = 0; i < RUN; ++i) raw[i] = row_x(min(r0 + i, (long)p.T - 1));
+#pragma unroll
+    for (int m = 0; m < H; ++m) before[m] = row_x(max(r0 - H + m, 0l));
+    uint64_t w[TAPS][2], win[TAPS][2];                       // win: rows t - taps + 1 .. t, row t at t % TAPS
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_pairs(p.conv + (long)j * p.C + c, w[j]);
     // portions are contiguous: rows that begin and end in the same one need no look at those between
     const int s_first = seq_of(r0);
     const bool same = s_first == seq_of(min(r0 + RUN, (long)p.T) - 1);
-    uint4 raw[HALF];
-#pragma unroll
-    for (int i = 0; i < HALF; ++i) raw[i] = r0 + i < p.T ? *reinterpret_cast<const uint4*>(x + (r0 + i) * p.ldx) : zero;
-    float w[TAPS][8], win[TAPS][8];                          // win: rows t - taps + 1 .. t, row t at t % TAPS
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) load8<float>(p.conv + (long)j * p.C + c, w[j]);
 #pragma unroll
     for (int i = 0; i < RUN; ++i) {
       const long row = r0 + i;
       if (row >= p.T) break;
-      if (i == HALF) {
-#pragma unroll
-        for (int k = 0; k < HALF; ++k) raw[k] = row + k < p.T ? *reinterpret_cast<const uint4*>(x + (row + k) * p.ldx) : zero;
-      }
       const int s = i == 0 || same ? s_first : seq_of(row);
       if (s != seq) {                                        // first row of the run or of a sequence
         enter(s);
         if (TAPS > 1) {
 #pragma unroll
           for (int m = 0; m < H; ++m) {
-            const uint4 q = raw_x((int)(row - q0) - H + m);
-            load8<bf16>(reinterpret_cast<const bf16*>(&q), win[(i + m + 1) % TAPS]);
+            const int b = (int)(row - q0) - H + m;
+            unpack4(b < 0 ? past(b) : (i == 0 ? before[m] : row_x(row - H + m)), win[(i + m + 1) % TAPS]);
           }
         }
       }
-      load8<bf16>(reinterpret_cast<const bf16*>(&raw[i % HALF]), win[i % TAPS]);
-      uint64_t o2[4];
+      unpack4(raw[i], win[i % TAPS]);
+      uint64_t o[2] = {bias[0], bias[1]};
 #pragma unroll
-      for (int e = 0; e < 4; ++e) o2[e] = pack2(bias[2 * e], bias[2 * e + 1]);
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          o2[e] = fma2(pack2(w[j][2 * e], w[j][2 * e + 1]), pack2(win[(i + j + 1) % TAPS][2 * e], win[(i + j + 1) % TAPS][2 * e + 1]), o2[e]);
-      float o[8];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) unpack2(o2[e], o[2 * e], o[2 * e + 1]);
+      for (int j = 0; j < TAPS; ++j) {
+        o[0] = fma2(w[j][0], win[(i + j + 1) % TAPS][0], o[0]);
+        o[1] = fma2(w[j][1], win[(i + j + 1) % TAPS][1], o[1]);
+      }
       finish(o, row);
       new_history(row);
     }
@@ -162,7 +167,7 @@ extern "C" int omni_conv_rows(const ConvRows* args, void* stream) {
   if (p.C <= 0 || (p.C & 7) || (p.ldx & 7) || p.ldx < p.C || p.taps < 1 || !p.conv || !p.x || !p.out || !p.row_seq || p.num_seqs <= 0 ||
       (reinterpret_cast<uintptr_t>(p.x) & 15) || (p.taps > 1 && (!p.hist || !p.state_in || !p.state_out || p.num_state <= 0)))
     return RC_BAD_ARG;
-  const long blocks = ((long)((p.T + 7) / 8) * (p.C / 8) + 127) / 128;
+  const long blocks = ((long)((p.T + 7) / 8) * (p.C / 4) + 127) / 128;
   if (blocks > 0x7fffffffl) return RC_BAD_ARG;
   cudaStream_t st = (cudaStream_t)stream;
   switch (p.taps) {

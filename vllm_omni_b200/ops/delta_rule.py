@@ -142,10 +142,7 @@ def delta_rule(proj, s: DeltaShape, seqs, rule, state, out, *, hist=None, decay=
     wide = s.dp * s.vp > 16384                              # a head's state does not fit the registers of one block
     raw = torch.empty(T, s.v_cols, dtype=proj.dtype, device=proj.device) if chunked or wide else None
     a.raw = P(raw)
-    if not chunked or seqs.n_decode:
-        a.n_list = seqs.n_decode if chunked else seqs.n_seqs
-        a.seq_list = P(seqs.decode_list) if chunked else 0  # none: every sequence
-        nv.check_rc(lib.omni_delta_steps(ctypes.byref(a), kind, bf, c_int(wide), st), "omni_delta_steps")
+    finish = lambda: nv.check_rc(lib.omni_delta_finish(ctypes.byref(a), kind, bf, st), "omni_delta_finish")
     if chunked:
         chunks = seqs.chunks(size)
         a.chunks, a.n_chunks, a.long_list, a.n_long = P(chunks.table), chunks.n, P(chunks.seqs), chunks.n_seqs
@@ -161,9 +158,14 @@ def delta_rule(proj, s: DeltaShape, seqs, rule, state, out, *, hist=None, decay=
             a.u, a.ldu = P(u), u.stride(0)
         a.mats, a.coef = P(mats), P(coef)
         nv.check_rc(nv.lib("delta_chunks").omni_delta_chunks(ctypes.byref(a), kind, c_int(size), st), "omni_delta_chunks")
-    if raw is not None:
-        # rows of single tokens are finished already unless their state was too wide
-        nv.check_rc(lib.omni_delta_finish(ctypes.byref(a), kind, bf, c_int(not wide), st), "omni_delta_finish")
+        if not wide:
+            finish()                                        # rows of single tokens are written over below
+    if not chunked or seqs.n_decode:
+        a.n_list = seqs.n_decode if chunked else seqs.n_seqs
+        a.seq_list = P(seqs.decode_list) if chunked else 0  # none: every sequence
+        nv.check_rc(lib.omni_delta_steps(ctypes.byref(a), kind, bf, c_int(wide), st), "omni_delta_steps")
+    if wide:
+        finish()
     return out
 
 
