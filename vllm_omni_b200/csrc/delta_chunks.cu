@@ -625,34 +625,43 @@ delta_sequence_kernel(const __grid_constant__ CUtensorMap tmU, const __grid_cons
       const uint4* mats = reinterpret_cast<const uint4*>(smem + so + lay.mats) + lane;
       // what the state gives for the chunk's keys (x) and queries (o)
       float x[M][2][4] = {}, o[M][2][4] = {};
-#pragma unroll
-      for (int k = 0; k < KW; ++k) {
-        if (!EXACT && (k0 + k) * 16 >= dp) break;
-        SplitB s;
-        s.from(S[k]);
-#pragma unroll
-        for (int m = 0; m < M; ++m) {
-          uint32_t a[4];
-          dc_ldsm4(st + at_a(0, m, k), a);
-          dc_mma(x[m][0], a, s.h0, s.h1);
-          dc_mma(x[m][1], a, s.l0, s.l1);
-          if (CHANNEL) {
-            dc_ldsm4(st + at_a(1, m, k), a);
-            dc_mma(x[m][1], a, s.h0, s.h1);
-          }
-        }
+      SplitB s[KW];
+      auto queries = [&](int k) {
 #pragma unroll
         for (int m = 0; m < M; ++m) {
           uint32_t a[4];
           dc_ldsm4(st + at_a(CHANNEL ? 2 : 1, m, k), a);
-          dc_mma(o[m][0], a, s.h0, s.h1);
-          dc_mma(o[m][1], a, s.l0, s.l1);
+          dc_mma(o[m][0], a, s[k].h0, s[k].h1);
+          dc_mma(o[m][1], a, s[k].l0, s[k].l1);
           if (CHANNEL) {
             dc_ldsm4(st + at_a(3, m, k), a);
-            dc_mma(o[m][1], a, s.h0, s.h1);
+            dc_mma(o[m][1], a, s[k].h0, s[k].h1);
           }
         }
+      };
+#pragma unroll
+      for (int k = 0; k < KW; ++k) {
+        if (!EXACT && (k0 + k) * 16 >= dp) break;
+        s[k].from(S[k]);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          uint32_t a[4];
+          dc_ldsm4(st + at_a(0, m, k), a);
+          dc_mma(x[m][0], a, s[k].h0, s[k].h1);
+          dc_mma(x[m][1], a, s[k].l0, s[k].l1);
+          if (CHANNEL) {
+            dc_ldsm4(st + at_a(1, m, k), a);
+            dc_mma(x[m][1], a, s[k].h0, s[k].h1);
+          }
+        }
+        if (SPLIT == 2) queries(k);                          // more chains side by side; with one warp they fill later gaps
       }
+      if (SPLIT == 1)
+#pragma unroll
+        for (int k = 0; k < KW; ++k) {
+          if (!EXACT && (k0 + k) * 16 >= dp) break;
+          queries(k);
+        }
 #pragma unroll
       for (int m = 0; m < M; ++m)
 #pragma unroll
@@ -661,19 +670,24 @@ delta_sequence_kernel(const __grid_constant__ CUtensorMap tmU, const __grid_cons
           o[m][0][e] += o[m][1][e];
           x[m][1][e] = o[m][1][e] = 0.f;
         }
-      if constexpr (SPLIT == 2) {
+      if constexpr (SPLIT == 2) {                            // what the other half of the key channels gives
         auto as4 = [](const float (&v)[4]) { return make_float4(v[0], v[1], v[2], v[3]); };
+        auto plus = [](float (&v)[4], const float4& a) {
+          v[0] += a.x;
+          v[1] += a.y;
+          v[2] += a.z;
+          v[3] += a.w;
+        };
         float4(*mine)[32] = s_ex[i & 1][warp], (*other)[32] = s_ex[i & 1][warp ^ GROUPS];
         mine[0][lane] = as4(x[0][0]);
         mine[1][lane] = as4(x[1][0]);
         mine[2][lane] = kh ? as4(o[0][0]) : as4(o[1][0]);
         asm volatile("bar.sync %0, 64;" ::"r"(1 + grp) : "memory");
-        const float4 a = other[0][lane], b = other[1][lane], c = other[2][lane];
-        x[0][0][0] += a.x; x[0][0][1] += a.y; x[0][0][2] += a.z; x[0][0][3] += a.w;
-        x[1][0][0] += b.x; x[1][0][1] += b.y; x[1][0][2] += b.z; x[1][0][3] += b.w;
-        float (&mo)[4] = o[0][0], (&so_)[4] = o[1][0];         // only one of the two is used
-        mo[0] += c.x; mo[1] += c.y; mo[2] += c.z; mo[3] += c.w;
-        so_[0] += c.x; so_[1] += c.y; so_[2] += c.z; so_[3] += c.w;
+        plus(x[0][0], other[0][lane]);
+        plus(x[1][0], other[1][lane]);
+        const float4 c = other[2][lane];                     // only one of the two tiles is finished here
+        plus(o[0][0], c);
+        plus(o[1][0], c);
       }
       if (SPLIT == 1 && warp == 0) {                         // into the place of chunk i - 1
         if (elect_one() && i + stages - 1 < n_chunks) copy(i + stages - 1);

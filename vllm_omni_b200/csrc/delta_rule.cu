@@ -214,15 +214,16 @@ delta_finish_kernel(const DeltaRule p, const int lph) {
   const int lane = threadIdx.x & (lph - 1), h = blockIdx.y;
   const int t0 = (blockIdx.x * (256 / lph) + threadIdx.x / lph) * ROWS;
   const float* gain = p.gain + (long)h * p.gain_hs;
-  auto opened = [&](float (&v)[8], const float (&z)[8], float s, int c) {
-    float gn[8];
-    load8<float>(gain + c, gn);
+  const float inv = 1.0f / (float)p.dv;
+  auto opened = [&](float (&v)[8], const float (&z)[8], const float (&gn)[8], float s) {
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
-      const float open = sizeof(T) == 4 ? dr_sigmoid(z[e]) : __fdividef(1.0f, 1.0f + __expf(-z[e]));
-      v[e] *= s * gn[e] * (CHANNEL ? open : z[e] * open);
+      const float open = sizeof(T) == 4 ? dr_sigmoid(z[e]) : dr_rcp(1.0f + dr_ex2(-1.4426950408889634f * z[e]));
+      v[e] *= (s * gn[e]) * (CHANNEL ? open : z[e] * open);
     }
   };
+  float gn[8];
+  if (ONE && lane * 8 < p.vp) load8<float>(gain + lane * 8, gn);
   float v[ROWS][8], z[ROWS][8], ss[ROWS];
 #pragma unroll
   for (int i = 0; i < ROWS; ++i) {
@@ -252,15 +253,17 @@ delta_finish_kernel(const DeltaRule p, const int lph) {
   for (int i = 0; i < ROWS; ++i) {
     const long row = t0 + i;
     if (row >= p.T) return;
-    const float s = rms_scale(ss[i], p.dv, p.eps);
+    const float s = sizeof(T) == 4 ? rms_scale(ss[i], p.dv, p.eps) : rsqrtf(fmaf(ss[i], inv, p.eps));
     T* out = static_cast<T*>(p.out) + row * p.ldo + (long)h * p.vp;
     for (int c = lane * 8; c < p.vp; c += lph * 8) {
       if (!ONE) {
         load8<T>(static_cast<const T*>(p.raw) + row * p.H * p.vp + (long)h * p.vp + c, v[i]);
         load8<T>(static_cast<const T*>(p.proj) + row * p.ldp + p.g_col + (long)h * p.vp + c, z[i]);
       }
-      opened(v[i], z[i], s, c);
+      if (!ONE) load8<float>(gain + c, gn);
+      opened(v[i], z[i], gn, s);
       store8<T>(out + c, v[i]);
+      if (ONE) break;
     }
   }
 }

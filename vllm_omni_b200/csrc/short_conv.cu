@@ -48,11 +48,9 @@ template <int TAPS>
 __global__ void __launch_bounds__(128)
 conv_rows_kernel(const ConvRows p) {
   constexpr int RUN = 8, H = TAPS > 1 ? TAPS - 1 : 1;
-  const int vecs = p.C / 4;
-  const long idx = (long)blockIdx.x * 128 + threadIdx.x;
-  const int c = (int)(idx % vecs) * 4;
-  const long r0 = idx / vecs * RUN;
-  if (r0 >= p.T) return;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 4;
+  const long r0 = (long)blockIdx.y * RUN;
+  if (c >= p.C) return;
   const int taps = TAPS > 0 ? TAPS : p.taps, h = taps - 1;
   const bf16* x = static_cast<const bf16*>(p.x) + c;
   bf16* hist = static_cast<bf16*>(p.hist) + c;
@@ -167,15 +165,15 @@ extern "C" int omni_conv_rows(const ConvRows* args, void* stream) {
   if (p.C <= 0 || (p.C & 7) || (p.ldx & 7) || p.ldx < p.C || p.taps < 1 || !p.conv || !p.x || !p.out || !p.row_seq || p.num_seqs <= 0 ||
       (reinterpret_cast<uintptr_t>(p.x) & 15) || (p.taps > 1 && (!p.hist || !p.state_in || !p.state_out || p.num_state <= 0)))
     return RC_BAD_ARG;
-  const long blocks = ((long)((p.T + 7) / 8) * (p.C / 4) + 127) / 128;
-  if (blocks > 0x7fffffffl) return RC_BAD_ARG;
+  const dim3 blocks((p.C / 4 + 127) / 128, (p.T + 7) / 8);
+  if (blocks.y > 65535) return RC_TOO_LARGE;
   cudaStream_t st = (cudaStream_t)stream;
   switch (p.taps) {
-    case 1: conv_rows_kernel<1><<<(unsigned)blocks, 128, 0, st>>>(p); break;
-    case 2: conv_rows_kernel<2><<<(unsigned)blocks, 128, 0, st>>>(p); break;
-    case 3: conv_rows_kernel<3><<<(unsigned)blocks, 128, 0, st>>>(p); break;
-    case 4: conv_rows_kernel<4><<<(unsigned)blocks, 128, 0, st>>>(p); break;
-    default: conv_rows_kernel<0><<<(unsigned)blocks, 128, 0, st>>>(p); break;
+    case 1: conv_rows_kernel<1><<<blocks, 128, 0, st>>>(p); break;
+    case 2: conv_rows_kernel<2><<<blocks, 128, 0, st>>>(p); break;
+    case 3: conv_rows_kernel<3><<<blocks, 128, 0, st>>>(p); break;
+    case 4: conv_rows_kernel<4><<<blocks, 128, 0, st>>>(p); break;
+    default: conv_rows_kernel<0><<<blocks, 128, 0, st>>>(p); break;
   }
   return (int)cudaGetLastError();
 }
