@@ -3,6 +3,7 @@ logits) against the plain restatements, one mechanism at a time."""
 import pytest
 import torch
 
+import fikizen_oracle as F
 import milivik_oracle as M
 import tavulix_oracle as O
 from vllm_omni_b200.models.seq_table import SeqTable
@@ -308,3 +309,66 @@ def test_scaled_logits(device, dtype):
     z = (torch.randn(3, 304) * 8).to(dtype)
     _close(lm.logit_softcap(z.to(device), None, 300, 0.4), 0.4 * z[:, :300].double(), torch.float32)
     _close(lm.logit_softcap(z.to(device), 5.0, 300, 0.4), O.soft_cap(0.4 * z[:, :300].double(), 5.0), torch.float32)
+
+
+# ------------------------------------------------------------------------------ row norms, rotation, pages
+@pytest.mark.parametrize("device,dtype", DEVICES)
+@pytest.mark.parametrize("shape", [(4, 2, 24, 20, 16), (3, 1, 18, 34, 18), (16, 4, 128, 128, 64), (6, 6, 10, 12, 2), (2, 1, 40, 136, 0), (40, 8, 128, 128, 128),
+                                   (1, 1, 2, 1, 2)])
+@pytest.mark.parametrize("normed", [False, True])
+def test_rotary_heads(device, dtype, shape, normed):
+    """Norms over all heads' channels at once, halves rotated against each other (stored as interleaved pairs), value heads
+    over their root mean square; rows without a slot leave no trace in the pages."""
+    from vllm_omni_b200.ops import stream
+    H, G, d, dv, rot = shape
+    T, BS, up = 11, 4, lambda n: (n + 15) // 16 * 16
+    hs = lm.HeadShape(H, G, d, dv, up(d), up(dv))
+    torch.manual_seed(H + d)
+    q, k, v = torch.randn(T, H, d).to(dtype), torch.randn(T, G, d).to(dtype), (0.3 * torch.randn(T, G, dv)).to(dtype)
+    order = torch.cat([torch.arange(rot).view(2, -1).T.reshape(-1), torch.arange(rot, d)]).long()      # stored channel <- checkpoint channel
+    pos = torch.arange(T) * 37
+    qg, kg = torch.rand(H, d) + 0.5, torch.rand(G, d) + 0.5
+    pad = lambda x, n: _pad(x.float(), n).reshape(x.shape[0], -1)
+    proj = torch.cat([pad(q[..., order], hs.dp), pad(k[..., order], hs.dp), pad(v, hs.vp), torch.full((T, 8), 5.0)], 1).to(device, dtype)
+    slots = torch.randperm(16)[:T].int()
+    slots[3] = -1
+    kc, vc = (torch.full((4, BS, G, n), 9.0, dtype=dtype, device=device) for n in (hs.dp, hs.vp))
+    turns = stream.rotary_rows(pos.to(device), 500.0, rot) if rot else None
+    kw = dict(q_gain=_pad(qg[:, order], hs.dp).reshape(-1).to(device), k_gain=_pad(kg[:, order], hs.dp).reshape(-1).to(device), v_norm=True,
+              v_mult=1.3, eps=1e-3) if normed else {}
+    out = lm.rotary_heads(proj, hs, slots.to(device), kc, vc, turns, rot, **kw)
+    qw, kw_, vw = q.double(), k.double(), v.double()
+    if normed:
+        qw = (F.rms_unit(qw.reshape(T, -1), 1e-3) * qg.double().reshape(-1)).reshape(T, H, d)
+        kw_ = (F.rms_unit(kw_.reshape(T, -1), 1e-3) * kg.double().reshape(-1)).reshape(T, G, d)
+        vw = 1.3 * F.rms_unit(vw, 1e-3)
+    qw, kw_ = (F.rotate_halves(x, pos.double(), 500.0, rot)[..., order] if rot else x for x in (qw, kw_))
+    _close(out[..., :d], qw, dtype)
+    assert not out[..., d:].any()
+    for t in range(T):
+        if slots[t] < 0:
+            continue
+        page, at = divmod(int(slots[t]), BS)
+        _close(kc[page, at, :, :d], kw_[t], dtype)
+        _close(vc[page, at, :, :dv], vw[t], dtype)
+    used = set(slots.tolist())
+    for s in set(range(16)) - used:
+        assert (kc.view(16, -1)[s] == 9).all() and (vc.view(16, -1)[s] == 9).all()
+
+
+@pytest.mark.parametrize("device,dtype", DEVICES)
+@pytest.mark.parametrize("act", ["tanh", "xielu"])
+@pytest.mark.parametrize("rows", [3, 300])
+def test_activations_of_a_product(device, dtype, act, rows):
+    """Small, ordinary and large arguments on either side of zero."""
+    from vllm_omni_b200.ops import gemm
+    torch.manual_seed(rows)
+    x, w = torch.randn(rows, 40).to(dtype), torch.randn(56, 40).to(dtype)
+    w *= torch.logspace(-6, 1, 56)[:, None].to(dtype)
+    p, q = torch.tensor(0.7), torch.tensor(-0.4)
+    coef = torch.stack([F.softplus(p), 0.5 + F.softplus(q)])
+    z = x.double() @ w.double().T
+    want = torch.tanh(z) if act == "tanh" else F.xielu(z, p.double(), q.double())
+    got = gemm.linear(x.to(device), w.to(device), act=act, coef=coef.to(device) if act == "xielu" else None).double().cpu()
+    err = (got - want).abs() / (want.abs() + 1e-9 + z.abs().mean(0) * 1e-6)
+    assert err.max() < (1e-4 if dtype == torch.float32 else 0.02), float(err.max())

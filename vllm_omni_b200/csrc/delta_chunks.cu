@@ -889,9 +889,9 @@ static int launch_sequence(const DeltaRule& p, cudaStream_t st) {
 
 template <bool CHANNEL, int KS>
 static int launch_exact(const DeltaRule& p, cudaStream_t st) {
-  // SMs to spare: two warps to eight columns
+  // few blocks: two warps to eight columns
   const long blocks = (long)((p.vp + 4 * DC_WARPS - 1) / (4 * DC_WARPS)) * p.H * p.n_long;
-  return blocks <= sm_count() ? launch_sequence<CHANNEL, KS, true, 2, 2>(p, st) : launch_sequence<CHANNEL, KS, true, 2, 1>(p, st);
+  return blocks <= (CHANNEL ? 1l : 2l) * sm_count() ? launch_sequence<CHANNEL, KS, true, 2, 2>(p, st) : launch_sequence<CHANNEL, KS, true, 2, 1>(p, st);
 }
 
 template <bool CHANNEL, int M>

@@ -292,11 +292,17 @@ class FikizenDecoder(PackedDecoder):
             t.update(layer.targets(f"l{i}.", D))
         return t
 
+    def load_weights(self, weights) -> set:
+        self._ranked = {}                                       # layers whose rank a tensor of this checkpoint has told
+        return super().load_weights(weights)
+
     def resize(self, name: str, shape) -> None:
-        mix = self.owners[name.split(".")[0][1:]].mix
+        i = name.split(".")[0][1:]
         n = shape[0] if name.endswith("w1") else shape[1]
-        if n != mix.rank:
-            mix.set_rank(n)
+        if self._ranked.setdefault(i, n) != n:
+            raise ValueError(f"{name}: rank {n}, but {self._ranked[i]} in the other tensor")
+        if n != self.owners[i].mix.rank:
+            self.owners[i].mix.set_rank(n)
 
     def weights_loaded(self) -> None:
         for layer in self.owners.values():
