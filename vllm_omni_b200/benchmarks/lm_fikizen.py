@@ -124,7 +124,7 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
     ids, emb = torch.randint(0, VOCAB, (T,), device=dev), rnd(VOCAB, width)
     row("embedding", "fikizen (table + norm)", lambda: stream.embed_rows(ids, emb, nxt), bytes_=8.0 * T * width)
     # ---- feed-forward
-    coef, up = torch.tensor([0.9, 1.3], device=dev), rnd(F_, width) * width ** -0.5
+    coef, up = (0.9, 1.3), rnd(F_, width) * width ** -0.5
     coef4 = torch.tensor([0.5, 0.3, 0.1, 0.0], device=dev)
     z = rnd(T, F_)
     for rows_, tag in ((T, "prompt"), (B, "64 rows")):

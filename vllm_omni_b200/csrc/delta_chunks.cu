@@ -896,7 +896,7 @@ static int launch_exact(const DeltaRule& p, cudaStream_t st) {
 
 template <bool CHANNEL, int M>
 static int launch_chunks(const DeltaRule& p, cudaStream_t st) {
-  if (CHANNEL) delta_prepare_channel_kernel<M><<<dim3(p.n_chunks, p.H), 32 * M, 0, st>>>(p);
+  if constexpr (CHANNEL) delta_prepare_channel_kernel<M><<<dim3(p.n_chunks, p.H), 32 * M, 0, st>>>(p);
   else delta_prepare_gated_kernel<M><<<dim3(p.n_chunks, (p.H * M + 3) / 4), 128, 0, st>>>(p);
   if (int e = (int)cudaGetLastError()) return e;
   if constexpr (M == 1) {

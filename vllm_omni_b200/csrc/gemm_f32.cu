@@ -16,7 +16,7 @@ struct GemmF32Batch {
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ A, long lda, const float* __restrict__ W, long ldw, float* __restrict__ C,
                 long ldc, int M, int N, int K, const float* __restrict__ bias, int act,
-                const float* __restrict__ coef, GemmF32Batch b) {
+                float c0, float c1, GemmF32Batch b) {
   A += blockIdx.z * b.a;
   W += blockIdx.z * b.w;
   C += blockIdx.z * b.c;
@@ -61,7 +61,7 @@ gemm_f32_kernel(const float* __restrict__ A, long lda, const float* __restrict__
         } else if (act == 4) {
           v = tanhf(v);
         } else if (act == 5) {                             // xIELU
-          v = fmaf(0.5f, v, v > 0.f ? coef[0] * v * v : coef[1] * (expm1f(v) - v));
+          v = fmaf(0.5f, v, v > 0.f ? c0 * v * v : c1 * (expm1f(v) - v));
         }
         C[(long)m * ldc + n] = v;
       }
@@ -71,21 +71,19 @@ gemm_f32_kernel(const float* __restrict__ A, long lda, const float* __restrict__
 }  // namespace omni
 
 // `batch` problems of one shape whose operands lie the given strides apart; act: 0 none, 3 squared ReLU, 4 tanh, 5 xIELU with
-// the two numbers `coef` (c0 z^2 + z / 2 above zero, c1 (e^z - 1 - z) + z / 2 below).
+// two numbers (c0 z^2 + z / 2 above zero, c1 (e^z - 1 - z) + z / 2 below).
 extern "C" int omni_gemm_f32_batched(const float* A, long lda, const float* W, long ldw, float* C, long ldc, int M, int N, int K,
                                      const float* bias, int act, int batch, long a_stride, long w_stride, long c_stride,
-                                     long bias_stride, const float* coef, void* stream) {
+                                     long bias_stride, float c0, float c1, void* stream) {
   if (M <= 0 || N <= 0 || batch <= 0) return omni::RC_OK;
-  if (K <= 0 || (M + omni::FB - 1) / omni::FB > 65535 || batch > 65535 || act < 0 || act == 1 || act == 2 || act > 5 ||
-      (act == 5 && !coef))
-    return omni::RC_BAD_ARG;
+  if (K <= 0 || (M + omni::FB - 1) / omni::FB > 65535 || batch > 65535 || act < 0 || act == 1 || act == 2 || act > 5) return omni::RC_BAD_ARG;
   dim3 grid((N + omni::FB - 1) / omni::FB, (M + omni::FB - 1) / omni::FB, batch);
   const omni::GemmF32Batch b = {a_stride, w_stride, c_stride, bias_stride};
-  omni::gemm_f32_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(A, lda, W, ldw, C, ldc, M, N, K, bias, act, coef, b);
+  omni::gemm_f32_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(A, lda, W, ldw, C, ldc, M, N, K, bias, act, c0, c1, b);
   return (int)cudaGetLastError();
 }
 
 extern "C" int omni_gemm_f32(const float* A, long lda, const float* W, long ldw, float* C, long ldc, int M, int N, int K,
                              const float* bias, void* stream) {
-  return omni_gemm_f32_batched(A, lda, W, ldw, C, ldc, M, N, K, bias, 0, 1, 0, 0, 0, 0, nullptr, stream);
+  return omni_gemm_f32_batched(A, lda, W, ldw, C, ldc, M, N, K, bias, 0, 1, 0, 0, 0, 0, 0.f, 0.f, stream);
 }

@@ -66,7 +66,7 @@ struct GemmEpilogue {
   // pointer already addresses the slot reserved for THIS rank's partial sums on the owner).
   int scatter_rows;
   __nv_bfloat16* peer_out[16];
-  const float* act_coef;          // ACT_XIELU: [2]
+  float act_c0, act_c1;           // ACT_XIELU
 };
 
 // Implicit-GEMM convolution (stride 1, "same" padding, NHWC bf16): the M dimension is the output
@@ -148,12 +148,19 @@ __device__ __forceinline__ __nv_bfloat16* epilogue_dest(int row, int col0, __nv_
   return cbase + (size_t)row * ldc + dcol;
 }
 
-// c0 z^2 + z / 2 above zero, c1 (e^z - 1 - z) + z / 2 below; near zero e^z - 1 - z from its series, where it would cancel
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// c0 z^2 + z / 2 above zero, c1 (e^z - 1 - z) + z / 2 below; near zero, where e^z - 1 - z would cancel, the first terms of its
+// series (the next one is below 1e-5 of the result)
 __device__ __forceinline__ float xielu(float z, float c0, float c1) {
-  const float m = fminf(z, 0.f);
-  const float series = m * m * fmaf(m, fmaf(m, fmaf(m, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
-  const float below = m > -0.125f ? series : __expf(m) - 1.0f - m;
-  return fmaf(0.5f, z, z > 0.f ? c0 * z * z : c1 * below);
+  // both branches are computed: a choice between numbers, not between paths
+  const float q = z * z, e = ex2_approx(1.4426950408889634f * fminf(z, 0.f));
+  const float far = c1 * ((e - 1.0f) - z), close = (c1 * q) * fmaf(z, 1.f / 6.f, 0.5f), above = c0 * q;
+  const float below = z > -0.03125f ? close : far;
+  return fmaf(0.5f, z, z > 0.f ? above : below);
 }
 
 // tanh for values that are rounded to bf16 next
@@ -198,9 +205,8 @@ __device__ __forceinline__ void epilogue_math32(const uint32_t (&v)[32], int row
 #pragma unroll
         for (int e = 0; e < 8; ++e) x[e] = tanh_short(x[e]);
       } else if (epi.act == ACT_XIELU) {
-        const float c0 = epi.act_coef[0], c1 = epi.act_coef[1];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = xielu(x[e], c0, c1);
+        for (int e = 0; e < 8; ++e) x[e] = xielu(x[e], epi.act_c0, epi.act_c1);
       }
       if (gate_row) {
         uint4 g = *reinterpret_cast<const uint4*>(gate_row + col0 + j * 8);
@@ -1052,15 +1058,14 @@ static int pick_bn(int M, int N, int ctas) {
 // choose the tile width.
 // `sync` (may be null): arrivals this launch waits for before reading A, and / or reports to the
 // group after its peer stores (see peer_signal.cuh).
-// `act_coef`: the two numbers of act 5 (xIELU).
+// `act_c0`, `act_c1`: the numbers of act 5 (xIELU).
 extern "C" int omni_gemm_bf16_coef(const void* A, int lda, const void* W, int ldw, void* C, int ldc,
                                    int M, int N, int K, const void* bias, const void* residual, int ldr,
                                    const void* gate, int gate_stride, int rows_per_batch, int act,
                                    int c_rows_per_batch, long c_batch_stride, int scatter_P, int scatter_G,
-                                   int scatter_rows, void* const* peer_out, int force_bn, const float* act_coef,
+                                   int scatter_rows, void* const* peer_out, int force_bn, float act_c0, float act_c1,
                                    const omni::OmniSync* sync, int* status, void* stream) {
   using namespace omni;
-  if (act == ACT_XIELU && act_coef == nullptr) return RC_BAD_ARG;
   if (M <= 0 || N <= 0 || K <= 0) return sync ? RC_BAD_ARG : RC_OK;
   if ((K & 7) || (N & 7) || (lda & 7) || (ldw & 7) || (ldc & 7) || (ldr & 7) || (gate_stride & 7))
     return RC_BAD_ARG;
@@ -1077,7 +1082,8 @@ extern "C" int omni_gemm_bf16_coef(const void* A, int lda, const void* W, int ld
   epi.gate_stride = gate_stride;
   epi.rows_per_batch = rows_per_batch > 0 ? rows_per_batch : 1;
   epi.act = act;
-  epi.act_coef = act_coef;
+  epi.act_c0 = act_c0;
+  epi.act_c1 = act_c1;
   epi.c_rows_per_batch = c_rows_per_batch;
   epi.c_batch_stride = c_batch_stride;
   if (c_rows_per_batch > 0 && (c_batch_stride & 7)) return RC_BAD_ARG;
@@ -1132,7 +1138,7 @@ extern "C" int omni_gemm_bf16_sync(const void* A, int lda, const void* W, int ld
                                    int scatter_rows, void* const* peer_out, int force_bn, const omni::OmniSync* sync,
                                    int* status, void* stream) {
   return omni_gemm_bf16_coef(A, lda, W, ldw, C, ldc, M, N, K, bias, residual, ldr, gate, gate_stride, rows_per_batch, act,
-                             c_rows_per_batch, c_batch_stride, scatter_P, scatter_G, scatter_rows, peer_out, force_bn, nullptr,
+                             c_rows_per_batch, c_batch_stride, scatter_P, scatter_G, scatter_rows, peer_out, force_bn, 0.f, 0.f,
                              sync, status, stream);
 }
 
@@ -1155,7 +1161,7 @@ extern "C" int omni_conv1d_nlc_bf16(const void* x, long ldx, long x_bs, const vo
                                     int T_out, int Cin, int Cout, int k, int dil, int pad, const void* bias,
                                     const void* residual, int ldr, int act, int* status, void* stream) {
   using namespace omni;
-  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has operands of its own
+  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has numbers of its own
   if (B <= 0 || T_in <= 0 || T_out <= 0 || Cin <= 0 || Cout <= 0) return RC_OK;
   if (k < 1 || k > 64 || dil < 1 || (Cout & 7) || (ldx & 7) || (x_bs & 7) || (ldy & 7) || (ldr & 7)) return RC_BAD_ARG;
   EncodeTiledFn enc = get_encode_tiled();
@@ -1213,7 +1219,7 @@ struct OmniGemmDesc {
 
 static int desc_epilogue(const OmniGemmDesc& d, omni::GemmEpilogue& epi) {
   if ((d.lda & 7) || (d.ldw & 7) || (d.ldc & 7) || (d.ldr & 7) || (d.gate_stride & 7)) return omni::RC_BAD_ARG;
-  if (d.act == omni::ACT_XIELU) return omni::RC_BAD_ARG;      // has operands of its own
+  if (d.act == omni::ACT_XIELU) return omni::RC_BAD_ARG;      // has numbers of its own
   if (d.gate && d.rows_per_batch <= 0) return omni::RC_BAD_ARG;
   if (d.c_rows_per_batch > 0 && (d.c_batch_stride & 7)) return omni::RC_BAD_ARG;
   epi = omni::GemmEpilogue{};
@@ -1288,7 +1294,7 @@ extern "C" int omni_gemm_bf16_grouped(const void* A, int lda, const void* W, int
                                       int M, int N, int K, const int* tile_expert, int act, int force_bn,
                                       int* status, void* stream) {
   using namespace omni;
-  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has operands of its own
+  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has numbers of its own
   if (M <= 0 || N <= 0 || K <= 0) return RC_OK;
   if ((K & 7) || (N & 7) || (lda & 7) || (ldc & 7) || (M % BM) || tile_expert == nullptr) return RC_BAD_ARG;
   CUtensorMap tmA;
@@ -1318,7 +1324,7 @@ extern "C" int omni_gemm_bf16_grouped_compact(const void* A, int lda, const void
                                               const int* tile_rows, int num_tiles, int act, int force_bn, int* status,
                                               void* stream) {
   using namespace omni;
-  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has operands of its own
+  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has numbers of its own
   if (M <= 0 || N <= 0 || K <= 0 || num_tiles <= 0) return RC_OK;
   if ((K & 7) || (N & 7) || (lda & 7) || (ldc & 7) || !tile_expert || !tile_row0 || !tile_rows) return RC_BAD_ARG;
   CUtensorMap tmA;
@@ -1350,7 +1356,7 @@ extern "C" int omni_conv2d_nhwc_bf16(const void* x, long ldx, const void* w, voi
                                      int Cin, int Cout, int ksize, const void* bias, const void* residual, int ldr,
                                      int act, int* status, void* stream) {
   using namespace omni;
-  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has operands of its own
+  if (act == ACT_XIELU) return RC_BAD_ARG;                   // has numbers of its own
   if (Nimg <= 0 || H <= 0 || W <= 0 || Cin <= 0 || Cout <= 0) return RC_OK;
   if ((ksize != 1 && ksize != 3) || (Cout & 7) || (ldx & 7) || (ldy & 7) || (ldr & 7)) return RC_BAD_ARG;
   EncodeTiledFn enc = get_encode_tiled();

@@ -560,34 +560,39 @@ struct RotaryHeads {
 };
 
 template <typename T, int NV>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(256)
 rotary_heads_kernel(const RotaryHeads p) {
   extern __shared__ float s_v[];                            // sums of squares of the value vectors
   __shared__ float sh[64];
   const long row = blockIdx.x;
   const int nq = p.H * p.dp, nk = p.G * p.dp, C = nq + nk + p.G * p.vp;
   const T* proj = static_cast<const T*>(p.proj) + row * p.ldp;
-  float v[NV][8];
-  float ss[2] = {0.f, 0.f};                                 // of the query row, of the key row
+  Raw8<T> raw[NV];                                          // as loaded: half the registers for bf16
+  int slot = p.slots[row];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * 8;
-    if (c >= C) continue;
-    load8<T>(proj + c, v[i]);
-    float s = 0.f;
-#pragma unroll
-    for (int e = 0; e < 8; ++e) s = fmaf(v[i][e], v[i][e], s);
-    if (c < nq) ss[0] += s;
-    else if (c < nq + nk) ss[1] += s;
-    else if (p.v_norm) s_v[(c - nq - nk) / 8] = s;
+    if (c < C) raw[i] = *reinterpret_cast<const Raw8<T>*>(proj + c);
   }
   float sq = 1.f, sk = 1.f;
   if (p.q_gain || p.k_gain || p.v_norm) {                   // uniform
+    float ss[2] = {0.f, 0.f};                               // of the query row, of the key row
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 8;
+      if (c >= C) continue;
+      float v[8], s = 0.f;
+      unraw8<T>(raw[i], v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
+      if (c < nq) ss[0] += s;
+      else if (c < nq + nk) ss[1] += s;
+      else if (p.v_norm) s_v[(c - nq - nk) / 8] = s;
+    }
     block_sum<2>(ss, sh);                                   // also: the value sums are in place
     sq = rms_scale(ss[0], p.nq, p.eps);
     sk = rms_scale(ss[1], p.nk, p.eps);
   }
-  int slot = p.slots[row];
   if (slot >= p.num_slots) {
     if (p.status) atomicCAS(p.status, 0, (int)ERR_BOUNDS);
     slot = -1;
@@ -597,6 +602,8 @@ rotary_heads_kernel(const RotaryHeads p) {
   for (int i = 0; i < NV; ++i) {
     const int c = (i * blockDim.x + threadIdx.x) * 8;
     if (c >= C) continue;
+    float v[8];
+    unraw8<T>(raw[i], v);
     if (c >= nq + nk) {
       const int cv = c - nq - nk;
       float s = p.v_mult;
@@ -607,27 +614,35 @@ rotary_heads_kernel(const RotaryHeads p) {
         s *= rms_scale(t, p.vdim, p.eps);
       }
 #pragma unroll
-      for (int e = 0; e < 8; ++e) v[i][e] *= s;
-      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + (long)slot * p.G * p.vp + cv, v[i]);
+      for (int e = 0; e < 8; ++e) v[e] *= s;
+      if (slot >= 0) store8<T>(static_cast<T*>(p.v_cache) + (long)slot * p.G * p.vp + cv, v);
       continue;
     }
     const bool is_q = c < nq;
     const int ck = is_q ? c : c - nq;
     const float* gain = is_q ? p.q_gain : p.k_gain;
-    if (gain) scale_gain8(v[i], is_q ? sq : sk, gain, 1, ck);
+    if (gain) scale_gain8(v, is_q ? sq : sk, gain, 1, ck);
     const int in = ck % p.dp;
-    if (in < p.rot) {
+    if (in + 8 <= p.rot && (p.rot & 3) == 0) {              // rows of turns on 16 bytes
+      float t[8];                                           // four pairs of cos and sin
+      load8<float>(turns + in, t);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        const float a = v[e], b = v[e + 1];
+        v[e] = a * t[e] - b * t[e + 1];
+        v[e + 1] = b * t[e] + a * t[e + 1];
+      }
+    } else {
 #pragma unroll
       for (int e = 0; e < 8; e += 2) {
         if (in + e >= p.rot) break;
-        const float2 t = *reinterpret_cast<const float2*>(turns + in + e);
-        const float a = v[i][e], b = v[i][e + 1];
-        v[i][e] = a * t.x - b * t.y;
-        v[i][e + 1] = b * t.x + a * t.y;
+        const float a = v[e], b = v[e + 1], co = turns[in + e], si = turns[in + e + 1];
+        v[e] = a * co - b * si;
+        v[e + 1] = b * co + a * si;
       }
     }
-    if (is_q) store8<T>(static_cast<T*>(p.q_out) + row * nq + ck, v[i]);
-    else if (slot >= 0) store8<T>(static_cast<T*>(p.k_cache) + (long)slot * nk + ck, v[i]);
+    if (is_q) store8<T>(static_cast<T*>(p.q_out) + row * nq + ck, v);
+    else if (slot >= 0) store8<T>(static_cast<T*>(p.k_cache) + (long)slot * nk + ck, v);
   }
 }
 
@@ -756,17 +771,19 @@ extern "C" int omni_rotary_heads(const RotaryHeads* args, int is_bf16, void* str
   if (p.H <= 0 || p.G <= 0 || (p.dp & 7) || (p.vp & 7) || p.dp <= 0 || p.vp <= 0 || (p.ldp & 7) || (p.rot & 1) || p.rot < 0 ||
       p.rot > p.dp || (p.rot && !p.turns) || !p.slots || !p.q_out || !p.k_cache || !p.v_cache || p.nq <= 0 || p.nk <= 0 || p.vdim <= 0)
     return RC_BAD_ARG;
-  const int C = (p.H + p.G) * p.dp + p.G * p.vp;
-  int threads, nv;
-  if (C > p.ldp || !row_shape(C, threads, nv)) return RC_BAD_ARG;
+  const int C = (p.H + p.G) * p.dp + p.G * p.vp, vec = C / 8;
+  if (C > p.ldp || vec > 256 * 16) return RC_BAD_ARG;
+  const int nv = vec <= 256 ? 1 : (vec <= 512 ? 2 : (vec <= 1024 ? 4 : 16));
+  const int threads = ((vec + nv - 1) / nv + 31) / 32 * 32;
   const int smem = p.v_norm ? p.G * p.vp / 8 * 4 : 0;
   if (smem > 47 * 1024) return RC_TOO_LARGE;
   cudaStream_t st = (cudaStream_t)stream;
-#define OMNI_ROTARY(ELT)                                                                \
+#define OMNI_ROTARY(ELT)                                                              \
   do {                                                                                \
-    if (nv == 1) rotary_heads_kernel<ELT, 1><<<p.T, threads, smem, st>>>(p);            \
-    else if (nv == 2) rotary_heads_kernel<ELT, 2><<<p.T, threads, smem, st>>>(p);       \
-    else rotary_heads_kernel<ELT, 4><<<p.T, threads, smem, st>>>(p);                    \
+    if (nv == 1) rotary_heads_kernel<ELT, 1><<<p.T, threads, smem, st>>>(p);          \
+    else if (nv == 2) rotary_heads_kernel<ELT, 2><<<p.T, threads, smem, st>>>(p);     \
+    else if (nv == 4) rotary_heads_kernel<ELT, 4><<<p.T, threads, smem, st>>>(p);     \
+    else rotary_heads_kernel<ELT, 16><<<p.T, threads, smem, st>>>(p);                 \
   } while (0)
   if (is_bf16) OMNI_ROTARY(bf16); else OMNI_ROTARY(float);
 #undef OMNI_ROTARY

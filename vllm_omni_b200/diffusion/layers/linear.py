@@ -44,7 +44,7 @@ class FusedLinear(nn.Module):
             y = gemm.linear(x, self.weight, self.bias)
             for (A, B, scale) in self.lora:
                 y = y + scale * gemm.linear(gemm.linear(x, A), B)
-            y = _epilogue(y, act, residual, gate, out, kw.get("coef"))
+            y = _epilogue(y, act, residual, gate, out, kw.get("coef", (0.0, 0.0)))
         else:
             y = gemm.linear(x, self.weight, self.bias, act=act, residual=residual, gate=gate, out=out, **kw)
         return y
@@ -53,7 +53,7 @@ class FusedLinear(nn.Module):
         return f"in={self.in_features}, out={self.out_features}, bias={self.bias is not None}"
 
 
-def _epilogue(y, act, residual, gate, out, coef=None):
+def _epilogue(y, act, residual, gate, out, coef=(0.0, 0.0)):
     import torch.nn.functional as F
     if act == "gelu_tanh":
         y = F.gelu(y.float(), approximate="tanh").to(y.dtype)

@@ -205,14 +205,16 @@ class _Dense(nn.Module):
         super().__init__()
         self.ff = ff
         self.up, self.down = _linear(cfg.hidden_size, ff, dtype, device), _linear(ff, cfg.hidden_size, dtype, device)
-        self.act, self.coef = (_zeros(2, dtype=torch.float32, device=device) for _ in range(2))
+        self.act = _zeros(2, dtype=torch.float32, device=device)
+        self.coef = (0.0, 0.5)                              # set with the weights
 
     def targets(self, p: str, D: int) -> dict:
         return {p + "up": [(self.up.weight[:self.ff, :D], _WHOLE)], p + "down": [(self.down.weight[:D, :self.ff], _WHOLE)],
                 p + "act": [(self.act, _WHOLE)]}
 
     def weights_loaded(self):
-        self.coef.copy_(F.softplus(self.act.double(), threshold=1e9) + self.act.new_tensor([0.0, 0.5]))
+        above, below = F.softplus(self.act.double(), threshold=1e9).tolist()
+        self.coef = (above, 0.5 + below)
 
     def forward(self, xn):
         return self.down(self.up(xn, act="xielu", coef=self.coef))

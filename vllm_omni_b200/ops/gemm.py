@@ -31,7 +31,7 @@ def xielu(z, coef):
     return torch.where(z > 0, coef[0] * z * z, coef[1] * (torch.expm1(z.clamp(max=0)) - z)) + 0.5 * z
 
 
-def linear_reference(x, w, bias=None, act=None, residual=None, gate=None, coef=None):
+def linear_reference(x, w, bias=None, act=None, residual=None, gate=None, coef=(0.0, 0.0)):
     """Plain PyTorch restatement (fp32 accumulate) used on CPU and as the test oracle.
 
     ``gate`` has shape [B, N] and ``x`` [B, S, K] (or [M, K] with B dividing M).
@@ -60,10 +60,10 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, a
            residual: torch.Tensor | None = None, gate: torch.Tensor | None = None,
            out: torch.Tensor | None = None, force_bn: int = 0,
            out_rows_per_batch: int = 0, out_batch_stride: int = 0, scatter=None, row_scatter=None,
-           sync=None, coef: torch.Tensor | None = None) -> torch.Tensor:
+           sync=None, coef: tuple[float, float] = (0.0, 0.0)) -> torch.Tensor:
     """y = residual + gate * act(x @ w.T + bias).
 
-    ``coef``: fp32 [2] on the device, the numbers of ``act="xielu"``.
+    ``coef``: the two numbers of ``act="xielu"``.
 
     ``out_rows_per_batch`` / ``out_batch_stride`` (elements): row r of the result is stored at
     ``out + (r // rpb) * batch_stride + (r % rpb) * out.stride(-2)``; used to write one stream's
@@ -135,19 +135,18 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, a
         rpb = M // gate.shape[0]
         gs = gate.stride(0) if gate.shape[0] > 1 else N
     st = nv.status_word(x.device)
-    assert act != "xielu" or (coef.dtype == torch.float32 and coef.numel() >= 2)
     rc = nv.lib("gemm_sm100").omni_gemm_bf16_coef(
         nv.ptr(x2), ctypes.c_int(x2.stride(0)), nv.ptr(w), ctypes.c_int(w.stride(0)),
         c_ptr, ctypes.c_int(ldc), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
         nv.ptr(bias), nv.ptr(res2), ctypes.c_int(ldr), nv.ptr(gate), ctypes.c_int(gs), ctypes.c_int(rpb),
         ctypes.c_int(ACT[act]), ctypes.c_int(out_rows_per_batch), ctypes.c_long(out_batch_stride),
         ctypes.c_int(sc_P), ctypes.c_int(sc_G), ctypes.c_int(sc_rows), sc_arr, ctypes.c_int(force_bn),
-        nv.ptr(coef), ctypes.byref(sync) if sync is not None else None, nv.ptr(st), nv.stream_ptr())
+        ctypes.c_float(coef[0]), ctypes.c_float(coef[1]), ctypes.byref(sync) if sync is not None else None, nv.ptr(st), nv.stream_ptr())
     nv.check_rc(rc, "omni_gemm_bf16")
     return None if to_peers else out
 
 
-def _linear_f32(x, w, bias, out, act=None, coef=None):
+def _linear_f32(x, w, bias, out, act=None, coef=(0.0, 0.0)):
     """Exact mode: true fp32 products on the CUDA cores (csrc/gemm_f32.cu); ``act(x @ w.T (+ bias))`` only."""
     K, N = x.shape[-1], w.shape[0]
     x2 = x.reshape(-1, K)
@@ -162,13 +161,13 @@ def _linear_f32(x, w, bias, out, act=None, coef=None):
 
 
 def batched_f32(a, w, out, *, bias=None, act=None, batch: int = 1, a_stride: int = 0, w_stride: int = 0, c_stride: int = 0,
-                bias_stride: int = 0, coef=None):
+                bias_stride: int = 0, coef=(0.0, 0.0)):
     """out[b] = act(a[b] @ w[b].T + bias[b]) in true fp32: 2-D operands of batch 0, element strides between batches."""
     rc = nv.lib("gemm_f32").omni_gemm_f32_batched(
         nv.ptr(a), ctypes.c_long(a.stride(0)), nv.ptr(w), ctypes.c_long(w.stride(0)), nv.ptr(out), ctypes.c_long(out.stride(0)),
         ctypes.c_int(a.shape[0]), ctypes.c_int(w.shape[0]), ctypes.c_int(w.shape[1]), nv.ptr(bias), ctypes.c_int(ACT[act]),
         ctypes.c_int(batch), ctypes.c_long(a_stride), ctypes.c_long(w_stride), ctypes.c_long(c_stride), ctypes.c_long(bias_stride),
-        nv.ptr(coef), nv.stream_ptr())
+        ctypes.c_float(coef[0]), ctypes.c_float(coef[1]), nv.stream_ptr())
     nv.check_rc(rc, "omni_gemm_f32_batched")
     return out
 
