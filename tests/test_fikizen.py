@@ -443,5 +443,5 @@ def test_the_checkpoint_tells_the_rank(first):
         W = weights(cfg, rank=rank)
         dec.load_weights(sorted(W.items(), reverse=bool(first)))
         mix = dec.layer(0).mix
-        assert mix.rank == rank and torch.equal(mix.w1.weight[:rank, :72], W["l0.mix.right.w1"].float())
+        assert mix.rank == rank and torch.equal(mix.proj.weight[mix.low_col:mix.low_col + rank, :72], W["l0.mix.right.w1"].float())
         assert torch.equal(mix.w2.weight[32:54, :rank], W["l0.mix.right.w2"][22:44].float())

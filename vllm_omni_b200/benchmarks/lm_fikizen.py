@@ -164,11 +164,10 @@ def kernel_rows(width: int, timer: Timer) -> list[dict]:
             row(f"of it, {tag}", "fikizen gated: convolution", lambda: conv_rows(pg, seqs, TAPS, gs.channels, gated.conv, hist, act="silu",
                 skip_single=True), bytes_=4.0 * rows_ * gs.channels)
     # ---- low-rank decay
-    w1, w2 = rnd(RANK, width) * width ** -0.5, rnd(rs.q_cols, RANK) * RANK ** -0.5
+    low, w2 = rnd(T, 4096 + RANK), rnd(rs.q_cols, RANK) * RANK ** -0.5
     for rows_, tag in ((T, "prompt"), (B, "64 rows")):
-        xr = rnd(rows_, width)
-        row(f"decay logits, {tag}", "fikizen (two GEMMs around a tanh)", lambda: gemm.linear(gemm.linear(xr, w1, act="tanh"), w2),
-            bytes_=2.0 * (rows_ * (width + 2 * RANK + rs.q_cols) + w1.numel() + w2.numel()), flops=2.0 * rows_ * RANK * (width + rs.q_cols))
+        row(f"decay logits, {tag}", "fikizen (tanh, GEMM)", lambda: gemm.linear(lm.tanh_cols(low[:rows_, 4096:]), w2),
+            bytes_=2.0 * (rows_ * (3 * RANK + rs.q_cols) + w2.numel()), flops=2.0 * rows_ * RANK * rs.q_cols)
         small = rnd(width, H * DIM)
         row(f"decay logits, {tag}", "output GEMM", lambda a=rnd(rows_, H * DIM): gemm.linear(a, small),
             bytes_=2.0 * (rows_ * (width + H * DIM) + small.numel()), flops=2.0 * rows_ * width * H * DIM)

@@ -58,9 +58,7 @@ gemm_f32_kernel(const float* __restrict__ A, long lda, const float* __restrict__
         if (act == 3) {                                    // squared ReLU
           v = fmaxf(v, 0.f);
           v *= v;
-        } else if (act == 4) {
-          v = tanhf(v);
-        } else if (act == 5) {                             // xIELU
+        } else if (act == 4) {                             // xIELU
           v = fmaf(0.5f, v, v > 0.f ? c0 * v * v : c1 * (expm1f(v) - v));
         }
         C[(long)m * ldc + n] = v;
@@ -70,13 +68,13 @@ gemm_f32_kernel(const float* __restrict__ A, long lda, const float* __restrict__
 
 }  // namespace omni
 
-// `batch` problems of one shape whose operands lie the given strides apart; act: 0 none, 3 squared ReLU, 4 tanh, 5 xIELU with
+// `batch` problems of one shape whose operands lie the given strides apart; act: 0 none, 3 squared ReLU, 4 xIELU with
 // two numbers (c0 z^2 + z / 2 above zero, c1 (e^z - 1 - z) + z / 2 below).
 extern "C" int omni_gemm_f32_batched(const float* A, long lda, const float* W, long ldw, float* C, long ldc, int M, int N, int K,
                                      const float* bias, int act, int batch, long a_stride, long w_stride, long c_stride,
                                      long bias_stride, float c0, float c1, void* stream) {
   if (M <= 0 || N <= 0 || batch <= 0) return omni::RC_OK;
-  if (K <= 0 || (M + omni::FB - 1) / omni::FB > 65535 || batch > 65535 || act < 0 || act == 1 || act == 2 || act > 5) return omni::RC_BAD_ARG;
+  if (K <= 0 || (M + omni::FB - 1) / omni::FB > 65535 || batch > 65535 || act < 0 || act == 1 || act == 2 || act > 4) return omni::RC_BAD_ARG;
   dim3 grid((N + omni::FB - 1) / omni::FB, (M + omni::FB - 1) / omni::FB, batch);
   const omni::GemmF32Batch b = {a_stride, w_stride, c_stride, bias_stride};
   omni::gemm_f32_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(A, lda, W, ldw, C, ldc, M, N, K, bias, act, c0, c1, b);

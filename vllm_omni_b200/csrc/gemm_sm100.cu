@@ -41,7 +41,7 @@ constexpr int BM = 128;
 constexpr int BK = 64;  // 64 bf16 = one 128-byte swizzle row
 constexpr int GEMM_THREADS = 320;  // warp 0 TMA, warp 1 MMA, warps 2-9 epilogue
 
-enum Act : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU2 = 3, ACT_TANH = 4, ACT_XIELU = 5 };
+enum Act : int { ACT_NONE = 0, ACT_GELU_TANH = 1, ACT_SILU = 2, ACT_RELU2 = 3, ACT_XIELU = 4 };
 
 struct GemmEpilogue {
   const __nv_bfloat16* bias;      // [N] or nullptr
@@ -163,13 +163,6 @@ __device__ __forceinline__ float xielu(float z, float c0, float c1) {
   return fmaf(0.5f, z, z > 0.f ? above : below);
 }
 
-// tanh for values that are rounded to bf16 next
-__device__ __forceinline__ float tanh_short(float z) {
-  const float a = fminf(fabsf(z), 15.f), q = a * a;
-  const float small = a * fmaf(q, fmaf(q, 2.f / 15.f, -1.f / 3.f), 1.f);
-  return copysignf(a < 0.125f ? small : 1.0f - __fdividef(2.0f, __expf(2.0f * a) + 1.0f), z);
-}
-
 // Fused epilogue math for 32 accumulator columns of one output row: bias, activation, gate,
 // residual, bf16 conversion.  o[j] holds columns [col0 + 8j, col0 + 8j + 8); groups at or past N
 // are left untouched.
@@ -201,9 +194,6 @@ __device__ __forceinline__ void epilogue_math32(const uint32_t (&v)[32], int row
           const float r = fmaxf(x[e], 0.f);
           x[e] = r * r;
         }
-      } else if (epi.act == ACT_TANH) {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = tanh_short(x[e]);
       } else if (epi.act == ACT_XIELU) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) x[e] = xielu(x[e], epi.act_c0, epi.act_c1);
@@ -1058,7 +1048,7 @@ static int pick_bn(int M, int N, int ctas) {
 // choose the tile width.
 // `sync` (may be null): arrivals this launch waits for before reading A, and / or reports to the
 // group after its peer stores (see peer_signal.cuh).
-// `act_c0`, `act_c1`: the numbers of act 5 (xIELU).
+// `act_c0`, `act_c1`: the numbers of act 4 (xIELU).
 extern "C" int omni_gemm_bf16_coef(const void* A, int lda, const void* W, int ldw, void* C, int ldc,
                                    int M, int N, int K, const void* bias, const void* residual, int ldr,
                                    const void* gate, int gate_stride, int rows_per_batch, int act,

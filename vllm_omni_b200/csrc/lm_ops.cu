@@ -10,6 +10,7 @@
 //                       the state pool
 //   omni_rotary_heads   norm of whole query and key rows, rotation of the first channels of every head, norm of value heads,
 //                       K/V rows written to their pages
+//   omni_tanh_cols      tanh of some columns of a projection, packed
 //   omni_logit_softcap  mult * logit, bounded to cap * tanh(. / cap) -> fp32
 //
 // Norm gains are fp32, either one number for the whole row (stride 0) or one per channel (stride 1).
@@ -646,6 +647,22 @@ rotary_heads_kernel(const RotaryHeads p) {
   }
 }
 
+// ------------------------------------------------------------------------------ tanh of columns
+template <typename T>
+__global__ void __launch_bounds__(256)
+tanh_cols_kernel(const T* __restrict__ in, long ldi, T* __restrict__ out, long rows, int n) {
+  const int vec = n / 8;
+  for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * vec; i += (long)gridDim.x * blockDim.x) {
+    const long r = i / vec;
+    const int c = (int)(i - r * vec) * 8;
+    float v[8];
+    load8<T>(in + r * ldi + c, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = tanhf(v[e]);
+    store8<T>(out + r * n + c, v);
+  }
+}
+
 // ------------------------------------------------------------------------------ logit cap
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -787,6 +804,17 @@ extern "C" int omni_rotary_heads(const RotaryHeads* args, int is_bf16, void* str
   } while (0)
   if (is_bf16) OMNI_ROTARY(bf16); else OMNI_ROTARY(float);
 #undef OMNI_ROTARY
+  return (int)cudaGetLastError();
+}
+
+extern "C" int omni_tanh_cols(const void* in, long ldi, void* out, long rows, int n, int is_bf16, void* stream) {
+  if (rows <= 0 || n <= 0) return RC_OK;
+  if ((n & 7) || (ldi & 7) || ldi < n || (reinterpret_cast<uintptr_t>(in) & 15)) return RC_BAD_ARG;
+  long blocks = (rows * (n / 8) + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (is_bf16) tanh_cols_kernel<bf16><<<(unsigned)blocks, 256, 0, st>>>((const bf16*)in, ldi, (bf16*)out, rows, n);
+  else tanh_cols_kernel<float><<<(unsigned)blocks, 256, 0, st>>>((const float*)in, ldi, (float*)out, rows, n);
   return (int)cudaGetLastError();
 }
 

@@ -61,8 +61,6 @@ def _epilogue(y, act, residual, gate, out, coef=(0.0, 0.0)):
         y = F.silu(y)
     elif act == "relu2":
         y = F.relu(y).square()
-    elif act == "tanh":
-        y = torch.tanh(y)
     elif act == "xielu":
         y = gemm.xielu(y.float(), coef).to(y.dtype)
     if gate is not None:

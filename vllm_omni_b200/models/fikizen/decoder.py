@@ -8,8 +8,8 @@ One step over a mixed batch (portions of prompts and decoded tokens), per layer:
                        its epilogue -> output GEMM
     gated delta        q | k | v | gate | step size | decay GEMM -> prompts: convolution and silu, chunk matrices, chunked
                        recurrence, norm and gate; decoded tokens: all of it in one kernel -> output GEMM
-    parallel           q | k | v | r | k | v | a | gate GEMM; low-rank decay: two GEMMs around a tanh -> row norms, rotation,
-                       value norm, pages (one kernel) -> attention; channel delta rule; both write one row -> output GEMM
+    parallel           q | k | v | r | k | v | a | gate | low-rank decay GEMM -> tanh, GEMM; row norms, rotation, value norm,
+                       pages (one kernel) -> attention; channel delta rule; both write one row -> output GEMM
     stream step        x += branch, next norm (one kernel)
     feed-forward       up GEMM with xIELU in its epilogue -> down GEMM
 
@@ -29,7 +29,7 @@ from ...ops import lm, stream
 from ...ops.delta_rule import ChannelDelta, DeltaShape, GatedDelta, delta_rule
 from ...ops.stream import RmsRows
 from ...ops.window_attention import ScoreRule, window_attention
-from ..packed_decoder import PackedDecoder, packed_linear as _linear, zeros_param as _zeros
+from ..packed_decoder import PackedDecoder, packed_linear as _linear, round_up, zeros_param as _zeros
 from ..qwen_decoder import ModelBatch
 from .config import AttentionMixer, DeltaMixer, FikizenConfig, LayerConfig, ParallelMixer
 
@@ -143,9 +143,9 @@ class _Parallel(nn.Module):
         super().__init__()
         self.m, self.hs, self.s, self.eps = m, m.left.head_shape, m.right, cfg.norm_eps
         hs, s, D = self.hs, self.s, cfg.hidden_size
-        self.width_, self.dtype_, self.device_ = D, dtype, device
+        self.make = lambda n_in, n_out, **kw: _linear(n_in, n_out, dtype, device, **kw)
+        self.width, self.low_col = D, hs.channels + 5 * s.q_cols
         f32 = lambda *sh: _zeros(*sh, dtype=torch.float32, device=device)
-        self.proj = _linear(D, hs.channels + 5 * s.q_cols, dtype, device, bias=True)
         self.q_gain, self.k_gain = f32(hs.heads * hs.dp), f32(hs.kv_heads * hs.dp)
         self.sink = f32(hs.heads)
         self.norm, self.removal = f32(s.v_cols), f32(s.q_cols)
@@ -155,10 +155,15 @@ class _Parallel(nn.Module):
         self.left_cols = hs.heads * hs.vp
         self.o = _linear(self.left_cols + s.v_cols, D, dtype, device)
 
+    @torch.no_grad()
     def set_rank(self, n: int):
-        self.rank = n
-        self.w1 = _linear(self.width_, n, self.dtype_, self.device_)
-        self.w2 = _linear(n, self.s.q_cols, self.dtype_, self.device_)
+        """Sizes of the low-rank decay: the last rows of the projection, and the matrix behind the tanh."""
+        old = getattr(self, "proj", None)
+        self.rank, self.rank_p, self.proj = n, round_up(n, 8), self.make(self.width, self.low_col + n, bias=True)
+        if old is not None:
+            self.proj.weight[:self.low_col].copy_(old.weight[:self.low_col])
+            self.proj.bias[:self.low_col].copy_(old.bias[:self.low_col])
+        self.w2 = self.make(n, self.s.q_cols)
 
     def targets(self, p: str, D: int) -> dict:
         m, hs, s, W = self.m, self.hs, self.s, self.proj.weight
@@ -173,7 +178,7 @@ class _Parallel(nn.Module):
         parts = _heads(s.dim, s.heads, s.dp)
         for n, w in (("a.b", self.removal), ("w0", self.decay_bias), ("norm", self.norm)):
             t[p + n] = [(w[d], a) for a, d in parts]
-        t[p + "w1"] = [(self.w1.weight[:self.rank, :D], _WHOLE)]
+        t[p + "w1"] = [(W[self.low_col:self.low_col + self.rank, :D], _WHOLE)]
         t[p + "w2"] = [(self.w2.weight[d, :self.rank], a) for a, d in parts]
         t[p + "o"] = [(self.o.weight[:D, self.left_cols + d.start:self.left_cols + d.stop], (_WHOLE, a)) for a, d in parts]
         return t
@@ -184,14 +189,14 @@ class _Parallel(nn.Module):
     def forward(self, xn, batch: ModelBatch, cache, turns):
         m, hs, s = self.m, self.hs, self.s
         proj = self.proj(xn)
-        decay = self.w2(self.w1(xn, act="tanh"))
+        decay = self.w2(lm.tanh_cols(proj[:, self.low_col:self.low_col + self.rank_p]))
         out = torch.empty(xn.shape[0], self.left_cols + s.v_cols, dtype=xn.dtype, device=xn.device)
         # the constant on the left branch rides on its values: the sink has none, so the result is linear in them
         q = lm.rotary_heads(proj, hs, batch.slot_mapping, cache[0], cache[1], turns(m.left), m.left.rot_dims, q_gain=self.q_gain,
                             k_gain=self.k_gain, v_norm=True, v_mult=m.left_scale, eps=self.eps)
         window_attention(q, cache[0], cache[1], batch.seqs, ScoreRule(m.left.scale, sink=self.sink, window=m.left.window),
                          out[:, :self.left_cols])
-        delta_rule(proj[:, hs.channels:], s, batch.seqs, self.rule, cache[2], out[:, self.left_cols:], decay=decay)
+        delta_rule(proj[:, hs.channels:self.low_col], s, batch.seqs, self.rule, cache[2], out[:, self.left_cols:], decay=decay)
         return self.o(out)
 
 

@@ -15,7 +15,7 @@ import torch.nn.functional as F
 
 from . import _native as nv
 
-ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3, "tanh": 4, "xielu": 5}
+ACT = {None: 0, "none": 0, "gelu_tanh": 1, "silu": 2, "relu2": 3, "xielu": 4}
 
 PAIR_BN = 512   # force_bn value that selects the CTA-pair (cta_group::2, 256 x 256 tile) kernel
 
@@ -43,8 +43,6 @@ def linear_reference(x, w, bias=None, act=None, residual=None, gate=None, coef=(
         y = F.silu(y)
     elif act == "relu2":
         y = F.relu(y).square()
-    elif act == "tanh":
-        y = torch.tanh(y)
     elif act == "xielu":
         y = xielu(y, coef)
     if gate is not None:
@@ -91,7 +89,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, a
             return out
         return y
     if x.dtype == torch.float32 and w.dtype == torch.float32:
-        assert act in (None, "relu2", "tanh", "xielu") and residual is None and gate is None and scatter is None and row_scatter is None
+        assert act in (None, "relu2", "xielu") and residual is None and gate is None and scatter is None and row_scatter is None
         return _linear_f32(x, w, bias, out, act, coef)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16, "tcgen05 GEMM path is bf16"
     K = x.shape[-1]

@@ -88,6 +88,17 @@ def poly_norm(z, coef, n: int, eps: float, out=None):
     return out
 
 
+def tanh_cols(x):
+    """tanh of a column view [T, n] (n a multiple of 8), packed."""
+    if not x.is_cuda:
+        return torch.tanh(x.float()).to(x.dtype)
+    assert x.stride(1) == 1
+    out = torch.empty(x.shape[0], x.shape[1], dtype=x.dtype, device=x.device)
+    nv.check_rc(nv.lib("lm_ops").omni_tanh_cols(nv.ptr(x), c_long(x.stride(0)), nv.ptr(out), c_long(x.shape[0]), c_int(x.shape[1]), _bf(x),
+                                                nv.stream_ptr()), "omni_tanh_cols")
+    return out
+
+
 def logit_softcap(logits, cap: float | None, n: int, mult: float = 1.0):
     """``mult`` times the first ``n`` columns of ``logits`` as fp32, bounded to cap * tanh(. / cap) when ``cap`` is set."""
     if not logits.is_cuda:
